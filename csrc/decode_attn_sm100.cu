@@ -21,6 +21,8 @@
 //
 // Cache layout: k_cache / v_cache = [num_slots, Hkv, D] bf16, slot = page * page_size + offset;
 // block_table[b, i] = page id of the i-th page of request b. page_size must be 16, 32, 64 or 128.
+#include <type_traits>
+
 #include "common.cuh"
 
 namespace sb {
@@ -55,14 +57,25 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return r;
 }
 
-template <int D, int G>
+// Windowed form (WIN): the query (the last token) sees the keys of its window and the first `keep_first` tokens, and scores
+// lose slopes[head] * distance. Only tiles with a visible key are visited: those of the kept tokens, then 128-key tiles from
+// the page that holds the window's first key. Head widths dk / dv may be smaller than D (the tensor maps read zeros past
+// them) and the group of query heads smaller than G (`group`; the surplus rows of Q are zero and never written out).
+struct DecWindow {
+  const float* slopes;  // [Hq] or null
+  int window, keep_first, group, dk, dv;
+};
+struct DecFull {};
+
+template <int D, int G, typename Win>
 __global__ void __launch_bounds__(DA_THREADS)
 decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                    const __nv_bfloat16* __restrict__ q, const int* __restrict__ block_table,
                    const int* __restrict__ seq_lens, __nv_bfloat16* __restrict__ out, float* __restrict__ part_o,
                    float* __restrict__ part_ml, int Hq, int Hkv, int page_size, int page_shift, int max_pages,
-                   int q_stride, int out_stride, int splits, float scale, int* status) {
+                   int q_stride, int out_stride, int splits, float scale, int* status, const Win win) {
   using S = DecSmem<D>;
+  constexpr bool WIN = std::is_same<Win, DecWindow>::value;
   constexpr int NCH = S::NCH;
   static_assert(G <= DA_MAXG, "at most 16 query heads per kv head");
   extern __shared__ uint8_t smem_raw[];
@@ -107,20 +120,56 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
   pdl_wait();
   pdl_launch_dependents();
   const int len = seq_lens[b];
-  const int per_split = ((len + splits - 1) / splits + DA_TILE - 1) & ~(DA_TILE - 1);
-  const int t_begin = sp * per_split;
-  const int t_end = min(len, t_begin + per_split);
-  const int ntiles = t_end > t_begin ? (t_end - t_begin + DA_TILE - 1) / DA_TILE : 0;
   const int* bt_row = block_table + static_cast<size_t>(b) * max_pages;
+  int t_begin, t_end, ntiles;
+  int n_keep = 0, win_base = 0, tile0 = 0, low = 0;  // windowed: tiles of kept tokens, first key of the others, this split's first
+  if constexpr (WIN) {
+    low = win.window >= len ? 0 : len - win.window;
+    win_base = (low >> page_shift) << page_shift;
+    n_keep = min((min(win.keep_first, len) + DA_TILE - 1) / DA_TILE, (win_base + DA_TILE - 1) / DA_TILE);
+    win_base = max(win_base, n_keep * DA_TILE);
+    const int total = n_keep + (len > win_base ? (len - win_base + DA_TILE - 1) / DA_TILE : 0);
+    const int per = (total + splits - 1) / splits;
+    tile0 = min(sp * per, total);
+    ntiles = min(total, tile0 + per) - tile0;
+    t_begin = 0;
+    t_end = len;
+  } else {
+    const int per_split = ((len + splits - 1) / splits + DA_TILE - 1) & ~(DA_TILE - 1);
+    t_begin = sp * per_split;
+    t_end = min(len, t_begin + per_split);
+    ntiles = t_end > t_begin ? (t_end - t_begin + DA_TILE - 1) / DA_TILE : 0;
+  }
+  // first key of this CTA's tile i
+  auto tile_key = [&](int i) -> int {
+    if constexpr (WIN) {
+      const int j = tile0 + i;
+      return j < n_keep ? j * DA_TILE : win_base + (j - n_keep) * DA_TILE;
+    } else {
+      return t_begin + i * DA_TILE;
+    }
+  };
   // one coalesced read of the page ids this CTA will need, so that issuing a tile's copies does not wait on them
-  const int my_pages = t_end > t_begin ? ((t_end - t_begin + page_size - 1) >> page_shift) : 0;
-  for (int i = tid; i < min(my_pages, DA_BT_CACHE); i += DA_THREADS) bt_s[i] = bt_row[(t_begin >> page_shift) + i];
+  const int ppt_shift = 7 - page_shift;  // log2 of the pages per tile
+  if constexpr (WIN) {
+    for (int i = tid; i < min(ntiles << ppt_shift, DA_BT_CACHE); i += DA_THREADS) {
+      const int page = (tile_key(i >> ppt_shift) >> page_shift) + (i & ((1 << ppt_shift) - 1));
+      bt_s[i] = page << page_shift < len ? bt_row[page] : 0;
+    }
+  } else {
+    const int my_pages = t_end > t_begin ? ((t_end - t_begin + page_size - 1) >> page_shift) : 0;
+    for (int i = tid; i < min(my_pages, DA_BT_CACHE); i += DA_THREADS) bt_s[i] = bt_row[(t_begin >> page_shift) + i];
+  }
   // Q rows (unscaled bf16; the scale is applied to the fp32 scores) in the canonical K-major 128B-swizzle layout:
   // 16-byte chunk j of row r sits at chunk position j ^ (r % 8).
   for (int i = tid; i < DA_MAXG * NCH * 8; i += DA_THREADS) {
     const int r = i / (NCH * 8), c = (i / 8) % NCH, j = i % 8;
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (r < G)
+    if constexpr (WIN) {
+      if (r < win.group && c * 64 + j * 8 < win.dk)
+        v = *reinterpret_cast<const uint4*>(q + static_cast<size_t>(b) * q_stride + static_cast<size_t>(kvh * win.group + r) * win.dk +
+                                            c * 64 + j * 8);
+    } else if (r < G)
       v = *reinterpret_cast<const uint4*>(q + static_cast<size_t>(b) * q_stride + static_cast<size_t>(kvh * G + r) * D +
                                           c * 64 + j * 8);
     *reinterpret_cast<uint4*>(sQ + c * (DA_MAXG * 128) + r * 128 + ((j ^ (r & 7)) << 4)) = v;
@@ -138,7 +187,7 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
   // V once that tile's O^T is done. With three stages K runs three tiles ahead of the softmax and V two.
   auto issue_half = [&](int i, bool is_k) {
     const int s = i % DA_STAGES;
-    const int t0 = t_begin + i * DA_TILE;
+    const int t0 = tile_key(i);
     const int valid = min(DA_TILE, t_end - t0);
     const int npages = (valid + page_size - 1) >> page_shift;
     uint8_t* dst = sKV + s * S::STAGE + (is_k ? S::KV_TILE : 0);
@@ -146,8 +195,8 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
     if (lane == 0) mbar_arrive_expect_tx(bar, static_cast<uint32_t>(npages * page_size * 128 * NCH));
     __syncwarp();
     if (lane < npages) {
-      const int pi = ((t0 - t_begin) >> page_shift) + lane;  // page index within this CTA's range
-      const int slot0 = (pi < DA_BT_CACHE ? bt_s[pi] : bt_row[(t_begin >> page_shift) + pi]) * page_size;
+      const int pi = WIN ? (i << ppt_shift) + lane : ((t0 - t_begin) >> page_shift) + lane;  // index into the cached ids
+      const int slot0 = (pi < DA_BT_CACHE ? bt_s[pi] : bt_row[(t0 >> page_shift) + lane]) * page_size;
 #pragma unroll
       for (int c = 0; c < NCH; ++c)
         tma_load_3d(dst + c * (DA_TILE * 128) + lane * page_size * 128, is_k ? &tmK : &tmV, bar, c * 64, kvh, slot0);
@@ -214,6 +263,12 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
     keep_prev[g] = 1.f;
     gain_prev[g] = 0.f;
   }
+  float slope2[WIN ? G : 1];
+  if constexpr (WIN) {
+#pragma unroll
+    for (int g = 0; g < G; ++g)
+      slope2[g] = (win.slopes != nullptr && g < win.group) ? win.slopes[kvh * win.group + g] * 1.4426950408889634f : 0.f;
+  }
   const bool merges = tid < D;  // warp-uniform: D is 64 or 128
   // merge tile j (O^T is ready once bar_o completes phase j); its V buffer is then free for tile j + DA_STAGES
   auto merge_tile = [&](int j) -> bool {
@@ -233,7 +288,7 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
 
   for (int i = 0; i < ntiles; ++i) {
     const int s = i % DA_STAGES, par = i & 1;
-    const int t0 = t_begin + i * DA_TILE;
+    const int t0 = tile_key(i);
     const int valid = min(DA_TILE, t_end - t0);
     // ---- scores of this thread's token (TMEM lane = tid) for the G heads
     if (ok) ok = mbar_wait(&bar_s[par], (i >> 1) & 1, cta_abort, status, ERR_WAIT_TMEM_FULL);
@@ -258,8 +313,16 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
 #pragma unroll
         for (int g = 0; g < 32; ++g) r[g] = 0;
       }
+      if constexpr (WIN) {
+        const int key = t0 + tid;
+        const bool see = tid < valid && (key >= low || key < win.keep_first);  // every visited tile has such a key
+        const float back = static_cast<float>(key - (len - 1));
 #pragma unroll
-      for (int g = 0; g < G; ++g) sc[g] = (tid < valid) ? __uint_as_float(r[g]) * scale_log2 : -INFINITY;
+        for (int g = 0; g < G; ++g) sc[g] = see ? fmaf(__uint_as_float(r[g]), scale_log2, slope2[g] * back) : -INFINITY;
+      } else {
+#pragma unroll
+        for (int g = 0; g < G; ++g) sc[g] = (tid < valid) ? __uint_as_float(r[g]) * scale_log2 : -INFINITY;
+      }
     }
 #pragma unroll
     for (int g = 0; g < G; ++g) {
@@ -337,10 +400,16 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
 #pragma unroll
     for (int g = 0; g < G; ++g) {
       const float l_run = red_l[0][g] + red_l[1][g] + red_l[2][g] + red_l[3][g];
-      const int h = kvh * G + g;
+      int h = kvh * G + g, width = D;
+      if constexpr (WIN) {
+        if (g >= win.group) break;
+        h = kvh * win.group + g;
+        width = win.dv;
+      }
       if (splits == 1) {
         const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-        out[static_cast<size_t>(b) * out_stride + static_cast<size_t>(h) * D + tid] = __float2bfloat16(acc[g] * inv);
+        if (!WIN || tid < width)
+          out[static_cast<size_t>(b) * out_stride + static_cast<size_t>(h) * width + tid] = __float2bfloat16(acc[g] * inv);
       } else {
         const size_t base = (static_cast<size_t>(b) * Hq + h) * splits + sp;
         part_o[base * D + tid] = acc[g];
@@ -365,8 +434,9 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
 }
 
 // out[b, h, :] = sum_s o_s exp(m_s - M) / sum_s l_s exp(m_s - M) over the splits of one (request, head).
+// dv: width of an output head (= D, or less where the kernel padded it).
 __global__ void decode_attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                           __nv_bfloat16* __restrict__ out, int D, int splits, int out_stride, int Hq) {
+                                           __nv_bfloat16* __restrict__ out, int D, int dv, int splits, int out_stride, int Hq) {
   pdl_wait();
   pdl_launch_dependents();
   const int bh = blockIdx.x, b = bh / Hq, h = bh % Hq;
@@ -377,11 +447,11 @@ __global__ void decode_attn_combine_kernel(const float* __restrict__ part_o, con
   for (int s = 0; s < splits; ++s)
     if (ml[2 * s] != -INFINITY) gl += ml[2 * s + 1] * __expf(ml[2 * s] - gm);
   const float inv = gl > 0.f ? 1.f / gl : 0.f;
-  for (int d = threadIdx.x; d < D; d += blockDim.x) {
+  for (int d = threadIdx.x; d < dv; d += blockDim.x) {
     float o = 0.f;
     for (int s = 0; s < splits; ++s)
       if (ml[2 * s] != -INFINITY) o += part_o[(static_cast<size_t>(bh) * splits + s) * D + d] * __expf(ml[2 * s] - gm);
-    out[static_cast<size_t>(b) * out_stride + static_cast<size_t>(h) * D + d] = __float2bfloat16(o * inv);
+    out[static_cast<size_t>(b) * out_stride + static_cast<size_t>(h) * dv + d] = __float2bfloat16(o * inv);
   }
 }
 
@@ -406,15 +476,15 @@ static CUtensorMap make_cache_tmap(const void* base, int num_slots, int Hkv, int
   return m;
 }
 
-template <int D, int G>
+template <int D, int G, typename Win = DecFull>
 static int launch_decode_attn(dim3 grid, cudaStream_t s, const CUtensorMap& tk, const CUtensorMap& tv, const __nv_bfloat16* q,
                               const int* bt, const int* sl, __nv_bfloat16* out, float* po, float* pml, int Hq, int Hkv,
                               int page_size, int page_shift, int max_pages, int q_stride, int out_stride, int splits,
-                              float scale, int* status) {
-  auto kern = decode_attn_kernel<D, G>;
+                              float scale, int* status, const Win& win = Win()) {
+  auto kern = decode_attn_kernel<D, G, Win>;
   if (cudaError_t e = ensure_dynamic_smem(reinterpret_cast<const void*>(kern), DecSmem<D>::TOTAL); e != cudaSuccess) return (int)e;
   return (int)launch_pdl(kern, grid, dim3(DA_THREADS), DecSmem<D>::TOTAL, s, tk, tv, q, bt, sl, out, po, pml, Hq, Hkv,
-                         page_size, page_shift, max_pages, q_stride, out_stride, splits, scale, status);
+                         page_size, page_shift, max_pages, q_stride, out_stride, splits, scale, status, win);
 }
 
 }  // namespace sb
@@ -451,6 +521,50 @@ extern "C" int sb_paged_decode_tc(const void* q, const void* k_cache, const void
     if (rc != 0) return rc;
     if (splits > 1)
       return (int)sb::launch_pdl(sb::decode_attn_combine_kernel, dim3(B * Hq), dim3(64), 0, s, part_o, part_ml, (bf16*)out, D,
+                                 D, splits, out_stride, Hq);
+    return (int)cudaGetLastError();
+  } catch (const std::exception& e) {
+    sb::set_last_error(e.what());
+    return (int)cudaErrorInvalidValue;
+  }
+}
+
+// Windowed form (see DecWindow): k_cache [num_slots, Hkv, DK], v_cache [num_slots, Hkv, DV] contiguous, q [B, Hq, DK] with row
+// pitch q_stride, out [B, Hq * DV]; part_o [B, Hq, splits, W] / part_ml [B, Hq, splits, 2] with W = 64 when both widths are at
+// most 64, else 128. Returns -1 for widths above 128 or no multiple of 8, groups above 16 heads, or a misaligned pointer.
+extern "C" int sb_paged_decode_window(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
+                                      const int* seq_lens, const float* slopes, void* out, float* part_o, float* part_ml, int B,
+                                      int Hq, int Hkv, int DK, int DV, int page_size, int max_pages, int num_slots, int q_stride,
+                                      int out_stride, int splits, float scale, int window, int keep_first, int* status,
+                                      cudaStream_t s) {
+  using bf16 = __nv_bfloat16;
+  if (B == 0) return 0;
+  if (Hkv <= 0 || Hq % Hkv != 0 || window < 1 || keep_first < 0 || splits < 1) return (int)cudaErrorInvalidValue;
+  const int G = Hq / Hkv;
+  if (G > 16 || DK <= 0 || DV <= 0 || DK > 128 || DV > 128 || DK % 8 || DV % 8) return -1;
+  int page_shift = 0;
+  while ((1 << page_shift) < page_size) ++page_shift;
+  if ((1 << page_shift) != page_size || page_size < 16 || page_size > 128) return -1;
+  if (((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache)) & 15) || (q_stride & 7))
+    return -1;
+  const int W = DK <= 64 && DV <= 64 ? 64 : 128;
+  try {
+    const CUtensorMap tk = sb::make_cache_tmap(k_cache, num_slots, Hkv, DK, page_size);
+    const CUtensorMap tv = sb::make_cache_tmap(v_cache, num_slots, Hkv, DV, page_size);
+    const sb::DecWindow win{slopes, window, keep_first, G, DK, DV};
+    const dim3 grid(B, Hkv, splits);
+    int rc = -1;
+#define SB_DW(WV, GV)                                                                                                       \
+  if (rc == -1 && W == WV && G <= GV)                                                                                       \
+    rc = sb::launch_decode_attn<WV, GV, sb::DecWindow>(grid, s, tk, tv, (const bf16*)q, block_table, seq_lens, (bf16*)out, part_o, \
+                                                       part_ml, Hq, Hkv, page_size, page_shift, max_pages, q_stride, out_stride,   \
+                                                       splits, scale, status, win);
+    SB_DW(64, 1) SB_DW(64, 2) SB_DW(64, 4) SB_DW(64, 8) SB_DW(64, 16)
+    SB_DW(128, 1) SB_DW(128, 2) SB_DW(128, 4) SB_DW(128, 8) SB_DW(128, 16)
+#undef SB_DW
+    if (rc != 0) return rc;
+    if (splits > 1)
+      return (int)sb::launch_pdl(sb::decode_attn_combine_kernel, dim3(B * Hq), dim3(64), 0, s, part_o, part_ml, (bf16*)out, W, DV,
                                  splits, out_stride, Hq);
     return (int)cudaGetLastError();
   } catch (const std::exception& e) {

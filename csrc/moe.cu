@@ -14,17 +14,17 @@
 
 namespace sb {
 
+// U: copy unit (uint4, or uint16_t for row widths that are no multiple of 8); H = row width in units
+template <typename U>
 __global__ void __launch_bounds__(256)
-moe_scatter_rows_kernel(const __nv_bfloat16* __restrict__ x, const int* __restrict__ dest, __nv_bfloat16* __restrict__ out,
-                        long slots, int k, int H) {
+moe_scatter_rows_kernel(const U* __restrict__ x, const int* __restrict__ dest, U* __restrict__ out, long slots, int k, int H) {
   const int lane = threadIdx.x & 31;
-  const int nvec = H >> 3;
   for (long s = static_cast<long>(blockIdx.x) * 8 + (threadIdx.x >> 5); s < slots; s += static_cast<long>(gridDim.x) * 8) {
     const int d = dest[s];
     if (d < 0) continue;
-    const uint4* src = reinterpret_cast<const uint4*>(x + (s / k) * H);
-    uint4* dst = reinterpret_cast<uint4*>(out + static_cast<long>(d) * H);
-    for (int c = lane; c < nvec; c += 32) dst[c] = src[c];
+    const U* src = x + (s / k) * H;
+    U* dst = out + static_cast<long>(d) * H;
+    for (int c = lane; c < H; c += 32) dst[c] = src[c];
   }
 }
 
@@ -91,7 +91,7 @@ moe_route_weight_grad_kernel(const __nv_bfloat16* __restrict__ rows, const int* 
 constexpr int TOPK_MAX_PER_LANE = 16;
 __global__ void __launch_bounds__(256)
 moe_topk_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int* __restrict__ idx, float* __restrict__ wts,
-                long T, int E, int k, int mode, int renorm, float scale) {
+                long T, int E, long ld, int k, int mode, int renorm, float scale) {
   const int lane = threadIdx.x & 31;
   for (long t = static_cast<long>(blockIdx.x) * 8 + (threadIdx.x >> 5); t < T; t += static_cast<long>(gridDim.x) * 8) {
     float raw[TOPK_MAX_PER_LANE], sel[TOPK_MAX_PER_LANE];
@@ -99,7 +99,7 @@ moe_topk_kernel(const float* __restrict__ logits, const float* __restrict__ bias
 #pragma unroll
     for (int i = 0; i < TOPK_MAX_PER_LANE; ++i) {
       const int e = lane + 32 * i;
-      raw[i] = e < E ? logits[t * E + e] : -INFINITY;
+      raw[i] = e < E ? logits[t * ld + e] : -INFINITY;
       mx = fmaxf(mx, raw[i]);
     }
     mx = warp_max(mx);
@@ -172,6 +172,85 @@ moe_topk_kernel(const float* __restrict__ logits, const float* __restrict__ bias
   }
 }
 
+// Expert-sorted, tile-padded layout of S = T * k routes in one launch of one CTA: every expert's rows start at a multiple
+// of 128, routes keep their order inside an expert. slot_dest[s] = padded row of route s (-1: served elsewhere),
+// tile_expert[i] = expert of the i-th 128-row tile (tiles past the last used one: the last expert).
+// Warp w owns a contiguous range of routes; two sweeps (count, place) with per-warp counters in shared memory, ranks inside
+// a warp by match_any: no atomics, so the layout is the same on every run.
+constexpr int LAYOUT_WARPS = 32;
+constexpr int LAYOUT_TILE = 128;
+__global__ void __launch_bounds__(LAYOUT_WARPS * 32)
+moe_layout_kernel(const int* __restrict__ idx, int* __restrict__ slot_dest, int* __restrict__ tile_expert, int S, int E, int first,
+                  int tiles) {
+  extern __shared__ int sm[];
+  int* cnt = sm;                       // [LAYOUT_WARPS][E]
+  int* pend = sm + LAYOUT_WARPS * E;   // [E] end of the expert's padded range
+  pdl_wait();
+  pdl_launch_dependents();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int i = threadIdx.x; i < LAYOUT_WARPS * E; i += blockDim.x) cnt[i] = 0;
+  __syncthreads();
+  const int per = ((S + LAYOUT_WARPS - 1) / LAYOUT_WARPS + 31) & ~31;
+  const int s0 = warp * per, s1 = min(S, s0 + per);
+  int* mine = cnt + warp * E;
+  for (int b = s0; b < s1; b += 32) {
+    const int s = b + lane;
+    int e = s < s1 ? idx[s] - first : -1;
+    if (e >= E) e = -1;
+    const unsigned peers = __match_any_sync(0xffffffffu, e);
+    if (e >= 0 && (peers & ((1u << lane) - 1)) == 0) mine[e] += __popc(peers);
+    __syncwarp();
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < E; e += blockDim.x) {  // counts -> exclusive prefix over the warps; total in pend
+    int run = 0;
+    for (int w = 0; w < LAYOUT_WARPS; ++w) {
+      const int c = cnt[w * E + e];
+      cnt[w * E + e] = run;
+      run += c;
+    }
+    pend[e] = (run + LAYOUT_TILE - 1) / LAYOUT_TILE * LAYOUT_TILE;
+  }
+  __syncthreads();
+  if (warp == 0) {  // inclusive scan of the padded sizes
+    int carry = 0;
+    for (int b = 0; b < E; b += 32) {
+      int v = b + lane < E ? pend[b + lane] : 0;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int u = __shfl_up_sync(0xffffffffu, v, o);
+        if (lane >= o) v += u;
+      }
+      if (b + lane < E) pend[b + lane] = v + carry;
+      carry += __shfl_sync(0xffffffffu, v, 31);
+    }
+  }
+  __syncthreads();
+  for (int b = s0; b < s1; b += 32) {
+    const int s = b + lane;
+    int e = s < s1 ? idx[s] - first : -1;
+    if (e >= E) e = -1;
+    const unsigned peers = __match_any_sync(0xffffffffu, e);
+    const int rank = __popc(peers & ((1u << lane) - 1));
+    int base = 0;
+    if (e >= 0) base = (e > 0 ? pend[e - 1] : 0) + mine[e];
+    __syncwarp();
+    if (e >= 0 && rank == 0) mine[e] += __popc(peers);
+    __syncwarp();
+    if (s < s1) slot_dest[s] = e >= 0 ? base + rank : -1;
+  }
+  for (int t = threadIdx.x; t < tiles; t += blockDim.x) {
+    const int row = t * LAYOUT_TILE;
+    int lo = 0, hi = E - 1;  // first expert whose range ends after `row`
+    while (lo < hi) {
+      const int mid = (lo + hi) >> 1;
+      if (pend[mid] > row) hi = mid;
+      else lo = mid + 1;
+    }
+    tile_expert[t] = lo;
+  }
+}
+
 static inline int moe_blocks(long items) {
   long b = (items + 7) / 8;
   return static_cast<int>(b < 1 ? 1 : (b > 148 * 16 ? 148 * 16 : b));
@@ -179,11 +258,15 @@ static inline int moe_blocks(long items) {
 
 }  // namespace sb
 
-// All row widths H must be multiples of 8 (16-byte vectors); pointers 16-byte aligned; rows contiguous (pitch H).
+// All row widths H must be multiples of 8 (16-byte vectors; sb_moe_scatter_rows takes any width, and rows of wider elements as
+// that many bf16); pointers 16-byte aligned; rows contiguous (pitch H).
 extern "C" int sb_moe_scatter_rows(const void* x, const int* dest, void* out, long slots, int k, int H, cudaStream_t s) {
   if (slots == 0) return 0;
-  if (H % 8 != 0 || k <= 0) return (int)cudaErrorInvalidValue;
-  sb::moe_scatter_rows_kernel<<<sb::moe_blocks(slots), 256, 0, s>>>((const __nv_bfloat16*)x, dest, (__nv_bfloat16*)out, slots, k, H);
+  if (k <= 0) return (int)cudaErrorInvalidValue;
+  if (H % 8 == 0)
+    sb::moe_scatter_rows_kernel<uint4><<<sb::moe_blocks(slots), 256, 0, s>>>((const uint4*)x, dest, (uint4*)out, slots, k, H / 8);
+  else
+    sb::moe_scatter_rows_kernel<uint16_t><<<sb::moe_blocks(slots), 256, 0, s>>>((const uint16_t*)x, dest, (uint16_t*)out, slots, k, H);
   return (int)cudaGetLastError();
 }
 
@@ -205,12 +288,22 @@ extern "C" int sb_moe_route_weight_grad(const void* rows, const int* dest, const
   return (int)cudaGetLastError();
 }
 
-// logits [T, E] fp32 (row-major, contiguous); bias [E] fp32 or null; idx [T, k] int32; weights [T, k] fp32. k <= 32.
-extern "C" int sb_moe_topk(const float* logits, const float* bias, int* idx, float* weights, long T, int E, int k, int mode,
+// logits [T, E] fp32 (row pitch ld); bias [E] fp32 or null; idx [T, k] int32; weights [T, k] fp32. k <= 32.
+extern "C" int sb_moe_topk(const float* logits, const float* bias, int* idx, float* weights, long T, int E, long ld, int k, int mode,
                            int renorm, float scale, cudaStream_t s) {
   if (T == 0) return 0;
   if (E <= 0 || E > 32 * sb::TOPK_MAX_PER_LANE || k <= 0 || k > 32 || k > E || mode < 0 || mode > 2)
     return (int)cudaErrorInvalidValue;
-  sb::moe_topk_kernel<<<sb::moe_blocks(T), 256, 0, s>>>(logits, bias, idx, weights, T, E, k, mode, renorm, scale);
+  sb::moe_topk_kernel<<<sb::moe_blocks(T), 256, 0, s>>>(logits, bias, idx, weights, T, E, ld, k, mode, renorm, scale);
   return (int)cudaGetLastError();
+}
+
+// idx [S] int32 expert ids; experts first .. first + E - 1 live here. tiles = rows of the padded buffer / 128.
+extern "C" int sb_moe_layout(const int* idx, int* slot_dest, int* tile_expert, int S, int E, int first, int tiles, cudaStream_t s) {
+  if (S == 0) return 0;
+  const int smem = (sb::LAYOUT_WARPS + 1) * E * 4;
+  if (E <= 0 || smem > 200 * 1024) return (int)cudaErrorInvalidValue;
+  if (cudaError_t e = sb::ensure_dynamic_smem(reinterpret_cast<const void*>(sb::moe_layout_kernel), 200 * 1024); e != cudaSuccess)
+    return (int)e;
+  return (int)sb::launch_pdl(sb::moe_layout_kernel, dim3(1), dim3(sb::LAYOUT_WARPS * 32), smem, s, idx, slot_dest, tile_expert, S, E, first, tiles);
 }

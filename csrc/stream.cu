@@ -1,0 +1,285 @@
+// Kernels around an fp32 residual stream, for layers that normalise before and after every sub-layer:
+//   * sb_stream_norm  one launch between two sub-layers: (mixture-of-experts combine, gated shared expert,) post-norm,
+//                     residual add in fp32, pre-norm of the next sub-layer. With `ids` it gathers embedding rows instead
+//                     and starts the stream.
+//   * sb_glu          activation of a feed-forward, gated or not (silu, tanh-gelu, squared relu)
+//   * sb_kv_scatter   new key / value rows into their cache slots, widths and element size free
+// Element types are bf16 or fp32 throughout (fp32: the engine's full-precision mode); all arithmetic is fp32.
+#include "common.cuh"
+
+namespace sb {
+
+template <typename T>
+__device__ __forceinline__ float to_f(T v);
+template <>
+__device__ __forceinline__ float to_f<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ float to_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T>
+__device__ __forceinline__ T from_f(float v);
+template <>
+__device__ __forceinline__ float from_f<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
+
+template <typename T, int VEC>
+__device__ __forceinline__ void load_vec(const T* p, float (&f)[VEC]) {
+  if constexpr (VEC == 8 && sizeof(T) == 2) {
+    const uint4 u = *reinterpret_cast<const uint4*>(p);
+    const float2 a = unpack_bf16x2(u.x), b = unpack_bf16x2(u.y), c = unpack_bf16x2(u.z), d = unpack_bf16x2(u.w);
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y; f[4] = c.x; f[5] = c.y; f[6] = d.x; f[7] = d.y;
+  } else if constexpr (VEC == 8) {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+  } else {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) f[i] = to_f(p[i]);
+  }
+}
+template <typename T, int VEC>
+__device__ __forceinline__ void store_vec(T* p, const float (&f)[VEC]) {
+  if constexpr (VEC == 8 && sizeof(T) == 2) {
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7]));
+  } else if constexpr (VEC == 8) {
+    reinterpret_cast<float4*>(p)[0] = make_float4(f[0], f[1], f[2], f[3]);
+    reinterpret_cast<float4*>(p)[1] = make_float4(f[4], f[5], f[6], f[7]);
+  } else {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) p[i] = from_f<T>(f[i]);
+  }
+}
+
+struct StreamNorm {
+  const void* y;         // sub-layer output [T, H]; with `ids` an embedding table; with `dest` the experts' rows
+  const int* ids;        // row of y per token (null: the token's own row); ids outside [0, y_rows) give a zero row
+  const int* dest;       // [T, k] rows of y of a token's experts, < 0: none (null: no mixture of experts)
+  const float* wts;      // [T, k] their weights
+  const void* shared;    // [T, H] shared expert's output, same type as y, or null
+  const float* gate;     // gate[t * gate_ld]: logit of the shared expert's gate, or null (gate 1)
+  const void* post_w;    // norm of the sub-layer output, or null
+  float* res;            // [T, H] residual stream, updated in place
+  const void* pre_w;     // norm of the next sub-layer's input, or null
+  void* h;               // [T, H] normed input of the next sub-layer
+  int k, y_rows, gate_ld, init, layer_norm, H;  // init: the stream starts here (res is written, not added to)
+  float eps;
+};
+
+// v <- norm(v) * w over the row held by the CTA (thread t holds vectors t, t + THREADS, ...).
+template <typename TW, int VEC, int MAXI, int THREADS>
+__device__ __forceinline__ void row_norm(float (&v)[MAXI][VEC], const TW* w, int H, int nvec, float eps, int layer_norm, float* scratch,
+                                         float (&o)[MAXI][VEC]) {
+  float mean = 0.f;
+  if (layer_norm) {
+    float s = 0.f;
+#pragma unroll
+    for (int j = 0; j < MAXI; ++j)
+      if (static_cast<int>(threadIdx.x) + j * THREADS < nvec)
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) s += v[j][i];
+    mean = block_sum<THREADS>(s, scratch) / H;
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < MAXI; ++j)
+    if (static_cast<int>(threadIdx.x) + j * THREADS < nvec)
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) {
+        const float d = v[j][i] - mean;
+        ss += d * d;
+      }
+  const float rstd = 1.f / sqrtf(block_sum<THREADS>(ss, scratch) / H + eps);
+#pragma unroll
+  for (int j = 0; j < MAXI; ++j) {
+    const int c = threadIdx.x + j * THREADS;
+    if (c < nvec) {
+      float g[VEC];
+      load_vec<TW, VEC>(w + static_cast<size_t>(c) * VEC, g);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) o[j][i] = (v[j][i] - mean) * rstd * g[i];
+    }
+  }
+}
+
+template <typename TY, typename TW, int VEC, int THREADS>
+__global__ void __launch_bounds__(THREADS) stream_norm_kernel(const __grid_constant__ StreamNorm a) {
+  constexpr int MAXI = 32 / VEC;
+  __shared__ float scratch[32];
+  pdl_wait();  // inputs come from the previous kernel in the stream
+  pdl_launch_dependents();
+  const size_t row = blockIdx.x;
+  const int H = a.H, nvec = H / VEC;
+  const TY* y = reinterpret_cast<const TY*>(a.y);
+  const TY* shared = reinterpret_cast<const TY*>(a.shared);
+  size_t src = row;
+  bool have = true;
+  if (a.ids != nullptr) {
+    const int id = a.ids[row];
+    have = id >= 0 && id < a.y_rows;
+    src = have ? id : 0;
+  }
+  const float gate = (shared != nullptr && a.gate != nullptr) ? 1.f / (1.f + expf(-a.gate[row * a.gate_ld])) : 1.f;
+  float v[MAXI][VEC];
+#pragma unroll
+  for (int j = 0; j < MAXI; ++j) {
+    const int c = threadIdx.x + j * THREADS;
+    if (c < nvec) {
+      const size_t off = static_cast<size_t>(c) * VEC;
+      if (a.dest != nullptr) {
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[j][i] = 0.f;
+        for (int r = 0; r < a.k; ++r) {  // route order: the same sum whatever the batch
+          const int d = a.dest[row * a.k + r];
+          if (d < 0) continue;
+          const float wt = a.wts[row * a.k + r];
+          float e[VEC];
+          load_vec<TY, VEC>(y + static_cast<size_t>(d) * H + off, e);
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) v[j][i] = fmaf(wt, e[i], v[j][i]);
+        }
+        if (shared != nullptr) {
+          float e[VEC];
+          load_vec<TY, VEC>(shared + row * H + off, e);
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) v[j][i] = fmaf(gate, e[i], v[j][i]);
+        }
+      } else if (have) {
+        load_vec<TY, VEC>(y + src * H + off, v[j]);
+      } else {
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[j][i] = 0.f;
+      }
+    }
+  }
+  if (a.post_w != nullptr)
+    row_norm<TW, VEC, MAXI, THREADS>(v, reinterpret_cast<const TW*>(a.post_w), H, nvec, a.eps, a.layer_norm, scratch, v);
+#pragma unroll
+  for (int j = 0; j < MAXI; ++j) {
+    const int c = threadIdx.x + j * THREADS;
+    if (c < nvec) {
+      float* rp = a.res + row * H + static_cast<size_t>(c) * VEC;
+      if (!a.init) {
+        float r[VEC];
+        load_vec<float, VEC>(rp, r);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[j][i] += r[i];
+      }
+      store_vec<float, VEC>(rp, v[j]);
+    }
+  }
+  if (a.pre_w != nullptr) {
+    float o[MAXI][VEC];
+    row_norm<TW, VEC, MAXI, THREADS>(v, reinterpret_cast<const TW*>(a.pre_w), H, nvec, a.eps, a.layer_norm, scratch, o);
+    TW* h = reinterpret_cast<TW*>(a.h);
+#pragma unroll
+    for (int j = 0; j < MAXI; ++j) {
+      const int c = threadIdx.x + j * THREADS;
+      if (c < nvec) store_vec<TW, VEC>(h + row * H + static_cast<size_t>(c) * VEC, o[j]);
+    }
+  }
+}
+
+template <typename TY, typename TW>
+static int launch_stream_norm(const StreamNorm& a, int T, bool vec, cudaStream_t s) {
+  if (vec && a.H <= 1024)
+    return (int)launch_pdl(stream_norm_kernel<TY, TW, 8, 128>, dim3(T), dim3(128), 0, s, a);
+  if (vec) return (int)launch_pdl(stream_norm_kernel<TY, TW, 8, 256>, dim3(T), dim3(256), 0, s, a);
+  return (int)launch_pdl(stream_norm_kernel<TY, TW, 1, 256>, dim3(T), dim3(256), 0, s, a);
+}
+
+enum : int { ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_RELU2 = 2 };
+
+__device__ __forceinline__ float activate(float z, int act) {
+  if (act == ACT_SILU) return z / (1.f + expf(-z));
+  if (act == ACT_GELU_TANH) return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  const float r = fmaxf(z, 0.f);
+  return r * r;
+}
+
+// out[t, f] = act(in[t, f]) * in[t, F + f] (gated, in [T, 2F]) or act(in[t, f]) (in [T, F])
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) glu_kernel(const T* __restrict__ in, T* __restrict__ out, long rows, int F, int gated, int act) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int nv = F / VEC;
+  const long n = rows * nv;
+  for (long i = static_cast<long>(blockIdx.x) * 256 + threadIdx.x; i < n; i += static_cast<long>(gridDim.x) * 256) {
+    const long t = i / nv;
+    const int c = static_cast<int>(i - t * nv) * VEC;
+    float g[VEC];
+    load_vec<T, VEC>(in + t * (gated ? 2 * F : F) + c, g);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) g[j] = activate(g[j], act);
+    if (gated) {
+      float u[VEC];
+      load_vec<T, VEC>(in + t * 2 * F + F + c, u);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) g[j] *= u[j];
+    }
+    store_vec<T, VEC>(out + t * F + c, g);
+  }
+}
+
+// One CTA per token: `kb` bytes of its key row and `vb` bytes of its value row to cache slot slots[t] (< 0: skipped).
+template <typename U>
+__global__ void __launch_bounds__(128)
+kv_scatter_kernel(const char* __restrict__ k, const char* __restrict__ v, const int* __restrict__ slots, char* __restrict__ k_cache,
+                  char* __restrict__ v_cache, int kb, int vb, long k_pitch, long v_pitch) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int slot = slots[blockIdx.x];
+  if (slot < 0) return;
+  const U* ks = reinterpret_cast<const U*>(k + blockIdx.x * k_pitch);
+  const U* vs = reinterpret_cast<const U*>(v + blockIdx.x * v_pitch);
+  U* kd = reinterpret_cast<U*>(k_cache + static_cast<long>(slot) * kb);
+  U* vd = reinterpret_cast<U*>(v_cache + static_cast<long>(slot) * vb);
+  const int nk = kb / sizeof(U), nv = vb / sizeof(U);
+  for (int c = threadIdx.x; c < nk + nv; c += blockDim.x) {
+    if (c < nk) kd[c] = ks[c];
+    else vd[c - nk] = vs[c - nk];
+  }
+}
+
+}  // namespace sb
+
+// Types: y_f32 / w_f32 (norm weights and h) = 1 for fp32, 0 for bf16; fp32 weights need fp32 y. H <= 8192.
+extern "C" int sb_stream_norm(const void* y, int y_f32, const int* ids, int y_rows, const int* dest, const float* wts, int k,
+                              const void* shared, const float* gate, int gate_ld, const void* post_w, float* res, int init,
+                              const void* pre_w, void* h, int w_f32, int T, int H, float eps, int layer_norm, cudaStream_t s) {
+  if (T == 0) return 0;
+  if (H <= 0 || H > 8192 || (w_f32 && !y_f32)) return (int)cudaErrorInvalidValue;
+  sb::StreamNorm a{y, ids, dest, wts, shared, gate, post_w, res, pre_w, h, k, y_rows, gate_ld, init, layer_norm, H, eps};
+  bool vec = H % 8 == 0;
+  for (const void* p : {y, shared, post_w, static_cast<const void*>(res), pre_w, static_cast<const void*>(h)})
+    vec = vec && (reinterpret_cast<uintptr_t>(p) & 15) == 0;
+  if (w_f32) return sb::launch_stream_norm<float, float>(a, T, vec, s);
+  if (y_f32) return sb::launch_stream_norm<float, __nv_bfloat16>(a, T, vec, s);
+  return sb::launch_stream_norm<__nv_bfloat16, __nv_bfloat16>(a, T, vec, s);
+}
+
+extern "C" int sb_glu(const void* in, void* out, long rows, int F, int gated, int act, int f32, cudaStream_t s) {
+  if (rows == 0 || F == 0) return 0;
+  if (act < 0 || act > 2) return (int)cudaErrorInvalidValue;
+  const bool vec = F % 8 == 0 && (reinterpret_cast<uintptr_t>(in) & 15) == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0;
+  const long n = rows * (vec ? F / 8 : F);
+  const long want = (n + 255) / 256;
+  const dim3 grid(static_cast<unsigned>(want < 148 * 16 ? want : 148 * 16));
+  using bf16 = __nv_bfloat16;
+  if (f32 && vec) return (int)sb::launch_pdl(sb::glu_kernel<float, 8>, grid, dim3(256), 0, s, (const float*)in, (float*)out, rows, F, gated, act);
+  if (f32) return (int)sb::launch_pdl(sb::glu_kernel<float, 1>, grid, dim3(256), 0, s, (const float*)in, (float*)out, rows, F, gated, act);
+  if (vec) return (int)sb::launch_pdl(sb::glu_kernel<bf16, 8>, grid, dim3(256), 0, s, (const bf16*)in, (bf16*)out, rows, F, gated, act);
+  return (int)sb::launch_pdl(sb::glu_kernel<bf16, 1>, grid, dim3(256), 0, s, (const bf16*)in, (bf16*)out, rows, F, gated, act);
+}
+
+// Row widths and pitches in bytes.
+extern "C" int sb_kv_scatter(const void* k, const void* v, const int* slots, void* k_cache, void* v_cache, int T, int kb, int vb,
+                             long k_pitch, long v_pitch, cudaStream_t s) {
+  if (T == 0) return 0;
+  const uintptr_t bits = reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v) | reinterpret_cast<uintptr_t>(k_cache) |
+                         reinterpret_cast<uintptr_t>(v_cache) | kb | vb | k_pitch | v_pitch;
+  const char *kp = (const char*)k, *vp = (const char*)v;
+  char *kc = (char*)k_cache, *vc = (char*)v_cache;
+  if (bits % 16 == 0) return (int)sb::launch_pdl(sb::kv_scatter_kernel<uint4>, dim3(T), dim3(128), 0, s, kp, vp, slots, kc, vc, kb, vb, k_pitch, v_pitch);
+  if (bits % 4 == 0) return (int)sb::launch_pdl(sb::kv_scatter_kernel<uint32_t>, dim3(T), dim3(128), 0, s, kp, vp, slots, kc, vc, kb, vb, k_pitch, v_pitch);
+  if (bits % 2 == 0) return (int)sb::launch_pdl(sb::kv_scatter_kernel<uint16_t>, dim3(T), dim3(128), 0, s, kp, vp, slots, kc, vc, kb, vb, k_pitch, v_pitch);
+  return (int)cudaErrorInvalidValue;
+}

@@ -19,6 +19,7 @@ release / resume memory by tag (weights | kv_cache | cuda_graph), weight update 
 
 from __future__ import annotations
 
+import dataclasses
 import heapq
 import threading
 import time
@@ -29,12 +30,29 @@ import torch
 
 from slime_b200 import ops
 from slime_b200.engine.kv_cache import OutOfPages, PagedKVCache, _hash_block
-from slime_b200.engine.model_runner import EngineWeights, ModelRunner
+from slime_b200.engine.model_runner import KV_KINDS, EngineWeights, ModelRunner
 from slime_b200.engine.request import ReqState, Request, SamplingParams
 from slime_b200.engine.server_args import ServerArgs
 from slime_b200.models.config import ModelConfig
+from slime_b200.ops.window_attention import ExtendBatch
 
 MEMORY_TAGS = ("weights", "kv_cache", "cuda_graph")
+
+
+@dataclasses.dataclass
+class _PackedTokens:
+    """New tokens of several requests laid end to end: ids, positions and cache slots, boundaries of the requests' new
+    tokens (``cu_q``) and contexts (``cu_k``), and the slots of all context tokens for models that gather them."""
+
+    ids: list = dataclasses.field(default_factory=list)
+    pos: list = dataclasses.field(default_factory=list)
+    slots: list = dataclasses.field(default_factory=list)
+    gather: list = dataclasses.field(default_factory=list)
+    cu_q: list = dataclasses.field(default_factory=lambda: [0])
+    cu_k: list = dataclasses.field(default_factory=lambda: [0])
+    fresh: bool = True
+    max_q: int = 0
+    max_k: int = 0
 
 
 class Engine:
@@ -46,6 +64,10 @@ class Engine:
             torch.device("cuda", torch.cuda.current_device()) if torch.cuda.is_available() else torch.device("cpu")
         )
         self.dtype = torch.bfloat16 if self.device.type == "cuda" else torch.float32
+        if self.args.dtype == "float32" and self.device.type == "cuda":
+            if cfg.layer_specs is None or self.args.quantization:
+                raise ValueError("full precision on a GPU (dtype float32) is available to unquantised models with layer_specs")
+            self.dtype = torch.float32
         self.tokenizer = tokenizer
         self.eos_ids: set[int] = set()
         if tokenizer is not None and getattr(tokenizer, "eos_token_id", None) is not None:
@@ -59,13 +81,12 @@ class Engine:
         if num_pages is None:
             num_pages = self._pages_from_memory()
         self.num_pages = num_pages
-        kv_heads, kv_dim, v_dim = self._kv_geometry()
-        self.kv = PagedKVCache(self._num_kv_layers(), kv_heads, kv_dim, num_pages, self.page_size, self.dtype,
-                               self.device, enable_prefix_cache=not self.args.disable_radix_cache, v_head_dim=v_dim)  # fmt: skip
+        self.kv = PagedKVCache(None, None, None, num_pages, self.page_size, self.dtype, self.device,
+                               enable_prefix_cache=not self.args.disable_radix_cache, geometry=self._kv_geometry())  # fmt: skip
         if self.args.enable_hierarchical_cache and not self.args.disable_radix_cache:
             from slime_b200.engine.kv_cache import HostKVTier
 
-            per_page = PagedKVCache.bytes_per_page(self._num_kv_layers(), kv_heads, kv_dim, self.page_size, self.dtype, v_head_dim=v_dim)
+            per_page = PagedKVCache.bytes_per_page(None, None, None, self.page_size, self.dtype, geometry=self._kv_geometry())
             host_pages = (self.args.hicache_size << 30) // per_page if self.args.hicache_size > 0 else int(num_pages * self.args.hicache_ratio)
             self.kv.allocator.host_tier = HostKVTier(self.kv, host_pages)
         self.runner = ModelRunner(cfg, self.weights, self.kv, self.max_running, self.max_context,
@@ -90,22 +111,26 @@ class Engine:
 
             self.spec = SpeculativeDecoder(self)
 
-    def _kv_geometry(self):
-        """(heads, key width, value width) of one cached token: latent attention caches a single vector per token (the
-        compressed key/value plus the shared rotary key) and no separate values."""
-        c = self.cfg
-        if c.multi_latent_attention:
-            return 1, c.kv_lora_rank + c.qk_pos_emb_head_dim + (c.index_head_dim if c.index_topk else 0), 0
-        return self.weights.hkv, c.head_dim, None
-
-    def _num_kv_layers(self) -> int:
-        """Layers that keep keys and values (delta-net layers keep a recurrent state per decode slot instead)."""
-        return sum(1 for L in self.weights.layers + self.weights.draft if L["kind"] in ("attention", "mla"))
+    def _kv_geometry(self) -> list[tuple[int, int, int]]:
+        """(heads, key width, value width) of one cached token, per layer that keeps keys and values (delta-net layers keep a
+        recurrent state per decode slot instead). Latent attention caches a single vector per token (the compressed
+        key/value plus the shared rotary key) and no separate values."""
+        c, out = self.cfg, []
+        for L in self.weights.layers + self.weights.draft:
+            if L["kind"] not in KV_KINDS:
+                continue
+            if L["kind"] == "window":
+                a = L["spec"].mixer
+                out.append((a.kv_heads // self.weights.tp, a.dim, a.vdim))
+            elif L["kind"] == "mla":
+                out.append((1, c.kv_lora_rank + c.qk_pos_emb_head_dim + (c.index_head_dim if c.index_topk else 0), 0))
+            else:
+                out.append((self.weights.hkv, c.head_dim, c.head_dim))
+        return out
 
     # ----------------------------------------------------------------- sizing
     def _pages_from_memory(self) -> int:
-        kv_heads, kv_dim, v_dim = self._kv_geometry()
-        per_page = PagedKVCache.bytes_per_page(self._num_kv_layers(), kv_heads, kv_dim, self.page_size, self.dtype, v_head_dim=v_dim)
+        per_page = PagedKVCache.bytes_per_page(None, None, None, self.page_size, self.dtype, geometry=self._kv_geometry())
         if self.args.max_total_tokens:
             return max(8, self.args.max_total_tokens // self.page_size)
         if self.device.type != "cuda":
@@ -241,56 +266,77 @@ class Engine:
         return [req.pages[p // ps] * ps + p % ps for p in range(start, end)]
 
     def _to_dev(self, x, dt=torch.int32):
-        host = torch.tensor(x, dtype=dt)
+        host = torch.from_numpy(np.ascontiguousarray(x)).to(dt) if isinstance(x, np.ndarray) else torch.tensor(x, dtype=dt)
         self.stats["h2d_bytes"] += host.numel() * host.element_size()
         if self.device.type == "cuda":
             host = host.pin_memory()
         return host.to(self.device, non_blocking=True)
 
-    def _run_prefill(self, batch) -> list[Request]:
-        t = self._to_dev
-        ids, pos, slots, cu_q, cu_k, gather, last_rows, samplers = [], [], [], [0], [0], [], [], []
-        fresh, max_q, max_k = True, 0, 0
-        want_all_rows = any(r.logprob_start_len >= 0 for r, _ in batch)
-        mrope = self.cfg.mrope_section is not None and any(r.mm is not None for r, _ in batch)
-        streams, emb_rows, emb_vecs, emb_deep = [], [], [], []
+    def _pack(self, batch) -> "_PackedTokens":
+        """The new tokens of ``batch`` (request, count) laid end to end, with where they and their context sit in the cache."""
+        p = _PackedTokens()
         for req, n in batch:
             s, e = req.num_computed, req.num_computed + n
-            ids += req.ctx_ids[s:e]
-            pos += list(range(s, e))
+            p.ids += req.ctx_ids[s:e]
+            p.pos += range(s, e)
+            p.slots += self._slots(req, s, e)
+            p.cu_q.append(p.cu_q[-1] + n)
+            p.cu_k.append(p.cu_k[-1] + e)
+            if not self.runner.layered:
+                p.gather += self._slots(req, 0, e)
+            p.fresh &= s == 0
+            p.max_q, p.max_k = max(p.max_q, n), max(p.max_k, e)
+        return p
+
+    def _extend_pass(self, batch, p: "_PackedTokens", rows, positions=None, embed_rows=None):
+        """One pass of the model over packed tokens -> (logits of ``rows`` or of all rows, the pass's device inputs)."""
+        t = self._to_dev
+        extend = None
+        if self.runner.layered:
+            starts = [r.num_computed for r, _ in batch]
+            extend = ExtendBatch.build([r.pages for r, _ in batch], starts, [n for _, n in batch], self.page_size, self.device, upload=t)
+            positions = extend.positions
+        states = [getattr(req, "gdn_state", None) for req, _ in batch] if self.runner.has_gdn else None
+        dev_in = (t(p.ids), t(p.pos) if positions is None else positions, t(p.slots), t(p.cu_q),
+                  None if p.fresh or self.runner.layered else t(p.gather, torch.long), t(p.cu_k))  # fmt: skip
+        logits = self.runner.prefill(*dev_in, p.max_q, p.max_k, rows, p.fresh, gdn_states=states, embed_rows=embed_rows, extend=extend)
+        if self.runner.has_gdn:
+            for (req, _), st in zip(batch, self.runner.last_gdn_states):
+                req.gdn_state = st
+        return logits, dev_in
+
+    def _run_prefill(self, batch) -> list[Request]:
+        t = self._to_dev
+        want_all_rows = any(r.logprob_start_len >= 0 for r, _ in batch)
+        mrope = self.cfg.mrope_section is not None and any(r.mm is not None for r, _ in batch)
+        p = self._pack(batch)
+        ids, cu_q, max_q, max_k, fresh = p.ids, p.cu_q, p.max_q, p.max_k, p.fresh
+        last_rows, samplers = [], []
+        streams, emb_rows, emb_vecs, emb_deep = [], [], [], []
+        for i, (req, n) in enumerate(batch):
+            s, e = req.num_computed, req.num_computed + n
             if req.mm is not None:
                 self._prepare_vision(req)
                 inside = (req.mm_rows >= s) & (req.mm_rows < e)
                 if bool(inside.any()):
-                    emb_rows.append(req.mm_rows[inside] - s + cu_q[-1])
+                    emb_rows.append(req.mm_rows[inside] - s + cu_q[i])
                     emb_vecs.append(req.mm_embeds[inside])
                     emb_deep.append([d[inside] for d in req.mm_deepstack])
             if mrope:
                 streams.append(self._position_streams(req, s, e))
-            slots += self._slots(req, s, e)
-            cu_q.append(cu_q[-1] + n)
-            cu_k.append(cu_k[-1] + e)
-            gather += self._slots(req, 0, e)
-            fresh &= s == 0
-            max_q, max_k = max(max_q, n), max(max_k, e)
             if e == len(req.ctx_ids):
-                last_rows.append(cu_q[-1] - 1)
+                last_rows.append(cu_q[i + 1] - 1)
                 samplers.append(req)
             if req.state == ReqState.WAITING:
                 req.state = ReqState.RUNNING
                 self.prefilling.append(req)
         rows = None if want_all_rows else t(last_rows, torch.long)
-        states = [getattr(req, "gdn_state", None) for req, _ in batch] if self.runner.has_gdn else None
-        dev_pos = torch.cat(streams, dim=1).to(self.device, torch.int32) if mrope else t(pos)
-        dev_in = (t(ids), dev_pos, t(slots), t(cu_q), None if fresh else t(gather, torch.long), t(cu_k))
+        positions = torch.cat(streams, dim=1).to(self.device, torch.int32) if mrope else None
         embed_rows = None
         if emb_rows:
             deep = [torch.cat([d[k] for d in emb_deep]) for k in range(len(emb_deep[0]))]
             embed_rows = (torch.cat(emb_rows).to(self.device), torch.cat(emb_vecs), deep)
-        logits = self.runner.prefill(*dev_in, max_q, max_k, rows, fresh, gdn_states=states, embed_rows=embed_rows)
-        if self.runner.has_gdn:
-            for (req, _), st in zip(batch, self.runner.last_gdn_states):
-                req.gdn_state = st
+        logits, dev_in = self._extend_pass(batch, p, rows, positions, embed_rows)
         self.stats["prefill_tokens"] += len(ids)
         routed = self.runner.take_routed()
         if routed is not None:
@@ -326,6 +372,69 @@ class Engine:
         if self.spec is not None:
             self.spec.after_prefill(batch, dev_in, cu_q, max_q, max_k, fresh)
         return finished
+
+    # ------------------------------------------------------------------- forced tokens (engine/trace.py, scoring drivers)
+    def open_stream(self, rid: str) -> Request:
+        """A request whose tokens the caller supplies step by step (``feed``). It holds a decode slot and grows its pages like
+        any other request, outside the scheduler's queues."""
+        with self.lock:
+            if not self.free_slots:
+                raise RuntimeError(f"all {self.max_running} request slots are taken")
+            req = Request(rid=rid, input_ids=[], sampling=SamplingParams(max_new_tokens=0), state=ReqState.RUNNING)
+            req.slot = heapq.heappop(self.free_slots)
+            return req
+
+    def close_stream(self, req: Request):
+        with self.lock:
+            heapq.heappush(self.free_slots, req.slot)
+            req.slot = None
+            self._finish(req, {"type": "length", "length": 0})
+
+    def feed(self, entries: list[tuple[Request, list[int], list[int]]]):
+        """One step over ``(stream, its next tokens, places among them whose logits are wanted)``: all entries run as one
+        batch. Single tokens of streams under way take the decode step (its kernels, its CUDA graph), anything else the
+        extend pass, in which portions of prompts and single tokens stand side by side. Returns fp32 logits
+        ``[wanted, vocab]`` in the order of the entries and places, or None when nothing is wanted."""
+        with self.lock:
+            for req, toks, _ in entries:
+                total = req.num_computed + len(toks)
+                if total > self.max_context:
+                    raise ValueError(f"stream {req.rid}: {total} tokens exceed the context length {self.max_context}")
+                need = -(-total // self.page_size) - len(req.pages)
+                if need > 0:
+                    req.pages += self.kv.allocator.alloc(need)
+                req.input_ids += toks
+                req.ctx_ids = req.input_ids
+            single = all(len(toks) == 1 and req.num_computed > 0 for req, toks, _ in entries)
+            logits = self._feed_decode(entries) if single and not self.runner.has_gdn else self._feed_extend(entries)
+            for req, toks, _ in entries:
+                req.num_computed += len(toks)
+            return logits
+
+    def _feed_extend(self, entries):
+        batch = [(req, len(toks)) for req, toks, _ in entries]
+        p = self._pack(batch)
+        rows = [a + w for a, (_, _, want) in zip(p.cu_q, entries) for w in want]
+        logits, _ = self._extend_pass(batch, p, self._to_dev(rows or [0], torch.long))
+        self.stats["prefill_tokens"] += len(p.ids)
+        return logits if rows else None
+
+    def _feed_decode(self, entries):
+        h = self.runner.host
+        for req, toks, _ in entries:
+            b = req.slot
+            h["active"][b], h["init_mask"][b] = 1, 1
+            h["init_ids"][b], h["init_pos"][b], h["init_out_pos"][b] = toks[0], req.num_computed, 0
+            h["block_table"][b, :] = 0
+            h["block_table"][b, : len(req.pages)] = req.pages
+        self.runner.upload_static()
+        self.runner.decode(max(req.slot for req, _, _ in entries) + 1, False)
+        for req, _, _ in entries:
+            self._deactivate(req.slot)
+        self.stats["decode_tokens"] += len(entries)
+        self.stats["decode_steps"] += 1
+        rows = [req.slot for req, _, want in entries for _ in want]
+        return self.runner.last_logits.index_select(0, self._to_dev(rows, torch.long)) if rows else None
 
     # ------------------------------------------------------------------------- vision inputs
     def _prepare_vision(self, req: Request):
@@ -393,10 +502,7 @@ class Engine:
         tokens, copied out of the paged cache (the pages can be released afterwards)."""
         if self.runner.has_gdn:
             raise NotImplementedError("prefill / decode disaggregation does not carry the recurrent state of delta-net layers")
-        slots = torch.tensor(self._slots(req, 0, req.num_computed), dtype=torch.long, device=self.device)
-        k = torch.stack([kl.index_select(0, slots) for kl in self.kv.k])
-        v = torch.stack([vl.index_select(0, slots) for vl in self.kv.v])
-        return k, v
+        return self.kv.export_slots(torch.tensor(self._slots(req, 0, req.num_computed), dtype=torch.long, device=self.device))
 
     def import_request(self, input_ids, first_token: int, first_logprob: float, kv, sampling: SamplingParams | dict | None = None,
                        rid: str | None = None, **kw) -> Request:  # fmt: skip
@@ -411,18 +517,12 @@ class Engine:
         self._req_counter = getattr(self, "_req_counter", 0) + 1
         req.seed = sp.sampling_seed if sp.sampling_seed is not None else (self.args.random_seed * 1000003 + self._req_counter) & 0x7FFFFFFFFFFF
         n = len(req.input_ids)
-        k, v = kv
-        if k.shape[1] != n or k.shape[0] != len(self.kv.k) or tuple(k.shape[2:]) != tuple(self.kv.k[0].shape[1:]):
-            raise ValueError(f"KV of shape {tuple(k.shape)} does not fit {n} tokens of this engine's cache "
-                             f"[{len(self.kv.k)}, *, {tuple(self.kv.k[0].shape[1:])}]")  # fmt: skip
+        self.kv.check_import(n, *kv)
         sp.max_new_tokens = max(0, min(sp.max_new_tokens, self.max_context - n))
         req.weight_version = self.weights.version
         with self.lock:
             req.pages = self.kv.allocator.alloc(-(-(n + 1) // self.page_size))
-            slots = torch.tensor(self._slots(req, 0, n), dtype=torch.long, device=self.device)
-            for li in range(len(self.kv.k)):
-                self.kv.k[li].index_copy_(0, slots, k[li].to(self.device, self.kv.k[li].dtype))
-                self.kv.v[li].index_copy_(0, slots, v[li].to(self.device, self.kv.v[li].dtype))
+            self.kv.import_slots(torch.tensor(self._slots(req, 0, n), dtype=torch.long, device=self.device), *kv)
             req.num_computed = n
             req.ctx_ids = list(req.input_ids)
             req.state = ReqState.RUNNING

@@ -157,11 +157,16 @@ class PagedKVCache:
     """Device tensors + allocator. Memory tag ``kv_cache``: released / re-created as a whole."""
 
     def __init__(self, num_layers, num_kv_heads, head_dim, num_pages, page_size, dtype, device, enable_prefix_cache=True,
-                 v_head_dim: int | None = None):  # fmt: skip
+                 v_head_dim: int | None = None, geometry: list[tuple[int, int, int]] | None = None):  # fmt: skip
         """``v_head_dim``: width of the value slab when it differs from the key slab's (0 for latent attention, whose
-        single cached vector per token serves as key and value)."""
-        self.num_layers, self.hkv, self.d = num_layers, num_kv_heads, head_dim
-        self.dv = head_dim if v_head_dim is None else v_head_dim
+        single cached vector per token serves as key and value). ``geometry``: (kv heads, key width, value width) of every
+        layer, for models whose layers differ; the other sizes are then not used."""
+        if geometry is None:
+            geometry = [(num_kv_heads, head_dim, head_dim if v_head_dim is None else v_head_dim)] * num_layers
+        self.geometry = [tuple(g) for g in geometry]
+        self.num_layers = len(self.geometry)
+        self.uniform = len(set(self.geometry)) <= 1
+        self.hkv, self.d, self.dv = self.geometry[0] if self.geometry else (num_kv_heads, head_dim, v_head_dim or head_dim)
         self.page_size, self.num_pages, self.dtype, self.device = page_size, num_pages, dtype, device
         self.allocator = PageAllocator(num_pages, page_size, enable_prefix_cache)
         self.k: list[torch.Tensor] = []
@@ -172,6 +177,11 @@ class PagedKVCache:
         if self.k:
             return
         slots = self.num_pages * self.page_size
+        if not self.uniform:
+            new = lambda h, w: torch.zeros(slots, h, w, dtype=self.dtype, device=self.device)  # noqa: E731
+            self.k = [new(h, d) for h, d, _ in self.geometry]
+            self.v = [new(h, dv) for h, _, dv in self.geometry]
+            return
         # one slab per kind so a layer's cache is a contiguous view
         self._k_slab = torch.zeros(self.num_layers, slots, self.hkv, self.d, dtype=self.dtype, device=self.device)
         self._v_slab = torch.zeros(self.num_layers, slots, self.hkv, self.dv, dtype=self.dtype, device=self.device)
@@ -188,10 +198,42 @@ class PagedKVCache:
         if torch.cuda.is_available():
             torch.cuda.empty_cache()
 
+    # ---- whole-request and whole-page copies (hand-over between engines, the host tier)
+    def export_slots(self, slots: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
+        """Keys and values of cache slots ``slots`` over all layers: ``[layers, n, kv heads, width]`` each, or, for layers of
+        different geometry, ``[1, n, 1, summed width]``."""
+        k, v = [x.index_select(0, slots) for x in self.k], [x.index_select(0, slots) for x in self.v]
+        if self.uniform:
+            return torch.stack(k), torch.stack(v)
+        flat = lambda xs: torch.cat([x.flatten(1) for x in xs], 1)[None, :, None]  # noqa: E731
+        return flat(k), flat(v)
+
+    def import_slots(self, slots: torch.Tensor, k: torch.Tensor, v: torch.Tensor):
+        """Write what ``export_slots`` of another cache of this geometry returned."""
+        n = slots.numel()
+        self.check_import(n, k, v)
+        for dst, src in ((self.k, k), (self.v, v)):
+            parts = src if self.uniform else src[0, :, 0].split([t[0].numel() for t in dst], dim=1)
+            for t, s in zip(dst, parts):
+                t.index_copy_(0, slots, s.reshape(n, *t.shape[1:]).to(self.device, t.dtype))
+
+    def check_import(self, n: int, k: torch.Tensor, v: torch.Tensor):
+        for dst, src in ((self.k, k), (self.v, v)):
+            want = (len(dst), n, *dst[0].shape[1:]) if self.uniform else (1, n, 1, sum(t[0].numel() for t in dst))
+            if tuple(src.shape) != want:
+                raise ValueError(f"KV of shape {tuple(src.shape)} does not fit {n} tokens of this engine's cache {want}")
+
+    def page_rows(self, page: int) -> list[torch.Tensor]:
+        """Views of one page, layers stacked where their geometry allows it (what the host tier copies)."""
+        rows = slice(page * self.page_size, (page + 1) * self.page_size)
+        return [self._k_slab[:, rows], self._v_slab[:, rows]] if self.uniform else [x[rows] for x in self.k + self.v]
+
     @staticmethod
-    def bytes_per_page(num_layers, num_kv_heads, head_dim, page_size, dtype=torch.bfloat16, v_head_dim: int | None = None) -> int:
-        width = head_dim + (head_dim if v_head_dim is None else v_head_dim)
-        return num_layers * page_size * num_kv_heads * width * torch.empty(0, dtype=dtype).element_size()
+    def bytes_per_page(num_layers, num_kv_heads, head_dim, page_size, dtype=torch.bfloat16, v_head_dim: int | None = None,
+                       geometry=None) -> int:  # fmt: skip
+        if geometry is None:
+            geometry = [(num_kv_heads, head_dim, head_dim if v_head_dim is None else v_head_dim)] * num_layers
+        return sum(h * (d + dv) for h, d, dv in geometry) * page_size * torch.empty(0, dtype=dtype).element_size()
 
 
 class HostKVTier:
@@ -209,57 +251,55 @@ class HostKVTier:
         self.index: collections.OrderedDict[bytes, int] = collections.OrderedDict()  # hash -> host slot, LRU order
         self.free = collections.deque(range(self.num_pages))
         self.hits = self.stores = 0
-        self.k = self.v = None
+        self.pools: list[torch.Tensor] | None = None  # one pinned tensor per view of ``PagedKVCache.page_rows``
         self.allocate()
 
     def allocate(self):
-        if self.k is not None:
+        if self.pools is not None:
             return
-        kv, pin = self.kv, self.kv.device.type == "cuda"
-        self.k = torch.empty(self.num_pages, kv.num_layers, kv.page_size, kv.hkv, kv.d, dtype=kv.dtype, pin_memory=pin)
-        self.v = torch.empty(self.num_pages, kv.num_layers, kv.page_size, kv.hkv, kv.dv, dtype=kv.dtype, pin_memory=pin)
+        pin = self.kv.device.type == "cuda"
+        self.pools = [torch.empty(self.num_pages, *x.shape, dtype=x.dtype, pin_memory=pin) for x in self.kv.page_rows(0)]
 
     def release(self):
         """Free the host pool (``--release-hicache``)."""
         self.flush()
-        self.k = self.v = None
+        self.pools = None
 
     def flush(self):
         self.index.clear()
         self.free = collections.deque(range(self.num_pages))
 
+    @property
+    def k(self) -> torch.Tensor | None:
+        """The pool of the first view (all keys, for layers of equal geometry); None when released."""
+        return None if self.pools is None else self.pools[0]
+
     def num_bytes(self) -> int:
-        return 0 if self.k is None else self.k.numel() * self.k.element_size() + self.v.numel() * self.v.element_size()
+        return sum(x.numel() * x.element_size() for x in self.pools or [])
 
     def touch(self, h: bytes) -> bool:
-        if self.k is None or h not in self.index:
+        if self.pools is None or h not in self.index:
             return False
         self.index.move_to_end(h)
         return True
 
-    def _rows(self, page: int) -> slice:
-        ps = self.kv.page_size
-        return slice(page * ps, (page + 1) * ps)
-
     def store(self, h: bytes, page: int):
-        if self.k is None or self.num_pages == 0 or not self.kv.k:
+        if self.pools is None or self.num_pages == 0 or not self.kv.k:
             return
         if h in self.index:
             self.index.move_to_end(h)
             return
         slot = self.free.popleft() if self.free else self.index.popitem(last=False)[1]
-        rows = self._rows(page)
-        self.k[slot].copy_(self.kv._k_slab[:, rows], non_blocking=True)
-        self.v[slot].copy_(self.kv._v_slab[:, rows], non_blocking=True)
+        for pool, rows in zip(self.pools, self.kv.page_rows(page)):
+            pool[slot].copy_(rows, non_blocking=True)
         self.index[h] = slot
         self.stores += 1
 
     def fetch(self, h: bytes, page: int) -> bool:
         slot = self.index.get(h)
-        if slot is None or self.k is None or not self.kv.k:
+        if slot is None or self.pools is None or not self.kv.k:
             return False
-        rows = self._rows(page)
-        self.kv._k_slab[:, rows].copy_(self.k[slot], non_blocking=True)
-        self.kv._v_slab[:, rows].copy_(self.v[slot], non_blocking=True)
+        for pool, rows in zip(self.pools, self.kv.page_rows(page)):
+            rows.copy_(pool[slot], non_blocking=True)
         self.hits += 1
         return True

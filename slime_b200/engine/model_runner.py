@@ -19,11 +19,18 @@ import torch
 from slime_b200 import ops
 from slime_b200.engine.kv_cache import PagedKVCache
 from slime_b200.models.config import ModelConfig
+from slime_b200.models.layer_spec import LayerSpec
+from slime_b200.ops import stream
 
 logger = logging.getLogger(__name__)
 
 _LAYER_RE = re.compile(r"^model\.layers\.(\d+)\.(.+)$")
+_LAYERED_RE = re.compile(r"^l(\d+)\.(.+)$")  # designs described layer by layer (models/layer_spec.py)
+_LAYERED_TOP = {"embed": "model.embed_tokens.weight", "head": "lm_head.weight", "final.norm": "model.norm.weight"}
 _MIMO_DRAFT_RE = re.compile(r"^model\.mtp_layers\.(\d+)\.(.+)$")
+
+
+KV_KINDS = ("attention", "mla", "window")  # layer kinds that keep keys and values in the paged cache
 
 
 class EngineWeights:
@@ -77,6 +84,9 @@ class EngineWeights:
         self.num_draft_layers = draft_layers
         for i in range(cfg.num_layers + draft_layers):
             kind = cfg.mixer(i)
+            if kind == "window_attention":
+                self.layers.append(self._specified_buffers(cfg.layer_specs[i], e, mat))
+                continue
             if kind not in ("attention", "general_attention", "gated_delta_net", "mla", "dsa"):
                 raise NotImplementedError(f"the rollout engine has no layer of kind {kind!r} (layer {i})")
             full_norm = cfg.qk_layernorm_full  # one weight per projection (sharded like it) instead of one per head
@@ -156,6 +166,78 @@ class EngineWeights:
             L["sinks"] = torch.zeros(self.hq, dtype=torch.float32, device=self.device)  # per-head logit in the denominator
         return L
 
+    def _specified_buffers(self, spec, e, mat) -> dict:
+        """Buffers of a layer that has its own ``LayerSpec``: fused q | k | v rows, gate and up rows stacked, the router's rows
+        followed by the shared expert's gate (one product computes both; rows padded to a multiple of 8)."""
+        h, a, m, tp = self.cfg.hidden_size, spec.mixer, spec.mlp, self.tp
+        if a.heads % tp or a.kv_heads % tp or self.cfg.padded_vocab_size % tp:
+            raise ValueError(f"{a.heads} query / {a.kv_heads} key-value heads and a vocabulary of {self.cfg.padded_vocab_size} do not "
+                             f"divide over {tp} tensor-parallel ranks")  # fmt: skip
+        hq, hkv = a.heads // tp, a.kv_heads // tp
+        parts = (hq * a.dim, (hq + hkv) * a.dim)
+        L = {"kind": "window", "spec": spec, "ln1": e(h), "post_attn_ln": e(h), "o": mat(h, hq * a.vdim),
+             "qkv": mat((hq + hkv) * a.dim + hkv * a.vdim, h, parts=parts)}  # fmt: skip
+        if m is None:
+            return L
+        L.update(ln2=e(h), post_mlp_ln=e(h))
+        up = 2 if m.gated else 1
+        if m.experts is None:
+            if m.ff % tp:
+                raise ValueError(f"a feed-forward of width {m.ff} does not divide over {tp} tensor-parallel ranks")
+            f = m.ff // tp
+            L.update(gate_up=mat(up * f, h, parts=(f,)), down=mat(h, f))
+            return L
+        if m.experts % self.ep or m.shared_ff % tp:
+            raise ValueError(f"{m.experts} experts / a shared expert of width {m.shared_ff} do not divide over {tp} ranks")
+        el, fs = m.experts // self.ep, m.shared_ff // tp
+        L.update(first_expert=0 if self.ep == 1 else self.rank * el, router=e(-(-(m.experts + 1) // 8) * 8, h),
+                 w13=mat(el, up * m.ff, h, parts=(m.ff,)), w2=mat(el, h, m.ff))  # fmt: skip
+        if m.shared_ff:
+            L.update(shared_gate_up=mat(up * fs, h, parts=(fs,)), shared_down=mat(h, fs))
+        return L
+
+    def _load_specified(self, L, sub: str, t, raw) -> bool:
+        """One tensor of a specified layer, addressed by its name behind ``l<i>.``."""
+        spec, h, tp = L["spec"], self.cfg.hidden_size, self.tp
+        a, m = spec.mixer, spec.mlp
+        norms = {"norm1": "ln1", "norm1b": "post_attn_ln", "norm2": "ln2", "norm2b": "post_mlp_ln"}
+        if sub in norms:
+            if norms[sub] not in L:
+                return False
+            L[norms[sub]].copy_(t)
+            return True
+        q, k, v = a.heads // tp * a.dim, a.kv_heads // tp * a.dim, a.kv_heads // tp * a.vdim
+        table = {"mix.q": ("qkv", 0, q, 0), "mix.k": ("qkv", q, k, 0), "mix.v": ("qkv", q + k, v, 0), "mix.o": ("o", 0, h, 1)}
+        if m is not None and m.experts is None:
+            f = m.ff // tp
+            table.update({"mlp.gate": ("gate_up", 0, f, 0), "mlp.up": ("gate_up", f if m.gated else 0, f, 0), "mlp.down": ("down", 0, h, 1)})
+        if m is not None and m.experts is not None:
+            if sub == "mlp.router":
+                L["router"][: m.experts].copy_(t)
+                return True
+            if sub == "mlp.shared.sg" and m.shared_gate:
+                L["router"][m.experts].copy_(t.view(-1))
+                return True
+            fs = m.shared_ff // tp
+            if m.shared_ff:
+                table.update({"mlp.shared.gate": ("shared_gate_up", 0, fs, 0), "mlp.shared.up": ("shared_gate_up", fs if m.gated else 0, fs, 0),
+                              "mlp.shared.down": ("shared_down", 0, h, 1)})  # fmt: skip
+            em = re.match(r"^mlp\.e(\d+)\.(gate|up|down)$", sub)
+            if em is not None and int(em.group(1)) < m.experts:
+                e, which = int(em.group(1)) - L["first_expert"], em.group(2)
+                if not 0 <= e < L["w2"].shape[0]:
+                    return True  # another rank's expert
+                if which == "down":
+                    self._put(L["w2"][e], 0, h, None, t, raw, scale=False)
+                else:
+                    self._put(L["w13"][e], m.ff if which == "up" and m.gated else 0, m.ff, None, t, raw, scale=False)
+                return True
+        if sub not in table or (sub.endswith(".gate") and not m.gated):
+            return False
+        key, r0, rows, cut = table[sub]
+        self._put(L[key], r0, rows, cut, t, raw, scale=False)
+        return True
+
     def num_bytes(self) -> int:
         seen, total = set(), 0
         for t in self.tensors():
@@ -172,7 +254,7 @@ class EngineWeights:
             yield from self.vision.parameters()
         for L in self.layers + self.draft:
             for v in L.values():
-                if v is None or isinstance(v, (str, int)):  # absent buffers, the layer's kind tag, the indexer's source layer
+                if v is None or isinstance(v, (str, int, LayerSpec)):  # absent buffers, kind tag, indexer's source layer, spec
                     continue
                 if hasattr(v, "tensors"):  # a quantised matrix: its bytes and its scales
                     yield from v.tensors()
@@ -186,6 +268,12 @@ class EngineWeights:
 
     def load_weight(self, name: str, t: torch.Tensor):
         cfg, d = self.cfg, self.cfg.head_dim
+        if cfg.layer_specs is not None:
+            m = _LAYERED_RE.match(name)
+            if m is not None:
+                return int(m.group(1)) < len(self.layers) and self._load_specified(
+                    self.layers[int(m.group(1))], m.group(2), t.to(self.device, self.dtype, non_blocking=True), t)
+            name = _LAYERED_TOP.get(name, name)
         if name.startswith("model.visual."):  # the image encoder keeps the checkpoint's parameter names
             if self.vision is None:
                 return True
@@ -434,8 +522,9 @@ class ModelRunner:
         self.max_batch, self.max_context = max_batch, max_context
         self.max_pages_per_req = -(-max_context // kv.page_size)
         # head dims other than 64 / 128 fall back to attention written with plain ops, which reads lengths on the host
-        self.use_cuda_graph = (use_cuda_graph and self.device.type == "cuda" and cfg.head_dim in (64, 128)
-                               and not cfg.multi_latent_attention and not cfg.softmax_sinks)  # fmt: skip
+        self.layered = cfg.layer_specs is not None  # fp32 residual stream, layers described one by one
+        self.use_cuda_graph = use_cuda_graph and self.device.type == "cuda" and (self.layered or (
+            cfg.head_dim in (64, 128) and not cfg.multi_latent_attention and not cfg.softmax_sinks))  # fmt: skip
         self.tp_group = tp_group
         # Row-parallel projections (attention output, MLP down) leave their result in fp32 when no cross-rank sum
         # follows: the fused add+RMSNorm reads it unrounded, and a skinny decode GEMM with a long K can then be cut
@@ -444,7 +533,7 @@ class ModelRunner:
         # Tensor-parallel decode: all-reduce + residual add + RMSNorm as one peer-memory kernel when the ranks share an
         # NVLink domain; otherwise NCCL all-reduce followed by the fused add+norm.
         self._fused_tp = None
-        if tp_group is not None and weights.tp > 1 and self.device.type == "cuda":
+        if tp_group is not None and weights.tp > 1 and self.device.type == "cuda" and not self.layered:
             from slime_b200.parallel import fused_tp
 
             if fused_tp.usable(weights.tp, self.device, cfg.hidden_size):
@@ -455,8 +544,8 @@ class ModelRunner:
         # KV slabs exist for the attention layers only; gated delta-net layers keep a recurrent state per decode slot
         self.kv_of, n_attn = [], 0
         for L in weights.layers + weights.draft:  # a draft head's layer number is num_layers + depth
-            self.kv_of.append(n_attn if L["kind"] in ("attention", "mla") else None)
-            n_attn += L["kind"] in ("attention", "mla")
+            self.kv_of.append(n_attn if L["kind"] in KV_KINDS else None)
+            n_attn += L["kind"] in KV_KINDS
         self.has_mla = any(L["kind"] == "mla" for L in weights.layers)
         self._dsa_masks: dict[int, torch.Tensor] = {}  # key choices of the indexer layers of the pass in flight
         self.has_gdn = any(L["kind"] == "gdn" for L in weights.layers)
@@ -474,7 +563,13 @@ class ModelRunner:
         self.rope_delta = torch.zeros(max_batch, dtype=torch.int32, device=self.device) if cfg.mrope_section else None
         self._mrope_axes = None
         rot = int(cfg.head_dim * cfg.rotary_percent) // 2 * 2
-        self.rope = ops.rope_table(cfg, max_context + 1, rot, self.device)
+        self.rope = None if self.layered else ops.rope_table(cfg, max_context + 1, rot, self.device)
+        self.slopes = []  # specified layers: distance-penalty factors of this rank's query heads
+        for L in weights.layers if self.layered else ():
+            sl, n = L["spec"].mixer.slopes(), L["spec"].mixer.heads // weights.tp
+            mine = None if sl is None else sl[weights.rank * n : (weights.rank + 1) * n]
+            self.slopes.append(None if mine is None else torch.tensor(mine, dtype=torch.float32, device=self.device))
+        self.stream_hook = None  # called with (layer, fp32 residual stream) after every specified layer (eager passes only)
         self.scale = 1.0 / math.sqrt(cfg.head_dim)
         if cfg.multi_latent_attention:
             from slime_b200.models import mixers
@@ -493,6 +588,7 @@ class ModelRunner:
                                            device=self.device)  # fmt: skip
         self._routed: list[torch.Tensor] = []
         self.last_routed = None
+        self.last_logits = None  # fp32 logits of the last decode step, one row per slot (a buffer of the graph)
         self.last_hidden = None  # residual stream before the final norm of the last prefill pass, all rows (draft heads read it)
 
     def take_routed(self):
@@ -813,6 +909,63 @@ class ModelRunner:
             self.gdn_S[li][slot].copy_(S)
             self.gdn_conv[li][slot].copy_(hist)
 
+    # ------------------------------------------------------------ specified layers (models/layer_spec.py)
+    def _specified_layers(self, ids, slots, attend):
+        """All layers of a model with ``layer_specs`` over the tokens ``ids`` -> the final norm's output. ``attend(li, spec, q)``
+        runs layer ``li``'s attention once its keys and values are in the cache: the only part that differs between a
+        prefill pass and a decode step. The residual stream is fp32; between two sub-layers there is one fused launch."""
+        cfg, w, eps = self.cfg, self.w, self.cfg.norm_epsilon
+        kind, f32 = cfg.norm_kind, torch.float32
+        first = w.layers[0]["ln1"]
+        if w.tp > 1:  # vocab-parallel table: rows of other ranks come out as zeros
+            x = self._tp_reduce(stream.stream_norm(w.embed, None, None, eps, ids=ids - w.rank * w.vocab_local)[1])
+            h, res = stream.stream_norm(x, None, first, eps, kind=kind)
+        else:
+            h, res = stream.stream_norm(w.embed, None, first, eps, kind=kind, ids=ids)
+        for li, L in enumerate(w.layers):
+            spec, a = L["spec"], L["spec"].mixer
+            hq, hkv = a.heads // w.tp, a.kv_heads // w.tp
+            qkv = _linear(h, L["qkv"])
+            nq, nk = hq * a.dim, hkv * a.dim
+            stream.kv_scatter(qkv[:, nq : nq + nk], qkv[:, nq + nk :], slots, self.kv.k[self.kv_of[li]], self.kv.v[self.kv_of[li]])
+            ctx = attend(li, a, qkv[:, :nq].unflatten(1, (hq, a.dim)))
+            y = self._tp_reduce(_linear(ctx.flatten(1), L["o"], out_dtype=f32))
+            after = w.layers[li + 1]["ln1"] if li + 1 < len(w.layers) else w.final_norm
+            h, _ = stream.stream_norm(y, res, after if spec.mlp is None else L["ln2"], eps, kind=kind, post_w=L["post_attn_ln"])
+            if spec.mlp is not None:
+                h, _ = stream.stream_norm(self._specified_mlp(L, spec.mlp, h), res, after, eps, kind=kind, post_w=L["post_mlp_ln"])
+            if self.stream_hook is not None:
+                self.stream_hook(li, res)
+        return h
+
+    def _specified_mlp(self, L, m, h):
+        """Feed-forward of a specified layer: fp32 output, or for experts the unfinished sum the next norm completes."""
+        w, f32 = self.w, torch.float32
+        if m.experts is None:
+            act = stream.feed_forward_act(_linear(h, L["gate_up"]), m.act, m.gated)
+            return self._tp_reduce(_linear(act, L["down"], out_dtype=f32))
+        from slime_b200.ops import grouped
+
+        # bf16 products are exact in fp32, so the tensor-core product is a 32-bit router too; the CUDA-core kernel is the
+        # faster one for a handful of tokens
+        big = h.is_cuda and h.dtype == torch.bfloat16 and h.shape[0] >= 256
+        logits = ops.gemm(h, L["router"], out_dtype=f32, splitk=1) if big else ops.router_gemm(h, L["router"])
+        probs, idx = grouped.route_topk(logits[:, : m.experts], m.top, score=m.score, renorm=m.renorm, raw_index=True)
+        if self.record_routed:
+            pad = self.cfg.moe_router_topk - m.top
+            self._routed.append(torch.nn.functional.pad(idx.to(torch.int32), (0, pad)) if pad else idx.to(torch.int32))
+        lay = grouped.DeviceLayout(idx, L["w13"].shape[0], L["first_expert"])
+        rows = _grouped_linear(stream.feed_forward_act(_grouped_linear(lay.pad(h), L["w13"], lay), m.act, m.gated), L["w2"], lay)
+        out = stream.ExpertSum(rows, lay.slot_dest, probs)
+        if m.shared_ff:
+            out.shared = _linear(stream.feed_forward_act(_linear(h, L["shared_gate_up"]), m.act, m.gated), L["shared_down"])
+            out.gate = logits[:, m.experts] if m.shared_gate else None
+        if w.ep > 1:  # this rank's experts and its part of the shared one travel in one reduction
+            return self._tp_reduce(stream.combine(out))
+        if w.tp > 1 and out.shared is not None:
+            out.shared = self._tp_reduce(out.shared)
+        return out
+
     def _post_norm(self, x, w):
         """GLM-4 sandwich norm: the sub-layer's output is normalised before it joins the residual stream."""
         return x if w is None else ops.rmsnorm(x, w, self.cfg.norm_epsilon)[0]
@@ -820,7 +973,7 @@ class ModelRunner:
     # --------------------------------------------------------------------- prefill
     @torch.no_grad()
     def prefill(self, ids, positions, slots, cu_q, kv_gather_slots, cu_k, max_q, max_k, last_rows, fresh: bool, gdn_states=None,
-                embed_rows=None):
+                embed_rows=None, extend=None):
         """Extend pass over packed new tokens.
 
         ids/positions/slots: [T] for the new tokens; ``cu_q`` their per-request boundaries.
@@ -831,8 +984,20 @@ class ModelRunner:
         None); the states after this pass are left in ``last_gdn_states``.
         Vision inputs: ``positions`` may be ``[3, T]`` (temporal / height / width streams) and ``embed_rows`` = (rows,
         vectors) replaces the embeddings of image placeholder tokens by the encoder's outputs.
+        Models with specified layers read the context from the cache pages: ``extend`` (``ops.window_attention.ExtendBatch``)
+        says where every row stands, ``kv_gather_slots`` is not used.
         """
         cfg, w, d = self.cfg, self.w, self.cfg.head_dim
+        if self.layered:
+            from slime_b200.ops import window_attention
+
+            def attend(li, a, q):
+                kv = self.kv_of[li]
+                return window_attention.window_extend(q, self.kv.k[kv], self.kv.v[kv], extend, a.scale, a.window, a.keep_first, self.slopes[li])
+
+            h = self._specified_layers(ids, slots, attend)
+            h = h if last_rows is None else h.index_select(0, last_rows)
+            return self._gather_logits(ops.gemm(h, w.lm_head, out_dtype=torch.float32))
         x = ops.embedding(ids, w.embed, w.rank * w.vocab_local)
         x = self._tp_reduce(x) if w.tp > 1 else x
         deepstack = []
@@ -987,8 +1152,9 @@ class ModelRunner:
         return stage.numel() * 4
 
     def _decode_step(self, n: int, filtered: bool, kept_cap: int):
-        """prepare -> model -> sample -> advance for slots [0, n). Returns (tokens, logprobs, kept_ids, kept_cnt)."""
-        cfg, w, d = self.cfg, self.w, self.cfg.head_dim
+        """prepare -> model -> sample -> advance for slots [0, n). Returns (tokens, logprobs, kept_ids, kept_cnt, routed
+        experts, logits)."""
+        w = self.w
         st, ds = self._static, self._dev_state
         ps, W = self.kv.page_size, self.max_pages_per_req
         ids, pos, seq_lens, slots = ds["ids_eff"][:n], ds["pos_eff"][:n], ds["seq_lens"][:n], ds["slots"][:n]
@@ -1003,6 +1169,35 @@ class ModelRunner:
                 P(ds["seq_lens"]), P(ds["slots"]), n, ps, W, _lib.stream()), "sb_decode_prepare")  # fmt: skip
         else:
             self._prepare_reference(n)
+        h = self._decode_layers(n, ids, pos, slots, bt, seq_lens)
+        logits = self._gather_logits(ops.gemm(h, w.lm_head, out_dtype=torch.float32))
+        tok, lp, kept_ids, kept_cnt = ops.sample(
+            logits, st["temperature"][:n], st["top_k"][:n] if filtered else None, st["top_p"][:n] if filtered else None,
+            st["min_p"][:n] if filtered else None, st["seeds"][:n], ds["out_pos"][:n], kept_cap,
+        )  # fmt: skip
+        routed = self.take_routed()
+        if self.device.type == "cuda":
+            _lib.check(_lib.lib().sb_decode_advance(P(ds["ids"]), P(ds["pos"]), P(ds["out_pos"]), P(st["active"]), P(tok), n,
+                                                    _lib.stream()), "sb_decode_advance")  # fmt: skip
+        else:
+            act = st["active"][:n].bool()
+            ds["ids"][:n] = torch.where(act, tok, ds["ids"][:n])
+            ds["pos"][:n] += act.int()
+            ds["out_pos"][:n] += act.int()
+        return tok, lp, kept_ids, kept_cnt, routed, logits
+
+    def _decode_layers(self, n, ids, pos, slots, bt, seq_lens):
+        """Embedding to final norm for one token per slot."""
+        cfg, w, d, ps = self.cfg, self.w, self.cfg.head_dim, self.kv.page_size
+        if self.layered:
+            from slime_b200.ops import window_attention
+
+            def attend(li, a, q):
+                kv = self.kv_of[li]
+                return window_attention.window_decode(q, self.kv.k[kv], self.kv.v[kv], bt, seq_lens, pos, ps, a.scale, a.window, a.keep_first,
+                                                      self.slopes[li], self.max_context)  # fmt: skip
+
+            return self._specified_layers(ids, slots, attend)
         if self.rope_delta is not None:
             pos = pos + self.rope_delta[:n]  # rotary position of a request that carries images
         x = ops.embedding(ids, w.embed, w.rank * w.vocab_local)
@@ -1033,22 +1228,7 @@ class ModelRunner:
                 normed, res = self._row_parallel_norm(act, L["down"], next_ln, res, n, post=L["post_mlp_ln"])
             else:
                 normed, res = ops.rmsnorm(self._post_norm(self._moe(L, normed), L["post_mlp_ln"]), next_ln, cfg.norm_epsilon, res)
-        h = normed
-        logits = self._gather_logits(ops.gemm(h, w.lm_head, out_dtype=torch.float32))
-        tok, lp, kept_ids, kept_cnt = ops.sample(
-            logits, st["temperature"][:n], st["top_k"][:n] if filtered else None, st["top_p"][:n] if filtered else None,
-            st["min_p"][:n] if filtered else None, st["seeds"][:n], ds["out_pos"][:n], kept_cap,
-        )  # fmt: skip
-        routed = self.take_routed()
-        if self.device.type == "cuda":
-            _lib.check(_lib.lib().sb_decode_advance(P(ds["ids"]), P(ds["pos"]), P(ds["out_pos"]), P(st["active"]), P(tok), n,
-                                                    _lib.stream()), "sb_decode_advance")  # fmt: skip
-        else:
-            act = st["active"][:n].bool()
-            ds["ids"][:n] = torch.where(act, tok, ds["ids"][:n])
-            ds["pos"][:n] += act.int()
-            ds["out_pos"][:n] += act.int()
-        return tok, lp, kept_ids, kept_cnt, routed
+        return normed
 
     def _prepare_reference(self, n):
         st, ds = self._static, self._dev_state
@@ -1072,7 +1252,7 @@ class ModelRunner:
         captured too: their expert-sorted layout is built on the device with static shapes. ``last_routed`` holds the
         step's expert choices when ``record_routed`` is set (a buffer of the graph: copy it before the next replay)."""
         if not self.use_cuda_graph:
-            *outs, self.last_routed = self._decode_step(n, filtered, kept_cap)
+            *outs, self.last_routed, self.last_logits = self._decode_step(n, filtered, kept_cap)
             return tuple(outs)
         bucket = next(b for b in self.graph_buckets if b >= n)
         key = (bucket, filtered, kept_cap)
@@ -1081,7 +1261,7 @@ class ModelRunner:
         graph, outs, n_kernels = self.graphs[key]
         self.replayed_launches += n_kernels
         graph.replay()
-        self.last_routed = outs[4]
+        self.last_routed, self.last_logits = outs[4], outs[5]
         return outs[:4]
 
     def _capture(self, bucket, filtered, kept_cap):

@@ -11,6 +11,7 @@ import json
 import os
 from dataclasses import dataclass
 
+from slime_b200.models.layer_spec import LAYERED_ARCHITECTURES, LayerSpec
 
 VISION_FIELDS = ("vision", "image_token_id", "video_token_id", "mrope_section", "mrope_interleaved")
 
@@ -91,6 +92,9 @@ class ModelConfig:
     index_head_dim: int | None = None
     index_topk_freq: int = 1  # a layer computes its own top-k when max(layer - offset, 0) % freq == 0, else reuses
     index_skip_topk_offset: int = 0
+    # designs whose layers differ (models/layer_spec.py): one spec per layer; the size fields above then hold maxima
+    layer_specs: list | None = None
+    norm_kind: str = "rms"  # rms | layer (weight only; models with layer_specs)
     # multi-token prediction (draft head)
     mtp_num_layers: int | None = None
     model_arch: str = "qwen2"
@@ -102,6 +106,10 @@ class ModelConfig:
             self.kv_channels = self.hidden_size // self.num_attention_heads
         if self.padded_vocab_size is None:
             self.padded_vocab_size = self.vocab_size
+        if self.layer_specs is not None:
+            self.layer_specs = [LayerSpec.of(x) for x in self.layer_specs]
+        elif self.norm_kind != "rms":
+            raise ValueError(f"norm_kind {self.norm_kind!r} is available to models with layer_specs only")
 
     @property
     def head_dim(self) -> int:
@@ -110,6 +118,9 @@ class ModelConfig:
     def is_moe_layer(self, layer: int) -> bool:
         if self.num_experts is None:
             return False
+        if self.layer_specs is not None:
+            mlp = self.layer_specs[layer].mlp
+            return mlp is not None and mlp.experts is not None
         f = self.moe_layer_freq
         if f is None:
             return True
@@ -119,7 +130,9 @@ class ModelConfig:
 
     def mixer(self, layer: int) -> str:
         """Token mixer of a layer: ``attention`` (the fused kernel path), ``general_attention`` (attention variants
-        composed from separate ops), ``gated_delta_net``, ``mla`` or ``dsa``."""
+        composed from separate ops), ``gated_delta_net``, ``mla``, ``dsa``, or ``window_attention`` (specified layers)."""
+        if self.layer_specs is not None:
+            return "window_attention"
         if self.full_attention_interval and (layer + 1) % self.full_attention_interval != 0:
             return "gated_delta_net"
         if self.multi_latent_attention:
@@ -132,6 +145,9 @@ class ModelConfig:
     def mixer_params(self, layer: int) -> int:
         h, d = self.hidden_size, self.head_dim
         kind = self.mixer(layer)
+        if kind == "window_attention":
+            a = self.layer_specs[layer].mixer
+            return h * (a.heads * (a.dim + a.vdim) + a.kv_heads * (a.dim + a.vdim))
         if kind == "gated_delta_net":
             kd, vd = self.linear_num_key_heads * self.linear_key_head_dim, self.linear_num_value_heads * self.linear_value_head_dim
             return (h * (2 * kd + 2 * vd) + h * 2 * self.linear_num_value_heads + (2 * kd + vd) * self.linear_conv_kernel_dim
@@ -153,6 +169,10 @@ class ModelConfig:
         h = self.hidden_size
         total = 0
         for i in range(self.num_layers):
+            if self.layer_specs is not None:
+                mlp = self.layer_specs[i].mlp
+                total += self.mixer_params(i) + (2 * h if mlp is None else 4 * h + mlp.params(h))
+                continue
             total += self.mixer_params(i) + 2 * h
             if self.is_moe_layer(i):
                 total += self.num_experts * 3 * h * self.moe_ffn_hidden_size + self.num_experts * h
@@ -191,6 +211,8 @@ class ModelConfig:
                 src = cls.from_hf(hf)
             except (KeyError, ValueError, OSError):
                 src = None
+            if src is not None and src.layer_specs is not None:
+                return src  # layers described one by one: nothing for size flags to say
             if src is not None and src.vision is not None:
                 kw.update({f: getattr(src, f) for f in VISION_FIELDS})
         return cls(**kw)
@@ -204,6 +226,8 @@ class ModelConfig:
         else:
             with open(os.path.join(path_or_dict, "config.json")) as f:
                 c = json.load(f)
+        if c.get("architecture") in LAYERED_ARCHITECTURES:
+            return cls(**LAYERED_ARCHITECTURES[c["architecture"]][0](c))
         top = c
         c = c.get("text_config", c)
         arch = (c.get("architectures") or top.get("architectures") or [c.get("model_type", "qwen2")])[0]
@@ -302,6 +326,8 @@ class ModelConfig:
         return cls(**kw)
 
     def to_hf_dict(self) -> dict:
+        if self.layer_specs is not None:
+            return LAYERED_ARCHITECTURES[self.model_arch][1](self)
         moe = self.num_experts is not None
         arch = self.model_arch if self.model_arch.endswith("ForCausalLM") else {
             "qwen2": "Qwen2ForCausalLM", "qwen3": "Qwen3ForCausalLM", "qwen3_moe": "Qwen3MoeForCausalLM",

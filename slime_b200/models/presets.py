@@ -150,6 +150,26 @@ MORE_PRESETS["qwen3-vl-8b"] = dict(
                 spatial_merge_size=2, out_hidden_size=4096, num_position_embeddings=2304, hidden_act="gelu_pytorch_tanh",
                 deepstack_visual_indexes=[8, 16, 24]))  # fmt: skip
 
+
+
+def _pefolix(layers: int, hidden: int, heads: int, kv_heads: int, dim: int, window: int, keep: int, ff: int, vocab: int, *, every: int = 0,
+             experts: int = 0, top: int = 0, expert_ff: int = 0, shared_ff: int = 0) -> dict:  # fmt: skip
+    """A Pefolix stack of equal attention layers; with ``every`` > 0 each ``every``-th layer is a mixture of experts."""
+    from slime_b200.models.layer_spec import AttentionSpec, FeedForwardSpec, LayerSpec, flat_sizes
+
+    mixer = AttentionSpec(heads, kv_heads, dim, dim, dim**-0.5, window, keep, "geometric")
+    dense = FeedForwardSpec(ff, "gelu_tanh")
+    moe = FeedForwardSpec(expert_ff, "relu2", False, experts, top, shared_ff=shared_ff, shared_gate=shared_ff > 0) if every else None
+    specs = [LayerSpec(mixer, moe if every and i % every == every - 1 else dense) for i in range(layers)]
+    return dict(flat_sizes(specs), layer_specs=specs, hidden_size=hidden, vocab_size=vocab, norm_epsilon=1e-5, norm_kind="layer",
+                post_self_attn_layernorm=True, post_mlp_layernorm=True, tie_word_embeddings=False, model_arch="Pefolix")  # fmt: skip
+
+
+# Pefolix at the sizes of the dense / MoE presets above (random weights: there is no published checkpoint)
+MORE_PRESETS["pefolix-4b"] = _pefolix(36, 2560, 32, 8, 128, 1024, 8, 9728, 151936)
+MORE_PRESETS["pefolix-a3b"] = _pefolix(24, 2048, 32, 4, 128, 1024, 8, 6144, 151936, every=2, experts=128, top=8, expert_ff=768, shared_ff=768)
+MORE_PRESETS["pefolix-tiny"] = _pefolix(3, 96, 4, 2, 32, 24, 3, 160, 512, every=3, experts=6, top=2, expert_ff=48, shared_ff=40)
+
 # name -> what is missing. The numbers of these families are in the recipes they come from; they are not repeated here
 # because a preset that cannot be instantiated correctly is worse than none.
 UNSUPPORTED: dict[str, str] = {}
@@ -173,6 +193,10 @@ def to_flags(cfg) -> list[str]:
                       "index_topk_freq", "index_skip_topk_offset", "rotary_scaling_type", "rotary_original_max_position",
                       "yarn_beta_fast", "yarn_beta_slow", "mscale", "mscale_all_dim", "rope_low_freq_factor", "rope_high_freq_factor", "index_rotary_interleaved") and v == base[f.name]:  # fmt: skip
             continue
+        if f.name == "norm_kind" or (f.name == "v_head_dim" and cfg.layer_specs is not None):
+            continue
+        if f.name == "layer_specs":
+            continue  # no flags: the layers are described by --hf-checkpoint (a preset or a config.json)
         if f.name in VISION_FIELDS:
             continue  # no flags: the trainer reads the image encoder's description from --hf-checkpoint
         flag = "--" + f.name.replace("_", "-")

@@ -116,6 +116,9 @@ def gemm(a, b, *, a_mn=False, b_mn=False, bias=None, out=None, out_dtype=None, a
         else:
             out.copy_(res.to(out.dtype))
         return out
+    if a.dtype == torch.float32 or (not a_mn and not b_mn and not accumulate and (a.shape[1] % 8)):
+        assert not (a_mn or b_mn or accumulate), "the CUDA-core GEMM takes row-major operands and overwrites its output"
+        return gemm_simt(a, b, bias=bias, out=out, out_dtype=out_dtype)
     assert a.dtype == torch.bfloat16 and b.dtype == torch.bfloat16, "sm_100a GEMM takes bf16 operands"
     assert out_dtype in (torch.bfloat16, torch.float32)
     if a.stride(-1) != 1:
@@ -143,6 +146,28 @@ def gemm(a, b, *, a_mn=False, b_mn=False, bias=None, out=None, out_dtype=None, a
         int(accumulate), bn, int(splitk), P(_lib.status_word(a.device)), _lib.sm_count(a.device), _lib.stream(),
     )  # fmt: skip
     _lib.check(rc, "sb_gemm_bf16")
+    return out
+
+
+def gemm_simt(a, b, bias=None, out=None, out_dtype=None, tile_boff=None, n=None):
+    """``a @ b^T`` on the CUDA cores: fp32 operands without any rounding (the engine's full-precision mode), or bf16 rows
+    whose length is no multiple of 8. ``tile_boff`` / ``n``: grouped form (first row of ``b`` per 128 rows of ``a``, rows per group)."""
+    M, K = a.shape
+    N = n if n is not None else b.shape[0]
+    assert a.dtype == b.dtype and b.shape[1] == K
+    a = a if a.stride(-1) == 1 else a.contiguous()
+    b = b if b.stride(-1) == 1 else b.contiguous()
+    if out is None:
+        out = torch.empty(M, N, dtype=out_dtype or a.dtype, device=a.device)
+    assert out.stride(-1) == 1
+    f32 = int(a.dtype == torch.float32)
+    rows = 65535 * 64  # row tiles of one launch
+    for m in range(0, M, rows):
+        part = a[m : m + rows]
+        rc = _lib.lib().sb_gemm_simt(P(part), P(b), P(out[m:]), P(bias), P(tile_boff[m // 128 :]) if tile_boff is not None else None,
+                                     part.shape[0], N, K, a.stride(0), b.stride(0), out.stride(0), f32,
+                                     int(out.dtype == torch.float32), _lib.stream())  # fmt: skip
+        _lib.check(rc, "sb_gemm_simt")
     return out
 
 
@@ -713,6 +738,8 @@ def router_gemm(x, w):
     """fp32 router logits ``x @ w^T`` with a batch-invariant reduction order (tokens in chunks of 16)."""
     if not _cuda(x):
         return x.float() @ w.float().t()
+    if x.dtype == torch.float32 or x.shape[1] % 8:
+        return gemm_simt(x, w, out_dtype=torch.float32)
     x = x.contiguous()
     T, K = x.shape
     E = w.shape[0]

@@ -34,13 +34,20 @@ _SIGS = {
     "sb_dp_reduce_shard": [P, I, I, I, L, L, P, P, P, P, P],
     "sb_dp_adam_bcast": [P, P, P, P, P, I, I, I, L, L, F, F, F, F, F, F, F, F, F, P, I, P],
     "sb_group_fp8_quant_1x128": [P, P, P, P, I, I, L, L, I, P],
-    "sb_moe_topk": [P, P, P, P, L, I, I, I, I, F, P],
+    "sb_moe_topk": [P, P, P, P, L, I, L, I, I, I, F, P],
+    "sb_moe_layout": [P, P, P, I, I, I, I, P],
+    "sb_stream_norm": [P, I, P, I, P, P, I, P, P, I, P, P, I, P, P, I, I, I, F, I, P],
+    "sb_glu": [P, P, L, I, I, I, I, P],
+    "sb_kv_scatter": [P, P, P, P, P, I, I, L, L, P],
+    "sb_gemm_simt": [P, P, P, P, P, I, I, I, L, L, L, I, I, P],
+    "sb_window_attn": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, L, L, F, I, I, I, P],
+    "sb_flash_window": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, L, L, F, I, I, P, P],
+    "sb_paged_decode_window": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, I, I, P, P],
     "sb_moe_scatter_rows": [P, P, P, L, I, I, P],
     "sb_moe_gather_sum": [P, P, P, P, L, I, I, I, P],
     "sb_moe_route_weight_grad": [P, P, P, P, L, I, I, P],
     "sb_gemm_fp8_block": [P, P, P, P, P, I, I, I, I, I, I, I, P, I, P],
     "sb_gemm_fp8_grouped": [P, P, P, P, P, P, I, I, I, I, I, I, I, I, P, I, P],
-    
     "sb_gemm_bf16_grouped": [P, P, P, P, I, I, I, I, I, I, I, I, I, I, P, I, P],
     "sb_gemm_bf16_splitk": [P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, P, I, P],
     "sb_rmsnorm_fwd": [P, P, P, P, P, P, I, I, F, P],
@@ -76,6 +83,14 @@ _SIGS = {
 
 class KernelLibraryMissing(RuntimeError):
     pass
+
+
+def use_library(path: str) -> None:
+    """Load ``path`` instead of the whole kernel library (``ops.build.ensure``); before the first kernel call."""
+    global _SO
+    if _lib is not None and path != _SO:
+        raise RuntimeError(f"the kernel library {_SO} is already loaded")
+    _SO = path
 
 
 def available() -> bool:

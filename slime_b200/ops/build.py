@@ -50,14 +50,51 @@ def sources() -> list[str]:
     return sorted(os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith(".cu"))
 
 
-def build(force: bool = False, verbose: bool = False) -> str:
-    srcs = sources()
-    headers = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cuh", ".h"))]
-    stamp = os.path.join(OBJ_DIR, "stamp.txt")
-    digest = _digest(srcs + headers)
-    if not force and os.path.exists(OUT) and os.path.exists(stamp) and open(stamp).read() == digest:
+# Parts of the library that can be built on their own (``ensure``): a process that only serves layered models has no use for
+# the training, fp8 and multi-GPU kernels, and a fresh checkout should not wait for them.
+GROUPS = {"serve": ("gemm_sm100", "gemm_simt", "stream", "window_attn", "flash_window_sm100", "decode_attn_sm100", "paged_attn", "moe",
+                    "quant", "elementwise", "sampling")}  # fmt: skip
+
+
+def _headers() -> list[str]:
+    return [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cuh", ".h"))]
+
+
+def _current(out: str, stamp: str, digest: str) -> bool:
+    if not os.path.exists(out) or not os.path.exists(stamp):
+        return False
+    with open(stamp) as f:
+        return f.read() == digest
+
+
+def ensure(group: str) -> str:
+    """Make sure the kernels of ``group`` are built and are what ``_lib`` loads: the whole library when it is there and
+    current, otherwise a library of the group's sources alone (compiled now if needed)."""
+    if _current(OUT, os.path.join(OBJ_DIR, "stamp.txt"), _digest(sources() + _headers())):
         return OUT
+    from slime_b200.ops import _lib
+
+    part = OUT.replace("_kernels.so", f"_kernels_{group}.so")
+    path = build(srcs=[os.path.join(CSRC, f + ".cu") for f in GROUPS[group]], out=part)
+    _lib.use_library(path)
+    return path
+
+
+def build(force: bool = False, verbose: bool = False, srcs: list[str] | None = None, out: str = OUT) -> str:
+    """Compile ``srcs`` (default: every source) and link them into ``out``. Processes that build at the same time take turns."""
+    import fcntl
+
     os.makedirs(OBJ_DIR, exist_ok=True)
+    with open(os.path.join(OBJ_DIR, "lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return _build(force, verbose, srcs or sources(), out)
+
+
+def _build(force: bool, verbose: bool, srcs: list[str], out: str) -> str:
+    stamp = os.path.join(OBJ_DIR, "stamp.txt" if out == OUT else os.path.basename(out) + ".stamp")
+    digest = _digest(srcs + _headers())
+    if not force and _current(out, stamp, digest):
+        return out
     nvcc = _nvcc()
 
     def compile_one(src):
@@ -75,13 +112,15 @@ def build(force: bool = False, verbose: bool = False) -> str:
 
     with concurrent.futures.ThreadPoolExecutor(max_workers=min(8, len(srcs))) as pool:
         objs = list(pool.map(compile_one, srcs))
-    link = [nvcc, "-shared", "-o", OUT, *objs, "-gencode", "arch=compute_100a,code=sm_100a"]
+    tmp = f"{out}.{os.getpid()}.tmp"  # renamed when complete: a process that has the old file loaded keeps it
+    link = [nvcc, "-shared", "-o", tmp, *objs, "-gencode", "arch=compute_100a,code=sm_100a"]
     res = subprocess.run(link, capture_output=True, text=True)
     if res.returncode != 0:
         raise RuntimeError("link failed:\n" + res.stdout + res.stderr)
+    os.replace(tmp, out)
     with open(stamp, "w") as f:
         f.write(digest)
-    return OUT
+    return out
 
 
 if __name__ == "__main__":

@@ -27,8 +27,9 @@ P = _lib.ptr
 
 
 def route_topk(logits: torch.Tensor, k: int, *, score: str = "softmax", pre_softmax: bool = False, renorm: bool = True,
-               bias: torch.Tensor | None = None, scale: float | None = None):
-    """Router logits [T, E] (fp32) -> ``(weights [T, k] fp32, indices [T, k] int64)`` in one kernel.
+               bias: torch.Tensor | None = None, scale: float | None = None, raw_index: bool = False):
+    """Router logits [T, E] (fp32) -> ``(weights [T, k] fp32, indices [T, k] int64)`` in one kernel (``raw_index``: the
+    kernel's own int32 indices on CUDA, which is what ``DeviceLayout`` reads).
 
     ``score="softmax"`` with ``renorm`` and not ``pre_softmax``: softmax over the k picked logits; with ``pre_softmax``
     or ``renorm=False``: full softmax, pick k, keep the probabilities. ``score="sigmoid"``: sigmoid scores, ``bias``
@@ -37,13 +38,14 @@ def route_topk(logits: torch.Tensor, k: int, *, score: str = "softmax", pre_soft
     T, E = logits.shape
     mode = 2 if score == "sigmoid" else (1 if (pre_softmax or not renorm) else 0)
     if logits.is_cuda and E <= 512 and k <= 32:
-        lg = logits.float().contiguous()
+        lg = logits.float()  # a column range of wider rows is fine
+        lg = lg if lg.stride(1) == 1 else lg.contiguous()
         idx = torch.empty(T, k, dtype=torch.int32, device=lg.device)
         w = torch.empty(T, k, dtype=torch.float32, device=lg.device)
         b = None if bias is None else bias.float().contiguous()
-        rc = _lib.lib().sb_moe_topk(P(lg), P(b), P(idx), P(w), T, E, k, mode, int(renorm), float(scale or 1.0), _lib.stream())
+        rc = _lib.lib().sb_moe_topk(P(lg), P(b), P(idx), P(w), T, E, lg.stride(0), k, mode, int(renorm), float(scale or 1.0), _lib.stream())
         _lib.check(rc, "sb_moe_topk")
-        return w, idx.long()
+        return w, idx if raw_index else idx.long()
     lg = logits.float()
     if mode == 2:
         scores = torch.sigmoid(lg)
@@ -63,8 +65,9 @@ def scatter_rows(x: torch.Tensor, dest: torch.Tensor, k: int, num_rows: int) -> 
     """``out[dest[s]] = x[s // k]`` for every route slot ``s`` with ``dest[s] >= 0``; other rows of ``out`` are zero."""
     _checks.index_range("scatter_rows", "dest", dest, upper=num_rows, lower=-(1 << 31))
     out = x.new_zeros(num_rows, x.shape[-1])
-    if x.is_cuda and x.dtype == torch.bfloat16 and x.shape[-1] % 8 == 0:
-        rc = _lib.lib().sb_moe_scatter_rows(P(x.contiguous()), P(dest), P(out), dest.numel(), k, x.shape[-1], _lib.stream())
+    if x.is_cuda and x.dtype in (torch.bfloat16, torch.float32):  # a copy: fp32 rows travel as twice as many bf16
+        width = x.shape[-1] * (x.element_size() // 2)
+        rc = _lib.lib().sb_moe_scatter_rows(P(x.contiguous()), P(dest), P(out), dest.numel(), k, width, _lib.stream())
         _lib.check(rc, "sb_moe_scatter_rows")
         return out
     keep = dest >= 0
@@ -187,6 +190,16 @@ class DeviceLayout:
         activations are replicated over the group and the outputs are summed over it afterwards."""
         T, k = idx.shape
         dev = idx.device
+        self.rows_padded = -(-(T * k + num_experts * (TILE - 1)) // TILE) * TILE
+        if idx.is_cuda and num_experts <= 1024:
+            self.k, self.num_experts = k, num_experts
+            tiles = self.rows_padded // TILE
+            self.slot_dest = torch.empty(T * k, dtype=torch.int32, device=dev)
+            self.tile_expert = torch.empty(tiles, dtype=torch.int32, device=dev)
+            ids = idx.to(torch.int32).contiguous()
+            rc = _lib.lib().sb_moe_layout(P(ids), P(self.slot_dest), P(self.tile_expert), T * k, num_experts, first_expert, tiles, _lib.stream())
+            _lib.check(rc, "sb_moe_layout")
+            return
         flat = idx.reshape(-1).long() - first_expert
         here = (flat >= 0) & (flat < num_experts)
         key = torch.where(here, flat, torch.full_like(flat, num_experts))  # routes served elsewhere sort to the end
@@ -203,7 +216,6 @@ class DeviceLayout:
         # the same destinations in slot order (slot s = token s // k, route s % k): what the permutation kernels index by
         self.slot_dest = torch.empty(flat.numel(), dtype=torch.int32, device=dev)
         self.slot_dest[self.order] = self.dest.to(torch.int32)
-        self.rows_padded = -(-(flat.numel() + num_experts * (TILE - 1)) // TILE) * TILE
         tiles = torch.arange(self.rows_padded // TILE, device=dev) * TILE
         self.tile_expert = torch.searchsorted(pend, tiles, right=True).clamp_(max=num_experts - 1).to(torch.int32)
         self.token = self.order // k
@@ -255,6 +267,11 @@ def grouped_gemm(a: torch.Tensor, w: torch.Tensor, lay, *, b_mn: bool = False, o
         return out.to(out_dtype)
     a = a.contiguous()
     w = w.contiguous()
+    if a.dtype == torch.float32 or (K % 8 and not b_mn):
+        assert not b_mn, "the CUDA-core grouped GEMM takes row-major weights"
+        from slime_b200.ops import gemm_simt
+
+        return gemm_simt(a, w.view(E * R, C), out_dtype=out_dtype, tile_boff=lay.tile_expert * R, n=N)
     out = torch.empty(M, N, dtype=out_dtype, device=a.device)
     if M == 0:
         return out

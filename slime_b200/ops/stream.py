@@ -1,0 +1,144 @@
+"""Ops around an fp32 residual stream (``csrc/stream.cu``): the fused step between two sub-layers of a decoder that
+normalises before and after each of them, feed-forward activations, and cache writes of any width.
+
+CUDA tensors run the kernels; CPU tensors run the definitions in this file.
+"""
+
+from __future__ import annotations
+
+import dataclasses
+
+import torch
+
+from slime_b200.ops import _checks, _lib
+
+P = _lib.ptr
+ACTS = {"silu": 0, "gelu_tanh": 1, "relu2": 2}
+
+
+@dataclasses.dataclass
+class ExpertSum:
+    """Unfinished output of a mixture-of-experts feed-forward: token t is ``sum_j weights[t, j] * rows[dest[t * k + j]]``
+    (``dest`` < 0: no row here) ``+ sigmoid(gate[t]) * shared[t]``. ``gate``: a column of the router's logits, or None."""
+
+    rows: torch.Tensor
+    dest: torch.Tensor
+    weights: torch.Tensor
+    shared: torch.Tensor | None = None
+    gate: torch.Tensor | None = None
+
+    def tokens(self) -> int:
+        return self.weights.shape[0]
+
+
+def _norm(v, w, eps, kind):
+    mean = v.mean(-1, keepdim=True) if kind == "layer" else 0.0
+    d = v - mean
+    return d * torch.rsqrt(d.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+
+
+def _combine(e: ExpertSum) -> torch.Tensor:
+    T, k = e.weights.shape
+    d = e.dest.view(T, k).long()
+    y = torch.zeros(T, e.rows.shape[-1], dtype=torch.float32, device=e.rows.device)
+    for j in range(k):
+        hit = (d[:, j] >= 0)[:, None]
+        y += torch.where(hit, e.weights[:, j : j + 1].float() * e.rows[d[:, j].clamp_min(0)].float(), torch.zeros_like(y))
+    if e.shared is not None:
+        s = e.shared.float()
+        y += s if e.gate is None else torch.sigmoid(e.gate.float())[:, None] * s
+    return y
+
+
+def stream_norm(y, res, pre_w, eps, *, kind="rms", post_w=None, ids=None):
+    """``res (+)= norm(y) * post_w`` and return ``norm(res) * pre_w``, in one launch.
+
+    ``y``: sub-layer output [T, H], an ``ExpertSum``, or an embedding table when ``ids`` [T] is given (ids outside the table give
+    zero rows: other ranks' part of a sharded vocabulary). ``res``: fp32 [T, H],
+    updated in place; None starts the stream (a new tensor is returned as second value). ``post_w`` None: no norm of the
+    sub-layer's output; ``pre_w`` None: nothing but the stream is wanted (the first value is None). ``kind``: "rms" or
+    "layer" (mean removed, no bias). Norms, sums and the stream are fp32 whatever the element types."""
+    moe = y if isinstance(y, ExpertSum) else None
+    src = moe.rows if moe is not None else y
+    T = moe.tokens() if moe is not None else (ids.numel() if ids is not None else y.shape[0])
+    H = src.shape[-1]
+    init = res is None
+    if moe is not None:
+        _checks.index_range("stream_norm", "dest", moe.dest, upper=src.shape[0], lower=-(1 << 31))
+    w_dtype = pre_w.dtype if pre_w is not None else (post_w.dtype if post_w is not None else src.dtype)
+    if not src.is_cuda:
+        if ids is not None:
+            i = ids.long()
+            v = src[i.clamp(0, src.shape[0] - 1)].float() * ((i >= 0) & (i < src.shape[0]))[:, None]
+        else:
+            v = _combine(moe) if moe is not None else src.float()
+        if post_w is not None:
+            v = _norm(v, post_w, eps, kind)
+        if init:
+            res = v.clone()
+        else:
+            res.add_(v)
+        return (None if pre_w is None else _norm(res, pre_w, eps, kind).to(w_dtype)), res
+    src = src.contiguous()
+    if init:
+        res = torch.empty(T, H, dtype=torch.float32, device=src.device)
+    assert res.dtype == torch.float32 and res.is_contiguous() and src.dtype in (torch.bfloat16, torch.float32)
+    h = torch.empty(T, H, dtype=w_dtype, device=src.device) if pre_w is not None else None
+    dest = wts = shared = gate = None
+    k = 1
+    if moe is not None:
+        k = moe.weights.shape[1]
+        dest, wts = moe.dest.contiguous(), moe.weights.contiguous()
+        assert dest.dtype == torch.int32 and wts.dtype == torch.float32
+        shared = None if moe.shared is None else moe.shared.contiguous()
+        assert shared is None or shared.dtype == src.dtype
+        gate = moe.gate if shared is not None else None
+        assert gate is None or gate.dtype == torch.float32
+    ids32 = None if ids is None else ids.to(torch.int32).contiguous()
+    rc = _lib.lib().sb_stream_norm(
+        P(src), int(src.dtype == torch.float32), P(ids32), src.shape[0], P(dest), P(wts), k, P(shared), P(gate),
+        gate.stride(0) if gate is not None else 0, P(post_w), P(res), int(init), P(pre_w), P(h), int(w_dtype == torch.float32),
+        T, H, float(eps), int(kind == "layer"), _lib.stream(),
+    )  # fmt: skip
+    _lib.check(rc, "sb_stream_norm")
+    return h, res
+
+
+def combine(e: ExpertSum) -> torch.Tensor:
+    """The sum an ``ExpertSum`` stands for, fp32 [T, H] (where a collective has to come before the norm)."""
+    return stream_norm(e, None, None, 0.0)[1]
+
+
+def feed_forward_act(x: torch.Tensor, act: str, gated: bool) -> torch.Tensor:
+    """``act(x[:, :F]) * x[:, F:]`` (gated) or ``act(x)``."""
+    F = x.shape[-1] // 2 if gated else x.shape[-1]
+    if not x.is_cuda:
+        g = x[..., :F].float()
+        if act == "silu":
+            g = g * torch.sigmoid(g)
+        elif act == "gelu_tanh":
+            g = torch.nn.functional.gelu(g, approximate="tanh")
+        else:
+            g = g.clamp_min(0).square()
+        return (g * x[..., F:].float() if gated else g).to(x.dtype)
+    x = x.contiguous()
+    out = torch.empty(x.shape[0], F, dtype=x.dtype, device=x.device)
+    rc = _lib.lib().sb_glu(P(x), P(out), x.shape[0], F, int(gated), ACTS[act], int(x.dtype == torch.float32), _lib.stream())
+    _lib.check(rc, "sb_glu")
+    return out
+
+
+def kv_scatter(k, v, slots, k_cache, v_cache):
+    """Rows ``k[t]`` [Hkv * D] and ``v[t]`` [Hkv * DV] (views with any row pitch) into cache slot ``slots[t]`` (< 0: skipped)."""
+    _checks.index_range("kv_scatter", "slots", slots, upper=k_cache.shape[0], lower=-(1 << 31))
+    if not k.is_cuda:
+        ok = slots >= 0
+        for src, dst in ((k, k_cache), (v, v_cache)):
+            dst.view(dst.shape[0], -1)[slots[ok].long()] = src[ok].to(dst.dtype)
+        return
+    assert k.stride(1) == 1 and v.stride(1) == 1 and k.dtype == k_cache.dtype and v.dtype == v_cache.dtype
+    assert k_cache.is_contiguous() and v_cache.is_contiguous()
+    es = k.element_size()
+    rc = _lib.lib().sb_kv_scatter(P(k), P(v), P(slots), P(k_cache), P(v_cache), k.shape[0], k.shape[1] * es, v.shape[1] * es,
+                                  k.stride(0) * es, v.stride(0) * es, _lib.stream())  # fmt: skip
+    _lib.check(rc, "sb_kv_scatter")

@@ -1,0 +1,169 @@
+"""Windowed attention over the paged KV cache, for prompts (``window_extend``) and single tokens (``window_decode``).
+
+A query at position i sees key j when ``j <= i`` and (``i - j < window`` or ``j < keep_first``); its score is
+``scale * q.k - slope[head] * (i - j)`` (``slopes`` None: no distance term). Keys and values are read from the cache only,
+so a prompt's later portions, portions of several requests and single tokens beside them are one launch.
+
+Dispatch on CUDA: bf16 with head widths that are multiples of 8 up to 128 run on the tensor cores
+(``csrc/flash_window_sm100.cu``, ``csrc/decode_attn_sm100.cu``), everything else, fp32 included, on the CUDA-core kernel
+``csrc/window_attn.cu``. CPU tensors run the definition below.
+"""
+
+from __future__ import annotations
+
+import dataclasses
+
+import numpy as np
+import torch
+
+from slime_b200.ops import _checks, _lib
+
+P = _lib.ptr
+NO_WINDOW = 2**31 - 1
+TILE = 128  # query rows (tokens x heads of one kv head) and keys per tile of the tensor-core kernels
+
+
+def tile_tokens(heads: int, kv_heads: int) -> int:
+    """Query tokens of one tile: the heads that share a kv head are stacked into the tile's rows."""
+    return TILE // (heads // kv_heads) if heads // kv_heads <= TILE else 0
+
+
+@dataclasses.dataclass
+class ExtendBatch:
+    """Where the packed new tokens of a pass stand: row t belongs to request ``row_req[t]`` at position ``positions[t]``;
+    request r's pages are ``block_table[r]``. ``starts`` / ``counts`` (host): first position and number of new tokens of
+    every request, from which the query tiles of a launch are cut."""
+
+    block_table: torch.Tensor  # [requests, pages] int32
+    row_req: torch.Tensor  # [T] int32
+    positions: torch.Tensor  # [T] int32
+    starts: list[int]
+    counts: list[int]
+    page_size: int
+    _tiles: dict = dataclasses.field(default_factory=dict)
+
+    @classmethod
+    def build(cls, pages: list[list[int]], starts, counts, page_size: int, device, upload=None):
+        """``upload(ndarray) -> int32 device tensor``; default: a plain copy."""
+        up = upload or (lambda a: torch.from_numpy(np.ascontiguousarray(a, dtype=np.int32)).to(device))
+        width = max(len(p) for p in pages)
+        table = np.zeros((len(pages), width), dtype=np.int32)
+        for r, p in enumerate(pages):
+            table[r, : len(p)] = p
+        req = np.repeat(np.arange(len(pages)), counts)
+        pos = np.concatenate([np.arange(s, s + n) for s, n in zip(starts, counts)])
+        return cls(up(table), up(req), up(pos), [int(s) for s in starts], [int(n) for n in counts], page_size)
+
+    def tiles(self, tokens: int) -> torch.Tensor:
+        """[n, 4] int32 (first row, tokens, first position, request) of query tiles of at most ``tokens`` tokens."""
+        if tokens not in self._tiles:
+            rows, row = [], 0
+            for r, (s, n) in enumerate(zip(self.starts, self.counts)):
+                off = np.arange(0, n, tokens)
+                rows.append(np.stack([row + off, np.minimum(tokens, n - off), s + off, np.full_like(off, r)], 1))
+                row += n
+            host = torch.from_numpy(np.concatenate(rows).astype(np.int32))
+            if self.row_req.is_cuda:
+                host = host.pin_memory()
+            self._tiles[tokens] = host.to(self.row_req.device, non_blocking=True)
+        return self._tiles[tokens]
+
+
+def _reference(q, k_cache, v_cache, table, row_req, positions, page_size, scale, window, keep_first, slopes):
+    T, Hq, _ = q.shape
+    Hkv, dv = k_cache.shape[1], v_cache.shape[2]
+    out = torch.empty(T, Hq, dv, dtype=q.dtype)
+    req = torch.arange(T) if row_req is None else row_req.long()
+    for r in req.unique().tolist():
+        rows = (req == r).nonzero().flatten()
+        pos = positions[rows].long()
+        j = torch.arange(int(pos.max()) + 1)
+        slots = table[r, j // page_size].long() * page_size + j % page_size
+        k, v = k_cache[slots].float(), v_cache[slots].float()
+        dist = pos[:, None] - j[None, :]
+        see = (dist >= 0) & ((dist < window) | (j[None, :] < keep_first))
+        qr = q[rows].float().view(len(rows), Hkv, Hq // Hkv, -1)
+        s = torch.einsum("tghd,jgd->tghj", qr, k) * scale
+        if slopes is not None:
+            s = s - slopes.view(1, Hkv, Hq // Hkv, 1) * dist[:, None, None, :].float()
+        p = s.masked_fill(~see[:, None, None, :], float("-inf")).softmax(-1)
+        out[rows] = torch.einsum("tghj,jgd->tghd", p, v).reshape(len(rows), Hq, dv).to(q.dtype)
+    return out
+
+
+def _tensor_core_shape(q, k_cache, v_cache, page_size) -> bool:
+    D, DV, G = q.shape[2], v_cache.shape[2], q.shape[1] // k_cache.shape[1]
+    return (q.dtype == torch.bfloat16 and D <= 128 and DV <= 128 and D % 8 == 0 and DV % 8 == 0 and G <= TILE and q.stride(0) % 8 == 0
+            and page_size in (16, 32, 64, 128))  # fmt: skip
+
+
+def _simt(q, k_cache, v_cache, table, row_req, positions, page_size, scale, window, keep_first, slopes, out):
+    T, Hq, D = q.shape
+    rc = _lib.lib().sb_window_attn(
+        P(q), P(k_cache), P(v_cache), P(table), P(row_req), P(positions), P(slopes), P(out), T, Hq, k_cache.shape[1], D,
+        v_cache.shape[2], page_size, table.stride(0), q.stride(0), out.stride(0), float(scale), window, keep_first,
+        int(q.dtype == torch.float32), _lib.stream(),
+    )  # fmt: skip
+    _lib.check(rc, "sb_window_attn")
+    return out
+
+
+def window_extend(q, k_cache, v_cache, batch: ExtendBatch, scale, window=None, keep_first=0, slopes=None):
+    """Attention of the packed rows ``q`` [T, Hq, D] (a strided view is fine) -> [T, Hq, DV]. The rows' own keys and values
+    must already be in the cache."""
+    w = NO_WINDOW if window is None else int(window)
+    T, Hq, D = q.shape
+    Hkv, DV = k_cache.shape[1], v_cache.shape[2]
+    _checks.index_range("window_extend", "block_table", batch.block_table, upper=k_cache.shape[0] // batch.page_size)
+    if not q.is_cuda:
+        return _reference(q, k_cache, v_cache, batch.block_table, batch.row_req, batch.positions, batch.page_size, scale, w, keep_first, slopes)
+    assert q.stride(2) == 1 and q.stride(1) == D and k_cache.is_contiguous() and v_cache.is_contiguous()
+    out = torch.empty(T, Hq, DV, dtype=q.dtype, device=q.device)
+    if _tensor_core_shape(q, k_cache, v_cache, batch.page_size):
+        tiles = batch.tiles(tile_tokens(Hq, Hkv))
+        rc = _lib.lib().sb_flash_window(
+            P(q), P(k_cache), P(v_cache), P(batch.block_table), P(tiles), P(slopes), P(out), tiles.shape[0], T, Hq, Hkv, D, DV,
+            batch.page_size, batch.block_table.stride(0), k_cache.shape[0], q.stride(0), out.stride(0), float(scale), w,
+            keep_first, P(_lib.status_word(q.device)), _lib.stream(),
+        )  # fmt: skip
+        if rc != -1:  # -1: an alignment the kernel does not take
+            _lib.check(rc, "sb_flash_window")
+            return out
+    return _simt(q, k_cache, v_cache, batch.block_table, batch.row_req, batch.positions, batch.page_size, scale, w, keep_first, slopes, out)
+
+
+def window_decode(q, k_cache, v_cache, block_table, seq_lens, positions, page_size, scale, window=None, keep_first=0, slopes=None,
+                  max_context: int | None = None):  # fmt: skip
+    """One query token per request: ``q`` [B, Hq, D] at ``positions`` = ``seq_lens - 1``, pages in ``block_table`` [B, W].
+    Static shapes, nothing read on the host (``max_context``: upper bound of the lengths, from which the number of splits
+    follows)."""
+    w = NO_WINDOW if window is None else int(window)
+    B, Hq, D = q.shape
+    Hkv, DV = k_cache.shape[1], v_cache.shape[2]
+    if _checks.enabled():
+        _checks.paged("window_decode", block_table, seq_lens, page_size, k_cache.shape[0])
+    if not q.is_cuda:
+        return _reference(q, k_cache, v_cache, block_table, None, positions, page_size, scale, w, keep_first, slopes)
+    assert q.stride(2) == 1 and q.stride(1) == D and k_cache.is_contiguous() and v_cache.is_contiguous()
+    out = torch.empty(B, Hq, DV, dtype=q.dtype, device=q.device)
+    if _tensor_core_shape(q, k_cache, v_cache, page_size) and Hq // Hkv <= 16:
+        from slime_b200 import ops
+
+        longest = min(max_context or block_table.shape[1] * page_size, block_table.shape[1] * page_size)
+        seen = min(longest, min(w, longest) + keep_first)
+        tiles = -(-seen // TILE) + 1  # a window rarely starts at a tile's edge
+        sms = _lib.sm_count(q.device)
+        splits = -(-tiles // 16) if ops.BATCH_INVARIANT else max(-(-tiles // 16), (2 * sms) // max(B * Hkv, 1))
+        splits = max(1, min(16, splits, tiles))
+        wd = 64 if max(D, DV) <= 64 else 128
+        part = torch.empty(B * Hq * splits * (wd + 2), dtype=torch.float32, device=q.device) if splits > 1 else None
+        ml = part[B * Hq * splits * wd :] if splits > 1 else None
+        rc = _lib.lib().sb_paged_decode_window(
+            P(q), P(k_cache), P(v_cache), P(block_table), P(seq_lens), P(slopes), P(out), P(part), P(ml), B, Hq, Hkv, D, DV, page_size,
+            block_table.stride(0), k_cache.shape[0], q.stride(0), out.stride(0), splits, float(scale), w, keep_first,
+            P(_lib.status_word(q.device)), _lib.stream(),
+        )  # fmt: skip
+        if rc != -1:
+            _lib.check(rc, "sb_paged_decode_window")
+            return out
+    return _simt(q, k_cache, v_cache, block_table, None, positions, page_size, scale, w, keep_first, slopes, out)

@@ -405,6 +405,11 @@ def _model_defaults_from_hf(args) -> None:
     else:
         with open(cfg_file) as f:
             cfg = json.load(f)
+    if "architecture" in cfg:  # designs described layer by layer: no per-size flags to reconcile
+        from slime_b200.models.config import ModelConfig, apply_to_args
+
+        apply_to_args(ModelConfig.from_hf(cfg), args)
+        return
     cfg = cfg.get("text_config", cfg)
     mapping = {
         "num_layers": "num_hidden_layers", "hidden_size": "hidden_size", "ffn_hidden_size": "intermediate_size",

@@ -124,8 +124,8 @@ def test_model_presets_round_trip_through_flags():
     for name in sorted(PRESETS):
         cfg = get_preset(name)
         args = parse_args(presets.to_flags(cfg) + ["--rollout-batch-size", "1", "--num-rollout", "1", "--debug-train-only"])
-        if cfg.vision:
-            args.hf_checkpoint = f"preset:{name}"  # the image encoder has no flags: it is read from the checkpoint's config
+        if cfg.vision or cfg.layer_specs:
+            args.hf_checkpoint = f"preset:{name}"  # no flags for image encoders and specified layers: read from the checkpoint's config
         back = ModelConfig.from_args(args)
         for f in dataclasses.fields(ModelConfig):
             if f.name in ("model_arch", "padded_vocab_size", "init_method_std"):
