@@ -79,6 +79,7 @@ class EngineWeights:
         self.embed = e(self.vocab_local, h)
         self.lm_head = self.embed if cfg.tie_word_embeddings else e(self.vocab_local, h)
         self.final_norm = e(h)
+        self._specified_tensors = None
         self.layers = []
         self.draft = []  # draft heads: an ordinary layer plus the two input norms, the joining projection and a final norm
         self.num_draft_layers = draft_layers
@@ -196,14 +197,39 @@ class EngineWeights:
             L.update(shared_gate_up=mat(up * fs, h, parts=(fs,)), shared_down=mat(h, fs))
         return L
 
+    def specified_tensors(self) -> dict[str, tuple[int, ...]]:
+        """Checkpoint tensors (name -> full shape) of a model with ``layer_specs``."""
+        if self._specified_tensors is None:
+            h, v = self.cfg.hidden_size, self.cfg.vocab_size
+            out = {"embed": (v, h), "head": (v, h), "final.norm": (h,)}
+            for i, s in enumerate(self.cfg.layer_specs):
+                a, m, p = s.mixer, s.mlp, f"l{i}."
+                out.update({p + "norm1": (h,), p + "norm1b": (h,), p + "mix.q": (a.heads * a.dim, h), p + "mix.k": (a.kv_heads * a.dim, h),
+                            p + "mix.v": (a.kv_heads * a.vdim, h), p + "mix.o": (h, a.heads * a.vdim)})  # fmt: skip
+                if m is None:
+                    continue
+                out.update({p + "norm2": (h,), p + "norm2b": (h,)})
+                stems = {p + "mlp": m.ff}
+                if m.experts is not None:
+                    stems = {f"{p}mlp.e{e}": m.ff for e in range(m.experts)}
+                    out[p + "mlp.router"] = (m.experts, h)
+                    if m.shared_ff:
+                        stems[p + "mlp.shared"] = m.shared_ff
+                    if m.shared_gate:
+                        out[p + "mlp.shared.sg"] = (1, h)
+                for stem, f in stems.items():
+                    out.update({stem + ".up": (f, h), stem + ".down": (h, f)})
+                    if m.gated:
+                        out[stem + ".gate"] = (f, h)
+            self._specified_tensors = out
+        return self._specified_tensors
+
     def _load_specified(self, L, sub: str, t, raw) -> bool:
-        """One tensor of a specified layer, addressed by its name behind ``l<i>.``."""
+        """One tensor of a specified layer, addressed by its name behind ``l<i>.`` (one of ``specified_tensors``)."""
         spec, h, tp = L["spec"], self.cfg.hidden_size, self.tp
         a, m = spec.mixer, spec.mlp
         norms = {"norm1": "ln1", "norm1b": "post_attn_ln", "norm2": "ln2", "norm2b": "post_mlp_ln"}
         if sub in norms:
-            if norms[sub] not in L:
-                return False
             L[norms[sub]].copy_(t)
             return True
         q, k, v = a.heads // tp * a.dim, a.kv_heads // tp * a.dim, a.kv_heads // tp * a.vdim
@@ -215,7 +241,7 @@ class EngineWeights:
             if sub == "mlp.router":
                 L["router"][: m.experts].copy_(t)
                 return True
-            if sub == "mlp.shared.sg" and m.shared_gate:
+            if sub == "mlp.shared.sg":
                 L["router"][m.experts].copy_(t.view(-1))
                 return True
             fs = m.shared_ff // tp
@@ -223,7 +249,7 @@ class EngineWeights:
                 table.update({"mlp.shared.gate": ("shared_gate_up", 0, fs, 0), "mlp.shared.up": ("shared_gate_up", fs if m.gated else 0, fs, 0),
                               "mlp.shared.down": ("shared_down", 0, h, 1)})  # fmt: skip
             em = re.match(r"^mlp\.e(\d+)\.(gate|up|down)$", sub)
-            if em is not None and int(em.group(1)) < m.experts:
+            if em is not None:
                 e, which = int(em.group(1)) - L["first_expert"], em.group(2)
                 if not 0 <= e < L["w2"].shape[0]:
                     return True  # another rank's expert
@@ -232,8 +258,6 @@ class EngineWeights:
                 else:
                     self._put(L["w13"][e], m.ff if which == "up" and m.gated else 0, m.ff, None, t, raw, scale=False)
                 return True
-        if sub not in table or (sub.endswith(".gate") and not m.gated):
-            return False
         key, r0, rows, cut = table[sub]
         self._put(L[key], r0, rows, cut, t, raw, scale=False)
         return True
@@ -269,6 +293,11 @@ class EngineWeights:
     def load_weight(self, name: str, t: torch.Tensor):
         cfg, d = self.cfg, self.cfg.head_dim
         if cfg.layer_specs is not None:
+            want = self.specified_tensors().get(name)
+            if want is None:
+                return False
+            if tuple(t.shape) != want:
+                raise ValueError(f"{name} has shape {tuple(t.shape)}, this model's is {want}")
             m = _LAYERED_RE.match(name)
             if m is not None:
                 return int(m.group(1)) < len(self.layers) and self._load_specified(
@@ -1111,13 +1140,11 @@ class ModelRunner:
         self._host_idx = 0
 
         def views(flat):
-            out, off = {}, 0
+            out, off = {"seeds": flat[: 2 * B].view(torch.int64)}, 2 * B  # 8-byte fields first: any number of slots is fine
             for f in self.HOST_FIELDS:
                 v = flat[off : off + B]
                 out[f] = v.view(torch.float32) if f in ("temperature", "top_p", "min_p") else v
                 off += B
-            out["seeds"] = flat[off : off + 2 * B].view(torch.int64)
-            off += 2 * B
             out["block_table"] = flat[off : off + B * W].view(B, W)
             return out
 

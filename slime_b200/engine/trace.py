@@ -34,6 +34,10 @@ def load_engine(model: str, dtype: str, max_tokens: int, page_size: int, max_req
     unknown = engine.update_weights([(n, reader.get(n)) for n in reader.keys() if not n.endswith("_scale_inv")])
     if unknown:
         raise ValueError(f"{model}: tensors this model has no place for: {unknown[:8]}")
+    if cfg.layer_specs is not None:
+        absent = sorted(set(engine.weights.specified_tensors()) - set(reader.keys()))
+        if absent:
+            raise ValueError(f"{model}: tensors missing from the checkpoint: {absent[:8]}")
     return engine
 
 

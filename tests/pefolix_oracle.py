@@ -104,3 +104,89 @@ def forward(config, tensors, tokens, dtype=torch.float64, layers_out=None):
         if layers_out is not None:
             layers_out.append(x.clone())
     return layer_norm(x, W("final.norm"), eps) @ W("head").t()
+
+
+# ------------------------------------------------------------------------------- models for the tests
+def attn(heads, kv_heads, dim, vdim, size, keep, scale=None):
+    return dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=scale if scale is not None else dim**-0.5,
+                mask=dict(size=size, keep_first=keep))  # fmt: skip
+
+
+def dense(ff):
+    return dict(kind="dense", ff=ff)
+
+
+def moe(ff, experts, top, shared=None):
+    d = dict(kind="moe", expert=dict(ff=ff), router=dict(experts=experts, top=top))
+    return dict(d, shared=dict(ff=shared)) if shared else d
+
+
+def model(width, vocab, layers, eps=1e-5):
+    return dict(architecture="Pefolix", width=width, vocab=vocab, norm=dict(eps=eps),
+                layers=[dict(type="attention", mixer=a, mlp=m) for a, m in layers])  # fmt: skip
+
+
+CONFIGS = {
+    # layers of different geometry, a mixer-only layer, several groupings, key and value heads of different width
+    "mixed": model(96, 203, [(attn(6, 2, 32, 24, 21, 4), dense(80)), (attn(4, 4, 16, 40, 9, 0), None),
+                             (attn(8, 1, 24, 16, 33, 2, scale=0.31), moe(40, 7, 2, shared=24)), (attn(2, 1, 64, 8, 1, 3), moe(16, 5, 1)),
+                             (attn(5, 5, 8, 72, 40, 20), dense(136))], eps=3e-4),
+    # equal layers (one cache slab), every token sees a single expert of two, the window reaches past the kept tokens
+    "equal": model(64, 128, [(attn(4, 2, 32, 32, 12, 5), moe(32, 2, 1, shared=48)), (attn(4, 2, 32, 32, 12, 5), dense(96)),
+                             (attn(4, 2, 32, 32, 12, 5), moe(32, 2, 2))]),
+    # widths that no 16-byte copy divides
+    "odd": model(90, 77, [(attn(3, 3, 10, 14, 17, 1), dense(50)), (attn(6, 3, 12, 22, 25, 6), moe(18, 6, 4, shared=30))], eps=1e-3),
+    # one head of each kind; eps large enough to matter
+    "single": model(40, 33, [(attn(1, 1, 16, 16, 5, 1), dense(24)), (attn(1, 1, 16, 48, 300, 0), moe(8, 4, 3, shared=8))], eps=0.1),
+}  # fmt: skip
+
+
+def random_tensors(config, seed=0, sharp=3.0, dtype=torch.float32):
+    """Random weights under the checkpoint's names. ``sharp`` scales queries and keys, so that single keys dominate the
+    softmax and a key too many or too few shows."""
+    g = torch.Generator().manual_seed(seed)
+    D, out = config["width"], {}
+
+    def mat(name, rows, cols, gain=1.0):
+        out[name] = torch.randn(rows, cols, generator=g) * gain * cols**-0.5
+
+    def norm(name):
+        out[name] = 1 + 0.3 * torch.randn(D, generator=g)
+
+    out["embed"] = torch.randn(config["vocab"], D, generator=g) + 0.5
+    for i, layer in enumerate(config["layers"]):
+        p, a, m = f"l{i}.", layer["mixer"], layer["mlp"]
+        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if m is not None else ()):
+            norm(p + n)
+        mat(p + "mix.q", a["heads"] * a["dim"], D, sharp)
+        mat(p + "mix.k", a["kv_heads"] * a["dim"], D, sharp)
+        mat(p + "mix.v", a["kv_heads"] * a["vdim"], D)
+        mat(p + "mix.o", D, a["heads"] * a["vdim"])
+        if m is None:
+            continue
+        if m["kind"] == "dense":
+            for n in ("gate", "up"):
+                mat(f"{p}mlp.{n}", m["ff"], D)
+            mat(p + "mlp.down", D, m["ff"])
+            continue
+        for e in [f"e{j}" for j in range(m["router"]["experts"])] + (["shared"] if m.get("shared") else []):
+            ff = m["shared"]["ff"] if e == "shared" else m["expert"]["ff"]
+            mat(f"{p}mlp.{e}.up", ff, D)
+            mat(f"{p}mlp.{e}.down", D, ff)
+        mat(p + "mlp.router", m["router"]["experts"], D, 2.0)
+        if m.get("shared"):
+            mat(p + "mlp.shared.sg", 1, D)
+    norm("final.norm")
+    mat("head", config["vocab"], D)
+    return {k: v.to(dtype) for k, v in out.items()}
+
+
+def random_tokens(config, n, seed=0):
+    return torch.randint(0, config["vocab"], (n,), generator=torch.Generator().manual_seed(seed)).tolist()
+
+
+def error(got, want):
+    """Largest root-mean-square difference of a row, mean taken off, relative to the rows' spread."""
+    d = got.double() - want.double()
+    d = d - d.mean(-1, keepdim=True)
+    return float((d.pow(2).mean(-1).sqrt() / want.double().std()).max())
