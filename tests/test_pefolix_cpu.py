@@ -323,3 +323,32 @@ def test_replay_writes_the_wanted_logits(tmp_path):
     assert not (tmp_path / "1.f32").exists() and not r.live and len(r.engine.free_slots) == 4
     with pytest.raises(ValueError, match="context length"):
         r.step({"step": 3, "entries": [{"id": "c", "tokens": a * 4, "want": []}], "end": []})
+
+
+def _rank_main(rank, port, config, tensors, tokens, want, ep):
+    import torch.distributed as dist
+
+    torch.set_num_threads(1)
+    dist.init_process_group("gloo", init_method=f"tcp://127.0.0.1:{port}", rank=rank, world_size=2)
+    args = ServerArgs(page_size=16, max_running_requests=4, context_length=128, ep_size=ep)
+    e = Engine(ModelConfig.from_hf(config), args, device="cpu", num_pages=16, tp_group=dist.group.WORLD, tp_size=2, tp_rank=rank)
+    assert not e.update_weights(tensors.items())
+    assert O.error(feed_all(e, [17, 2, 20], tokens), want) < TOL
+    dist.destroy_process_group()
+
+
+@pytest.mark.parametrize("ep", [1, 2])
+def test_two_tensor_parallel_ranks(ep):
+    import socket
+
+    config = O.model(48, 70, [(O.attn(4, 2, 16, 24, 14, 3), O.dense(40)), (O.attn(6, 2, 8, 16, 30, 0), O.moe(24, 6, 3, shared=20)),
+                              (O.attn(2, 2, 16, 16, 9, 9), O.moe(16, 4, 1))])  # fmt: skip
+    tensors, tokens = O.random_tensors(config, seed=3), O.random_tokens(config, 44, seed=3)
+    with socket.socket() as s:
+        s.bind(("127.0.0.1", 0))
+        port = s.getsockname()[1]
+    want = O.forward(config, tensors, tokens)
+    torch.multiprocessing.spawn(_rank_main, args=(port, config, tensors, tokens, want, ep), nprocs=2)
+    with pytest.raises(ValueError, match="divide"):
+        cfg = ModelConfig.from_hf(O.CONFIGS["odd"])
+        Engine(cfg, ServerArgs(), device="cpu", num_pages=4, tp_size=2)
