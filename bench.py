@@ -62,6 +62,9 @@ def parse():
     p.add_argument("--recompute", type=str, default=None, choices=["full", "none", "auto"])
     p.add_argument("--e2e-steps", type=int, default=None, help="steps of the end-to-end arm (default: --steps)")
     p.add_argument("--no-e2e", action="store_true")
+    p.add_argument("--workload", type=str, default="grpo", choices=["grpo", "serve"],
+                   help="serve: prefill / decode throughput of Pefolix beside the closest existing models (slime_b200/engine/serve_bench.py)")
+    p.add_argument("--pair", type=str, default=None, help="serve: only the model pairs whose name contains this")
     a = p.parse_args()
     for k, v in CONFIGS[a.config].items():
         if getattr(a, k, None) is None:
@@ -173,6 +176,11 @@ def main():
     a = parse()
     if a.impl == "reference":
         return reference_arm(a)
+    if a.workload == "serve":
+        assert a.gpus == 1 and a.impl == "ours", "the serve workload runs on one GPU"
+        from slime_b200.engine import serve_bench
+
+        return serve_bench.main(a.steps, a.warmup, ClockSampler(0), a.pair)
     if a.impl == "library":
         os.environ["SLIME_B200_LIBRARY_OPS"] = "1"  # read by slime_b200.ops at import: see ops.library_mode()
 

@@ -1,4 +1,4 @@
-"""Kernel micro-benchmarks: ``python -m slime_b200.ops.microbench {gemm,decode,norm} [options]``.
+"""Kernel micro-benchmarks: ``python -m slime_b200.ops.microbench {gemm,decode,norm,...} [options]``.
 
 Every number is a CUDA-event time on the launching stream after warm-up, median over ``--iters`` timed
 repetitions with an L2 flush (a 256 MiB memset) between them. One JSON object per line on stdout.
@@ -7,6 +7,7 @@ repetitions with an L2 flush (a 256 MiB memset) between them. One JSON object pe
     decode  each kernel of one rollout decode step at a given batch and context length
     norm    RMSNorm forward/backward bandwidth
     attn    flash attention forward / backward (own kernels; the flash-attn library on the same tensors for comparison)
+    window  kernels of models with specified layers, each beside the like kernel of the existing models
     fused_emul  the peer-memory kernels (DP reduce / Adam, TP all-reduce + norm) with all ranks emulated on one GPU
 
 ``--small`` shrinks the working set to a case suitable for a profiler capture (a few launches, < 1 GB).
@@ -342,6 +343,107 @@ def bench_attn(a):
     _lib.check_status("cuda")
 
 
+def _peaks() -> tuple[float, float]:
+    """(copy GB/s, bf16 TFLOP/s burst) of this pool, measured or an earlier measurement."""
+    try:
+        with open(os.path.join(os.path.dirname(__file__), "..", "..", "MEASURED_PEAKS.json")) as f:
+            d = json.load(f)
+        return d["hbm_gbs"], d["bf16_tflops"]
+    except OSError:
+        return 6650.0, 1590.0
+
+
+def _window_keys(n: int, window: int, keep: int) -> int:
+    """Visible (query, key) pairs of one fresh prompt of ``n`` tokens."""
+    return sum(min(i + 1, window) + min(keep, max(0, i + 1 - window)) for i in range(n))
+
+
+def bench_window(a):
+    from slime_b200.ops import attention, stream
+    from slime_b200.ops import window_attention as wa
+
+    gbs, tf = _peaks()
+    ps, keep, dev, bf16 = 64, 8, "cuda", torch.bfloat16
+    rnd = lambda *sh: (torch.randn(*sh, device=dev) * 0.5).to(bf16)  # noqa: E731
+
+    def pair(what, t_new, t_old, work_new, work_old, peak, **kw):
+        f_new, f_old = work_new / t_new / peak, work_old / t_old / peak
+        _emit(kind=what, us=round(t_new * 1e3, 2), like_us=round(t_old * 1e3, 2), of_peak=round(f_new, 3), like_of_peak=round(f_old, 3),
+              times_further=round(f_old / f_new, 2), **kw)  # fmt: skip
+
+    for hq, hkv, d in ((32, 8, 128), (32, 8, 64), (32, 4, 128)) if not a.small else ((32, 8, 128),):
+        slopes = torch.tensor([2.0 ** (-8 * (h + 1) / hq) for h in range(hq)], device=dev)
+        for n, nseq, window in ((1024, 8, 1024), (4096, 2, 1024), (4096, 2, 4096)) if not a.small else ((2048, 1, 1024),):
+            T = n * nseq
+            x = rnd(T, hq + 2 * hkv, d)
+            q, k, v = x[:, :hq], x[:, hq : hq + hkv], x[:, hq + hkv :]
+            pages = [list(range(i * n // ps, (i + 1) * n // ps)) for i in range(nseq)]
+            batch = wa.ExtendBatch.build(pages, [0] * nseq, [n] * nseq, ps, dev)
+            kc, vc = k.contiguous(), v.contiguous()
+            seg = attention.segments_from_cu_seqlens(torch.arange(0, T + 1, n, dtype=torch.int32, device=dev))
+            t = time_ms(lambda: wa.window_extend(q, kc, vc, batch, d**-0.5, window, keep, slopes), a.iters)
+            t2 = time_ms(lambda: attention.flash_fwd(q, k, v, seg, d**-0.5), a.iters)
+            per = 4.0 * d * hq * nseq / 1e9
+            pair("attention_prefill", t, t2, per * _window_keys(n, window, keep), per * n * (n + 1) / 2, tf, heads=f"{hq}/{hkv}x{d}",
+                 prompts=f"{nseq}x{n}", window=window)  # fmt: skip
+        for B, ctx, window in ((64, 1024, 1024), (64, 4096, 1024), (64, 4096, 4096), (4, 1024, 1024)) if not a.small else ((64, 1024, 1024),):
+            npg = ctx // ps
+            kc, vc = rnd(B * npg * ps, hkv, d), rnd(B * npg * ps, hkv, d)
+            bt = torch.randperm(B * npg, device=dev).to(torch.int32).view(B, npg)
+            sl = torch.full((B,), ctx, dtype=torch.int32, device=dev)
+            q = rnd(B, hq, d)
+            t = time_ms(lambda: wa.window_decode(q, kc, vc, bt, sl, sl - 1, ps, d**-0.5, window, keep, slopes), a.iters)
+            t2 = time_ms(lambda: ops.paged_decode_attention(q, kc, vc, bt, sl, ps, d**-0.5), a.iters)
+            per = B * hkv * d * 4 / 1e6
+            seen = min(ctx, window) + (keep if ctx > window else 0)
+            pair("attention_decode", t, t2, per * seen, per * ctx, gbs, heads=f"{hq}/{hkv}x{d}", batch=B, context=ctx, window=window)
+    for T, H in ((8192, 2560), (64, 2560), (8192, 2048), (4, 2048)) if not a.small else ((8192, 2560),):
+        y, res, w, r16 = torch.randn(T, H, device=dev), torch.randn(T, H, device=dev), rnd(H), rnd(T, H)
+        t = time_ms(lambda: stream.stream_norm(y, res, w, 1e-5, kind="layer", post_w=w), a.iters)
+        t2 = time_ms(lambda: ops.rmsnorm(y, w, 1e-6, r16), a.iters)
+        pair("stream_norm", t, t2, T * H * 14 / 1e6, T * H * 10 / 1e6, gbs, rows=T, width=H)
+        F = 8192
+        gu = rnd(T, 2 * F)
+        t = time_ms(lambda: stream.feed_forward_act(gu, "gelu_tanh", True), a.iters)
+        t2 = time_ms(lambda: ops.swiglu(gu), a.iters)
+        pair("activation", t, t2, T * F * 6 / 1e6, T * F * 6 / 1e6, gbs, rows=T, width=F)
+        kv, slots = rnd(T, 48 * 128), torch.randperm(T, device=dev).to(torch.int32)
+        kc, vc = rnd(T, 8, 128), rnd(T, 8, 128)
+        table, pos = torch.randn(T, 128, device=dev), torch.arange(T, dtype=torch.int32, device=dev)
+        t = time_ms(lambda: stream.kv_scatter(kv[:, 4096:5120], kv[:, 5120:], slots, kc, vc), a.iters)
+        t2 = time_ms(lambda: ops.rope_kv_write(kv, pos, table, slots, kc, vc, 32, 8, 128), a.iters)
+        pair("cache_write", t, t2, T * 8 * 128 * 8 / 1e6, T * (40 * 128 * 4 + 8 * 128 * 6) / 1e6, gbs, rows=T)
+    from slime_b200.ops import grouped
+
+    E, H, F, k = 128, 2048, 768, 8
+    w1, w13, w2, router = rnd(E, F, H), rnd(E, 2 * F, H), rnd(E, H, F), rnd(136, H)
+    for T in (8192, 64, 4) if not a.small else (64,):
+        x, sh, res, w = rnd(T, H), rnd(T, H), torch.randn(T, H, device=dev), rnd(H)
+        logits = ops.gemm(x, router, out_dtype=torch.float32)
+        probs, idx = grouped.route_topk(logits[:, :E], k, renorm=False, raw_index=True)
+        lay = grouped.DeviceLayout(idx, E)
+        full = rnd(lay.rows_padded, H)
+        hit = min(E, T * k) * H * 2 / 1e6
+
+        def new():
+            return grouped.grouped_gemm(stream.feed_forward_act(grouped.grouped_gemm(lay.pad(x), w1, lay), "relu2", False), w2, lay)
+
+        def old():
+            return grouped.grouped_gemm(ops.swiglu(grouped.grouped_gemm(lay.pad(x), w13, lay)), w2, lay)
+
+        t, t2 = time_ms(new, a.iters), time_ms(old, a.iters)
+        if T >= 1024:
+            pair("experts", t, t2, 4.0 * T * k * H * F / 1e9, 6.0 * T * k * H * F / 1e9, tf, tokens=T)
+        else:
+            pair("experts", t, t2, 2 * F * hit, 3 * F * hit, gbs, tokens=T)
+        t = time_ms(lambda: stream.stream_norm(stream.ExpertSum(full, lay.slot_dest, probs, sh, logits[:, E]), res, w, 1e-5, kind="layer", post_w=w), a.iters)
+        t2 = time_ms(lambda: ops.rmsnorm(grouped.gather_sum(full, lay.slot_dest, probs, k), w, 1e-6, sh), a.iters)
+        pair("experts_sum_norm", t, t2, T * H * (2 * k + 2 + 10) / 1e6, T * H * (2 * k + 10) / 1e6, gbs, tokens=T)
+        t = time_ms(lambda: grouped.DeviceLayout(idx, E), a.iters)
+        _emit(kind="layout", us=round(t * 1e3, 2), tokens=T)
+    _lib.check_status("cuda")
+
+
 def bench_fused_emul(a):
     """The peer-memory kernels with every "rank" a buffer of THIS GPU (profilers attach to one process on one GPU, and
     kernels that wait on one another must not run as separate launches on one device): the data path, instruction mix
@@ -398,7 +500,7 @@ def bench_fused_emul(a):
 
 def main(argv=None):
     p = argparse.ArgumentParser(prog="python -m slime_b200.ops.microbench")
-    p.add_argument("what", choices=["gemm", "decode", "norm", "fp8", "moe", "attn", "fused_emul"])
+    p.add_argument("what", choices=["gemm", "decode", "norm", "fp8", "moe", "attn", "window", "fused_emul"])
     p.add_argument("--iters", type=int, default=20)
     p.add_argument("--reps", type=int, default=20, help="back-to-back launches per timed repetition (decode)")
     p.add_argument("--small", action="store_true")
@@ -412,7 +514,7 @@ def main(argv=None):
     from slime_b200.ops import build
 
     build.build()
-    {"gemm": bench_gemm, "decode": bench_decode, "norm": bench_norm, "fp8": bench_fp8, "moe": bench_moe, "attn": bench_attn, "fused_emul": bench_fused_emul}[a.what](a)
+    {"gemm": bench_gemm, "decode": bench_decode, "norm": bench_norm, "fp8": bench_fp8, "moe": bench_moe, "attn": bench_attn, "window": bench_window, "fused_emul": bench_fused_emul}[a.what](a)
 
 
 if __name__ == "__main__":
