@@ -14,6 +14,11 @@
 // visits only key tiles that some row of its tile can see: the tiles that hold the kept first tokens, then 128-key tiles
 // from the page that holds the first key of the window up to the last token. Rows with nothing visible yet keep a running
 // maximum of -inf; the first tile that shows them a key corrects it like any later rise.
+//
+// The distance penalty costs the softmax nothing per element. Inside a key tile it is slope * (key0 - i) + slope * c for
+// column c: the first term is one number per row and tile, the second is one more k-step of the score product, with
+// (hi, mid, lo) of slope / scale in the row's three extra query columns and (c, c, c) in the extra key columns. The three
+// bf16 parts carry all 24 bits of the factor, c <= 127 is exact, and the extra key columns are the same for every tile.
 #include "common.cuh"
 
 namespace sb {
@@ -29,7 +34,8 @@ struct FwSmem {
   static constexpr int K_BYTES = FW_BN * 128 * KCH;
   static constexpr int V_BYTES = FW_BN * 128 * VCH;
   static constexpr int P_BYTES = FW_BM * FW_BN * 2;
-  static constexpr int TOTAL = Q_BYTES + FW_STAGES * (K_BYTES + V_BYTES) + P_BYTES + 256 + 1024;  // + barriers, alignment
+  static constexpr int X_BYTES = FW_BM * 128;  // extra columns: k-step 0 of row r = query row r's, k-step 1 = key column r's
+  static constexpr int TOTAL = Q_BYTES + FW_STAGES * (K_BYTES + V_BYTES) + P_BYTES + X_BYTES + 256 + 1024;  // + barriers, alignment
   static constexpr int TMEM_COLS = 512;  // S0 @0, S1 @128, O @256
 };
 
@@ -37,6 +43,11 @@ __device__ __forceinline__ float fw_exp2(float x) {
   float r;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
   return r;
+}
+
+// The n lowest bits (n <= 0: none, n >= 32: all).
+__device__ __forceinline__ uint32_t fw_below(int n) {
+  return n <= 0 ? 0u : (n >= 32 ? 0xffffffffu : (1u << n) - 1);
 }
 
 struct FwArgs {
@@ -62,7 +73,8 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   uint8_t* sK = sQ + S::Q_BYTES;
   uint8_t* sV = sK + FW_STAGES * S::K_BYTES;
   uint8_t* sP = sV + FW_STAGES * S::V_BYTES;
-  uint64_t* q_full = reinterpret_cast<uint64_t*>(sP + S::P_BYTES);
+  uint8_t* sX = sP + S::P_BYTES;
+  uint64_t* q_full = reinterpret_cast<uint64_t*>(sX + S::X_BYTES);
   uint64_t* k_full = q_full + 1;
   uint64_t* k_empty = k_full + FW_STAGES;
   uint64_t* v_full = k_empty + FW_STAGES;
@@ -102,6 +114,23 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   }
   pdl_wait();
   pdl_launch_dependents();
+  if (a.slopes != nullptr && warp >= 2) {
+    const int r = threadIdx.x - 64;
+    const float f = r < bq * G ? a.slopes[kvh * G + r % G] / a.scale : 0.f;
+    const __nv_bfloat16 hi = __float2bfloat16(f);
+    const float f1 = f - __bfloat162float(hi);
+    const __nv_bfloat16 mid = __float2bfloat16(f1);
+    const float f2 = f1 - __bfloat162float(mid);
+    const float c = static_cast<float>(r);
+    uint8_t* x = sX + r * 128;
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    *reinterpret_cast<uint4*>(x + ((0 ^ (r & 7)) << 4)) =
+        make_uint4(pack_bf16x2(__bfloat162float(hi), __bfloat162float(mid)), pack_bf16x2(f2, 0.f), 0, 0);
+    *reinterpret_cast<uint4*>(x + ((1 ^ (r & 7)) << 4)) = zero;
+    *reinterpret_cast<uint4*>(x + ((2 ^ (r & 7)) << 4)) = make_uint4(pack_bf16x2(c, c), pack_bf16x2(c, 0.f), 0, 0);
+    *reinterpret_cast<uint4*>(x + ((3 ^ (r & 7)) << 4)) = zero;
+    fence_proxy_async();  // plain stores -> visible to the tensor core
+  }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -158,7 +187,7 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     if (lane == 0) {
       constexpr uint32_t idesc_s = make_idesc(FW_BM, FW_BN, 1, 1, 0, 0);
       constexpr uint32_t idesc_o = make_idesc(FW_BM, DV, 1, 1, 0, 1);  // B = V read MN-major
-      const uint32_t q_addr = smem_u32(sQ), p_addr = smem_u32(sP);
+      const uint32_t q_addr = smem_u32(sQ), p_addr = smem_u32(sP), x_addr = smem_u32(sX);
       auto issue_s = [&](int j) {
         const uint32_t k_addr = smem_u32(sK + (j % FW_STAGES) * S::K_BYTES);
 #pragma unroll
@@ -167,6 +196,9 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           umma_f16(tmem_base + (j & 1) * FW_BN, make_smem_desc(q_addr + off, 16, 1024, UMMA_SWIZZLE_128B),
                    make_smem_desc(k_addr + off, 16, 1024, UMMA_SWIZZLE_128B), idesc_s, k != 0 ? 1u : 0u);
         }
+        if (a.slopes != nullptr)
+          umma_f16(tmem_base + (j & 1) * FW_BN, make_smem_desc(x_addr, 16, 1024, UMMA_SWIZZLE_128B),
+                   make_smem_desc(x_addr + 32, 16, 1024, UMMA_SWIZZLE_128B), idesc_s, 1u);
         umma_commit(&k_empty[j % FW_STAGES]);
         umma_commit(&s_full[j & 1]);
       };
@@ -220,10 +252,14 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       const int key0 = key0_of(j);
       // every row sees the whole tile: no element tests (rows past the tile's tokens never do: their scores are garbage)
       const bool masked = key0 + FW_BN - 1 > p0 || key0 < low_last || ntok < bq || row >= bq * G;
-      const int up = valid ? pos - key0 : -1;       // column c is visible iff c <= up and (c >= dn or c < kp)
-      const int dn = low - key0, kp = a.keep_first - key0;
+      // bit i of vis[w]: column 32 w + i is visible: c <= up and (c >= dn or c < kp)
+      const int up = valid ? pos - key0 : -1, dn = low - key0, kp = a.keep_first - key0;
+      uint32_t vis[FW_BN / 32];
+#pragma unroll
+      for (int w = 0; w < FW_BN / 32; ++w)
+        vis[w] = fw_below(up + 1 - 32 * w) & (~fw_below(dn - 32 * w) | fw_below(kp - 32 * w));
       const float rowb = slope2 * static_cast<float>(key0 - pos);
-      float mx = -INFINITY;
+      float mx = -INFINITY;  // of the raw products: scale > 0 and rowb is the same for the whole row
 #pragma unroll
       for (int c4 = 0; c4 < FW_BN / 32; ++c4) {
         uint32_t r[32];
@@ -231,17 +267,14 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         tmem_ld_wait();
         if (masked) {
 #pragma unroll
-          for (int i = 0; i < 32; ++i) {
-            const int c = c4 * 32 + i;
-            const float x = fmaf(__uint_as_float(r[i]), c_log2, fmaf(slope2, static_cast<float>(c), rowb));
-            if (c <= up && (c >= dn || c < kp)) mx = fmaxf(mx, x);
-          }
+          for (int i = 0; i < 32; ++i)
+            if (vis[c4] >> i & 1) mx = fmaxf(mx, __uint_as_float(r[i]));
         } else {
 #pragma unroll
-          for (int i = 0; i < 32; ++i)
-            mx = fmaxf(mx, fmaf(__uint_as_float(r[i]), c_log2, fmaf(slope2, static_cast<float>(c4 * 32 + i), rowb)));
+          for (int i = 0; i < 32; ++i) mx = fmaxf(mx, __uint_as_float(r[i]));
         }
       }
+      mx = fmaf(mx, c_log2, rowb);
       const float m_new = fmaxf(m_run, mx);
       bool raise = false;
       if (j == 0) m_run = m_new;
@@ -258,12 +291,11 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         const float off = rowb - m_sub;
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
-          const int c = c4 * 32 + i;
-          float q0 = fw_exp2(fmaf(__uint_as_float(r[i]), c_log2, fmaf(slope2, static_cast<float>(c), off)));
-          float q1 = fw_exp2(fmaf(__uint_as_float(r[i + 1]), c_log2, fmaf(slope2, static_cast<float>(c + 1), off)));
+          float q0 = fw_exp2(fmaf(__uint_as_float(r[i]), c_log2, off));
+          float q1 = fw_exp2(fmaf(__uint_as_float(r[i + 1]), c_log2, off));
           if (masked) {
-            if (!(c <= up && (c >= dn || c < kp))) q0 = 0.f;
-            if (!(c + 1 <= up && (c + 1 >= dn || c + 1 < kp))) q1 = 0.f;
+            if (!(vis[c4] >> i & 1)) q0 = 0.f;
+            if (!(vis[c4] >> (i + 1) & 1)) q1 = 0.f;
           }
           lsum += q0 + q1;
           pk[c4 * 16 + (i >> 1)] = pack_bf16x2(q0, q1);
@@ -412,6 +444,7 @@ extern "C" int sb_flash_window(const void* q, const void* k_cache, const void* v
   if (ntiles <= 0 || T <= 0) return 0;
   if (Hkv <= 0 || Hq % Hkv != 0 || window < 1 || keep_first < 0) return (int)cudaErrorInvalidValue;
   const int G = Hq / Hkv;
+  if (!(scale > 0.f)) return -1;
   if (G > sb::FW_BM || D <= 0 || DV <= 0 || D > 128 || DV > 128 || D % 8 || DV % 8) return -1;
   int shift = 0;
   while ((1 << shift) < page_size) ++shift;

@@ -179,6 +179,7 @@ moe_topk_kernel(const float* __restrict__ logits, const float* __restrict__ bias
 // a warp by match_any: no atomics, so the layout is the same on every run.
 constexpr int LAYOUT_WARPS = 32;
 constexpr int LAYOUT_TILE = 128;
+constexpr int LAYOUT_AHEAD = 8;
 __global__ void __launch_bounds__(LAYOUT_WARPS * 32)
 moe_layout_kernel(const int* __restrict__ idx, int* __restrict__ slot_dest, int* __restrict__ tile_expert, int S, int E, int first,
                   int tiles) {
@@ -193,13 +194,21 @@ moe_layout_kernel(const int* __restrict__ idx, int* __restrict__ slot_dest, int*
   const int per = ((S + LAYOUT_WARPS - 1) / LAYOUT_WARPS + 31) & ~31;
   const int s0 = warp * per, s1 = min(S, s0 + per);
   int* mine = cnt + warp * E;
-  for (int b = s0; b < s1; b += 32) {
-    const int s = b + lane;
-    int e = s < s1 ? idx[s] - first : -1;
-    if (e >= E) e = -1;
-    const unsigned peers = __match_any_sync(0xffffffffu, e);
-    if (e >= 0 && (peers & ((1u << lane) - 1)) == 0) mine[e] += __popc(peers);
-    __syncwarp();
+  // eight groups of 32 routes per round: their loads overlap
+  for (int b = s0; b < s1; b += 32 * LAYOUT_AHEAD) {
+    int es[LAYOUT_AHEAD];
+#pragma unroll
+    for (int u = 0; u < LAYOUT_AHEAD; ++u) {
+      const int s = b + u * 32 + lane;
+      es[u] = s < s1 ? idx[s] - first : -1;
+      if (es[u] >= E) es[u] = -1;
+    }
+#pragma unroll
+    for (int u = 0; u < LAYOUT_AHEAD; ++u) {
+      const unsigned peers = __match_any_sync(0xffffffffu, es[u]);
+      if (es[u] >= 0 && (peers & ((1u << lane) - 1)) == 0) mine[es[u]] += __popc(peers);
+      __syncwarp();
+    }
   }
   __syncthreads();
   for (int e = threadIdx.x; e < E; e += blockDim.x) {  // counts -> exclusive prefix over the warps; total in pend
@@ -226,18 +235,25 @@ moe_layout_kernel(const int* __restrict__ idx, int* __restrict__ slot_dest, int*
     }
   }
   __syncthreads();
-  for (int b = s0; b < s1; b += 32) {
-    const int s = b + lane;
-    int e = s < s1 ? idx[s] - first : -1;
-    if (e >= E) e = -1;
-    const unsigned peers = __match_any_sync(0xffffffffu, e);
-    const int rank = __popc(peers & ((1u << lane) - 1));
-    int base = 0;
-    if (e >= 0) base = (e > 0 ? pend[e - 1] : 0) + mine[e];
-    __syncwarp();
-    if (e >= 0 && rank == 0) mine[e] += __popc(peers);
-    __syncwarp();
-    if (s < s1) slot_dest[s] = e >= 0 ? base + rank : -1;
+  for (int b = s0; b < s1; b += 32 * LAYOUT_AHEAD) {
+    int es[LAYOUT_AHEAD];
+#pragma unroll
+    for (int u = 0; u < LAYOUT_AHEAD; ++u) {
+      const int s = b + u * 32 + lane;
+      es[u] = s < s1 ? idx[s] - first : -1;
+      if (es[u] >= E) es[u] = -1;
+    }
+#pragma unroll
+    for (int u = 0; u < LAYOUT_AHEAD; ++u) {
+      const int s = b + u * 32 + lane, e = es[u];
+      const unsigned peers = __match_any_sync(0xffffffffu, e);
+      const int rank = __popc(peers & ((1u << lane) - 1));
+      const int base = e >= 0 ? (e > 0 ? pend[e - 1] : 0) + mine[e] : 0;
+      __syncwarp();
+      if (e >= 0 && rank == 0) mine[e] += __popc(peers);
+      __syncwarp();
+      if (s < s1) slot_dest[s] = e >= 0 ? base + rank : -1;
+    }
   }
   for (int t = threadIdx.x; t < tiles; t += blockDim.x) {
     const int row = t * LAYOUT_TILE;
