@@ -61,8 +61,10 @@ __device__ __forceinline__ float fast_exp2(float x) {
 // lose slopes[head] * distance. Only tiles with a visible key are visited: those of the kept tokens, then 128-key tiles from
 // the page that holds the window's first key. Head widths dk / dv may be smaller than D (the tensor maps read zeros past
 // them) and the group of query heads smaller than G (`group`; the surplus rows of Q are zero and never written out).
+// sinks: score of an extra softmax column without a value, per head; the output is multiplied by out_scale.
 struct DecWindow {
-  const float* slopes;  // [Hq] or null
+  const float *slopes, *sinks;  // [Hq] or null
+  float out_scale;
   int window, keep_first, group, dk, dv;
 };
 struct DecFull {};
@@ -399,15 +401,19 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
   if (all_ok && merges) {
 #pragma unroll
     for (int g = 0; g < G; ++g) {
-      const float l_run = red_l[0][g] + red_l[1][g] + red_l[2][g] + red_l[3][g];
+      float l_run = red_l[0][g] + red_l[1][g] + red_l[2][g] + red_l[3][g], gain = 1.f;
       int h = kvh * G + g, width = D;
       if constexpr (WIN) {
         if (g >= win.group) break;
         h = kvh * win.group + g;
         width = win.dv;
+        if (splits == 1) {
+          if (win.sinks != nullptr) l_run += fast_exp2(fmaf(win.sinks[h], 1.4426950408889634f, -m_thr[g]));
+          gain = win.out_scale;
+        }
       }
       if (splits == 1) {
-        const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+        const float inv = l_run > 0.f ? gain / l_run : 0.f;
         if (!WIN || tid < width)
           out[static_cast<size_t>(b) * out_stride + static_cast<size_t>(h) * width + tid] = __float2bfloat16(acc[g] * inv);
       } else {
@@ -434,9 +440,10 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
 }
 
 // out[b, h, :] = sum_s o_s exp(m_s - M) / sum_s l_s exp(m_s - M) over the splits of one (request, head).
-// dv: width of an output head (= D, or less where the kernel padded it).
+// dv: width of an output head (= D, or less where the kernel padded it). sinks / out_scale: as in DecWindow.
 __global__ void decode_attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                           __nv_bfloat16* __restrict__ out, int D, int dv, int splits, int out_stride, int Hq) {
+                                           __nv_bfloat16* __restrict__ out, int D, int dv, int splits, int out_stride, int Hq,
+                                           const float* __restrict__ sinks, float out_scale) {
   pdl_wait();
   pdl_launch_dependents();
   const int bh = blockIdx.x, b = bh / Hq, h = bh % Hq;
@@ -446,7 +453,8 @@ __global__ void decode_attn_combine_kernel(const float* __restrict__ part_o, con
   float gl = 0.f;
   for (int s = 0; s < splits; ++s)
     if (ml[2 * s] != -INFINITY) gl += ml[2 * s + 1] * __expf(ml[2 * s] - gm);
-  const float inv = gl > 0.f ? 1.f / gl : 0.f;
+  if (sinks != nullptr) gl += __expf(sinks[h] - gm);
+  const float inv = gl > 0.f ? out_scale / gl : 0.f;
   for (int d = threadIdx.x; d < dv; d += blockDim.x) {
     float o = 0.f;
     for (int s = 0; s < splits; ++s)
@@ -521,7 +529,7 @@ extern "C" int sb_paged_decode_tc(const void* q, const void* k_cache, const void
     if (rc != 0) return rc;
     if (splits > 1)
       return (int)sb::launch_pdl(sb::decode_attn_combine_kernel, dim3(B * Hq), dim3(64), 0, s, part_o, part_ml, (bf16*)out, D,
-                                 D, splits, out_stride, Hq);
+                                 D, splits, out_stride, Hq, static_cast<const float*>(nullptr), 1.f);
     return (int)cudaGetLastError();
   } catch (const std::exception& e) {
     sb::set_last_error(e.what());
@@ -533,10 +541,10 @@ extern "C" int sb_paged_decode_tc(const void* q, const void* k_cache, const void
 // pitch q_stride, out [B, Hq * DV]; part_o [B, Hq, splits, W] / part_ml [B, Hq, splits, 2] with W = 64 when both widths are at
 // most 64, else 128. Returns -1 for widths above 128 or no multiple of 8, groups above 16 heads, or a misaligned pointer.
 extern "C" int sb_paged_decode_window(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
-                                      const int* seq_lens, const float* slopes, void* out, float* part_o, float* part_ml, int B,
+                                      const int* seq_lens, const float* slopes, const float* sinks, void* out, float* part_o, float* part_ml, int B,
                                       int Hq, int Hkv, int DK, int DV, int page_size, int max_pages, int num_slots, int q_stride,
-                                      int out_stride, int splits, float scale, int window, int keep_first, int* status,
-                                      cudaStream_t s) {
+                                      int out_stride, int splits, float scale, float out_scale, int window, int keep_first,
+                                      int* status, cudaStream_t s) {
   using bf16 = __nv_bfloat16;
   if (B == 0) return 0;
   if (Hkv <= 0 || Hq % Hkv != 0 || window < 1 || keep_first < 0 || splits < 1) return (int)cudaErrorInvalidValue;
@@ -551,7 +559,7 @@ extern "C" int sb_paged_decode_window(const void* q, const void* k_cache, const 
   try {
     const CUtensorMap tk = sb::make_cache_tmap(k_cache, num_slots, Hkv, DK, page_size);
     const CUtensorMap tv = sb::make_cache_tmap(v_cache, num_slots, Hkv, DV, page_size);
-    const sb::DecWindow win{slopes, window, keep_first, G, DK, DV};
+    const sb::DecWindow win{slopes, sinks, out_scale, window, keep_first, G, DK, DV};
     const dim3 grid(B, Hkv, splits);
     int rc = -1;
 #define SB_DW(WV, GV)                                                                                                       \
@@ -565,7 +573,7 @@ extern "C" int sb_paged_decode_window(const void* q, const void* k_cache, const 
     if (rc != 0) return rc;
     if (splits > 1)
       return (int)sb::launch_pdl(sb::decode_attn_combine_kernel, dim3(B * Hq), dim3(64), 0, s, part_o, part_ml, (bf16*)out, W, DV,
-                                 splits, out_stride, Hq);
+                                 splits, out_stride, Hq, sinks, out_scale);
     return (int)cudaGetLastError();
   } catch (const std::exception& e) {
     sb::set_last_error(e.what());

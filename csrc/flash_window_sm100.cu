@@ -4,6 +4,8 @@
 //
 //     row at position i sees key j   iff   j <= i  and  (i - j < window  or  j < keep_first)
 //     score = scale * q.k - slope[head] * (i - j)                                     (slopes null: no penalty)
+// sinks: score of an extra softmax column that has no value, per head (null: none); it joins the sum once, at the end. The
+// output is multiplied by out_scale.
 //
 // Two things differ in structure. Keys and values come straight from the cache pages (one TMA box per page and 64-wide
 // chunk), so a later portion of a prompt, portions of several requests and single tokens beside them are one launch without
@@ -53,11 +55,11 @@ __device__ __forceinline__ uint32_t fw_below(int n) {
 struct FwArgs {
   const int* block_table;
   const int4* tiles;
-  const float* slopes;
+  const float *slopes, *sinks;
   __nv_bfloat16* out;
   int Hkv, G, dv, page_size, page_shift, max_pages;
   long out_stride;
-  float scale;
+  float scale, out_scale;
   int window, keep_first;
   int* status;
 };
@@ -360,7 +362,8 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     }
     if (ok) {
       tc_fence_after();
-      const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      if (valid && a.sinks != nullptr) l_run += fw_exp2(fmaf(a.sinks[head], 1.4426950408889634f, -m_run));
+      const float inv = l_run > 0.f ? a.out_scale / l_run : 0.f;
       uint8_t* orow = sP + row * (DV * 2);
 #pragma unroll
       for (int c4 = 0; c4 < DV / 32; ++c4) {
@@ -438,9 +441,9 @@ static int launch_flash_window(dim3 grid, const CUtensorMap& q, const CUtensorMa
 // slopes [Hq] fp32 or null; out [T, Hq * DV] with row pitch out_stride. D, DV multiples of 8 up to 128.
 // Returns 0, a cudaError_t value, or -1 when the shape or an alignment is outside what the kernel takes.
 extern "C" int sb_flash_window(const void* q, const void* k_cache, const void* v_cache, const int* block_table, const int* tiles,
-                               const float* slopes, void* out, int ntiles, int T, int Hq, int Hkv, int D, int DV, int page_size,
-                               int max_pages, int num_slots, long q_stride, long out_stride, float scale, int window,
-                               int keep_first, int* status, cudaStream_t s) {
+                               const float* slopes, const float* sinks, void* out, int ntiles, int T, int Hq, int Hkv, int D, int DV, int page_size,
+                               int max_pages, int num_slots, long q_stride, long out_stride, float scale, float out_scale,
+                               int window, int keep_first, int* status, cudaStream_t s) {
   if (ntiles <= 0 || T <= 0) return 0;
   if (Hkv <= 0 || Hq % Hkv != 0 || window < 1 || keep_first < 0) return (int)cudaErrorInvalidValue;
   const int G = Hq / Hkv;
@@ -456,8 +459,8 @@ extern "C" int sb_flash_window(const void* q, const void* k_cache, const void* v
     const CUtensorMap tq = sb::fw_map(q, D, Hq, T, q_stride, G, sb::FW_BM / G);
     const CUtensorMap tk = sb::fw_map(k_cache, D, Hkv, num_slots, long(Hkv) * D, 1, page_size);
     const CUtensorMap tv = sb::fw_map(v_cache, DV, Hkv, num_slots, long(Hkv) * DV, 1, page_size);
-    const sb::FwArgs a{block_table, reinterpret_cast<const int4*>(tiles), slopes, (__nv_bfloat16*)out, Hkv, G, DV, page_size, shift,
-                       max_pages, out_stride, scale, window, keep_first, status};
+    const sb::FwArgs a{block_table, reinterpret_cast<const int4*>(tiles), slopes, sinks, (__nv_bfloat16*)out, Hkv, G, DV, page_size, shift,
+                       max_pages, out_stride, scale, out_scale, window, keep_first, status};
     const dim3 grid(ntiles, Hkv);
     if (D <= 64 && DV <= 64) return sb::launch_flash_window<64, 64>(grid, tq, tk, tv, a, s);
     if (D <= 64) return sb::launch_flash_window<64, 128>(grid, tq, tk, tv, a, s);

@@ -247,7 +247,8 @@ extern "C" int sb_paged_decode(const void* q, const void* k_cache, const void* v
 // ---------------------------------------------------------------- decode step state
 // Device-owned per-slot decode state (ids, pos, out_pos) lets consecutive decode steps be launched
 // without a host round trip: the sampled token becomes the next input on the device. The host owns
-// the block table, the active mask and "init" records for slots that start decoding this step.
+// the block table, the active mask and "init" records for slots that start decoding this step. prev (null: not kept): the
+// token in front of each slot's current one.
 namespace sb {
 
 __global__ void decode_prepare_kernel(int* __restrict__ ids, int* __restrict__ pos, int* __restrict__ out_pos,
@@ -255,7 +256,8 @@ __global__ void decode_prepare_kernel(int* __restrict__ ids, int* __restrict__ p
                                       const int* __restrict__ init_pos, const int* __restrict__ init_out_pos,
                                       const int* __restrict__ active, const int* __restrict__ block_table,
                                       int* __restrict__ ids_eff, int* __restrict__ pos_eff, int* __restrict__ seq_lens,
-                                      int* __restrict__ slots, int B, int page_size, int max_pages) {
+                                      int* __restrict__ slots, int* __restrict__ prev, const int* __restrict__ init_prev,
+                                      int* __restrict__ prev_eff, int B, int page_size, int max_pages) {
   pdl_wait();  // inputs come from the previous kernel in the stream
   pdl_launch_dependents();
   const int b = blockIdx.x * blockDim.x + threadIdx.x;
@@ -264,7 +266,9 @@ __global__ void decode_prepare_kernel(int* __restrict__ ids, int* __restrict__ p
     ids[b] = init_ids[b];
     pos[b] = init_pos[b];
     out_pos[b] = init_out_pos[b];
+    if (prev != nullptr) prev[b] = init_prev[b];
   }
+  if (prev != nullptr) prev_eff[b] = active[b] ? prev[b] : -1;
   if (active[b]) {
     const int p = pos[b];
     ids_eff[b] = ids[b];
@@ -280,11 +284,13 @@ __global__ void decode_prepare_kernel(int* __restrict__ ids, int* __restrict__ p
 }
 
 __global__ void decode_advance_kernel(int* __restrict__ ids, int* __restrict__ pos, int* __restrict__ out_pos,
-                                      const int* __restrict__ active, const int* __restrict__ sampled, int B) {
+                                      const int* __restrict__ active, const int* __restrict__ sampled, int* __restrict__ prev,
+                                      int B) {
   pdl_wait();  // inputs come from the previous kernel in the stream
   pdl_launch_dependents();
   const int b = blockIdx.x * blockDim.x + threadIdx.x;
   if (b >= B || !active[b]) return;
+  if (prev != nullptr) prev[b] = ids[b];
   ids[b] = sampled[b];
   pos[b] += 1;
   out_pos[b] += 1;
@@ -294,17 +300,17 @@ __global__ void decode_advance_kernel(int* __restrict__ ids, int* __restrict__ p
 
 extern "C" int sb_decode_prepare(int* ids, int* pos, int* out_pos, const int* init_mask, const int* init_ids,
                                  const int* init_pos, const int* init_out_pos, const int* active, const int* block_table,
-                                 int* ids_eff, int* pos_eff, int* seq_lens, int* slots, int B, int page_size,
-                                 int max_pages, cudaStream_t s) {
+                                 int* ids_eff, int* pos_eff, int* seq_lens, int* slots, int* prev, const int* init_prev,
+                                 int* prev_eff, int B, int page_size, int max_pages, cudaStream_t s) {
   if (B == 0) return 0;
   return (int)sb::launch_pdl(sb::decode_prepare_kernel, dim3((B + 127) / 128), dim3(128), 0, s, ids, pos, out_pos, init_mask,
-                             init_ids, init_pos, init_out_pos, active, block_table, ids_eff, pos_eff, seq_lens, slots, B,
-                             page_size, max_pages);
+                             init_ids, init_pos, init_out_pos, active, block_table, ids_eff, pos_eff, seq_lens, slots, prev,
+                             init_prev, prev_eff, B, page_size, max_pages);
 }
 
-extern "C" int sb_decode_advance(int* ids, int* pos, int* out_pos, const int* active, const int* sampled, int B,
+extern "C" int sb_decode_advance(int* ids, int* pos, int* out_pos, const int* active, const int* sampled, int* prev, int B,
                                  cudaStream_t s) {
   if (B == 0) return 0;
   return (int)sb::launch_pdl(sb::decode_advance_kernel, dim3((B + 127) / 128), dim3(128), 0, s, ids, pos, out_pos, active,
-                             sampled, B);
+                             sampled, prev, B);
 }

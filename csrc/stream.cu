@@ -1,9 +1,10 @@
 // Kernels around an fp32 residual stream, for layers that normalise before and after every sub-layer:
 //   * sb_stream_norm  one launch between two sub-layers: (mixture-of-experts combine, gated shared expert,) post-norm,
 //                     residual add in fp32, pre-norm of the next sub-layer. With `ids` it gathers embedding rows instead
-//                     and starts the stream.
+//                     and starts the stream; a second table can add a row chosen by (previous token, token).
 //   * sb_glu          activation of a feed-forward, gated or not (silu, tanh-gelu, squared relu)
 //   * sb_kv_scatter   new key / value rows into their cache slots, widths and element size free
+//   * sb_heads        per-head RMS norm and rotation of new queries and keys; keys and values into their cache slots
 // Element types are bf16 or fp32 throughout (fp32: the engine's full-precision mode); all arithmetic is fp32.
 #include "common.cuh"
 
@@ -61,13 +62,19 @@ struct StreamNorm {
   const void* pre_w;     // norm of the next sub-layer's input, or null
   void* h;               // [T, H] normed input of the next sub-layer
   int k, y_rows, gate_ld, init, layer_norm, H;  // init: the stream starts here (res is written, not added to)
-  float eps;
+  float eps, w_off;      // w_off is added to every norm weight
+  // second embedding table: row (prev * mul_prev + token * mul_cur) mod pair_rows is added to the sub-layer output, row
+  // pair_rows where there is no previous token (prev < 0)
+  const void* pair;      // same type as y, or null
+  const int *pair_ids, *prev;
+  long mul_prev, mul_cur;
+  int pair_rows;
 };
 
 // v <- norm(v) * w over the row held by the CTA (thread t holds vectors t, t + THREADS, ...).
 template <typename TW, int VEC, int MAXI, int THREADS>
-__device__ __forceinline__ void row_norm(float (&v)[MAXI][VEC], const TW* w, int H, int nvec, float eps, int layer_norm, float* scratch,
-                                         float (&o)[MAXI][VEC]) {
+__device__ __forceinline__ void row_norm(float (&v)[MAXI][VEC], const TW* w, int H, int nvec, float eps, float w_off, int layer_norm,
+                                         float* scratch, float (&o)[MAXI][VEC]) {
   float mean = 0.f;
   if (layer_norm) {
     float s = 0.f;
@@ -95,7 +102,7 @@ __device__ __forceinline__ void row_norm(float (&v)[MAXI][VEC], const TW* w, int
       float g[VEC];
       load_vec<TW, VEC>(w + static_cast<size_t>(c) * VEC, g);
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) o[j][i] = (v[j][i] - mean) * rstd * g[i];
+      for (int i = 0; i < VEC; ++i) o[j][i] = (v[j][i] - mean) * rstd * (g[i] + w_off);
     }
   }
 }
@@ -116,6 +123,16 @@ __global__ void __launch_bounds__(THREADS) stream_norm_kernel(const __grid_const
     const int id = a.ids[row];
     have = id >= 0 && id < a.y_rows;
     src = have ? id : 0;
+  }
+  const TY* pair = nullptr;
+  if (a.pair != nullptr) {
+    const int id = a.pair_ids[row], prev = a.prev[row];
+    long r = a.pair_rows;
+    if (prev >= 0) {
+      r = (prev * a.mul_prev + id * a.mul_cur) % a.pair_rows;
+      if (r < 0) r += a.pair_rows;
+    }
+    pair = reinterpret_cast<const TY*>(a.pair) + r * H;
   }
   const float gate = (shared != nullptr && a.gate != nullptr) ? 1.f / (1.f + expf(-a.gate[row * a.gate_ld])) : 1.f;
   float v[MAXI][VEC];
@@ -148,10 +165,16 @@ __global__ void __launch_bounds__(THREADS) stream_norm_kernel(const __grid_const
 #pragma unroll
         for (int i = 0; i < VEC; ++i) v[j][i] = 0.f;
       }
+      if (pair != nullptr) {
+        float e[VEC];
+        load_vec<TY, VEC>(pair + off, e);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[j][i] += e[i];
+      }
     }
   }
   if (a.post_w != nullptr)
-    row_norm<TW, VEC, MAXI, THREADS>(v, reinterpret_cast<const TW*>(a.post_w), H, nvec, a.eps, a.layer_norm, scratch, v);
+    row_norm<TW, VEC, MAXI, THREADS>(v, reinterpret_cast<const TW*>(a.post_w), H, nvec, a.eps, a.w_off, a.layer_norm, scratch, v);
 #pragma unroll
   for (int j = 0; j < MAXI; ++j) {
     const int c = threadIdx.x + j * THREADS;
@@ -168,7 +191,7 @@ __global__ void __launch_bounds__(THREADS) stream_norm_kernel(const __grid_const
   }
   if (a.pre_w != nullptr) {
     float o[MAXI][VEC];
-    row_norm<TW, VEC, MAXI, THREADS>(v, reinterpret_cast<const TW*>(a.pre_w), H, nvec, a.eps, a.layer_norm, scratch, o);
+    row_norm<TW, VEC, MAXI, THREADS>(v, reinterpret_cast<const TW*>(a.pre_w), H, nvec, a.eps, a.w_off, a.layer_norm, scratch, o);
     TW* h = reinterpret_cast<TW*>(a.h);
 #pragma unroll
     for (int j = 0; j < MAXI; ++j) {
@@ -195,9 +218,10 @@ __device__ __forceinline__ float activate(float z, int act) {
   return r * r;
 }
 
-// out[t, f] = act(in[t, f]) * in[t, F + f] (gated, in [T, 2F]) or act(in[t, f]) (in [T, F])
+// out[t, f] = act(in[t, f]) * up[t, f], or act(in[t, f]) where up is null; rows of in and up are in_pitch apart
 template <typename T, int VEC>
-__global__ void __launch_bounds__(256) glu_kernel(const T* __restrict__ in, T* __restrict__ out, long rows, int F, int gated, int act) {
+__global__ void __launch_bounds__(256)
+glu_kernel(const T* __restrict__ in, const T* __restrict__ up, T* __restrict__ out, long rows, int F, long in_pitch, long out_pitch, int act) {
   pdl_wait();
   pdl_launch_dependents();
   const int nv = F / VEC;
@@ -206,16 +230,16 @@ __global__ void __launch_bounds__(256) glu_kernel(const T* __restrict__ in, T* _
     const long t = i / nv;
     const int c = static_cast<int>(i - t * nv) * VEC;
     float g[VEC];
-    load_vec<T, VEC>(in + t * (gated ? 2 * F : F) + c, g);
+    load_vec<T, VEC>(in + t * in_pitch + c, g);
 #pragma unroll
     for (int j = 0; j < VEC; ++j) g[j] = activate(g[j], act);
-    if (gated) {
+    if (up != nullptr) {
       float u[VEC];
-      load_vec<T, VEC>(in + t * 2 * F + F + c, u);
+      load_vec<T, VEC>(up + t * in_pitch + c, u);
 #pragma unroll
       for (int j = 0; j < VEC; ++j) g[j] *= u[j];
     }
-    store_vec<T, VEC>(out + t * F + c, g);
+    store_vec<T, VEC>(out + t * out_pitch + c, g);
   }
 }
 
@@ -239,35 +263,122 @@ kv_scatter_kernel(const char* __restrict__ k, const char* __restrict__ v, const 
   }
 }
 
+// New queries, keys and values of one attention layer. One warp per (token, head): query heads first, then key heads, then value
+// heads. Query and key heads: RMS norm over D times q_norm / k_norm (null: none), then the first `dims` coordinates turned by
+// the position's angles (table [positions, dims] = cos | sin of the dims / 2 pairs; pair i is (2i, 2i + 1) when interleaved,
+// else (i, i + dims / 2)). Queries are written back in place, keys and values to cache slot slots[t] (< 0: nowhere).
+struct Heads {
+  void *q;
+  const void *k, *v;
+  const void *q_norm, *k_norm;
+  const float* table;
+  const int *positions, *slots;
+  void *k_cache, *v_cache;
+  int Hq, Hkv, D, DV, dims, interleaved;
+  long q_pitch, k_pitch, v_pitch;
+  float eps;
+};
+constexpr int HEADS_MAX_D = 512;
+
+template <typename T>
+__global__ void __launch_bounds__(128) heads_kernel(const __grid_constant__ Heads a) {
+  __shared__ float x_s[4][HEADS_MAX_D];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int lane = threadIdx.x & 31, vec = blockIdx.y * 4 + (threadIdx.x >> 5);
+  if (vec >= a.Hq + 2 * a.Hkv) return;
+  const long t = blockIdx.x;
+  const int slot = a.slots[t];
+  if (vec >= a.Hq + a.Hkv) {
+    const int h = vec - a.Hq - a.Hkv;
+    if (slot < 0) return;
+    const T* src = reinterpret_cast<const T*>(a.v) + t * a.v_pitch + static_cast<long>(h) * a.DV;
+    T* dst = reinterpret_cast<T*>(a.v_cache) + (static_cast<long>(slot) * a.Hkv + h) * a.DV;
+    for (int d = lane; d < a.DV; d += 32) dst[d] = src[d];
+    return;
+  }
+  const bool is_q = vec < a.Hq;
+  const int h = is_q ? vec : vec - a.Hq;
+  const T* src = is_q ? reinterpret_cast<const T*>(a.q) + t * a.q_pitch : reinterpret_cast<const T*>(a.k) + t * a.k_pitch;
+  src += static_cast<long>(h) * a.D;
+  const T* w = reinterpret_cast<const T*>(is_q ? a.q_norm : a.k_norm);
+  float* x = x_s[threadIdx.x >> 5];
+  float ss = 0.f;
+  for (int d = lane; d < a.D; d += 32) {
+    x[d] = to_f(src[d]);
+    ss = fmaf(x[d], x[d], ss);
+  }
+  if (w != nullptr) {
+    const float r = 1.f / sqrtf(warp_sum(ss) / a.D + a.eps);
+    for (int d = lane; d < a.D; d += 32) x[d] *= r * to_f(w[d]);
+  }
+  __syncwarp();
+  T* dst = is_q ? reinterpret_cast<T*>(a.q) + t * a.q_pitch + static_cast<long>(h) * a.D
+                : reinterpret_cast<T*>(a.k_cache) + (static_cast<long>(slot < 0 ? 0 : slot) * a.Hkv + h) * a.D;
+  if (!is_q && slot < 0) return;
+  const int half = a.dims / 2;
+  const float* cs = half > 0 ? a.table + static_cast<long>(a.positions[t]) * a.dims : nullptr;
+  for (int d = lane; d < a.D; d += 32) {
+    float y = x[d];
+    if (d < a.dims) {
+      const int i = a.interleaved ? d >> 1 : (d < half ? d : d - half);
+      const bool second = a.interleaved ? d & 1 : d >= half;
+      const float other = x[a.interleaved ? d ^ 1 : (second ? d - half : d + half)];
+      y = second ? fmaf(other, cs[half + i], y * cs[i]) : fmaf(-other, cs[half + i], y * cs[i]);
+    }
+    dst[d] = from_f<T>(y);
+  }
+}
+
 }  // namespace sb
+
+extern "C" int sb_heads(void* q, const void* k, const void* v, const void* q_norm, const void* k_norm, const float* table,
+                        const int* positions, const int* slots, void* k_cache, void* v_cache, int T, int Hq, int Hkv, int D, int DV,
+                        int dims, int interleaved, long q_pitch, long k_pitch, long v_pitch, float eps, int f32, cudaStream_t s) {
+  if (T == 0) return 0;
+  if (D <= 0 || D > sb::HEADS_MAX_D || DV <= 0 || dims < 0 || dims > D || dims % 2 || Hq <= 0 || Hkv <= 0) return (int)cudaErrorInvalidValue;
+  const sb::Heads a{q, k, v, q_norm, k_norm, table, positions, slots, k_cache, v_cache, Hq, Hkv, D, DV, dims, interleaved, q_pitch, k_pitch,
+                    v_pitch, eps};
+  const dim3 grid(T, (Hq + 2 * Hkv + 3) / 4);
+  if (f32) return (int)sb::launch_pdl(sb::heads_kernel<float>, grid, dim3(128), 0, s, a);
+  return (int)sb::launch_pdl(sb::heads_kernel<__nv_bfloat16>, grid, dim3(128), 0, s, a);
+}
 
 // Types: y_f32 / w_f32 (norm weights and h) = 1 for fp32, 0 for bf16; fp32 weights need fp32 y. H <= 8192.
 extern "C" int sb_stream_norm(const void* y, int y_f32, const int* ids, int y_rows, const int* dest, const float* wts, int k,
                               const void* shared, const float* gate, int gate_ld, const void* post_w, float* res, int init,
-                              const void* pre_w, void* h, int w_f32, int T, int H, float eps, int layer_norm, cudaStream_t s) {
+                              const void* pre_w, void* h, int w_f32, int T, int H, float eps, float w_off, int layer_norm,
+                              const void* pair, const int* pair_ids, const int* prev, long mul_prev, long mul_cur, int pair_rows,
+                              cudaStream_t s) {
   if (T == 0) return 0;
-  if (H <= 0 || H > 8192 || (w_f32 && !y_f32)) return (int)cudaErrorInvalidValue;
-  sb::StreamNorm a{y, ids, dest, wts, shared, gate, post_w, res, pre_w, h, k, y_rows, gate_ld, init, layer_norm, H, eps};
+  if (H <= 0 || H > 8192 || (w_f32 && !y_f32) || (pair != nullptr && pair_rows <= 0)) return (int)cudaErrorInvalidValue;
+  sb::StreamNorm a{y, ids, dest, wts, shared, gate, post_w, res, pre_w, h, k, y_rows, gate_ld, init, layer_norm, H, eps, w_off,
+                   pair, pair_ids, prev, mul_prev, mul_cur, pair_rows};
   bool vec = H % 8 == 0;
-  for (const void* p : {y, shared, post_w, static_cast<const void*>(res), pre_w, static_cast<const void*>(h)})
+  for (const void* p : {y, pair, shared, post_w, static_cast<const void*>(res), pre_w, static_cast<const void*>(h)})
     vec = vec && (reinterpret_cast<uintptr_t>(p) & 15) == 0;
   if (w_f32) return sb::launch_stream_norm<float, float>(a, T, vec, s);
   if (y_f32) return sb::launch_stream_norm<float, __nv_bfloat16>(a, T, vec, s);
   return sb::launch_stream_norm<__nv_bfloat16, __nv_bfloat16>(a, T, vec, s);
 }
 
-extern "C" int sb_glu(const void* in, void* out, long rows, int F, int gated, int act, int f32, cudaStream_t s) {
+extern "C" int sb_glu(const void* in, const void* up, void* out, long rows, int F, long in_pitch, long out_pitch, int act, int f32,
+                      cudaStream_t s) {
   if (rows == 0 || F == 0) return 0;
   if (act < 0 || act > 2) return (int)cudaErrorInvalidValue;
-  const bool vec = F % 8 == 0 && (reinterpret_cast<uintptr_t>(in) & 15) == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0;
+  const uintptr_t bits = reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(up) | reinterpret_cast<uintptr_t>(out);
+  const bool vec = F % 8 == 0 && (bits & 15) == 0 && in_pitch % 8 == 0 && out_pitch % 8 == 0;
   const long n = rows * (vec ? F / 8 : F);
   const long want = (n + 255) / 256;
-  const dim3 grid(static_cast<unsigned>(want < 148 * 16 ? want : 148 * 16));
+  const dim3 grid(static_cast<unsigned>(want < 148 * 16 ? want : 148 * 16)), block(256);
   using bf16 = __nv_bfloat16;
-  if (f32 && vec) return (int)sb::launch_pdl(sb::glu_kernel<float, 8>, grid, dim3(256), 0, s, (const float*)in, (float*)out, rows, F, gated, act);
-  if (f32) return (int)sb::launch_pdl(sb::glu_kernel<float, 1>, grid, dim3(256), 0, s, (const float*)in, (float*)out, rows, F, gated, act);
-  if (vec) return (int)sb::launch_pdl(sb::glu_kernel<bf16, 8>, grid, dim3(256), 0, s, (const bf16*)in, (bf16*)out, rows, F, gated, act);
-  return (int)sb::launch_pdl(sb::glu_kernel<bf16, 1>, grid, dim3(256), 0, s, (const bf16*)in, (bf16*)out, rows, F, gated, act);
+#define SB_GLU(T, V) \
+  return (int)sb::launch_pdl(sb::glu_kernel<T, V>, grid, block, 0, s, (const T*)in, (const T*)up, (T*)out, rows, F, in_pitch, out_pitch, act)
+  if (f32 && vec) SB_GLU(float, 8);
+  if (f32) SB_GLU(float, 1);
+  if (vec) SB_GLU(bf16, 8);
+  SB_GLU(bf16, 1);
+#undef SB_GLU
 }
 
 // Row widths and pitches in bytes.

@@ -4,6 +4,7 @@
 //
 // Query row t belongs to request row_req[t] (null: request t) and stands at position row_pos[t]; it sees the keys j <= pos
 // with pos - j < window or j < keep_first, and its scores are  scale * q.k - slope[head] * (pos - j).
+// sinks: score of an extra softmax column without a value, per head (null: none). The output is multiplied by out_scale.
 // Cache layout as everywhere: [num_slots, Hkv, D], slot = page * page_size + offset, pages from block_table[request].
 #include "common.cuh"
 
@@ -22,8 +23,9 @@ template <typename T>
 __global__ void __launch_bounds__(WA_WARPS * 32)
 window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                    const int* __restrict__ block_table, const int* __restrict__ row_req, const int* __restrict__ row_pos,
-                   const float* __restrict__ slopes, T* __restrict__ out, int Hq, int Hkv, int D, int DV, int page_size,
-                   int max_pages, long q_stride, long out_stride, float scale, int window, int keep_first) {
+                   const float* __restrict__ slopes, const float* __restrict__ sinks, T* __restrict__ out, int Hq, int Hkv, int D, int DV, int page_size,
+                   int max_pages, long q_stride, long out_stride, float scale, float out_scale, int window,
+                   int keep_first) {
   __shared__ float q_s[WA_WARPS][WA_MAX_D];
   pdl_wait();
   pdl_launch_dependents();
@@ -73,7 +75,8 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const
         if (lane + 32 * i < DV) acc[i] = fmaf(pj, wa_load(vr + lane + 32 * i), acc[i]);
     }
   }
-  const float inv = 1.f / l;  // a row always sees its own key: l > 0
+  if (sinks != nullptr) l += expf(sinks[h] - m);
+  const float inv = out_scale / l;  // a row always sees its own key: l > 0
 #pragma unroll
   for (int i = 0; i < WA_ACC; ++i)
     if (lane + 32 * i < DV) wa_store(out + t * out_stride + static_cast<long>(h) * DV + lane + 32 * i, acc[i] * inv);
@@ -82,9 +85,9 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const
 }  // namespace sb
 
 extern "C" int sb_window_attn(const void* q, const void* k_cache, const void* v_cache, const int* block_table, const int* row_req,
-                              const int* row_pos, const float* slopes, void* out, int T, int Hq, int Hkv, int D, int DV,
-                              int page_size, int max_pages, long q_stride, long out_stride, float scale, int window,
-                              int keep_first, int f32, cudaStream_t s) {
+                              const int* row_pos, const float* slopes, const float* sinks, void* out, int T, int Hq, int Hkv, int D, int DV,
+                              int page_size, int max_pages, long q_stride, long out_stride, float scale, float out_scale,
+                              int window, int keep_first, int f32, cudaStream_t s) {
   if (T == 0) return 0;
   if (Hkv <= 0 || Hq % Hkv != 0 || D <= 0 || DV <= 0 || D > sb::WA_MAX_D || DV > sb::WA_MAX_D || window < 1 || keep_first < 0)
     return (int)cudaErrorInvalidValue;
@@ -92,9 +95,9 @@ extern "C" int sb_window_attn(const void* q, const void* k_cache, const void* v_
   using bf16 = __nv_bfloat16;
   if (f32)
     return (int)sb::launch_pdl(sb::window_attn_kernel<float>, grid, dim3(sb::WA_WARPS * 32), 0, s, (const float*)q, (const float*)k_cache,
-                               (const float*)v_cache, block_table, row_req, row_pos, slopes, (float*)out, Hq, Hkv, D, DV, page_size,
-                               max_pages, q_stride, out_stride, scale, window, keep_first);
+                               (const float*)v_cache, block_table, row_req, row_pos, slopes, sinks, (float*)out, Hq, Hkv, D, DV, page_size,
+                               max_pages, q_stride, out_stride, scale, out_scale, window, keep_first);
   return (int)sb::launch_pdl(sb::window_attn_kernel<bf16>, grid, dim3(sb::WA_WARPS * 32), 0, s, (const bf16*)q, (const bf16*)k_cache,
-                             (const bf16*)v_cache, block_table, row_req, row_pos, slopes, (bf16*)out, Hq, Hkv, D, DV, page_size,
-                             max_pages, q_stride, out_stride, scale, window, keep_first);
+                             (const bf16*)v_cache, block_table, row_req, row_pos, slopes, sinks, (bf16*)out, Hq, Hkv, D, DV, page_size,
+                             max_pages, q_stride, out_stride, scale, out_scale, window, keep_first);
 }

@@ -69,6 +69,12 @@ class SafetensorReader:
         return t
 
 
+def tensor_shapes(path: str) -> dict[str, tuple[int, ...]]:
+    """Shapes of a checkpoint directory's tensors, from the file headers."""
+    reader = SafetensorReader(path)
+    return {k: tuple(reader._file(k).get_slice(k).get_shape()) for k in reader.keys()}
+
+
 def supports_hf_weight_loading(path: str) -> bool:
     try:
         with open(os.path.join(path, "config.json")) as f:

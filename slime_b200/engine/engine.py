@@ -30,9 +30,10 @@ import torch
 
 from slime_b200 import ops
 from slime_b200.engine.kv_cache import OutOfPages, PagedKVCache, _hash_block
-from slime_b200.engine.model_runner import KV_KINDS, EngineWeights, ModelRunner
+from slime_b200.engine.model_runner import EngineWeights, ModelRunner, cached_mixers
 from slime_b200.engine.request import ReqState, Request, SamplingParams
 from slime_b200.engine.server_args import ServerArgs
+from slime_b200.engine.state_cache import RecurrentStates
 from slime_b200.models.config import ModelConfig
 from slime_b200.ops.window_attention import ExtendBatch
 
@@ -45,6 +46,7 @@ class _PackedTokens:
     tokens (``cu_q``) and contexts (``cu_k``), and the slots of all context tokens for models that gather them."""
 
     ids: list = dataclasses.field(default_factory=list)
+    prev: list = dataclasses.field(default_factory=list)  # the token in front of each, -1 at a sequence's start
     pos: list = dataclasses.field(default_factory=list)
     slots: list = dataclasses.field(default_factory=list)
     gather: list = dataclasses.field(default_factory=list)
@@ -78,6 +80,9 @@ class Engine:
         self.max_context = self.args.context_length or min(cfg.max_position_embeddings, 32768)
         self.page_size = self.args.page_size
         self.max_running = self.args.max_running_requests
+        # recurrent mixers keep a state per live request instead of keys and values per token
+        geometry = self.weights.state_geometry()
+        self.states = RecurrentStates(geometry, self.max_running, self.dtype, self.device) if geometry else None
         if num_pages is None:
             num_pages = self._pages_from_memory()
         self.num_pages = num_pages
@@ -90,7 +95,7 @@ class Engine:
             host_pages = (self.args.hicache_size << 30) // per_page if self.args.hicache_size > 0 else int(num_pages * self.args.hicache_ratio)
             self.kv.allocator.host_tier = HostKVTier(self.kv, host_pages)
         self.runner = ModelRunner(cfg, self.weights, self.kv, self.max_running, self.max_context,
-                                  use_cuda_graph=not self.args.disable_cuda_graph, tp_group=tp_group)  # fmt: skip
+                                  use_cuda_graph=not self.args.disable_cuda_graph, tp_group=tp_group, states=self.states)  # fmt: skip
         self.runner._alloc_static()
         self.runner.record_routed = bool(self.args.enable_return_routed_experts) and cfg.num_experts is not None
         self.routed_hist: dict[int, torch.Tensor] = {}  # decode step -> [slots, moe layers * k] int32 on the host
@@ -112,16 +117,14 @@ class Engine:
             self.spec = SpeculativeDecoder(self)
 
     def _kv_geometry(self) -> list[tuple[int, int, int]]:
-        """(heads, key width, value width) of one cached token, per layer that keeps keys and values (delta-net layers keep a
-        recurrent state per decode slot instead). Latent attention caches a single vector per token (the compressed
+        """(heads, key width, value width) of one cached token, per mixer that keeps keys and values. Latent attention caches a single vector per token (the compressed
         key/value plus the shared rotary key) and no separate values."""
         c, out = self.cfg, []
         for L in self.weights.layers + self.weights.draft:
-            if L["kind"] not in KV_KINDS:
+            if L["kind"] == "specified":
+                out += [(a.kv_heads // self.weights.tp, a.dim, a.vdim) for a in cached_mixers(L)]
+            elif not cached_mixers(L):
                 continue
-            if L["kind"] == "window":
-                a = L["spec"].mixer
-                out.append((a.kv_heads // self.weights.tp, a.dim, a.vdim))
             elif L["kind"] == "mla":
                 out.append((1, c.kv_lora_rank + c.qk_pos_emb_head_dim + (c.index_head_dim if c.index_topk else 0), 0))
             else:
@@ -133,6 +136,8 @@ class Engine:
         per_page = PagedKVCache.bytes_per_page(None, None, None, self.page_size, self.dtype, geometry=self._kv_geometry())
         if self.args.max_total_tokens:
             return max(8, self.args.max_total_tokens // self.page_size)
+        if per_page == 0:  # no mixer keeps keys and values: pages only count tokens
+            return self.max_running * -(-self.max_context // self.page_size) + 1
         if self.device.type != "cuda":
             return 512
         free, total = torch.cuda.mem_get_info(self.device)
@@ -219,7 +224,8 @@ class Engine:
         still_waiting = []
         admitted = 0
         for req in self.waiting:
-            if budget <= 0 or len(self.running) + len(self.prefilling) + admitted >= self.max_running:
+            no_state = self.states is not None and not self.states.free
+            if budget <= 0 or no_state or len(self.running) + len(self.prefilling) + admitted >= self.max_running:
                 still_waiting.append(req)
                 continue
             if req.sampling.max_new_tokens == 0 and req.logprob_start_len < 0:
@@ -236,7 +242,7 @@ class Engine:
             # (a recurrent layer's state at a page boundary is not kept, so hybrid models do not reuse prefixes either)
             # (image placeholder tokens look the same for every image: such prompts neither reuse nor offer prefixes)
             want_cache = (req.logprob_start_len < 0 and not (req.return_routed_experts and self.runner.record_routed)
-                          and not self.runner.has_gdn and req.mm is None)  # fmt: skip
+                          and not self.runner.recurrent and req.mm is None)  # fmt: skip
             pages, chain = self.kv.allocator.match_prefix(ctx) if want_cache else ([], b"")
             cached = len(pages) * ps
             total_pages = -(-(len(ctx) + 1) // ps)
@@ -248,6 +254,8 @@ class Engine:
                 budget = 0
                 continue
             req.pages = pages + new_pages
+            if self.states is not None:
+                req.state_slot = self.states.take()
             req.num_cached_tokens = req.num_computed = cached
             req.committed_pages, req.chain_hash = len(pages), chain
             req.first_scheduled = req.first_scheduled or time.time()
@@ -278,6 +286,8 @@ class Engine:
         for req, n in batch:
             s, e = req.num_computed, req.num_computed + n
             p.ids += req.ctx_ids[s:e]
+            if self.cfg.bigram:
+                p.prev += req.ctx_ids[s - 1 : e - 1] if s > 0 else [-1] + req.ctx_ids[: e - 1]
             p.pos += range(s, e)
             p.slots += self._slots(req, s, e)
             p.cu_q.append(p.cu_q[-1] + n)
@@ -288,21 +298,21 @@ class Engine:
             p.max_q, p.max_k = max(p.max_q, n), max(p.max_k, e)
         return p
 
+    def _extend_batch(self, batch) -> ExtendBatch:
+        reqs = [r for r, _ in batch]
+        return ExtendBatch.build([r.pages for r in reqs], [r.num_computed for r in reqs], [n for _, n in batch], self.page_size, self.device,
+                                 self._to_dev, [r.state_slot for r in reqs] if self.runner.recurrent else None)  # fmt: skip
+
     def _extend_pass(self, batch, p: "_PackedTokens", rows, positions=None, embed_rows=None):
         """One pass of the model over packed tokens -> (logits of ``rows`` or of all rows, the pass's device inputs)."""
         t = self._to_dev
-        extend = None
+        extend = self._extend_batch(batch) if self.runner.layered or self.runner.recurrent else None
         if self.runner.layered:
-            starts = [r.num_computed for r, _ in batch]
-            extend = ExtendBatch.build([r.pages for r, _ in batch], starts, [n for _, n in batch], self.page_size, self.device, upload=t)
             positions = extend.positions
-        states = [getattr(req, "gdn_state", None) for req, _ in batch] if self.runner.has_gdn else None
         dev_in = (t(p.ids), t(p.pos) if positions is None else positions, t(p.slots), t(p.cu_q),
                   None if p.fresh or self.runner.layered else t(p.gather, torch.long), t(p.cu_k))  # fmt: skip
-        logits = self.runner.prefill(*dev_in, p.max_q, p.max_k, rows, p.fresh, gdn_states=states, embed_rows=embed_rows, extend=extend)
-        if self.runner.has_gdn:
-            for (req, _), st in zip(batch, self.runner.last_gdn_states):
-                req.gdn_state = st
+        prev = t(p.prev) if self.cfg.bigram else None
+        logits = self.runner.prefill(*dev_in, p.max_q, p.max_k, rows, p.fresh, prev=prev, embed_rows=embed_rows, extend=extend)
         return logits, dev_in
 
     def _run_prefill(self, batch) -> list[Request]:
@@ -382,6 +392,8 @@ class Engine:
                 raise RuntimeError(f"all {self.max_running} request slots are taken")
             req = Request(rid=rid, input_ids=[], sampling=SamplingParams(max_new_tokens=0), state=ReqState.RUNNING)
             req.slot = heapq.heappop(self.free_slots)
+            if self.states is not None:
+                req.state_slot = self.states.take()
             return req
 
     def close_stream(self, req: Request):
@@ -406,7 +418,7 @@ class Engine:
                 req.input_ids += toks
                 req.ctx_ids = req.input_ids
             single = all(len(toks) == 1 and req.num_computed > 0 for req, toks, _ in entries)
-            logits = self._feed_decode(entries) if single and not self.runner.has_gdn else self._feed_extend(entries)
+            logits = self._feed_decode(entries) if single else self._feed_extend(entries)
             for req, toks, _ in entries:
                 req.num_computed += len(toks)
             return logits
@@ -425,6 +437,7 @@ class Engine:
             b = req.slot
             h["active"][b], h["init_mask"][b] = 1, 1
             h["init_ids"][b], h["init_pos"][b], h["init_out_pos"][b] = toks[0], req.num_computed, 0
+            h["init_prev"][b], h["state_slot"][b] = req.ctx_ids[req.num_computed - 1], req.state_slot or 0
             h["block_table"][b, :] = 0
             h["block_table"][b, : len(req.pages)] = req.pages
         self.runner.upload_static()
@@ -500,8 +513,8 @@ class Engine:
     def export_kv(self, req: Request):
         """``(k, v)``, each ``[layers, tokens, kv heads, head dim]``: the cached keys and values of the request's computed
         tokens, copied out of the paged cache (the pages can be released afterwards)."""
-        if self.runner.has_gdn:
-            raise NotImplementedError("prefill / decode disaggregation does not carry the recurrent state of delta-net layers")
+        if self.runner.recurrent:
+            raise NotImplementedError("prefill / decode disaggregation does not carry the recurrent state of a request")
         return self.kv.export_slots(torch.tensor(self._slots(req, 0, req.num_computed), dtype=torch.long, device=self.device))
 
     def import_request(self, input_ids, first_token: int, first_logprob: float, kv, sampling: SamplingParams | dict | None = None,
@@ -512,6 +525,8 @@ class Engine:
         the reference's PD-disaggregated rollout servers (slime/ray/rollout.py:46-219, worker types prefill / decode)."""
         if self.spec is not None:
             raise NotImplementedError("a speculating engine cannot adopt a prompt: the draft head's keys are not part of the hand-over")
+        if self.runner.recurrent:
+            raise NotImplementedError("prefill / decode disaggregation does not carry the recurrent state of a request")
         sp = sampling if isinstance(sampling, SamplingParams) else SamplingParams.from_dict(sampling)
         req = Request(rid=rid or uuid.uuid4().hex, input_ids=list(input_ids), sampling=sp, **kw)
         self._req_counter = getattr(self, "_req_counter", 0) + 1
@@ -581,11 +596,9 @@ class Engine:
         self.slot_req[b] = r
         if self.runner.rope_delta is not None:
             self.runner.rope_delta[b] = r.rope_delta
-        if self.runner.has_gdn:
-            self.runner.load_gdn_state(b, r.gdn_state)
-            r.gdn_state = None
         h["active"][b], h["init_mask"][b] = 1, 1
         h["init_ids"][b], h["init_pos"][b], h["init_out_pos"][b] = r.output_ids[-1], L - 1, len(r.output_ids)
+        h["init_prev"][b], h["state_slot"][b] = (r.output_ids[-2] if len(r.output_ids) > 1 else r.input_ids[-1]), r.state_slot or 0
         h["top_k"][b], h["temperature"][b] = max(r.sampling.top_k, 0), r.sampling.temperature
         h["top_p"][b], h["min_p"][b], h["seeds"][b] = r.sampling.top_p, r.sampling.min_p, r.seed
         bt = h["block_table"][b]
@@ -783,12 +796,17 @@ class Engine:
         r.num_computed = len(r.input_ids) + len(r.output_ids) - 1
         self._commit_pages(r, None)
 
+    def _give_state(self, req: Request):
+        if req.state_slot is not None:
+            self.states.give(req.state_slot)
+            req.state_slot = None
+
     def _retract(self, req: Request):
         """Return a decoding request to the queue: tokens generated so far are kept and re-prefilled later."""
         self._harvest(req, self.processed)
         self._release_slot(req)
         req.routed_experts = []  # the re-prefill computes every position again
-        req.gdn_state = None
+        self._give_state(req)
         req.spec_draft, req.spec_hidden = [], None
         self.kv.allocator.release(req.pages)
         req.pages, req.num_computed, req.committed_pages, req.chain_hash = [], 0, 0, b""
@@ -842,6 +860,7 @@ class Engine:
         if req.pages:
             self.kv.allocator.release(req.pages)
             req.pages = []
+        self._give_state(req)
         if req.done_event is not None:
             req.done_event.set()
         if req.on_token is not None and reason.get("type") == "abort":
@@ -885,6 +904,8 @@ class Engine:
                 if tag == "kv_cache":
                     self.abort(abort_all=True)
                     self.kv.release()
+                    if self.states is not None:
+                        self.states.release()
                     if self.args.release_hicache and self.kv.allocator.host_tier is not None:
                         self.kv.allocator.host_tier.release()  # the host pool goes too; without the switch it survives
                 elif tag == "cuda_graph":
@@ -903,6 +924,8 @@ class Engine:
                     continue
                 if tag == "kv_cache":
                     self.kv.allocate()
+                    if self.states is not None:
+                        self.states.allocate()
                     if self.kv.allocator.host_tier is not None:
                         self.kv.allocator.host_tier.allocate()
                     if 0 in self.kv.allocator.free:

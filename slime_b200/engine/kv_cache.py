@@ -166,7 +166,7 @@ class PagedKVCache:
         self.geometry = [tuple(g) for g in geometry]
         self.num_layers = len(self.geometry)
         self.uniform = len(set(self.geometry)) <= 1
-        self.hkv, self.d, self.dv = self.geometry[0] if self.geometry else (num_kv_heads, head_dim, v_head_dim or head_dim)
+        self.hkv, self.d, self.dv = self.geometry[0] if self.geometry else (1, 0, 0)  # (no layer: pages only count tokens)
         self.page_size, self.num_pages, self.dtype, self.device = page_size, num_pages, dtype, device
         self.allocator = PageAllocator(num_pages, page_size, enable_prefix_cache)
         self.k: list[torch.Tensor] = []

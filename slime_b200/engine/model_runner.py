@@ -18,19 +18,30 @@ import torch
 
 from slime_b200 import ops
 from slime_b200.engine.kv_cache import PagedKVCache
+from slime_b200.engine.projections import LayerProjections
+from slime_b200.engine.state_cache import RecurrentStates
 from slime_b200.models.config import ModelConfig
-from slime_b200.models.layer_spec import LayerSpec
-from slime_b200.ops import stream
+from slime_b200.models.layer_spec import AttentionSpec, DeltaSpec
+from slime_b200.ops import delta, stream
 
 logger = logging.getLogger(__name__)
 
 _LAYER_RE = re.compile(r"^model\.layers\.(\d+)\.(.+)$")
 _LAYERED_RE = re.compile(r"^l(\d+)\.(.+)$")  # designs described layer by layer (models/layer_spec.py)
 _LAYERED_TOP = {"embed": "model.embed_tokens.weight", "head": "lm_head.weight", "final.norm": "model.norm.weight"}
+_NORMS = {"norm1": "ln1", "norm1b": "post_attn_ln", "norm2": "ln2", "norm2b": "post_mlp_ln"}  # of a specified layer
 _MIMO_DRAFT_RE = re.compile(r"^model\.mtp_layers\.(\d+)\.(.+)$")
 
 
-KV_KINDS = ("attention", "mla", "window")  # layer kinds that keep keys and values in the paged cache
+KV_KINDS = ("attention", "mla")  # layer kinds that keep keys and values in the paged cache
+
+
+def cached_mixers(L) -> list[AttentionSpec | None]:
+    """What layer ``L`` keeps keys and values for: the attention mixers of a specified layer, one unnamed entry of another
+    attention layer, nothing for a recurrent one."""
+    if L["kind"] == "specified":
+        return [m for _, m, _ in L["spec"].branches() if isinstance(m, AttentionSpec)]
+    return [None] if L["kind"] in KV_KINDS else []
 
 
 class EngineWeights:
@@ -79,13 +90,14 @@ class EngineWeights:
         self.embed = e(self.vocab_local, h)
         self.lm_head = self.embed if cfg.tie_word_embeddings else e(self.vocab_local, h)
         self.final_norm = e(h)
+        self.bigram = e(cfg.bigram["buckets"] + 1, h) if cfg.bigram else None  # replicated over tensor-parallel ranks
         self._specified_tensors = None
         self.layers = []
         self.draft = []  # draft heads: an ordinary layer plus the two input norms, the joining projection and a final norm
         self.num_draft_layers = draft_layers
         for i in range(cfg.num_layers + draft_layers):
             kind = cfg.mixer(i)
-            if kind == "window_attention":
+            if kind == "specified":
                 self.layers.append(self._specified_buffers(cfg.layer_specs[i], e, mat))
                 continue
             if kind not in ("attention", "general_attention", "gated_delta_net", "mla", "dsa"):
@@ -168,19 +180,30 @@ class EngineWeights:
         return L
 
     def _specified_buffers(self, spec, e, mat) -> dict:
-        """Buffers of a layer that has its own ``LayerSpec``: fused q | k | v rows, gate and up rows stacked, the router's rows
-        followed by the shared expert's gate (one product computes both; rows padded to a multiple of 8)."""
-        h, a, m, tp = self.cfg.hidden_size, spec.mixer, spec.mlp, self.tp
-        if a.heads % tp or a.kv_heads % tp or self.cfg.padded_vocab_size % tp:
-            raise ValueError(f"{a.heads} query / {a.kv_heads} key-value heads and a vocabulary of {self.cfg.padded_vocab_size} do not "
-                             f"divide over {tp} tensor-parallel ranks")  # fmt: skip
-        hq, hkv = a.heads // tp, a.kv_heads // tp
-        parts = (hq * a.dim, (hq + hkv) * a.dim)
-        L = {"kind": "window", "spec": spec, "ln1": e(h), "post_attn_ln": e(h), "o": mat(h, hq * a.vdim),
-             "qkv": mat((hq + hkv) * a.dim + hkv * a.vdim, h, parts=parts)}  # fmt: skip
-        if m is None:
+        """Buffers of a layer that has its own ``LayerSpec``: the fused matrices of ``LayerProjections``; for a feed-forward behind
+        the mixer gate and up rows stacked, and the router's rows followed by the shared expert's gate (one product
+        computes both; rows padded to a multiple of 8)."""
+        h, m, tp = self.cfg.hidden_size, spec.mlp, self.tp
+        if self.cfg.padded_vocab_size % tp:
+            raise ValueError(f"a vocabulary of {self.cfg.padded_vocab_size} does not divide over {tp} tensor-parallel ranks")
+        lay = LayerProjections(spec, tp)
+        attention_only = all(isinstance(x, AttentionSpec) for _, x, _ in spec.branches())
+        L = {"kind": "specified", "spec": spec, "proj": lay}
+        L.update({_NORMS[n]: e(h) for n in spec.norms(self.cfg.post_self_attn_layernorm)})
+        # block-scaled fp8 covers plain attention projections; what enters a recurrence keeps its precision
+        L["in"] = mat(lay.in_rows, h, parts=[r for r, _ in lay.ins.values() if r]) if attention_only else e(lay.in_rows, h)
+        L["out"] = mat(h, lay.out_cols) if attention_only and len(lay.outs) == 1 else e(h, lay.out_cols)
+        f32 = lambda n: torch.zeros(n, dtype=torch.float32, device=self.device)  # noqa: E731
+        for p, x, _ in spec.branches():
+            if isinstance(x, DeltaSpec):
+                L.update({p + "conv": e(x.channels // tp, x.conv), p + "A_log": f32(x.heads // tp), p + "dt_bias": f32(x.decays // tp),
+                          p + "norm": e(x.vdim)})  # fmt: skip
+                if p in lay.low:
+                    L[p + "low"] = e(lay.low[p][2], lay.low[p][1])
+            elif x.qk_norm:
+                L.update({p + "q.norm": e(x.dim), p + "k.norm": e(x.dim)})
+        if m is None or spec.parallel_ff:
             return L
-        L.update(ln2=e(h), post_mlp_ln=e(h))
         up = 2 if m.gated else 1
         if m.experts is None:
             if m.ff % tp:
@@ -202,13 +225,14 @@ class EngineWeights:
         if self._specified_tensors is None:
             h, v = self.cfg.hidden_size, self.cfg.vocab_size
             out = {"embed": (v, h), "head": (v, h), "final.norm": (h,)}
+            if self.cfg.bigram:
+                out["bigram"] = (self.cfg.bigram["buckets"] + 1, h)
             for i, s in enumerate(self.cfg.layer_specs):
-                a, m, p = s.mixer, s.mlp, f"l{i}."
-                out.update({p + "norm1": (h,), p + "norm1b": (h,), p + "mix.q": (a.heads * a.dim, h), p + "mix.k": (a.kv_heads * a.dim, h),
-                            p + "mix.v": (a.kv_heads * a.vdim, h), p + "mix.o": (h, a.heads * a.vdim)})  # fmt: skip
-                if m is None:
+                m, p = s.mlp, f"l{i}."
+                out.update({p + n: (h,) for n in s.norms(self.cfg.post_self_attn_layernorm)})
+                out.update({p + n: shape for n, shape in LayerProjections(s).tensors(h).items()})
+                if m is None or s.parallel_ff:
                     continue
-                out.update({p + "norm2": (h,), p + "norm2b": (h,)})
                 stems = {p + "mlp": m.ff}
                 if m.experts is not None:
                     stems = {f"{p}mlp.e{e}": m.ff for e in range(m.experts)}
@@ -224,20 +248,53 @@ class EngineWeights:
             self._specified_tensors = out
         return self._specified_tensors
 
+    def _load_mixer(self, L, sub: str, t, raw) -> bool:
+        """A tensor of a specified layer's mixers, or of a feed-forward beside them; False when it is neither."""
+        lay, h = L["proj"], self.cfg.hidden_size
+        if sub in lay.ins:
+            r0, rows = lay.ins[sub]
+            self._put(L["in"], r0, rows, None if sub in lay.whole else 0, t, raw, scale=False)
+            return True
+        if sub in lay.outs:
+            c0, cols = lay.outs[sub]
+            if isinstance(L["out"], torch.Tensor):
+                L["out"][:, c0 : c0 + cols].copy_(t[:, self.rank * cols : (self.rank + 1) * cols])
+            else:
+                self._put(L["out"], 0, h, 1, t, raw, scale=False)
+            return True
+        for p, (_, _, _, parts) in lay.low.items():
+            if sub in parts:
+                r0, rows, c0, cols = parts[sub]
+                L[p + "low"][r0 : r0 + rows, c0 : c0 + cols].copy_(self._rows(t, rows))
+                return True
+        for p, m, _ in L["spec"].branches():
+            if sub in (p + "q.conv", p + "k.conv", p + "v.conv"):
+                g, v = m.kv_heads // self.tp * m.dim, m.heads // self.tp * m.vdim
+                r0, rows = {"q": (0, g), "k": (g, g), "v": (2 * g, v)}[sub[len(p)]]
+                L[p + "conv"][r0 : r0 + rows].copy_(self._rows(t, rows))
+                return True
+            if sub in (p + "A_log", p + "dt_bias"):
+                L[sub].copy_(self._rows(raw, L[sub].numel()))
+                return True
+            if sub in (p + "norm", p + "q.norm", p + "k.norm"):
+                L[sub].copy_(t)
+                return True
+        return False
+
     def _load_specified(self, L, sub: str, t, raw) -> bool:
         """One tensor of a specified layer, addressed by its name behind ``l<i>.`` (one of ``specified_tensors``)."""
         spec, h, tp = L["spec"], self.cfg.hidden_size, self.tp
-        a, m = spec.mixer, spec.mlp
-        norms = {"norm1": "ln1", "norm1b": "post_attn_ln", "norm2": "ln2", "norm2b": "post_mlp_ln"}
-        if sub in norms:
-            L[norms[sub]].copy_(t)
+        m = spec.mlp
+        if sub in _NORMS:
+            L[_NORMS[sub]].copy_(t)
             return True
-        q, k, v = a.heads // tp * a.dim, a.kv_heads // tp * a.dim, a.kv_heads // tp * a.vdim
-        table = {"mix.q": ("qkv", 0, q, 0), "mix.k": ("qkv", q, k, 0), "mix.v": ("qkv", q + k, v, 0), "mix.o": ("o", 0, h, 1)}
-        if m is not None and m.experts is None:
+        if self._load_mixer(L, sub, t, raw):
+            return True
+        table = {}
+        if m.experts is None:
             f = m.ff // tp
-            table.update({"mlp.gate": ("gate_up", 0, f, 0), "mlp.up": ("gate_up", f if m.gated else 0, f, 0), "mlp.down": ("down", 0, h, 1)})
-        if m is not None and m.experts is not None:
+            table = {"mlp.gate": ("gate_up", 0, f, 0), "mlp.up": ("gate_up", f if m.gated else 0, f, 0), "mlp.down": ("down", 0, h, 1)}
+        else:
             if sub == "mlp.router":
                 L["router"][: m.experts].copy_(t)
                 return True
@@ -262,6 +319,16 @@ class EngineWeights:
         self._put(L[key], r0, rows, cut, t, raw, scale=False)
         return True
 
+    def state_geometry(self) -> list[tuple[int, int, int, int, int]]:
+        """(heads, key width, value width, convolution channels, taps) of this rank's recurrent mixers, in layer order."""
+        c, out = self.cfg, []
+        for L in self.layers:
+            if L["kind"] == "gdn":
+                out.append((c.linear_num_value_heads, c.linear_key_head_dim, c.linear_value_head_dim, L["gdn_conv"].shape[0], L["gdn_conv"].shape[1]))
+            if L["kind"] == "specified":
+                out += [(m.heads // self.tp, m.dim, m.vdim, m.channels // self.tp, m.conv) for _, m, _ in L["spec"].branches() if isinstance(m, DeltaSpec)]
+        return out
+
     def num_bytes(self) -> int:
         seen, total = set(), 0
         for t in self.tensors():
@@ -271,19 +338,21 @@ class EngineWeights:
         return total
 
     def tensors(self):
+        from slime_b200.engine.quant import Fp8Weight
+
         yield self.embed
         yield self.lm_head
         yield self.final_norm
+        if self.bigram is not None:
+            yield self.bigram
         if self.vision is not None:
             yield from self.vision.parameters()
         for L in self.layers + self.draft:
             for v in L.values():
-                if v is None or isinstance(v, (str, int, LayerSpec)):  # absent buffers, kind tag, indexer's source layer, spec
-                    continue
-                if hasattr(v, "tensors"):  # a quantised matrix: its bytes and its scales
-                    yield from v.tensors()
-                else:
+                if isinstance(v, torch.Tensor):
                     yield v
+                elif isinstance(v, Fp8Weight):  # a quantised matrix: its bytes and its scales
+                    yield from v.tensors()
 
     # -- loading -----------------------------------------------------------------------
     def _rows(self, t, n_local):
@@ -302,6 +371,9 @@ class EngineWeights:
             if m is not None:
                 return int(m.group(1)) < len(self.layers) and self._load_specified(
                     self.layers[int(m.group(1))], m.group(2), t.to(self.device, self.dtype, non_blocking=True), t)
+            if name == "bigram":
+                self.bigram.copy_(t.to(self.device, self.dtype))
+                return True
             name = _LAYERED_TOP.get(name, name)
         if name.startswith("model.visual."):  # the image encoder keeps the checkpoint's parameter names
             if self.vision is None:
@@ -508,9 +580,6 @@ class EngineWeights:
 
         g = torch.Generator(device=self.device).manual_seed(seed)
         quantised = [v for L in self.layers + self.draft for v in L.values() if isinstance(v, Fp8Weight)]
-        for L in self.layers:  # the decay parameter of delta-net layers must start in its valid range
-            if "gdn_A_log" in L:
-                L["gdn_A_log"].copy_(torch.empty_like(L["gdn_A_log"]).uniform_(1e-3, 16.0, generator=g).log())
         skip = {t.data_ptr() for v in quantised for t in v.tensors()}
         for t in self.tensors():
             if t.data_ptr() in skip:
@@ -521,6 +590,13 @@ class EngineWeights:
                 t.copy_(torch.empty(t.shape, dtype=torch.float32, device=self.device).normal_(0, std, generator=g))
         for v in quantised:
             v.fill_random_(std, g)
+        stream_norms = [self.final_norm] + [L[k] for L in self.layers for k in _NORMS.values() if L.get(k) is not None]
+        for t in stream_norms if self.cfg.norm_offset else ():  # stored as the difference from the offset
+            t.fill_(1.0 - self.cfg.norm_offset)
+        for L in self.layers:
+            for k, t in L.items():
+                if k.endswith("A_log"):  # the decay parameter of the delta rule must start in its valid range
+                    t.copy_(torch.empty_like(t).uniform_(1e-3, 16.0, generator=g).log())
         for L in self.layers + self.draft:
             if L.get("qkv_bias") is not None:
                 L["qkv_bias"].zero_()
@@ -545,8 +621,11 @@ def _grouped_linear(x, w, lay):
 
 class ModelRunner:
     def __init__(self, cfg: ModelConfig, weights: EngineWeights, kv: PagedKVCache, max_batch: int, max_context: int,
-                 use_cuda_graph: bool = True, tp_group=None):  # fmt: skip
-        self.cfg, self.w, self.kv = cfg, weights, kv
+                 use_cuda_graph: bool = True, tp_group=None, states: RecurrentStates | None = None):  # fmt: skip
+        """``states``: recurrent states of the live requests, for models whose weights have a ``state_geometry``."""
+        self.cfg, self.w, self.kv, self.states = cfg, weights, kv, states
+        self.recurrent = bool(weights.state_geometry())
+        assert not self.recurrent or states is not None
         self.device = weights.device
         self.max_batch, self.max_context = max_batch, max_context
         self.max_pages_per_req = -(-max_context // kv.page_size)
@@ -570,22 +649,16 @@ class ModelRunner:
                     self._fused_tp = fused_tp.FusedAllReduceNorm(tp_group, max_batch, cfg.hidden_size, self.device)
                 except Exception as e:  # noqa: BLE001
                     logger.warning("fused tensor-parallel all-reduce unavailable (%r): using NCCL", e)
-        # KV slabs exist for the attention layers only; gated delta-net layers keep a recurrent state per decode slot
-        self.kv_of, n_attn = [], 0
+        # KV slabs exist for the attention layers only; recurrent mixers keep a state per request (``states``)
+        self.kv_of, self.state_of, n_attn, n_state = [], [], 0, 0  # per layer: number of its first slab / state
         for L in weights.layers + weights.draft:  # a draft head's layer number is num_layers + depth
-            self.kv_of.append(n_attn if L["kind"] in KV_KINDS else None)
-            n_attn += L["kind"] in KV_KINDS
+            n = len(cached_mixers(L))
+            r = len(L["spec"].branches()) - n if L["kind"] == "specified" else int(L["kind"] == "gdn")
+            self.kv_of.append(n_attn if n else None)
+            self.state_of.append(n_state if r else None)
+            n_attn, n_state = n_attn + n, n_state + r
         self.has_mla = any(L["kind"] == "mla" for L in weights.layers)
         self._dsa_masks: dict[int, torch.Tensor] = {}  # key choices of the indexer layers of the pass in flight
-        self.has_gdn = any(L["kind"] == "gdn" for L in weights.layers)
-        self.gdn_S, self.gdn_conv, self.last_gdn_states = {}, {}, None
-        if self.has_gdn:
-            hv, dk, dv = cfg.linear_num_value_heads, cfg.linear_key_head_dim, cfg.linear_value_head_dim
-            C, K = 2 * cfg.linear_num_key_heads * dk + hv * dv, cfg.linear_conv_kernel_dim
-            for li, L in enumerate(weights.layers):
-                if L["kind"] == "gdn":
-                    self.gdn_S[li] = torch.zeros(max_batch, hv, dk, dv, dtype=torch.float32, device=self.device)
-                    self.gdn_conv[li] = torch.zeros(max_batch, K - 1, C, dtype=weights.dtype, device=self.device)
         self._composed_attention = cfg.rotary_percent < 1.0 or cfg.rotary_interleaved or cfg.qk_layernorm_full or bool(cfg.mrope_section)
         # vision inputs: decode positions are the token index plus a per-request offset (an image advances the position
         # by its larger grid side only), prefill positions are three streams
@@ -593,11 +666,16 @@ class ModelRunner:
         self._mrope_axes = None
         rot = int(cfg.head_dim * cfg.rotary_percent) // 2 * 2
         self.rope = None if self.layered else ops.rope_table(cfg, max_context + 1, rot, self.device)
-        self.slopes = []  # specified layers: distance-penalty factors of this rank's query heads
+        # specified attention mixers, by slab: this rank's distance-penalty factors, scores of the column without a value
+        self.slopes, self.sinks, self.rotary = [], [], {}
         for L in weights.layers if self.layered else ():
-            sl, n = L["spec"].mixer.slopes(), L["spec"].mixer.heads // weights.tp
-            mine = None if sl is None else sl[weights.rank * n : (weights.rank + 1) * n]
-            self.slopes.append(None if mine is None else torch.tensor(mine, dtype=torch.float32, device=self.device))
+            for a in cached_mixers(L):
+                n, sl = a.heads // weights.tp, a.slopes()
+                f32 = lambda x: torch.tensor(x, dtype=torch.float32, device=self.device)  # noqa: E731
+                self.slopes.append(None if sl is None else f32(sl[weights.rank * n : (weights.rank + 1) * n]))
+                self.sinks.append(None if a.sink is None else f32([a.sink] * n))
+                if a.rot is not None and a.rot.dims and a.rot not in self.rotary:
+                    self.rotary[a.rot] = stream.rotary_table(max_context + 1, a.rot.dims, a.rot.base, self.device)
         self.stream_hook = None  # called with (layer, fp32 residual stream) after every specified layer (eager passes only)
         self.scale = 1.0 / math.sqrt(cfg.head_dim)
         if cfg.multi_latent_attention:
@@ -877,95 +955,101 @@ class ModelRunner:
             return mixed, z.reshape(T, hv, dv), b.reshape(T, hv), a.reshape(T, hv)
         return ops.gemm(x, L["gdn_qkv"]), ops.gemm(x, L["gdn_z"]).view(T, hv, dv), ops.gemm(x, L["gdn_b"]), ops.gemm(x, L["gdn_a"])
 
-    def _gdn_finish(self, L, o, z):
-        """Gated RMSNorm of the delta-rule output and the output projection."""
-        from slime_b200.models import mixers
-
-        T = o.shape[0]
-        y = mixers._rms(o, L["gdn_norm"], self.cfg.norm_epsilon).float() * torch.nn.functional.silu(z.float())
-        return ops.gemm(y.to(self.w.dtype).reshape(T, -1), L["gdn_out"])
-
-    def _gdn_gates(self, L, b, a):
-        beta = torch.sigmoid(b.float())
-        g = -L["gdn_A_log"].float().exp() * torch.nn.functional.softplus(a.float() + L["gdn_dt_bias"].float())
-        return g, beta
-
-    def _gdn_heads(self, mixed):
-        cfg, T = self.cfg, mixed.shape[0]
+    def _gdn(self, L, li, x, recur):
+        """Delta-net layer; ``recur`` as in ``_specified_layers``."""
+        cfg, T = self.cfg, x.shape[0]
         hk, hv, dk, dv = cfg.linear_num_key_heads, cfg.linear_num_value_heads, cfg.linear_key_head_dim, cfg.linear_value_head_dim
-        q, k, v = mixed.split([hk * dk, hk * dk, hv * dv], dim=-1)
-        q, k, v = q.view(T, hk, dk), k.view(T, hk, dk), v.view(T, hv, dv)
-        if hv // hk > 1:
-            q, k = q.repeat_interleave(hv // hk, dim=1), k.repeat_interleave(hv // hk, dim=1)
-        return q, k, v
+        mixed, z, b, a = self._gdn_project(L, x)
+        q, k, v = mixed.contiguous().split([hk * dk, hk * dk, hv * dv], dim=-1)
+        inputs = delta.DeltaInputs(q, k, v, a, b, L["gdn_conv"], L["gdn_A_log"], L["gdn_dt_bias"])
+        return ops.gemm(recur(self.state_of[li], inputs, z.reshape(T, -1), L["gdn_norm"], "silu", 1.0, None), L["gdn_out"])
 
-    def _gdn_prefill(self, L, li, x, positions_in_call, cu_q, states_in, states_out):
-        """Delta-net layer over the new tokens of every request; ``states_in[i][li]`` = (state, convolution history) the
-        request arrived with (None at its first chunk); the states after the chunk go to ``states_out[i][li]``."""
-        from slime_b200.models import mixers
+    def _extend_recurrence(self, extend):
+        """``recur(state number, inputs, gate, norm weight, gate activation, output factor, output view or None)`` of an extend pass."""
 
-        K = self.cfg.linear_conv_kernel_dim
-        mixed_in, z, b, a = self._gdn_project(L, x)
-        n_req = cu_q.numel() - 1
-        S_in = [None if states_in is None or states_in[i] is None else states_in[i][li][0] for i in range(n_req)]
-        h_in = [None if states_in is None or states_in[i] is None else states_in[i][li][1] for i in range(n_req)]
-        mixed = mixers.causal_short_conv(mixed_in, L["gdn_conv"], positions_in_call, history=h_in if any(h is not None for h in h_in) else None,
-                                         cu_seqlens=cu_q)  # fmt: skip
-        q, k, v = self._gdn_heads(mixed)
-        g, beta = self._gdn_gates(L, b, a)
-        o, finals = mixers.gated_delta_rule_chunked(q, k, v, g, beta, cu_q, initial_states=S_in, return_final_states=True)
-        bounds = cu_q.tolist()
-        for i, (lo, hi) in enumerate(zip(bounds[:-1], bounds[1:])):
-            prev = h_in[i] if h_in[i] is not None else mixed_in.new_zeros(K - 1, mixed_in.shape[1])
-            hist = torch.cat([prev.to(mixed_in.dtype), mixed_in[lo:hi]])[-(K - 1):]
-            states_out[i][li] = (finals[i], hist)
-        return self._gdn_finish(L, o.to(self.w.dtype), z)
+        def recur(n, inputs, z, w, act, scale, out):
+            o = delta.delta_extend(inputs, self.states.state[n], self.states.ring[n], extend)
+            return delta.head_gate(o, z, w, act, self.cfg.norm_epsilon, scale, out)
 
-    def _gdn_decode(self, L, li, x, n):
-        from slime_b200.models import mixers
+        return recur
 
-        mixed_in, z, b, a = self._gdn_project(L, x)
-        mixed = mixers.short_conv_step(mixed_in, L["gdn_conv"], self.gdn_conv[li][:n])
-        q, k, v = self._gdn_heads(mixed)
-        g, beta = self._gdn_gates(L, b, a)
-        o = mixers.gated_delta_rule_step(q, k, v, g, beta, self.gdn_S[li][:n])
-        return self._gdn_finish(L, o.to(self.w.dtype), z)
+    def _step_recurrence(self, n_rows: int, positions):
+        """The same of a decode step: idle rows touch no state."""
+        slots, active = self._static["state_slot"][:n_rows], self._static["active"][:n_rows]
 
-    def load_gdn_state(self, slot: int, states: dict | None):
-        """Put a request's recurrent states (from its prefill) into decode slot ``slot``."""
-        for li in self.gdn_S:
-            S, hist = states[li]
-            self.gdn_S[li][slot].copy_(S)
-            self.gdn_conv[li][slot].copy_(hist)
+        def recur(n, inputs, z, w, act, scale, out):
+            return delta.delta_step(inputs, self.states.state[n], self.states.ring[n], slots, active, positions, z, w, act,
+                                    self.cfg.norm_epsilon, scale, out)  # fmt: skip
+
+        return recur
 
     # ------------------------------------------------------------ specified layers (models/layer_spec.py)
-    def _specified_layers(self, ids, slots, attend):
-        """All layers of a model with ``layer_specs`` over the tokens ``ids`` -> the final norm's output. ``attend(li, spec, q)``
-        runs layer ``li``'s attention once its keys and values are in the cache: the only part that differs between a
-        prefill pass and a decode step. The residual stream is fp32; between two sub-layers there is one fused launch."""
-        cfg, w, eps = self.cfg, self.w, self.cfg.norm_epsilon
-        kind, f32 = cfg.norm_kind, torch.float32
+    def _specified_layers(self, ids, prev, positions, slots, attend, recur):
+        """All layers of a model with ``layer_specs`` over the tokens ``ids`` (``prev``: the tokens in front of them, -1 at a
+        sequence's start; read by models with a bigram table) -> the final norm's output. ``attend(slab, spec, q, factor, out)`` runs an
+        attention mixer once its keys and values are in the cache, ``recur`` (``_extend_recurrence``) a recurrent one: the
+        only parts that differ between a prefill pass and a decode step. The residual stream is fp32; between two
+        sub-layers there is one fused launch."""
+        cfg, w = self.cfg, self.w
+        norm = dict(kind=cfg.norm_kind, offset=cfg.norm_offset)
+        f32, eps = torch.float32, cfg.norm_epsilon
         first = w.layers[0]["ln1"]
+        pair = None
+        if cfg.bigram:
+            pair = stream.PairTable(w.bigram, ids.to(torch.int32), prev, cfg.bigram["mul_prev"], cfg.bigram["mul_cur"])
         if w.tp > 1:  # vocab-parallel table: rows of other ranks come out as zeros
             x = self._tp_reduce(stream.stream_norm(w.embed, None, None, eps, ids=ids - w.rank * w.vocab_local)[1])
-            h, res = stream.stream_norm(x, None, first, eps, kind=kind)
+            if pair is not None:
+                x = x + pair.table[pair.rows()].float()
+            h, res = stream.stream_norm(x, None, first, eps, **norm)
         else:
-            h, res = stream.stream_norm(w.embed, None, first, eps, kind=kind, ids=ids)
+            h, res = stream.stream_norm(w.embed, None, first, eps, ids=ids, pair=pair, **norm)
         for li, L in enumerate(w.layers):
-            spec, a = L["spec"], L["spec"].mixer
-            hq, hkv = a.heads // w.tp, a.kv_heads // w.tp
-            qkv = _linear(h, L["qkv"])
-            nq, nk = hq * a.dim, hkv * a.dim
-            stream.kv_scatter(qkv[:, nq : nq + nk], qkv[:, nq + nk :], slots, self.kv.k[self.kv_of[li]], self.kv.v[self.kv_of[li]])
-            ctx = attend(li, a, qkv[:, :nq].unflatten(1, (hq, a.dim)))
-            y = self._tp_reduce(_linear(ctx.flatten(1), L["o"], out_dtype=f32))
+            spec = L["spec"]
+            y = self._tp_reduce(_linear(self._specified_mixers(L, li, h, positions, slots, attend, recur), L["out"], out_dtype=f32))
             after = w.layers[li + 1]["ln1"] if li + 1 < len(w.layers) else w.final_norm
-            h, _ = stream.stream_norm(y, res, after if spec.mlp is None else L["ln2"], eps, kind=kind, post_w=L["post_attn_ln"])
-            if spec.mlp is not None:
-                h, _ = stream.stream_norm(self._specified_mlp(L, spec.mlp, h), res, after, eps, kind=kind, post_w=L["post_mlp_ln"])
+            behind = spec.mlp is not None and not spec.parallel_ff
+            h, _ = stream.stream_norm(y, res, L["ln2"] if behind else after, eps, post_w=L.get("post_attn_ln"), **norm)
+            if behind:
+                h, _ = stream.stream_norm(self._specified_mlp(L, spec.mlp, h), res, after, eps, post_w=L.get("post_mlp_ln"), **norm)
             if self.stream_hook is not None:
                 self.stream_hook(li, res)
         return h
+
+    def _specified_mixers(self, L, li, h, positions, slots, attend, recur):
+        """What goes into a layer's output projection: the heads of its mixers, scaled, and the hidden units of a feed-forward
+        beside them, side by side as in ``LayerProjections.outs``."""
+        spec, lay, T = L["spec"], L["proj"], h.shape[0]
+        x = _linear(h, L["in"])
+        cols = lambda name: x[:, lay.ins[name][0] : sum(lay.ins[name])]  # noqa: E731
+        y = (torch.zeros if lay.padded(lay.outs) else torch.empty)(T, lay.out_cols, dtype=h.dtype, device=h.device)
+        slab, number = self.kv_of[li], self.state_of[li]
+        for p, m, factor in spec.branches():
+            c0, n = lay.outs[p + "o"]
+            out = y[:, c0 : c0 + n]
+            if isinstance(m, AttentionSpec):
+                q = stream.place_heads(cols(p + "q"), cols(p + "k"), cols(p + "v"), slots, self.kv.k[slab], self.kv.v[slab],
+                                       q_norm=L.get(p + "q.norm"), k_norm=L.get(p + "k.norm"), eps=self.cfg.norm_epsilon,
+                                       table=self.rotary.get(m.rot), positions=positions, interleaved=m.rot is None or m.rot.interleaved)  # fmt: skip
+                attend(slab, m, q, factor, out)
+                slab += 1
+                continue
+            a, z = (cols(p + s) if p + s in lay.ins else None for s in "ag")
+            if p in lay.low:
+                r0, inner, _, parts = lay.low[p]
+                second = _linear(x[:, r0 : r0 + inner], L[p + "low"])
+                if p + "a2" in parts:
+                    a = second[:, parts[p + "a2"][0] : sum(parts[p + "a2"][:2])]
+                if p + "g2" in parts:
+                    z = second[:, parts[p + "g2"][0] : sum(parts[p + "g2"][:2])]
+            inputs = delta.DeltaInputs(cols(p + "q"), cols(p + "k"), cols(p + "v"), a, cols(p + "b"), L[p + "conv"], L[p + "A_log"], L[p + "dt_bias"])
+            recur(number, inputs, z, L[p + "norm"], m.gate, factor, out)
+            number += 1
+        if spec.parallel_ff and spec.mlp is not None:
+            m, (c0, n) = spec.mlp, lay.outs["mlp.down"]
+            r0 = lay.ins["mlp.gate" if m.gated else "mlp.up"][0]
+            stream.feed_forward_act(x[:, r0 : r0 + (2 * n if m.gated else n)], m.act, m.gated, out=y[:, c0 : c0 + n])
+        return y
 
     def _specified_mlp(self, L, m, h):
         """Feed-forward of a specified layer: fp32 output, or for experts the unfinished sum the next norm completes."""
@@ -1001,7 +1085,7 @@ class ModelRunner:
 
     # --------------------------------------------------------------------- prefill
     @torch.no_grad()
-    def prefill(self, ids, positions, slots, cu_q, kv_gather_slots, cu_k, max_q, max_k, last_rows, fresh: bool, gdn_states=None,
+    def prefill(self, ids, positions, slots, cu_q, kv_gather_slots, cu_k, max_q, max_k, last_rows, fresh: bool, prev=None,
                 embed_rows=None, extend=None):
         """Extend pass over packed new tokens.
 
@@ -1009,22 +1093,22 @@ class ModelRunner:
         ``kv_gather_slots``/``cu_k``: cache slots of every context token (cached prefix + new) per
         request, used when some context is already cached (``fresh`` False). Returns logits
         ``[len(last_rows), V/tp]`` fp32 for the requested rows and, when ``last_rows`` is None, all rows.
-        Models with delta-net layers: ``gdn_states[i]`` is request i's recurrent state from its earlier chunks (or
-        None); the states after this pass are left in ``last_gdn_states``.
+        ``prev``: the token in front of each row (-1 at a sequence's start), for models with a bigram table.
         Vision inputs: ``positions`` may be ``[3, T]`` (temporal / height / width streams) and ``embed_rows`` = (rows,
         vectors) replaces the embeddings of image placeholder tokens by the encoder's outputs.
-        Models with specified layers read the context from the cache pages: ``extend`` (``ops.window_attention.ExtendBatch``)
-        says where every row stands, ``kv_gather_slots`` is not used.
+        Models with specified layers read the context from the cache pages, models with recurrent mixers continue each
+        request's state: ``extend`` (``ops.window_attention.ExtendBatch``) says where every row stands. With specified layers
+        ``kv_gather_slots`` is not used.
         """
         cfg, w, d = self.cfg, self.w, self.cfg.head_dim
         if self.layered:
             from slime_b200.ops import window_attention
 
-            def attend(li, a, q):
-                kv = self.kv_of[li]
-                return window_attention.window_extend(q, self.kv.k[kv], self.kv.v[kv], extend, a.scale, a.window, a.keep_first, self.slopes[li])
+            def attend(n, a, q, factor, out):
+                return window_attention.window_extend(q, self.kv.k[n], self.kv.v[n], extend, a.scale, a.window, a.keep_first, self.slopes[n],
+                                                      self.sinks[n], factor, out)  # fmt: skip
 
-            h = self._specified_layers(ids, slots, attend)
+            h = self._specified_layers(ids, prev, positions, slots, attend, self._extend_recurrence(extend))
             h = h if last_rows is None else h.index_select(0, last_rows)
             return self._gather_logits(ops.gemm(h, w.lm_head, out_dtype=torch.float32))
         x = ops.embedding(ids, w.embed, w.rank * w.vocab_local)
@@ -1035,17 +1119,13 @@ class ModelRunner:
             deepstack = embed_rows[2] if len(embed_rows) > 2 else []
         res = None
         T = ids.numel()
-        if self.has_gdn:
-            from slime_b200.models.gpt import positions_from_cu_seqlens
-
-            in_call = positions_from_cu_seqlens(cu_q, T)  # position inside this pass (a later chunk starts at 0 again)
-            self.last_gdn_states = [dict() for _ in range(cu_q.numel() - 1)]
+        recur = self._extend_recurrence(extend)
         for li, L in enumerate(w.layers):
             if 0 < li <= len(deepstack):  # vision vectors that join the stream after layer li - 1 (stream = x + res)
                 x = x.index_add(0, embed_rows[0], deepstack[li - 1].to(x.dtype))
             normed, res = ops.rmsnorm(x, L["ln1"], cfg.norm_epsilon, res)
             if L["kind"] == "gdn":
-                x = self._gdn_prefill(L, li, normed, in_call, cu_q, gdn_states, self.last_gdn_states)
+                x = self._gdn(L, li, normed, recur)
                 normed, res = ops.rmsnorm(x, L["ln2"], cfg.norm_epsilon, res)
                 x = self._mlp(L, normed)
                 continue
@@ -1128,7 +1208,7 @@ class ModelRunner:
     # lags one step behind reading results. The host owns the block table, the active mask, sampling
     # parameters and "init" records for slots that start decoding; those live in one flat pinned buffer
     # (double-buffered) uploaded with a single copy per step.
-    HOST_FIELDS = ("active", "init_mask", "init_ids", "init_pos", "init_out_pos", "top_k", "temperature", "top_p", "min_p")
+    HOST_FIELDS = ("active", "init_mask", "init_ids", "init_pos", "init_out_pos", "init_prev", "state_slot", "top_k", "temperature", "top_p", "min_p")
 
     def _alloc_static(self):
         B, W, dev = self.max_batch, self.max_pages_per_req, self.device
@@ -1159,6 +1239,8 @@ class ModelRunner:
         i32 = lambda *sh: torch.zeros(*sh, dtype=torch.int32, device=dev)  # noqa: E731
         self._dev_state = dict(ids=i32(B), pos=i32(B), out_pos=i32(B), ids_eff=i32(B), pos_eff=i32(B), seq_lens=i32(B) + 1,
                                slots=i32(B))  # fmt: skip
+        if self.cfg.bigram:  # the token in front of each slot's current one
+            self._dev_state.update(prev=i32(B) - 1, prev_eff=i32(B) - 1)
 
     def upload_static(self):
         """Copy the scheduler's host state to the device through a pinned staging buffer that is not in
@@ -1193,7 +1275,7 @@ class ModelRunner:
             _lib.check(_lib.lib().sb_decode_prepare(
                 P(ds["ids"]), P(ds["pos"]), P(ds["out_pos"]), P(st["init_mask"]), P(st["init_ids"]), P(st["init_pos"]),
                 P(st["init_out_pos"]), P(st["active"]), P(st["block_table"]), P(ds["ids_eff"]), P(ds["pos_eff"]),
-                P(ds["seq_lens"]), P(ds["slots"]), n, ps, W, _lib.stream()), "sb_decode_prepare")  # fmt: skip
+                P(ds["seq_lens"]), P(ds["slots"]), P(ds.get("prev")), P(st["init_prev"]), P(ds.get("prev_eff")), n, ps, W, _lib.stream()), "sb_decode_prepare")  # fmt: skip
         else:
             self._prepare_reference(n)
         h = self._decode_layers(n, ids, pos, slots, bt, seq_lens)
@@ -1204,10 +1286,12 @@ class ModelRunner:
         )  # fmt: skip
         routed = self.take_routed()
         if self.device.type == "cuda":
-            _lib.check(_lib.lib().sb_decode_advance(P(ds["ids"]), P(ds["pos"]), P(ds["out_pos"]), P(st["active"]), P(tok), n,
-                                                    _lib.stream()), "sb_decode_advance")  # fmt: skip
+            _lib.check(_lib.lib().sb_decode_advance(P(ds["ids"]), P(ds["pos"]), P(ds["out_pos"]), P(st["active"]), P(tok),
+                                                    P(ds.get("prev")), n, _lib.stream()), "sb_decode_advance")  # fmt: skip
         else:
             act = st["active"][:n].bool()
+            if "prev" in ds:
+                ds["prev"][:n] = torch.where(act, ds["ids"][:n], ds["prev"][:n])
             ds["ids"][:n] = torch.where(act, tok, ds["ids"][:n])
             ds["pos"][:n] += act.int()
             ds["out_pos"][:n] += act.int()
@@ -1219,12 +1303,13 @@ class ModelRunner:
         if self.layered:
             from slime_b200.ops import window_attention
 
-            def attend(li, a, q):
-                kv = self.kv_of[li]
-                return window_attention.window_decode(q, self.kv.k[kv], self.kv.v[kv], bt, seq_lens, pos, ps, a.scale, a.window, a.keep_first,
-                                                      self.slopes[li], self.max_context)  # fmt: skip
+            def attend(i, a, q, factor, out):
+                return window_attention.window_decode(q, self.kv.k[i], self.kv.v[i], bt, seq_lens, pos, ps, a.scale, a.window, a.keep_first,
+                                                      self.slopes[i], self.max_context, self.sinks[i], factor, out)  # fmt: skip
 
-            return self._specified_layers(ids, slots, attend)
+            prev = self._dev_state["prev_eff"][:n] if cfg.bigram else None
+            return self._specified_layers(ids, prev, pos, slots, attend, self._step_recurrence(n, pos))
+        recur = self._step_recurrence(n, pos)  # (a state's position counts tokens, whatever the rotary position is)
         if self.rope_delta is not None:
             pos = pos + self.rope_delta[:n]  # rotary position of a request that carries images
         x = ops.embedding(ids, w.embed, w.rank * w.vocab_local)
@@ -1236,7 +1321,7 @@ class ModelRunner:
         normed, res = ops.rmsnorm(x, w.layers[0]["ln1"], cfg.norm_epsilon, None)
         for li, L in enumerate(w.layers):
             if L["kind"] == "gdn":
-                normed, res = ops.rmsnorm(self._gdn_decode(L, li, normed, n), L["ln2"], cfg.norm_epsilon, res)
+                normed, res = ops.rmsnorm(self._gdn(L, li, normed, recur), L["ln2"], cfg.norm_epsilon, res)
             elif L["kind"] == "mla":
                 ctx = self._mla_decode(L, li, normed, pos, slots, bt, seq_lens, n)
                 normed, res = self._row_parallel_norm(ctx, L["o"], L["ln2"], res, n)
@@ -1264,6 +1349,9 @@ class ModelRunner:
         for dst, src in (("ids", "init_ids"), ("pos", "init_pos"), ("out_pos", "init_out_pos")):
             ds[dst][:n] = torch.where(init, st[src][:n], ds[dst][:n])
         act = st["active"][:n].bool()
+        if "prev" in ds:
+            ds["prev"][:n] = torch.where(init, st["init_prev"][:n], ds["prev"][:n])
+            ds["prev_eff"][:n] = torch.where(act, ds["prev"][:n], torch.full_like(ds["prev"][:n], -1))
         p = ds["pos"][:n].long()
         slot = st["block_table"][:n].gather(1, (p // ps)[:, None]).squeeze(1).long() * ps + p % ps
         idle = torch.arange(n) % ps

@@ -1,0 +1,98 @@
+"""Where the matrices of a specified layer (``models/layer_spec.py``) lie in the engine's fused buffers.
+
+Everything that reads a layer's normed input is one matrix ``in`` (rows: the projections of all its mixers, and of the
+feed-forward when it runs beside them), everything that ends in the residual stream is one matrix ``out`` (columns: the
+mixers' heads, the feed-forward's hidden units). So a layer costs two large products whatever it is made of, the products'
+sum over mixers and feed-forward is the second one's inner product, and one all-reduce covers it. Two-factor projections
+share a third, block-diagonal matrix ``low`` that reads a column range of the first product.
+
+Every range starts at a multiple of 8 (16 bytes in bf16); what is in between is zero in the matrices.
+"""
+
+from __future__ import annotations
+
+from slime_b200.models.layer_spec import AttentionSpec, DeltaSpec, LayerSpec
+
+
+def up8(n: int) -> int:
+    return -(-n // 8) * 8
+
+
+class LayerProjections:
+    """``ins[name] = (first row, rows)`` and ``outs[name] = (first column, columns)`` of this rank's part of checkpoint tensor
+    ``name`` (behind ``l<i>.``); ``whole``: names that every rank holds completely. ``low[prefix]``: the second factors of mixer
+    ``prefix``: (first column in the first product, inner width, rows, {name: (first row, rows, first column, columns)})."""
+
+    def __init__(self, spec: LayerSpec, tp: int = 1):
+        self.spec, self.tp = spec, tp
+        self.ins: dict[str, tuple[int, int]] = {}
+        self.outs: dict[str, tuple[int, int]] = {}
+        self.low: dict[str, tuple[int, int, int, dict]] = {}
+        self.whole: set[str] = set()
+        self.in_rows = self.out_cols = 0
+        for p, m, _ in spec.branches():
+            if m.heads % tp or m.kv_heads % tp:
+                raise ValueError(f"{m.heads} and {m.kv_heads} heads do not divide over {tp} tensor-parallel ranks")
+            h, g = m.heads // tp, m.kv_heads // tp
+            self._in(p + "q", (h if isinstance(m, AttentionSpec) else g) * m.dim)
+            self._in(p + "k", g * m.dim)
+            self._in(p + "v", (g if isinstance(m, AttentionSpec) else h) * m.vdim)
+            if isinstance(m, DeltaSpec):
+                self._delta(p, m, h)
+            self._out(p + "o", h * m.vdim)
+        m = spec.mlp
+        if m is not None and spec.parallel_ff:
+            if m.ff % tp:
+                raise ValueError(f"a feed-forward of width {m.ff} does not divide over {tp} tensor-parallel ranks")
+            f = m.ff // tp
+            if m.gated:  # gate and up rows without a gap: the activation reads them as one range
+                self.ins["mlp.gate"] = (self.in_rows, f)
+                self.ins["mlp.up"] = (self.in_rows + f, f)
+                self.in_rows += up8(2 * f)
+            else:
+                self._in("mlp.up", f)
+            self._out("mlp.down", f)
+
+    def _in(self, name: str, rows: int):
+        self.ins[name] = (self.in_rows, rows)
+        self.in_rows += up8(rows)
+
+    def _out(self, name: str, cols: int):
+        self.outs[name] = (self.out_cols, cols)
+        self.out_cols += up8(cols)
+
+    def _delta(self, p: str, m: DeltaSpec, h: int):
+        self._in(p + "b", h)
+        pairs = [("a", m.decay_rank, m.decays // self.tp), ("g", m.gate_rank, h * m.vdim)]
+        for n, rank, rows in pairs:
+            if rank is None:
+                self._in(p + n, rows)
+        first, inner, total, parts = self.in_rows, 0, 0, {}
+        for n, rank, rows in pairs:
+            if rank is not None:
+                self._in(p + n + "1", rank)
+                self.whole.add(p + n + "1")
+                parts[p + n + "2"] = (total, rows, inner, rank)
+                inner, total = inner + up8(rank), total + up8(rows)
+        if parts:
+            self.low[p] = (first, inner, total, parts)
+
+    def padded(self, ranges: dict) -> bool:
+        return any(n % 8 for _, n in ranges.values())
+
+    # ------------------------------------------------------------------ the checkpoint's side
+    def tensors(self, width: int) -> dict[str, tuple[int, ...]]:
+        """Shapes of the mixers' tensors (and of a feed-forward beside them) in the checkpoint; tp must be 1."""
+        assert self.tp == 1
+        out = {n: (rows, width) for n, (_, rows) in self.ins.items()}
+        out.update({n: (width, cols) for n, (_, cols) in self.outs.items()})
+        for _, _, _, parts in self.low.values():
+            out.update({n: (rows, cols) for n, (_, rows, _, cols) in parts.items()})
+        for p, m, _ in self.spec.branches():
+            if isinstance(m, DeltaSpec):
+                g, h = m.kv_heads * m.dim, m.heads * m.vdim
+                out.update({p + "q.conv": (g, m.conv), p + "k.conv": (g, m.conv), p + "v.conv": (h, m.conv), p + "A_log": (m.heads,),
+                            p + "dt_bias": (m.decays,), p + "norm": (m.vdim,)})  # fmt: skip
+            elif m.qk_norm:
+                out.update({p + "q.norm": (m.dim,), p + "k.norm": (m.dim,)})
+        return out

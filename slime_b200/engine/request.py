@@ -62,7 +62,7 @@ class Request:
     stream: bool = False
     prefill_only: bool = False  # prefill / decode disaggregation: stop after the first token and export the prompt's KV
     kv_export: Any = None  # (k, v) [layers, tokens, kv heads, head dim] of a finished prefill-only request
-    gdn_state: Any = None  # {layer: (recurrent state, convolution history)} between prefill chunks, until a decode slot takes it
+    state_slot: int | None = None  # where its recurrent states live (engine/state_cache.py), from admission to the end
     mm: dict | None = None  # vision inputs: pixel_values + image_grid_thw (and the video pair) for the placeholder tokens of input_ids
     extra_meta: dict = field(default_factory=dict)  # added verbatim to meta_info (e.g. the pd_* transfer figures)
     # ---- engine state ----

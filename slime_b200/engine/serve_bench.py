@@ -70,12 +70,9 @@ def _prefill_ms(e: Engine, lengths: list[int], steps: int, warmup: int) -> float
     p = e._pack(batch)
     rows = e._to_dev([c - 1 for c in p.cu_q[1:]], torch.long)
     _, dev_in = e._extend_pass(batch, p, rows)
-    extend = None
-    if e.runner.layered:
-        from slime_b200.ops.window_attention import ExtendBatch
-
-        extend = ExtendBatch.build([r.pages for r, _ in batch], [0] * len(batch), lengths, e.page_size, e.device)
-    ms = _timed(lambda: e.runner.prefill(*dev_in, p.max_q, p.max_k, rows, True, extend=extend), steps, warmup)
+    extend = e._extend_batch(batch) if e.runner.layered or e.runner.recurrent else None
+    prev = e._to_dev(p.prev) if e.cfg.bigram else None
+    ms = _timed(lambda: e.runner.prefill(*dev_in, p.max_q, p.max_k, rows, True, prev=prev, extend=extend), steps, warmup)
     for r, _ in batch:
         e.kv.allocator.release(r.pages)
     return ms

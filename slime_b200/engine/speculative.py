@@ -49,7 +49,7 @@ class SpeculativeDecoder:
             raise NotImplementedError("a separate draft model is not supported: the draft head is the checkpoint's own")
         if not engine.weights.draft:
             raise ValueError("speculative decoding needs a model with a draft head (mtp_num_layers >= 1)")
-        if engine.runner.has_gdn:
+        if engine.runner.recurrent:
             raise NotImplementedError("speculative decoding over recurrent (delta-net) layers would need state rollback")
         self.eng = engine
         self.k = max(1, int(a.speculative_num_steps))

@@ -95,6 +95,10 @@ class ModelConfig:
     # designs whose layers differ (models/layer_spec.py): one spec per layer; the size fields above then hold maxima
     layer_specs: list | None = None
     norm_kind: str = "rms"  # rms | layer (weight only; models with layer_specs)
+    norm_offset: float = 0.0  # added to the stored weight of the stream's norms (1: stored around zero; models with layer_specs)
+    # second embedding table (models with layer_specs): row (previous token * mul_prev + token * mul_cur) mod buckets is added,
+    # row ``buckets`` for a sequence's first token
+    bigram: dict | None = None
     # multi-token prediction (draft head)
     mtp_num_layers: int | None = None
     model_arch: str = "qwen2"
@@ -108,8 +112,8 @@ class ModelConfig:
             self.padded_vocab_size = self.vocab_size
         if self.layer_specs is not None:
             self.layer_specs = [LayerSpec.of(x) for x in self.layer_specs]
-        elif self.norm_kind != "rms":
-            raise ValueError(f"norm_kind {self.norm_kind!r} is available to models with layer_specs only")
+        elif self.norm_kind != "rms" or self.norm_offset or self.bigram:
+            raise ValueError("norm_kind, norm_offset and bigram are available to models with layer_specs only")
 
     @property
     def head_dim(self) -> int:
@@ -130,9 +134,9 @@ class ModelConfig:
 
     def mixer(self, layer: int) -> str:
         """Token mixer of a layer: ``attention`` (the fused kernel path), ``general_attention`` (attention variants
-        composed from separate ops), ``gated_delta_net``, ``mla``, ``dsa``, or ``window_attention`` (specified layers)."""
+        composed from separate ops), ``gated_delta_net``, ``mla``, ``dsa``, or ``specified`` (layer_specs)."""
         if self.layer_specs is not None:
-            return "window_attention"
+            return "specified"
         if self.full_attention_interval and (layer + 1) % self.full_attention_interval != 0:
             return "gated_delta_net"
         if self.multi_latent_attention:
@@ -145,9 +149,8 @@ class ModelConfig:
     def mixer_params(self, layer: int) -> int:
         h, d = self.hidden_size, self.head_dim
         kind = self.mixer(layer)
-        if kind == "window_attention":
-            a = self.layer_specs[layer].mixer
-            return h * (a.heads * (a.dim + a.vdim) + a.kv_heads * (a.dim + a.vdim))
+        if kind == "specified":
+            return self.layer_specs[layer].mixer.params(h)
         if kind == "gated_delta_net":
             kd, vd = self.linear_num_key_heads * self.linear_key_head_dim, self.linear_num_value_heads * self.linear_value_head_dim
             return (h * (2 * kd + 2 * vd) + h * 2 * self.linear_num_value_heads + (2 * kd + vd) * self.linear_conv_kernel_dim
@@ -170,8 +173,8 @@ class ModelConfig:
         total = 0
         for i in range(self.num_layers):
             if self.layer_specs is not None:
-                mlp = self.layer_specs[i].mlp
-                total += self.mixer_params(i) + (2 * h if mlp is None else 4 * h + mlp.params(h))
+                spec = self.layer_specs[i]
+                total += self.mixer_params(i) + len(spec.norms(self.post_self_attn_layernorm)) * h + (spec.mlp.params(h) if spec.mlp else 0)
                 continue
             total += self.mixer_params(i) + 2 * h
             if self.is_moe_layer(i):
@@ -181,6 +184,8 @@ class ModelConfig:
             else:
                 total += 3 * h * self.ffn_hidden_size
         total += self.vocab_size * h * (1 if self.tie_word_embeddings else 2) + h
+        if self.bigram:
+            total += (self.bigram["buckets"] + 1) * h
         if self.vision:
             v = self.vision
             d, inter, big = v["hidden_size"], v["intermediate_size"], v["hidden_size"] * v.get("spatial_merge_size", 2) ** 2
@@ -218,7 +223,9 @@ class ModelConfig:
         return cls(**kw)
 
     @classmethod
-    def from_hf(cls, path_or_dict) -> "ModelConfig":
+    def from_hf(cls, path_or_dict, shapes: dict | None = None) -> "ModelConfig":
+        """``shapes``: tensor shapes by name for designs that state a size by a tensor only (default: those of the files in
+        the checkpoint directory)."""
         if isinstance(path_or_dict, dict):
             c = path_or_dict
         elif isinstance(path_or_dict, str) and path_or_dict.startswith("preset:"):
@@ -227,7 +234,11 @@ class ModelConfig:
             with open(os.path.join(path_or_dict, "config.json")) as f:
                 c = json.load(f)
         if c.get("architecture") in LAYERED_ARCHITECTURES:
-            return cls(**LAYERED_ARCHITECTURES[c["architecture"]][0](c))
+            if shapes is None and isinstance(path_or_dict, str):
+                from slime_b200.checkpoint.hf_loader import tensor_shapes
+
+                shapes = tensor_shapes(path_or_dict)
+            return cls(**LAYERED_ARCHITECTURES[c["architecture"]][0](c, shapes))
         top = c
         c = c.get("text_config", c)
         arch = (c.get("architectures") or top.get("architectures") or [c.get("model_type", "qwen2")])[0]

@@ -4,6 +4,9 @@
 widths, window or feed-forward carries a list of ``LayerSpec`` instead (``ModelConfig.layer_specs``); the flat fields then
 hold the largest value of each size, for code that only budgets memory. The specs are mechanism parameters, not a model:
 any architecture whose layers are built from these pieces can use them.
+
+A layer is a mixer (``AttentionSpec``, ``DeltaSpec``, or two of them side by side: ``ParallelSpec``) and a feed-forward, one
+after the other with a residual sum each, or both reading one normed input (``LayerSpec.parallel_ff``).
 """
 
 from __future__ import annotations
@@ -13,10 +16,26 @@ from dataclasses import dataclass
 
 
 @dataclass(frozen=True)
+class RotarySpec:
+    """Rotation of the first ``dims`` coordinates of a query / key head by ``position * base^(-2i / dims)`` for pair i;
+    ``interleaved``: pair i is (2i, 2i + 1), otherwise (i, i + dims / 2)."""
+
+    dims: int
+    base: float
+    interleaved: bool = True
+
+    def __post_init__(self):
+        if self.dims < 0 or self.dims % 2:
+            raise ValueError(f"a rotation of {self.dims} coordinates: they come in pairs")
+
+
+@dataclass(frozen=True)
 class AttentionSpec:
-    """Grouped-query attention without rotation. ``window``: a query at position i sees keys j with i - j < window (None:
+    """Grouped-query attention. ``window``: a query at position i sees keys j with i - j < window (None:
     all earlier ones) and, whatever the distance, the first ``keep_first`` tokens of the sequence. ``distance_bias``
-    "geometric": head h of H subtracts ``2^(-8 (h + 1) / H) * (i - j)`` from its scores."""
+    "geometric": head h of H subtracts ``2^(-8 (h + 1) / H) * (i - j)`` from its scores. ``qk_norm``: RMS norm of every query
+    and key head (one weight each, shared by the heads) before the rotation ``rot``. ``sink``: score of an extra column of
+    the softmax that has no value (None: no such column)."""
 
     heads: int
     kv_heads: int
@@ -26,8 +45,15 @@ class AttentionSpec:
     window: int | None = None
     keep_first: int = 0
     distance_bias: str | None = None
+    qk_norm: bool = False
+    rot: RotarySpec | None = None
+    sink: float | None = None
 
     def __post_init__(self):
+        if isinstance(self.rot, dict):
+            object.__setattr__(self, "rot", RotarySpec(**self.rot))
+        if self.rot is not None and self.rot.dims > self.dim:
+            raise ValueError(f"a rotation of {self.rot.dims} coordinates in a head of {self.dim}")
         if self.heads % self.kv_heads:
             raise ValueError(f"{self.heads} query heads do not divide over {self.kv_heads} key/value heads")
         if self.window is not None and self.window < 1:
@@ -40,6 +66,72 @@ class AttentionSpec:
         if self.distance_bias is None:
             return None
         return [2.0 ** (-8.0 * (h + 1) / self.heads) for h in range(self.heads)]
+
+    def params(self, width: int) -> int:
+        return width * (self.heads + self.kv_heads) * (self.dim + self.vdim) + (2 * self.dim if self.qk_norm else 0)
+
+
+@dataclass(frozen=True)
+class DeltaSpec:
+    """Gated delta rule. Per head a state S [dim, vdim] follows ``S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q``; q, k and
+    v come from a causal convolution over ``conv`` tokens per channel and silu, q and k as unit vectors (q times dim^-1/2).
+    ``decay``: g = exp(-exp(A_log) softplus(projection + dt_bias)) is one number per "head" or one per key "channel".
+    The output is RMS normed per head and multiplied by ``gate``(projection). ``decay_rank`` / ``gate_rank``: inner width
+    of a two-factor projection (None: one full matrix)."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+    decay: str = "head"
+    gate: str = "silu"
+    decay_rank: int | None = None
+    gate_rank: int | None = None
+
+    def __post_init__(self):
+        if self.heads % self.kv_heads:
+            raise ValueError(f"{self.heads} heads do not divide over {self.kv_heads} query/key heads")
+        if self.decay not in ("head", "channel") or self.gate not in ("silu", "sigmoid"):
+            raise ValueError(f"unknown decay {self.decay!r} or gate {self.gate!r}")
+        if self.conv < 1:
+            raise ValueError(f"a convolution over {self.conv} tokens")
+
+    @property
+    def decays(self) -> int:
+        """Decay factors of one token."""
+        return self.heads * (self.dim if self.decay == "channel" else 1)
+
+    @property
+    def channels(self) -> int:
+        """Channels that pass the convolution: q, k, v."""
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+    def params(self, width: int) -> int:
+        pair = lambda n, r: n * width if r is None else r * (width + n)  # noqa: E731
+        n = self.channels * (width + self.conv) + self.heads * (width + 1) + self.decays + self.vdim
+        return n + pair(self.decays, self.decay_rank) + pair(self.heads * self.vdim, self.gate_rank) + width * self.heads * self.vdim
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """Two mixers that read the same input; the result is ``left_scale * left + right_scale * right``."""
+
+    left: AttentionSpec | DeltaSpec
+    right: AttentionSpec | DeltaSpec
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+
+    def params(self, width: int) -> int:
+        return self.left.params(width) + self.right.params(width)
+
+
+def _mixer_of(x):
+    if not isinstance(x, dict):
+        return x
+    if "left" in x:
+        return ParallelSpec(**{**x, "left": _mixer_of(x["left"]), "right": _mixer_of(x["right"])})
+    return DeltaSpec(**x) if "conv" in x else AttentionSpec(**x)
 
 
 @dataclass(frozen=True)
@@ -77,25 +169,44 @@ class FeedForwardSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: AttentionSpec
+    mixer: AttentionSpec | DeltaSpec | ParallelSpec
     mlp: FeedForwardSpec | None = None  # None: the layer is its mixer only
+    parallel_ff: bool = False  # mixer and feed-forward read the same normed input and join the stream in one sum
+
+    def __post_init__(self):
+        if self.parallel_ff and self.mlp is not None and self.mlp.experts is not None:
+            raise ValueError("a feed-forward beside the mixer is dense: experts have no form of it")
 
     @classmethod
     def of(cls, x) -> "LayerSpec":
         """Accepts a ``LayerSpec`` or its ``dataclasses.asdict`` form (presets, argument namespaces read from JSON)."""
         if isinstance(x, cls):
             return x
-        mixer, mlp = x["mixer"], x.get("mlp")
-        return cls(mixer if isinstance(mixer, AttentionSpec) else AttentionSpec(**mixer),
-                   mlp if mlp is None or isinstance(mlp, FeedForwardSpec) else FeedForwardSpec(**mlp))  # fmt: skip
+        mlp = x.get("mlp")
+        return cls(_mixer_of(x["mixer"]), mlp if mlp is None or isinstance(mlp, FeedForwardSpec) else FeedForwardSpec(**mlp),
+                   x.get("parallel_ff", False))  # fmt: skip
 
     def to_dict(self) -> dict:
         return dataclasses.asdict(self)
 
+    def branches(self) -> list[tuple[str, AttentionSpec | DeltaSpec, float]]:
+        """(prefix of its tensors behind ``l<i>.``, mixer, factor of its output) of every mixer of the layer."""
+        m = self.mixer
+        if isinstance(m, ParallelSpec):
+            return [("mix.left.", m.left, m.left_scale), ("mix.right.", m.right, m.right_scale)]
+        return [("mix.", m, 1.0)]
+
+    def norms(self, post: bool) -> list[str]:
+        """Names of the layer's norms (``post``: every sub-layer's output has one too)."""
+        subs = ["norm1"] if self.mlp is None or self.parallel_ff else ["norm1", "norm2"]
+        return [n + x for n in subs for x in (("", "b") if post else ("",))]
+
 
 def flat_sizes(specs: list[LayerSpec]) -> dict:
     """The ``ModelConfig`` size fields of a specified stack: the largest value of each over the layers."""
-    at, ff = [s.mixer for s in specs], [s.mlp for s in specs if s.mlp is not None]
+    mixers = [m for s in specs for _, m, _ in s.branches()]
+    at = [m for m in mixers if isinstance(m, AttentionSpec)] or mixers
+    ff = [s.mlp for s in specs if s.mlp is not None]
     moe = [m for m in ff if m.experts is not None]
     out = dict(num_layers=len(specs), num_attention_heads=max(a.heads for a in at), num_query_groups=max(a.kv_heads for a in at),
                kv_channels=max(a.dim for a in at), v_head_dim=max(a.vdim for a in at),
@@ -112,7 +223,7 @@ def flat_sizes(specs: list[LayerSpec]) -> dict:
 # squared-relu experts weighted by their own softmax score, geometric distance bias. Everything else is in config.json.
 
 
-def pefolix_config(c: dict) -> dict:
+def pefolix_config(c: dict, shapes: dict | None = None) -> dict:
     """``config.json`` of a Pefolix model -> ``ModelConfig`` arguments."""
     specs = []
     for i, layer in enumerate(c["layers"]):
@@ -154,5 +265,67 @@ def pefolix_json(cfg) -> dict:
     return dict(architecture="Pefolix", layers=layers, norm=dict(eps=cfg.norm_epsilon), vocab=cfg.vocab_size, width=cfg.hidden_size)
 
 
-# ``config.json`` files that name their design in "architecture": name -> (reader, writer)
-LAYERED_ARCHITECTURES = {"Pefolix": (pefolix_config, pefolix_json)}
+# ------------------------------------------------------------------------------------------------- Ledazen
+# Fixed by the design: one norm per layer (RMS, weight stored around zero) whose output mixer and feed-forward both read,
+# squared-relu feed-forward without a gate, rotation of interleaved pairs, q / k norms and a sink of score 0 in attention,
+# the two forms of the delta rule (alone: a decay per head, silu gate; beside attention: a decay per key channel, sigmoid
+# gate, both through two-factor projections), a bigram table added to the embedding.
+
+
+def _inner_width(shapes: dict | None, name: str, m: dict, key: str) -> int:
+    """Inner width of a two-factor projection: the checkpoint's tensor says it, or ``key`` of the mixer's description."""
+    if shapes and name in shapes:
+        return int(shapes[name][0])
+    if key in m:
+        return int(m[key])
+    raise ValueError(f"the inner width of {name} is not in config.json: give the checkpoint's tensor shapes, or {key!r} in the mixer")
+
+
+def ledazen_config(c: dict, shapes: dict | None = None) -> dict:
+    """``config.json`` of a Ledazen model (and the shapes of its tensors by name) -> ``ModelConfig`` arguments."""
+    sizes = lambda m: (m["heads"], m["kv_heads"], m["dim"], m["vdim"])  # noqa: E731
+    specs = []
+    for i, layer in enumerate(c["layers"]):
+        m, f = layer["mixer"], layer.get("mlp")
+        if layer["type"] == "delta":
+            mixer = DeltaSpec(*sizes(m), m["conv"])
+        elif layer["type"] == "parallel":
+            a, d = m["left"], m["right"]
+            rot = RotarySpec(a["rot"]["dims"], float(a["rot"]["base"])) if a.get("rot") else None
+            left = AttentionSpec(*sizes(a), float(a["scale"]), qk_norm=True, rot=rot, sink=0.0)
+            p = f"l{i}.mix.right."
+            right = DeltaSpec(*sizes(d), d["conv"], "channel", "sigmoid", _inner_width(shapes, p + "a1", d, "decay_rank"),
+                              _inner_width(shapes, p + "g1", d, "gate_rank"))  # fmt: skip
+            mixer = ParallelSpec(left, right, float(m["left_scale"]), float(m["right_scale"]))
+        else:
+            raise ValueError(f"layer {i}: a Ledazen model has no mixer of type {layer['type']!r}")
+        if f is not None and f["kind"] != "dense":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
+        specs.append(LayerSpec(mixer, None if f is None else FeedForwardSpec(f["ff"], "relu2", gated=False), parallel_ff=True))
+    b = c["embedding"]["bigram"]
+    return dict(flat_sizes(specs), layer_specs=specs, hidden_size=c["width"], vocab_size=c["vocab"], norm_epsilon=c["norm"]["eps"],
+                norm_offset=1.0, bigram=dict(buckets=b["buckets"], mul_prev=b["mul_prev"], mul_cur=b["mul_cur"]),
+                tie_word_embeddings=False, model_arch="Ledazen")  # fmt: skip
+
+
+def ledazen_json(cfg) -> dict:
+    """The ``config.json`` of a Ledazen ``ModelConfig`` (inverse of ``ledazen_config``; carries the inner widths too)."""
+    sizes = lambda m: dict(heads=m.heads, kv_heads=m.kv_heads, dim=m.dim, vdim=m.vdim)  # noqa: E731
+    layers = []
+    for s in cfg.layer_specs:
+        m = s.mixer
+        if isinstance(m, DeltaSpec):
+            kind, mixer = "delta", dict(sizes(m), conv=m.conv)
+        else:
+            left = dict(sizes(m.left), scale=m.left.scale)
+            if m.left.rot is not None:
+                left["rot"] = dict(dims=m.left.rot.dims, base=m.left.rot.base)
+            right = dict(sizes(m.right), conv=m.right.conv, decay_rank=m.right.decay_rank, gate_rank=m.right.gate_rank)
+            kind, mixer = "parallel", dict(left=left, right=right, left_scale=m.left_scale, right_scale=m.right_scale)
+        layers.append(dict(type=kind, mixer=mixer, mlp=None if s.mlp is None else dict(kind="dense", ff=s.mlp.ff)))
+    return dict(architecture="Ledazen", embedding=dict(bigram=dict(cfg.bigram)), layers=layers, norm=dict(eps=cfg.norm_epsilon),
+                vocab=cfg.vocab_size, width=cfg.hidden_size)  # fmt: skip
+
+
+# ``config.json`` files that name their design in "architecture": name -> (reader(config, tensor shapes or None), writer)
+LAYERED_ARCHITECTURES = {"Pefolix": (pefolix_config, pefolix_json), "Ledazen": (ledazen_config, ledazen_json)}

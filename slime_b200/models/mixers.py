@@ -677,7 +677,7 @@ def build_mixer(cfg: ModelConfig, layer_number: int, dtype, device, sequence_par
         if custom is not None:
             return custom
     kind = cfg.mixer(layer_number)
-    if kind == "window_attention":
+    if kind == "specified":
         raise NotImplementedError(f"{cfg.model_arch} models run in the rollout engine only: their layers have no backward pass here")
     if kind == "attention":
         from slime_b200.models.gpt import SelfAttention

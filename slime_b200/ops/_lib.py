@@ -36,13 +36,18 @@ _SIGS = {
     "sb_group_fp8_quant_1x128": [P, P, P, P, I, I, L, L, I, P],
     "sb_moe_topk": [P, P, P, P, L, I, L, I, I, I, F, P],
     "sb_moe_layout": [P, P, P, I, I, I, I, P],
-    "sb_stream_norm": [P, I, P, I, P, P, I, P, P, I, P, P, I, P, P, I, I, I, F, I, P],
-    "sb_glu": [P, P, L, I, I, I, I, P],
+    "sb_stream_norm": [P, I, P, I, P, P, I, P, P, I, P, P, I, P, P, I, I, I, F, F, I, P, P, P, L, L, I, P],
+    "sb_glu": [P, P, P, L, I, L, L, I, I, P],
+    "sb_heads": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, L, L, L, F, I, P],
     "sb_kv_scatter": [P, P, P, P, P, I, I, L, L, P],
     "sb_gemm_simt": [P, P, P, P, P, I, I, I, L, L, L, I, I, P],
-    "sb_window_attn": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, L, L, F, I, I, I, P],
-    "sb_flash_window": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, L, L, F, I, I, P, P],
-    "sb_paged_decode_window": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, I, I, P, P],
+    "sb_window_attn": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, L, L, F, F, I, I, I, P],
+    "sb_flash_window": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, L, L, F, F, I, I, P, P],
+    "sb_paged_decode_window": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, F, I, I, P, P],
+    "sb_delta_prep": [P, P, P, P, P, L, L, L, P, P, P, P, P, P, I, P, P, P, P, P, P, I, I, I, I, I, I, I, P],
+    "sb_delta_scan": [P, P, P, L, P, P, P, I, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P],
+    "sb_delta_step": [P, P, P, P, P, L, L, L, P, P, P, P, P, P, P, P, P, P, P, L, L, F, F, I, I, I, I, I, I, I, I, I, P],
+    "sb_head_gate": [P, P, P, P, I, I, I, L, L, F, F, I, I, P],
     "sb_moe_scatter_rows": [P, P, P, L, I, I, P],
     "sb_moe_gather_sum": [P, P, P, P, L, I, I, I, P],
     "sb_moe_route_weight_grad": [P, P, P, P, L, I, I, P],
@@ -68,8 +73,8 @@ _SIGS = {
     "sb_sample": [P, I, L, I, I, P, P, P, P, P, P, P, P, P, P, I, P],
     "sb_kv_write": [P, P, P, P, P, I, I, I, I, P],
     "sb_rope_kv_write": [P, P, P, P, P, P, P, P, I, I, I, I, I, F, P],
-    "sb_decode_prepare": [P, P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, P],
-    "sb_decode_advance": [P, P, P, P, P, I, P],
+    "sb_decode_prepare": [P, P, P, P, P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, P],
+    "sb_decode_advance": [P, P, P, P, P, P, I, P],
     "sb_paged_decode": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P],
     "sb_paged_decode_tc": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, P, P],
     "sb_paged_decode_ws": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, P, I, L, L, P],

@@ -31,10 +31,27 @@ class ExpertSum:
         return self.weights.shape[0]
 
 
-def _norm(v, w, eps, kind):
+@dataclasses.dataclass
+class PairTable:
+    """Second embedding table: token t adds row ``(prev * mul_prev + token * mul_cur) mod (rows - 1)`` of ``table``, the last row
+    where it has no predecessor (``prev`` < 0)."""
+
+    table: torch.Tensor
+    ids: torch.Tensor
+    prev: torch.Tensor
+    mul_prev: int
+    mul_cur: int
+
+    def rows(self) -> torch.Tensor:
+        n = self.table.shape[0] - 1
+        r = (self.prev.long() * self.mul_prev + self.ids.long() * self.mul_cur) % n
+        return torch.where(self.prev >= 0, r, torch.full_like(r, n))
+
+
+def _norm(v, w, eps, kind, offset=0.0):
     mean = v.mean(-1, keepdim=True) if kind == "layer" else 0.0
     d = v - mean
-    return d * torch.rsqrt(d.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+    return d * torch.rsqrt(d.pow(2).mean(-1, keepdim=True) + eps) * (w.float() + offset)
 
 
 def _combine(e: ExpertSum) -> torch.Tensor:
@@ -50,14 +67,15 @@ def _combine(e: ExpertSum) -> torch.Tensor:
     return y
 
 
-def stream_norm(y, res, pre_w, eps, *, kind="rms", post_w=None, ids=None):
+def stream_norm(y, res, pre_w, eps, *, kind="rms", post_w=None, ids=None, offset=0.0, pair: PairTable | None = None):
     """``res (+)= norm(y) * post_w`` and return ``norm(res) * pre_w``, in one launch.
 
     ``y``: sub-layer output [T, H], an ``ExpertSum``, or an embedding table when ``ids`` [T] is given (ids outside the table give
     zero rows: other ranks' part of a sharded vocabulary). ``res``: fp32 [T, H],
     updated in place; None starts the stream (a new tensor is returned as second value). ``post_w`` None: no norm of the
     sub-layer's output; ``pre_w`` None: nothing but the stream is wanted (the first value is None). ``kind``: "rms" or
-    "layer" (mean removed, no bias). Norms, sums and the stream are fp32 whatever the element types."""
+    "layer" (mean removed, no bias); ``offset`` is added to the norm weights in fp32. ``pair``: rows of a second table added to
+    ``y``. Norms, sums and the stream are fp32 whatever the element types."""
     moe = y if isinstance(y, ExpertSum) else None
     src = moe.rows if moe is not None else y
     T = moe.tokens() if moe is not None else (ids.numel() if ids is not None else y.shape[0])
@@ -72,13 +90,15 @@ def stream_norm(y, res, pre_w, eps, *, kind="rms", post_w=None, ids=None):
             v = src[i.clamp(0, src.shape[0] - 1)].float() * ((i >= 0) & (i < src.shape[0]))[:, None]
         else:
             v = _combine(moe) if moe is not None else src.float()
+        if pair is not None:
+            v = v + pair.table[pair.rows()].float()
         if post_w is not None:
-            v = _norm(v, post_w, eps, kind)
+            v = _norm(v, post_w, eps, kind, offset)
         if init:
             res = v.clone()
         else:
             res.add_(v)
-        return (None if pre_w is None else _norm(res, pre_w, eps, kind).to(w_dtype)), res
+        return (None if pre_w is None else _norm(res, pre_w, eps, kind, offset).to(w_dtype)), res
     src = src.contiguous()
     if init:
         res = torch.empty(T, H, dtype=torch.float32, device=src.device)
@@ -95,10 +115,15 @@ def stream_norm(y, res, pre_w, eps, *, kind="rms", post_w=None, ids=None):
         gate = moe.gate if shared is not None else None
         assert gate is None or gate.dtype == torch.float32
     ids32 = None if ids is None else ids.to(torch.int32).contiguous()
+    if pair is not None:
+        assert pair.table.is_contiguous() and pair.table.dtype == src.dtype and pair.table.shape[1] == H
+        assert pair.ids.dtype == pair.prev.dtype == torch.int32 and pair.ids.is_contiguous() and pair.prev.is_contiguous()
     rc = _lib.lib().sb_stream_norm(
         P(src), int(src.dtype == torch.float32), P(ids32), src.shape[0], P(dest), P(wts), k, P(shared), P(gate),
         gate.stride(0) if gate is not None else 0, P(post_w), P(res), int(init), P(pre_w), P(h), int(w_dtype == torch.float32),
-        T, H, float(eps), int(kind == "layer"), _lib.stream(),
+        T, H, float(eps), float(offset), int(kind == "layer"), P(pair.table) if pair else None, P(pair.ids) if pair else None,
+        P(pair.prev) if pair else None, pair.mul_prev if pair else 0, pair.mul_cur if pair else 0, pair.table.shape[0] - 1 if pair else 0,
+        _lib.stream(),
     )  # fmt: skip
     _lib.check(rc, "sb_stream_norm")
     return h, res
@@ -109,8 +134,8 @@ def combine(e: ExpertSum) -> torch.Tensor:
     return stream_norm(e, None, None, 0.0)[1]
 
 
-def feed_forward_act(x: torch.Tensor, act: str, gated: bool) -> torch.Tensor:
-    """``act(x[:, :F]) * x[:, F:]`` (gated) or ``act(x)``."""
+def feed_forward_act(x: torch.Tensor, act: str, gated: bool, out: torch.Tensor | None = None) -> torch.Tensor:
+    """``act(x[:, :F]) * x[:, F:]`` (gated) or ``act(x)``; ``x`` and ``out`` may be column ranges of wider matrices."""
     F = x.shape[-1] // 2 if gated else x.shape[-1]
     if not x.is_cuda:
         g = x[..., :F].float()
@@ -120,12 +145,66 @@ def feed_forward_act(x: torch.Tensor, act: str, gated: bool) -> torch.Tensor:
             g = torch.nn.functional.gelu(g, approximate="tanh")
         else:
             g = g.clamp_min(0).square()
-        return (g * x[..., F:].float() if gated else g).to(x.dtype)
-    x = x.contiguous()
-    out = torch.empty(x.shape[0], F, dtype=x.dtype, device=x.device)
-    rc = _lib.lib().sb_glu(P(x), P(out), x.shape[0], F, int(gated), ACTS[act], int(x.dtype == torch.float32), _lib.stream())
+        y = (g * x[..., F:].float() if gated else g).to(x.dtype)
+        return y if out is None else out.copy_(y)
+    x = x if x.stride(-1) == 1 else x.contiguous()
+    if out is None:
+        out = torch.empty(x.shape[0], F, dtype=x.dtype, device=x.device)
+    assert out.dtype == x.dtype and out.stride(-1) == 1 and out.shape == (x.shape[0], F)
+    rc = _lib.lib().sb_glu(P(x), P(x[:, F:]) if gated else None, P(out), x.shape[0], F, x.stride(0), out.stride(0), ACTS[act],
+                           int(x.dtype == torch.float32), _lib.stream())  # fmt: skip
     _lib.check(rc, "sb_glu")
     return out
+
+
+def rotary_table(positions: int, dims: int, base: float, device=None) -> torch.Tensor:
+    """fp32 ``[positions, dims]`` = cos | sin of ``p * base^(-2i / dims)`` for the dims / 2 pairs i (computed in fp64)."""
+    f = base ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)
+    angle = torch.arange(positions, dtype=torch.float64)[:, None] * f
+    return torch.cat([angle.cos(), angle.sin()], 1).float().to(device)
+
+
+def _turn(x, table, positions, interleaved):
+    half = table.shape[1] // 2
+    cos, sin = table[positions.long()][:, None].split(half, dim=-1)
+    pair = slice(0, 2 * half, 2), slice(1, 2 * half, 2)
+    if not interleaved:
+        pair = slice(0, half), slice(half, 2 * half)
+    out = x.clone()
+    u, v = x[..., pair[0]], x[..., pair[1]]
+    out[..., pair[0]], out[..., pair[1]] = u * cos - v * sin, v * cos + u * sin
+    return out
+
+
+def place_heads(q, k, v, slots, k_cache, v_cache, *, q_norm=None, k_norm=None, eps=0.0, table=None, positions=None, interleaved=True):
+    """New queries ``q`` [T, Hq * D], keys [T, Hkv * D] and values [T, Hkv * DV] (column ranges of a projection are fine): RMS norm
+    per query / key head (``q_norm`` / ``k_norm`` [D]; None: none), rotation by ``table`` (``rotary_table``; None: none) at
+    ``positions``. Queries are changed in place and returned [T, Hq, D]; keys and values go to cache slot ``slots[t]`` (< 0:
+    nowhere)."""
+    T, (Hkv, D), DV = q.shape[0], k_cache.shape[1:], v_cache.shape[2]
+    Hq = q.shape[1] // D
+    _checks.index_range("place_heads", "slots", slots, upper=k_cache.shape[0], lower=-(1 << 31))
+    if table is not None:
+        _checks.index_range("place_heads", "positions", positions, upper=table.shape[0])
+    if q_norm is None and table is None:
+        kv_scatter(k, v, slots, k_cache, v_cache)
+        return q.unflatten(1, (Hq, D))
+    if not q.is_cuda:
+        out = []
+        for x, w in ((q, q_norm), (k, k_norm)):
+            y = x.unflatten(1, (-1, D)).float()
+            y = y if w is None else _norm(y, w, eps, "rms")
+            out.append((y if table is None else _turn(y, table, positions, interleaved)).flatten(1).to(x.dtype))
+        q.copy_(out[0])
+        kv_scatter(out[1], v, slots, k_cache, v_cache)
+        return q.unflatten(1, (Hq, D))
+    assert q.stride(1) == k.stride(1) == v.stride(1) == 1 and q.dtype == k.dtype == v.dtype == k_cache.dtype == v_cache.dtype
+    assert k_cache.is_contiguous() and v_cache.is_contiguous() and (q_norm is None or q_norm.dtype == k_norm.dtype == q.dtype)
+    rc = _lib.lib().sb_heads(P(q), P(k), P(v), P(q_norm), P(k_norm), P(table), P(positions), P(slots), P(k_cache), P(v_cache), T, Hq, Hkv, D, DV,
+                             0 if table is None else table.shape[1], int(interleaved), q.stride(0), k.stride(0), v.stride(0), float(eps),
+                             int(q.dtype == torch.float32), _lib.stream())  # fmt: skip
+    _lib.check(rc, "sb_heads")
+    return q.unflatten(1, (Hq, D))
 
 
 def kv_scatter(k, v, slots, k_cache, v_cache):

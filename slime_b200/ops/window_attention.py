@@ -1,7 +1,8 @@
 """Windowed attention over the paged KV cache, for prompts (``window_extend``) and single tokens (``window_decode``).
 
 A query at position i sees key j when ``j <= i`` and (``i - j < window`` or ``j < keep_first``); its score is
-``scale * q.k - slope[head] * (i - j)`` (``slopes`` None: no distance term). Keys and values are read from the cache only,
+``scale * q.k - slope[head] * (i - j)`` (``slopes`` None: no distance term). ``sinks`` [Hq]: score of an extra softmax column
+without a value (None: no such column); ``out_scale`` multiplies the output, ``out`` may be a column range of a wider matrix. Keys and values are read from the cache only,
 so a prompt's later portions, portions of several requests and single tokens beside them are one launch.
 
 Dispatch on CUDA: bf16 with head widths that are multiples of 8 up to 128 run on the tensor cores
@@ -32,7 +33,8 @@ def tile_tokens(heads: int, kv_heads: int) -> int:
 class ExtendBatch:
     """Where the packed new tokens of a pass stand: row t belongs to request ``row_req[t]`` at position ``positions[t]``;
     request r's pages are ``block_table[r]``. ``starts`` / ``counts`` (host): first position and number of new tokens of
-    every request, from which the query tiles of a launch are cut."""
+    every request, from which the query tiles of a launch are cut. ``state_slots`` (host): slot of every request's recurrent
+    state, for models that have one."""
 
     block_table: torch.Tensor  # [requests, pages] int32
     row_req: torch.Tensor  # [T] int32
@@ -40,10 +42,11 @@ class ExtendBatch:
     starts: list[int]
     counts: list[int]
     page_size: int
+    state_slots: list[int] | None = None
     _tiles: dict = dataclasses.field(default_factory=dict)
 
     @classmethod
-    def build(cls, pages: list[list[int]], starts, counts, page_size: int, device, upload=None):
+    def build(cls, pages: list[list[int]], starts, counts, page_size: int, device, upload=None, state_slots=None):
         """``upload(ndarray) -> int32 device tensor``; default: a plain copy."""
         up = upload or (lambda a: torch.from_numpy(np.ascontiguousarray(a, dtype=np.int32)).to(device))
         width = max(len(p) for p in pages)
@@ -52,7 +55,8 @@ class ExtendBatch:
             table[r, : len(p)] = p
         req = np.repeat(np.arange(len(pages)), counts)
         pos = np.concatenate([np.arange(s, s + n) for s, n in zip(starts, counts)])
-        return cls(up(table), up(req), up(pos), [int(s) for s in starts], [int(n) for n in counts], page_size)
+        return cls(up(table), up(req), up(pos), [int(s) for s in starts], [int(n) for n in counts], page_size,
+                   state_slots)
 
     def tiles(self, tokens: int) -> torch.Tensor:
         """[n, 4] int32 (first row, tokens, first position, request) of query tiles of at most ``tokens`` tokens."""
@@ -68,8 +72,18 @@ class ExtendBatch:
             self._tiles[tokens] = host.to(self.row_req.device, non_blocking=True)
         return self._tiles[tokens]
 
+    def segments(self) -> torch.Tensor:
+        """[requests, 4] int32: first row, tokens, first position, state slot."""
+        if "segments" not in self._tiles:
+            first = np.concatenate([[0], np.cumsum(self.counts)[:-1]])
+            host = torch.from_numpy(np.stack([first, self.counts, self.starts, self.state_slots], 1).astype(np.int32))
+            if self.row_req.is_cuda:
+                host = host.pin_memory()
+            self._tiles["segments"] = host.to(self.row_req.device, non_blocking=True)
+        return self._tiles["segments"]
 
-def _reference(q, k_cache, v_cache, table, row_req, positions, page_size, scale, window, keep_first, slopes):
+
+def _reference(q, k_cache, v_cache, table, row_req, positions, page_size, scale, window, keep_first, slopes, sinks, out_scale):
     T, Hq, _ = q.shape
     Hkv, dv = k_cache.shape[1], v_cache.shape[2]
     out = torch.empty(T, Hq, dv, dtype=q.dtype)
@@ -86,7 +100,10 @@ def _reference(q, k_cache, v_cache, table, row_req, positions, page_size, scale,
         s = torch.einsum("tghd,jgd->tghj", qr, k) * scale
         if slopes is not None:
             s = s - slopes.view(1, Hkv, Hq // Hkv, 1) * dist[:, None, None, :].float()
-        p = s.masked_fill(~see[:, None, None, :], float("-inf")).softmax(-1)
+        s = s.masked_fill(~see[:, None, None, :], float("-inf"))
+        if sinks is not None:
+            s = torch.cat([s, sinks.view(1, Hkv, Hq // Hkv, 1).expand(len(rows), -1, -1, 1)], -1)
+        p = s.softmax(-1)[..., : len(j)] * out_scale
         out[rows] = torch.einsum("tghj,jgd->tghd", p, v).reshape(len(rows), Hq, dv).to(q.dtype)
     return out
 
@@ -97,18 +114,31 @@ def _tensor_core_shape(q, k_cache, v_cache, page_size) -> bool:
             and page_size in (16, 32, 64, 128))  # fmt: skip
 
 
-def _simt(q, k_cache, v_cache, table, row_req, positions, page_size, scale, window, keep_first, slopes, out):
+def _simt(q, k_cache, v_cache, table, row_req, positions, page_size, scale, window, keep_first, slopes, sinks, out_scale, out):
     T, Hq, D = q.shape
     rc = _lib.lib().sb_window_attn(
-        P(q), P(k_cache), P(v_cache), P(table), P(row_req), P(positions), P(slopes), P(out), T, Hq, k_cache.shape[1], D,
-        v_cache.shape[2], page_size, table.stride(0), q.stride(0), out.stride(0), float(scale), window, keep_first,
-        int(q.dtype == torch.float32), _lib.stream(),
+        P(q), P(k_cache), P(v_cache), P(table), P(row_req), P(positions), P(slopes), P(sinks), P(out), T, Hq, k_cache.shape[1], D,
+        v_cache.shape[2], page_size, table.stride(0), q.stride(0), out.stride(0), float(scale), float(out_scale), window,
+        keep_first, int(q.dtype == torch.float32), _lib.stream(),
     )  # fmt: skip
     _lib.check(rc, "sb_window_attn")
     return out
 
 
-def window_extend(q, k_cache, v_cache, batch: ExtendBatch, scale, window=None, keep_first=0, slopes=None):
+def _output(out, T, Hq, DV, q):
+    """[T, Hq, DV] view of ``out`` [T, Hq * DV], or a new tensor."""
+    if out is None:
+        return torch.empty(T, Hq, DV, dtype=q.dtype, device=q.device)
+    assert out.dtype == q.dtype and out.stride(1) == 1 and out.shape == (T, Hq * DV)
+    return out.unflatten(1, (Hq, DV))
+
+
+def _into(out, res):
+    return res if out is None else out.copy_(res.flatten(1)).unflatten(1, res.shape[1:])
+
+
+def window_extend(q, k_cache, v_cache, batch: ExtendBatch, scale, window=None, keep_first=0, slopes=None, sinks=None, out_scale=1.0,
+                  out=None):  # fmt: skip
     """Attention of the packed rows ``q`` [T, Hq, D] (a strided view is fine) -> [T, Hq, DV]. The rows' own keys and values
     must already be in the cache."""
     w = NO_WINDOW if window is None else int(window)
@@ -116,24 +146,26 @@ def window_extend(q, k_cache, v_cache, batch: ExtendBatch, scale, window=None, k
     Hkv, DV = k_cache.shape[1], v_cache.shape[2]
     _checks.index_range("window_extend", "block_table", batch.block_table, upper=k_cache.shape[0] // batch.page_size)
     if not q.is_cuda:
-        return _reference(q, k_cache, v_cache, batch.block_table, batch.row_req, batch.positions, batch.page_size, scale, w, keep_first, slopes)
+        return _into(out, _reference(q, k_cache, v_cache, batch.block_table, batch.row_req, batch.positions, batch.page_size, scale, w,
+                                     keep_first, slopes, sinks, out_scale))  # fmt: skip
     assert q.stride(2) == 1 and q.stride(1) == D and k_cache.is_contiguous() and v_cache.is_contiguous()
-    out = torch.empty(T, Hq, DV, dtype=q.dtype, device=q.device)
+    out = _output(out, T, Hq, DV, q)
     if _tensor_core_shape(q, k_cache, v_cache, batch.page_size):
         tiles = batch.tiles(tile_tokens(Hq, Hkv))
         rc = _lib.lib().sb_flash_window(
-            P(q), P(k_cache), P(v_cache), P(batch.block_table), P(tiles), P(slopes), P(out), tiles.shape[0], T, Hq, Hkv, D, DV,
-            batch.page_size, batch.block_table.stride(0), k_cache.shape[0], q.stride(0), out.stride(0), float(scale), w,
-            keep_first, P(_lib.status_word(q.device)), _lib.stream(),
+            P(q), P(k_cache), P(v_cache), P(batch.block_table), P(tiles), P(slopes), P(sinks), P(out), tiles.shape[0], T, Hq, Hkv, D, DV,
+            batch.page_size, batch.block_table.stride(0), k_cache.shape[0], q.stride(0), out.stride(0), float(scale),
+            float(out_scale), w, keep_first, P(_lib.status_word(q.device)), _lib.stream(),
         )  # fmt: skip
         if rc != -1:  # -1: an alignment the kernel does not take
             _lib.check(rc, "sb_flash_window")
             return out
-    return _simt(q, k_cache, v_cache, batch.block_table, batch.row_req, batch.positions, batch.page_size, scale, w, keep_first, slopes, out)
+    return _simt(q, k_cache, v_cache, batch.block_table, batch.row_req, batch.positions, batch.page_size, scale, w, keep_first, slopes, sinks,
+                 out_scale, out)  # fmt: skip
 
 
 def window_decode(q, k_cache, v_cache, block_table, seq_lens, positions, page_size, scale, window=None, keep_first=0, slopes=None,
-                  max_context: int | None = None):  # fmt: skip
+                  max_context: int | None = None, sinks=None, out_scale=1.0, out=None):  # fmt: skip
     """One query token per request: ``q`` [B, Hq, D] at ``positions`` = ``seq_lens - 1``, pages in ``block_table`` [B, W].
     Static shapes, nothing read on the host (``max_context``: upper bound of the lengths, from which the number of splits
     follows)."""
@@ -143,9 +175,10 @@ def window_decode(q, k_cache, v_cache, block_table, seq_lens, positions, page_si
     if _checks.enabled():
         _checks.paged("window_decode", block_table, seq_lens, page_size, k_cache.shape[0])
     if not q.is_cuda:
-        return _reference(q, k_cache, v_cache, block_table, None, positions, page_size, scale, w, keep_first, slopes)
+        return _into(out, _reference(q, k_cache, v_cache, block_table, None, positions, page_size, scale, w, keep_first, slopes, sinks,
+                                     out_scale))  # fmt: skip
     assert q.stride(2) == 1 and q.stride(1) == D and k_cache.is_contiguous() and v_cache.is_contiguous()
-    out = torch.empty(B, Hq, DV, dtype=q.dtype, device=q.device)
+    out = _output(out, B, Hq, DV, q)
     if _tensor_core_shape(q, k_cache, v_cache, page_size) and Hq // Hkv <= 16:
         from slime_b200 import ops
 
@@ -159,11 +192,11 @@ def window_decode(q, k_cache, v_cache, block_table, seq_lens, positions, page_si
         part = torch.empty(B * Hq * splits * (wd + 2), dtype=torch.float32, device=q.device) if splits > 1 else None
         ml = part[B * Hq * splits * wd :] if splits > 1 else None
         rc = _lib.lib().sb_paged_decode_window(
-            P(q), P(k_cache), P(v_cache), P(block_table), P(seq_lens), P(slopes), P(out), P(part), P(ml), B, Hq, Hkv, D, DV, page_size,
-            block_table.stride(0), k_cache.shape[0], q.stride(0), out.stride(0), splits, float(scale), w, keep_first,
-            P(_lib.status_word(q.device)), _lib.stream(),
+            P(q), P(k_cache), P(v_cache), P(block_table), P(seq_lens), P(slopes), P(sinks), P(out), P(part), P(ml), B, Hq, Hkv, D, DV, page_size,
+            block_table.stride(0), k_cache.shape[0], q.stride(0), out.stride(0), splits, float(scale), float(out_scale), w,
+            keep_first, P(_lib.status_word(q.device)), _lib.stream(),
         )  # fmt: skip
         if rc != -1:
             _lib.check(rc, "sb_paged_decode_window")
             return out
-    return _simt(q, k_cache, v_cache, block_table, None, positions, page_size, scale, w, keep_first, slopes, out)
+    return _simt(q, k_cache, v_cache, block_table, None, positions, page_size, scale, w, keep_first, slopes, sinks, out_scale, out)

@@ -126,7 +126,7 @@ def test_hybrid_engine_carries_recurrent_state_through_chunked_prefill_and_batch
                                max_prefill_tokens=7), device="cpu", num_pages=64)  # fmt: skip
     hf = [x for n, p in model.named_parameters() for x in convert.convert_to_hf(cfg, n, p.detach())]
     assert not e.weights.load_weights(hf)
-    assert e.kv.num_layers == 2 and e.runner.has_gdn  # two of the four layers keep keys and values
+    assert e.kv.num_layers == 2 and e.runner.recurrent  # two of the four layers keep keys and values
     g = torch.Generator().manual_seed(2)
     prompts = [torch.randint(0, cfg.vocab_size, (n,), generator=g).tolist() for n in (13, 3, 9)]
     reqs = e.generate(prompts, [dict(max_new_tokens=5 + i, temperature=0, ignore_eos=True) for i in range(3)])
