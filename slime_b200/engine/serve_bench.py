@@ -5,8 +5,9 @@
 Random weights, one GPU, bf16. ``prefill``: one extend pass over packed fresh prompts (logits of the last row of each), tokens
 per second. ``decode``: replays of the captured decode step (sampling included) at a fixed batch and context, tokens per
 second. Device time by CUDA events around exactly K passes after W warm-up ones; the weights and the cache a pass streams are
-several times the L2. Both models of a pair have the same widths, head counts, layer count and vocabulary; at the context of
-``window`` tokens they also read the same keys. Prints one JSON line.
+several times the L2. The models of a Pefolix pair have the same widths, head counts, layer count and vocabulary; at the context of
+``window`` tokens they also read the same keys. A Ledazen pair has the same width, heads, layers and vocabulary; its feed-forward
+width is chosen for an equal number of weights in the layers. Prints one JSON line.
 """
 
 from __future__ import annotations
@@ -20,7 +21,7 @@ from slime_b200.engine.engine import Engine
 from slime_b200.engine.request import Request
 from slime_b200.engine.server_args import ServerArgs
 from slime_b200.models.config import ModelConfig, get_preset
-from slime_b200.models.presets import _pefolix
+from slime_b200.models.presets import _ledazen, _pefolix
 
 LAYERS = 8  # of the 24 to 36 layers of the models the widths are taken from: per-layer cost is what is compared
 
@@ -35,7 +36,16 @@ def _pairs() -> dict[str, tuple[ModelConfig, ModelConfig]]:
                       vocab_size=151936, rotary_base=1e6, tie_word_embeddings=False, qk_layernorm=True, num_experts=128,
                       moe_ffn_hidden_size=768, moe_router_topk=8, moe_layer_freq=[0, 1] * (LAYERS // 2),
                       moe_shared_expert_intermediate_size=768, moe_shared_expert_gate=True, model_arch="Qwen3MoeForCausalLM")  # fmt: skip
+    # delta-net layers with attention in every fourth, against attention beside the delta rule in every fourth
+    hybrid = ModelConfig(num_layers=LAYERS, hidden_size=2560, num_attention_heads=32, num_query_groups=8, kv_channels=128, ffn_hidden_size=9216,
+                         vocab_size=151936, rotary_base=1e6, tie_word_embeddings=False, qk_layernorm=True, full_attention_interval=4,
+                         linear_num_key_heads=16, linear_num_value_heads=32, linear_key_head_dim=128, linear_value_head_dim=128,
+                         model_arch="Qwen3_5ForCausalLM")  # fmt: skip
+    llama = get_preset("llama-3.2-1b")
+    llama.num_layers, llama.tie_word_embeddings = LAYERS, False
     return {
+        "ledazen-hybrid": (ModelConfig(**_ledazen("dddp" * (LAYERS // 4), 2560, 32, 8, 128, 11776, 151936, 32, 16, 128, 128, 128, 65521)), hybrid),
+        "ledazen-d64": (ModelConfig(**_ledazen("p" * LAYERS, 2048, 32, 8, 64, 9984, 128256, 16, 16, 64, 64, 64, 32749)), llama),
         "d128-dense": (ModelConfig(**_pefolix(LAYERS, 2560, 32, 8, 128, 1024, 8, 9728, 151936)), dense),
         "d64-dense": (ModelConfig(**_pefolix(LAYERS, 2048, 32, 8, 64, 1024, 8, 8192, 128256)), small),
         "d128-moe": (ModelConfig(**_pefolix(LAYERS, 2048, 32, 4, 128, 1024, 8, 6144, 151936, every=2, experts=128, top=8, expert_ff=768,

@@ -170,6 +170,24 @@ MORE_PRESETS["pefolix-4b"] = _pefolix(36, 2560, 32, 8, 128, 1024, 8, 9728, 15193
 MORE_PRESETS["pefolix-a3b"] = _pefolix(24, 2048, 32, 4, 128, 1024, 8, 6144, 151936, every=2, experts=128, top=8, expert_ff=768, shared_ff=768)
 MORE_PRESETS["pefolix-tiny"] = _pefolix(3, 96, 4, 2, 32, 24, 3, 160, 512, every=3, experts=6, top=2, expert_ff=48, shared_ff=40)
 
+def _ledazen(kinds: str, hidden: int, heads: int, kv_heads: int, dim: int, ff: int, vocab: int, rule_heads: int, rule_kv_heads: int, rule_dim: int,
+             rule_vdim: int, rank: int, buckets: int) -> dict:  # fmt: skip
+    """A Ledazen stack: one letter per layer, "d" the delta rule alone, "p" attention beside it."""
+    from slime_b200.models.layer_spec import AttentionSpec, DeltaSpec, FeedForwardSpec, LayerSpec, ParallelSpec, RotarySpec, flat_sizes
+
+    sizes = (rule_heads, rule_kv_heads, rule_dim, rule_vdim, 4)
+    left = AttentionSpec(heads, kv_heads, dim, dim, dim**-0.5, qk_norm=True, rot=RotarySpec(dim, 1e6), sink=0.0)
+    both = ParallelSpec(left, DeltaSpec(*sizes, "channel", "sigmoid", rank, rank), 0.5, 0.5)
+    specs = [LayerSpec(both if k == "p" else DeltaSpec(*sizes), FeedForwardSpec(ff, "relu2", gated=False), parallel_ff=True) for k in kinds]
+    return dict(flat_sizes(specs), layer_specs=specs, hidden_size=hidden, vocab_size=vocab, norm_epsilon=1e-5, norm_offset=1.0,
+                bigram=dict(buckets=buckets, mul_prev=1000003, mul_cur=8191), tie_word_embeddings=False, model_arch="Ledazen")  # fmt: skip
+
+
+# Ledazen at the sizes of the dense and hybrid presets above (random weights: there is no published checkpoint)
+MORE_PRESETS["ledazen-4b"] = _ledazen("dddp" * 9, 2560, 32, 8, 128, 10240, 151936, 32, 16, 128, 128, 128, 65521)
+MORE_PRESETS["ledazen-1b"] = _ledazen("pp" * 8, 2048, 32, 8, 64, 6144, 128256, 16, 16, 64, 64, 64, 32749)
+MORE_PRESETS["ledazen-tiny"] = _ledazen("pd" * 2, 96, 4, 2, 24, 160, 512, 4, 2, 24, 16, 8, 61)
+
 # name -> what is missing. The numbers of these families are in the recipes they come from; they are not repeated here
 # because a preset that cannot be instantiated correctly is worse than none.
 UNSUPPORTED: dict[str, str] = {}

@@ -444,6 +444,104 @@ def bench_window(a):
     _lib.check_status("cuda")
 
 
+def bench_delta(a):
+    """Kernels of recurrent layers beside the torch ops of the trainer's delta-net layer (the form the engine used for it), and
+    the other kernels of Ledazen layers beside their nearest relatives. Fractions of the copy bandwidth."""
+    from slime_b200.models import mixers
+    from slime_b200.ops import delta, stream
+    from slime_b200.ops import window_attention as wa
+
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    gbs, _ = _peaks()
+    rnd = lambda *s, dt=bf: torch.randn(*s, device=dev).to(dt)  # noqa: E731
+
+    def emit(what, t, t2, mb, **kw):
+        _emit(kind=what, us=round(t * 1e3, 2), of_peak=round(mb / t / gbs, 4), like_us=None if t2 is None else round(t2 * 1e3, 2), **kw)
+
+    for H, G, D, DV, pc in ((32, 16, 128, 128, False), (32, 16, 128, 128, True), (16, 16, 64, 64, True)):
+        C = 2 * G * D + H * DV
+        conv, rate, bias, w = rnd(C, 4), torch.randn(H, device=dev), torch.randn(H * D if pc else H, device=dev) - 3, rnd(DV)
+        tag = dict(heads=H, qk_heads=G, dim=D, vdim=DV, per_channel=pc)
+
+        def inputs(T):
+            x, ab, z = rnd(T, C), rnd(T, bias.numel() + 64), rnd(T, H * DV)
+            q, k, v = x.split([G * D, G * D, H * DV], 1)
+            return x, z, delta.DeltaInputs(q, k, v, ab[:, : bias.numel()], ab[:, bias.numel() : bias.numel() + H], conv, rate, bias)
+
+        for n, L in ((8, 1024), (2, 4096)) if not a.small else ((8, 1024),):
+            T = n * L
+            x, z, inp = inputs(T)
+            state, ring = torch.zeros(n, H, D, DV, device=dev), rnd(n, 4, C)
+            batch = wa.ExtendBatch.build([[0]] * n, [0] * n, [L] * n, 8192, dev, state_slots=list(range(n)))
+            out = rnd(T, H * DV)
+            prof = {}
+
+            def new():
+                o = delta.delta_extend(inp, state, ring, batch)
+                delta.head_gate(o, z, w, "silu", 1e-5, 1.0, out)
+                prof["o"] = o
+
+            t = time_ms(new, a.iters)
+            cu = torch.arange(0, T + 1, L, device=dev, dtype=torch.int32)
+            pos = torch.arange(T, device=dev) % L
+
+            def old():
+                y = mixers.causal_short_conv(x, conv, pos)
+                q, k, v = y.split([G * D, G * D, H * DV], -1)
+                q, k = (s.view(T, G, D).repeat_interleave(H // G, 1) for s in (q, k))
+                g = -rate.exp() * torch.nn.functional.softplus(inp.a.float() + bias)
+                o = mixers.gated_delta_rule_chunked(q, k, v.view(T, H, DV), g, torch.sigmoid(inp.b.float()), cu)
+                (mixers._rms(o, w, 1e-5).float() * torch.nn.functional.silu(z.view(T, H, DV).float())).to(bf)
+
+            t2 = None if pc else time_ms(old, 3)  # the torch form has no decay per key channel
+            mb = T * 2 * (C + 2 * H * DV + bias.numel() + H) / 1e6 + n * H * D * DV * 4 / 1e6
+            emit("delta_extend", t, t2, mb, tokens=T, requests=n, **tag)
+            o = prof["o"]
+            t = time_ms(lambda: delta.head_gate(o, z, w, "silu", 1e-5, 1.0, out), a.iters)
+            emit("head_gate", t, None, T * H * DV * 8 / 1e6, tokens=T, **tag)
+        for B in (64, 4):
+            x, z, inp = inputs(B)
+            state, ring = torch.zeros(4 * 64, H, D, DV, device=dev), rnd(4 * 64, 4, C)  # rotating slots: states come from memory
+            i32 = lambda v: torch.as_tensor(v, dtype=torch.int32, device=dev)  # noqa: E731
+            sets = [i32(range(j * B, (j + 1) * B)) for j in range(4 * 64 // B)]
+            one, at, turn, out = i32([1] * B), i32([77] * B), [0], rnd(B, H * DV)
+
+            def new():
+                turn[0] = (turn[0] + 1) % len(sets)
+                delta.delta_step(inp, state, ring, sets[turn[0]], one, at, z, w, "silu", 1e-5, 1.0, out)
+
+            S, hist = torch.zeros(B, H, D, DV, device=dev), rnd(B, 3, C)
+
+            def old():
+                y = mixers.short_conv_step(x, conv, hist)
+                q, k, v = y.split([G * D, G * D, H * DV], -1)
+                q, k = (s.view(B, G, D).repeat_interleave(H // G, 1) for s in (q, k))
+                g = -rate.exp() * torch.nn.functional.softplus(inp.a.float() + bias)
+                o = mixers.gated_delta_rule_step(q, k, v.view(B, H, DV), g, torch.sigmoid(inp.b.float()), S)
+                (mixers._rms(o.to(bf), w, 1e-5).float() * torch.nn.functional.silu(z.view(B, H, DV).float())).to(bf)
+
+            t, t2 = time_ms(new, a.iters), None if pc else time_ms(old, a.iters)
+            emit("delta_step", t, t2, B * (H * D * DV * 8 + C * 10 + H * DV * 4) / 1e6, rows=B, **tag)
+    for T in (8192, 64):
+        kv, slots = rnd(T, 48 * 128), torch.randperm(T, device=dev).to(torch.int32)
+        kc, vc = rnd(T, 8, 128), rnd(T, 8, 128)
+        pos, qn = torch.arange(T, dtype=torch.int32, device=dev), rnd(128)
+        table = stream.rotary_table(T, 128, 1e6, dev)
+        t = time_ms(lambda: stream.place_heads(kv[:, :4096], kv[:, 4096:5120], kv[:, 5120:], slots, kc, vc, q_norm=qn, k_norm=qn, eps=1e-6,
+                                               table=table, positions=pos), a.iters)  # fmt: skip
+        t2 = time_ms(lambda: ops.rope_kv_write(kv, pos, table, slots, kc, vc, 32, 8, 128, qn, qn, 1e-6), a.iters)
+        emit("heads_to_cache", t, t2, T * (40 * 128 * 4 + 8 * 128 * 4) / 1e6, rows=T)
+        y, res, r16, w = torch.randn(T, 2560, device=dev), torch.randn(T, 2560, device=dev), rnd(T, 2560), rnd(2560)
+        t = time_ms(lambda: stream.stream_norm(y, res, w, 1e-5, offset=1.0), a.iters)
+        t2 = time_ms(lambda: ops.rmsnorm(y, w, 1e-6, r16), a.iters)
+        emit("stream_norm", t, t2, T * 2560 * 14 / 1e6, rows=T, like_of_peak=round(T * 2560 * 10 / 1e6 / t2 / gbs, 4))
+        up, out, gu = rnd(T, 10240 + 256), rnd(T, 10240 + 4096), rnd(T, 2 * 6912)
+        t = time_ms(lambda: stream.feed_forward_act(up[:, 256:], "relu2", False, out[:, 4096:]), a.iters)
+        t2 = time_ms(lambda: ops.swiglu(gu), a.iters)
+        emit("activation", t, t2, T * 10240 * 4 / 1e6, rows=T, like_of_peak=round(T * 6912 * 6 / 1e6 / t2 / gbs, 4))
+    _lib.check_status("cuda")
+
+
 def bench_fused_emul(a):
     """The peer-memory kernels with every "rank" a buffer of THIS GPU (profilers attach to one process on one GPU, and
     kernels that wait on one another must not run as separate launches on one device): the data path, instruction mix
@@ -500,7 +598,7 @@ def bench_fused_emul(a):
 
 def main(argv=None):
     p = argparse.ArgumentParser(prog="python -m slime_b200.ops.microbench")
-    p.add_argument("what", choices=["gemm", "decode", "norm", "fp8", "moe", "attn", "window", "fused_emul"])
+    p.add_argument("what", choices=["gemm", "decode", "norm", "fp8", "moe", "attn", "window", "delta", "fused_emul"])
     p.add_argument("--iters", type=int, default=20)
     p.add_argument("--reps", type=int, default=20, help="back-to-back launches per timed repetition (decode)")
     p.add_argument("--small", action="store_true")
@@ -514,7 +612,7 @@ def main(argv=None):
     from slime_b200.ops import build
 
     build.build()
-    {"gemm": bench_gemm, "decode": bench_decode, "norm": bench_norm, "fp8": bench_fp8, "moe": bench_moe, "attn": bench_attn, "window": bench_window, "fused_emul": bench_fused_emul}[a.what](a)
+    {"gemm": bench_gemm, "decode": bench_decode, "norm": bench_norm, "fp8": bench_fp8, "moe": bench_moe, "attn": bench_attn, "window": bench_window, "delta": bench_delta, "fused_emul": bench_fused_emul}[a.what](a)
 
 
 if __name__ == "__main__":

@@ -156,3 +156,98 @@ def error(got, want):
     d = got.double() - want.double()
     d = d - d.mean(-1, keepdim=True)
     return float((d.pow(2).mean(-1).sqrt() / want.double().std()).max())
+
+
+# ------------------------------------------------------------------------------- models for the tests
+def attn(heads, kv_heads, dim, vdim, dims, base=1e4, scale=None):
+    return dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, rot=dict(dims=dims, base=base), scale=scale if scale is not None else dim**-0.5)
+
+
+def rule(heads, kv_heads, dim, vdim, conv):
+    return dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, conv=conv)
+
+
+def both(left, right, left_scale=0.8, right_scale=0.7):
+    return dict(left=left, right=right, left_scale=left_scale, right_scale=right_scale)
+
+
+def model(width, vocab, bigram, layers, eps=1e-5):
+    """``bigram``: (buckets, mul_prev, mul_cur); ``layers``: (mixer, width of the feed-forward or None)."""
+    return dict(architecture="Ledazen", width=width, vocab=vocab, norm=dict(eps=eps),
+                embedding=dict(bigram=dict(zip(("buckets", "mul_prev", "mul_cur"), bigram))),
+                layers=[dict(type="parallel" if "left" in m else "delta", mixer=m, mlp=None if ff is None else dict(kind="dense", ff=ff))
+                        for m, ff in layers])  # fmt: skip
+
+
+CONFIGS = {
+    # layers of different geometry and order, layers without a feed-forward, partial rotation, several groupings and taps
+    "mixed": model(96, 203, (41, 13, 5), [
+        (both(attn(6, 2, 32, 24, 20, scale=0.4), rule(6, 3, 24, 40, 4)), 80), (rule(4, 2, 16, 40, 3), None),
+        (rule(6, 1, 40, 16, 5), 56), (both(attn(5, 5, 16, 48, 16, 5e5), rule(2, 2, 40, 8, 2), 1.3, -0.4), None)], eps=3e-4),
+    # equal attention heads (one cache slab), one tap: no convolution state
+    "equal": model(64, 128, (64, 3, 1), [(both(attn(4, 1, 32, 32, 32), rule(2, 1, 16, 32, 1)), 96),
+                                         (both(attn(4, 1, 32, 32, 32), rule(4, 4, 32, 16, 4)), 64)]),
+    # widths that no 16-byte copy divides
+    "odd": model(90, 77, (23, 7, 11), [(rule(3, 3, 10, 14, 4), 50), (both(attn(6, 3, 10, 22, 6), rule(3, 1, 9, 7, 3), 0.5, 1.0), 45)], eps=1e-3),
+    # one head of each kind; eps large enough to matter
+    "single": model(40, 33, (9, 2, 3), [(both(attn(1, 1, 16, 48, 4, 100.0), rule(1, 1, 16, 24, 6), 1.0, 1.0), 24)], eps=0.1),
+    # no attention: nothing is kept per token
+    "rules": model(48, 60, (31, 5, 7), [(rule(2, 1, 24, 24, 4), 40), (rule(3, 3, 16, 32, 2), None)]),
+}  # fmt: skip
+
+
+def random_tensors(config, seed=0, sharp=2.5, dtype=torch.float32):
+    """Random weights under the checkpoint's names. ``sharp`` scales the query and key norms, so that single keys dominate
+    the softmax; decays are close to one, so that old writes are still read."""
+    g = torch.Generator().manual_seed(seed)
+    D, out, b = config["width"], {}, config["embedding"]["bigram"]
+
+    def rand(*s, gain=1.0, mean=0.0):
+        return torch.randn(*s, generator=g) * gain + mean
+
+    def mat(name, rows, cols, gain=1.0):
+        out[name] = rand(rows, cols, gain=gain * cols**-0.5)
+
+    out["embed"], out["bigram"] = rand(config["vocab"], D, mean=0.3), rand(b["buckets"] + 1, D)
+    for i, layer in enumerate(config["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        out[p + "norm1"] = rand(D, gain=0.3)
+        if layer["type"] == "parallel":
+            a, q = m["left"], p + "mix.left."
+            mat(q + "q", a["heads"] * a["dim"], D)
+            mat(q + "k", a["kv_heads"] * a["dim"], D)
+            mat(q + "v", a["kv_heads"] * a["vdim"], D)
+            mat(q + "o", D, a["heads"] * a["vdim"])
+            for n in "qk":
+                out[f"{q}{n}.norm"] = rand(a["dim"], gain=0.3, mean=1.0) * sharp**0.5
+        r, q = (m["right"], p + "mix.right.") if layer["type"] == "parallel" else (m, p + "mix.")
+        H, dv = r["heads"], r["vdim"]
+        for n, rows in (("q", r["kv_heads"] * r["dim"]), ("k", r["kv_heads"] * r["dim"]), ("v", H * dv)):
+            mat(q + n, rows, D)
+            out[f"{q}{n}.conv"] = rand(rows, r["conv"], gain=0.6)
+        mat(q + "b", H, D)
+        out[q + "A_log"], out[q + "norm"] = rand(H, gain=0.5), rand(dv, gain=0.3, mean=1.0)
+        if layer["type"] == "parallel":
+            for n, rows, rank in (("a", H * r["dim"], 5 + i), ("g", H * dv, 11 - i)):  # inner widths are a matter of the tensors
+                mat(f"{q}{n}1", rank, D)
+                mat(f"{q}{n}2", rows, rank)
+            out[q + "dt_bias"] = rand(H * r["dim"], mean=-3.5)
+        else:
+            mat(q + "a", H, D)
+            mat(q + "g", H * dv, D)
+            out[q + "dt_bias"] = rand(H, mean=-3.5)
+        mat(q + "o", D, H * dv)
+        if layer["mlp"] is not None:
+            mat(p + "mlp.up", layer["mlp"]["ff"], D)
+            mat(p + "mlp.down", D, layer["mlp"]["ff"], 0.7)
+    out["final.norm"] = rand(D, gain=0.3)
+    mat("head", config["vocab"], D)
+    return {k: v.to(dtype) for k, v in out.items()}
+
+
+def shapes(tensors):
+    return {k: tuple(v.shape) for k, v in tensors.items()}
+
+
+def random_tokens(config, n, seed=0):
+    return torch.randint(0, config["vocab"], (n,), generator=torch.Generator().manual_seed(seed)).tolist()
