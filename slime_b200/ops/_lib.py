@@ -39,7 +39,7 @@ _SIGS = {
     "sb_stream_norm": [P, I, P, I, P, P, I, P, P, I, P, P, I, P, P, I, I, I, F, F, I, P, P, P, L, L, I, P],
     "sb_glu": [P, P, P, L, I, L, L, I, I, P],
     "sb_heads": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, L, L, L, F, I, P],
-    "sb_kv_scatter": [P, P, P, P, P, I, I, L, L, P],
+    "sb_kv_scatter": [P, P, P, P, P, I, I, I, L, L, P],
     "sb_gemm_simt": [P, P, P, P, P, I, I, I, L, L, L, I, I, P],
     "sb_window_attn": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, L, L, F, F, I, I, I, P],
     "sb_flash_window": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, L, L, F, F, I, I, P, P],
