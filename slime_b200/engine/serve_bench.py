@@ -71,8 +71,16 @@ def _place(e: Engine, lengths: list[int]) -> list[Request]:
     for i, n in enumerate(lengths):
         r = Request(rid=str(i), input_ids=[(7 * i + j) % 1000 for j in range(n)], sampling=None)
         r.ctx_ids, r.pages = r.input_ids, e.kv.allocator.alloc(-(-n // e.page_size))
+        if e.states is not None:
+            r.state_slot = e.states.take()
         out.append(r)
     return out
+
+
+def _give_back(e: Engine, reqs: list[Request]):
+    for r in reqs:
+        e.kv.allocator.release(r.pages)
+        e._give_state(r)
 
 
 def _prefill_ms(e: Engine, lengths: list[int], steps: int, warmup: int) -> float:
@@ -83,8 +91,7 @@ def _prefill_ms(e: Engine, lengths: list[int], steps: int, warmup: int) -> float
     extend = e._extend_batch(batch) if e.runner.layered or e.runner.recurrent else None
     prev = e._to_dev(p.prev) if e.cfg.bigram else None
     ms = _timed(lambda: e.runner.prefill(*dev_in, p.max_q, p.max_k, rows, True, prev=prev, extend=extend), steps, warmup)
-    for r, _ in batch:
-        e.kv.allocator.release(r.pages)
+    _give_back(e, [r for r, _ in batch])
     return ms
 
 
@@ -95,13 +102,14 @@ def _decode_ms(e: Engine, batch: int, context: int, steps: int, warmup: int) -> 
     for b, r in enumerate(reqs):
         h["active"][b], h["init_mask"][b], h["init_ids"][b], h["init_pos"][b] = 1, 1, 5, context
         h["block_table"][b, : len(r.pages)] = r.pages
+        h["state_slot"][b] = r.state_slot or 0
     e.runner.upload_static()
     e.runner.decode(batch, False)
     e.runner.upload_static()  # init records are consumed: from here on the device advances the slots itself
     ms = _timed(lambda: e.runner.decode(batch, False), steps, warmup)
-    for b, r in enumerate(reqs):
+    for b in range(batch):
         e._deactivate(b)
-        e.kv.allocator.release(r.pages)
+    _give_back(e, reqs)
     return ms
 
 
