@@ -117,10 +117,169 @@ delta_prep_kernel(const __grid_constant__ DeltaIn a, const int4* __restrict__ ru
   }
 }
 
+// V adjacent elements as floats, and back.
+template <int V>
+__device__ __forceinline__ void dr_load_v(const float* p, float (&f)[V]) {
+  if constexpr (V == 4) {
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    f[0] = x.x; f[1] = x.y; f[2] = x.z; f[3] = x.w;
+  } else {
+    const float2 x = *reinterpret_cast<const float2*>(p);
+    f[0] = x.x; f[1] = x.y;
+  }
+}
+template <int V>
+__device__ __forceinline__ void dr_load_v(const __nv_bfloat16* p, float (&f)[V]) {
+  if constexpr (V == 4) {
+    const uint2 x = *reinterpret_cast<const uint2*>(p);
+    const float2 a = unpack_bf16x2(x.x), b = unpack_bf16x2(x.y);
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  } else {
+    const float2 a = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(p));
+    f[0] = a.x; f[1] = a.y;
+  }
+}
+template <int V>
+__device__ __forceinline__ void dr_store_v(float* p, const float (&f)[V]) {
+  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  else *reinterpret_cast<float2*>(p) = make_float2(f[0], f[1]);
+}
+template <int V>
+__device__ __forceinline__ void dr_store_v(__nv_bfloat16* p, const float (&f)[V]) {
+  if constexpr (V == 4) *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]));
+  else *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(f[0], f[1]);
+}
+// Activations of projections may be as exact as their storage: bf16 results take the fast exponential.
+template <typename T>
+__device__ __forceinline__ float dr_act(float z) {
+  if constexpr (sizeof(T) == 2) return __fdividef(z, 1.f + __expf(-z));
+  return dr_silu(z);
+}
+
+// Convolution of V adjacent channels of one projection, token after token, its last inputs in registers.
+template <typename T, int V>
+struct ConvLine {
+  static constexpr int TAPS = 4;
+  float w[TAPS][V], past[TAPS - 1][V];
+  const T* x;
+
+  __device__ __forceinline__ void start(const DeltaIn& a, const void* proj, int col, const T* ring, int c, int pos, const int4& seg, bool on) {
+    const int taps = a.taps, C = 2 * a.G * a.D + a.H * a.DV;
+    const T* conv = reinterpret_cast<const T*>(a.conv) + static_cast<long>(c) * taps;
+    x = reinterpret_cast<const T*>(proj) + col;
+#pragma unroll
+    for (int s = 0; s < TAPS; ++s) {
+      const int at = pos - s;
+#pragma unroll
+      for (int i = 0; i < V; ++i) {
+        w[s][i] = (on && s < taps) ? dr_load(conv + i * taps + taps - 1 - s) : 0.f;
+        if (s > 0) past[s > 0 ? s - 1 : 0][i] = 0.f;
+      }
+      if (s > 0 && on && s < taps && at >= 0)
+        dr_load_v<V>(at >= seg.z ? x + (static_cast<long>(seg.x) + at - seg.z) * a.pitch : ring + static_cast<long>(at % taps) * C + c,
+                     past[s > 0 ? s - 1 : 0]);
+    }
+  }
+  __device__ __forceinline__ void next(const DeltaIn& a, long row, bool on, float (&y)[V]) {
+    float cur[V];
+#pragma unroll
+    for (int i = 0; i < V; ++i) cur[i] = 0.f;
+    if (on) dr_load_v<V>(x + row * a.pitch, cur);
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      float t = w[0][i] * cur[i];
+#pragma unroll
+      for (int s = 1; s < TAPS; ++s) t = fmaf(w[s][i], past[s - 1][i], t);
+      y[i] = dr_act<T>(t);
+#pragma unroll
+      for (int s = TAPS - 2; s > 0; --s) past[s][i] = past[s - 1][i];
+      past[0][i] = cur[i];
+    }
+  }
+};
+
+// The usual sizes: heads of at most 32 V channels, at most 4 taps, everything aligned for V-wide accesses.
+template <typename T, int V>
+__global__ void __launch_bounds__(128)
+delta_prep_wide_kernel(const __grid_constant__ DeltaIn a, const int4* __restrict__ runs, const int4* __restrict__ segs,
+                       float* __restrict__ q_out, float* __restrict__ k_out, float* __restrict__ v_out, float* __restrict__ g_out,
+                       float* __restrict__ beta_out, float* __restrict__ qk_out) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int lane = threadIdx.x & 31, vec = blockIdx.y * 4 + (threadIdx.x >> 5);
+  if (vec >= a.G + 2 * a.H) return;
+  const int4 run = runs[blockIdx.x], seg = segs[run.w];
+  const int H = a.H, G = a.G, D = a.D, DV = a.DV, d = lane * V;
+  const T* ring = reinterpret_cast<const T*>(a.ring) + static_cast<long>(seg.w) * a.taps * (2 * G * D + H * DV);
+  if (vec < G) {
+    const bool on = d < D;
+    ConvLine<T, V> lq, lk;
+    lq.start(a, a.q, vec * D + d, ring, vec * D + d, run.z, seg, on);
+    lk.start(a, a.k, vec * D + d, ring, (G + vec) * D + d, run.z, seg, on);
+    const float dim = 1.f / sqrtf(static_cast<float>(D));
+    for (int i = 0; i < run.y; ++i) {
+      const long row = run.x + i;
+      float q[V], k[V], qq = 0.f, kk = 0.f, qk = 0.f;
+      lq.next(a, row, on, q);
+      lk.next(a, row, on, k);
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        qq = fmaf(q[j], q[j], qq);
+        kk = fmaf(k[j], k[j], kk);
+        qk = fmaf(q[j], k[j], qk);
+      }
+      const float rq = dim / sqrtf(warp_sum(qq) + 1e-6f), rk = 1.f / sqrtf(warp_sum(kk) + 1e-6f);
+      qk = warp_sum(qk) * rq * rk;
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        q[j] *= rq;
+        k[j] *= rk;
+      }
+      if (on) {
+        dr_store_v<V>(q_out + (row * G + vec) * D + d, q);
+        dr_store_v<V>(k_out + (row * G + vec) * D + d, k);
+      }
+      if (lane == 0) qk_out[row * G + vec] = qk;
+    }
+  } else if (vec < G + H) {
+    const int h = vec - G;
+    const bool on = d < DV;
+    ConvLine<T, V> lv;
+    lv.start(a, a.v, h * DV + d, ring, 2 * G * D + h * DV + d, run.z, seg, on);
+    if (lane < run.y) beta_out[(run.x + lane) * H + h] = dr_sigmoid(dr_load(reinterpret_cast<const T*>(a.b) + (static_cast<long>(run.x) + lane) * a.b_pitch + h));
+    for (int i = 0; i < run.y; ++i) {
+      const long row = run.x + i;
+      float v[V];
+      lv.next(a, row, on, v);
+      if (on) dr_store_v<V>(v_out + (row * H + h) * DV + d, v);
+    }
+  } else {
+    const int h = vec - G - H;
+    const float rate = expf(a.A_log[h]);
+    const T* ap = reinterpret_cast<const T*>(a.a);
+    if (!a.per_channel) {
+      const long row = run.x + lane;
+      if (lane < run.y) g_out[row * H + h] = dr_decay(rate, dr_load(ap + row * a.a_pitch + h) + a.dt_bias[h]);
+    } else if (d < D) {
+      float bias[V];
+      dr_load_v<V>(a.dt_bias + h * D + d, bias);
+      for (int i = 0; i < run.y; ++i) {
+        const long row = run.x + i;
+        float z[V];
+        dr_load_v<V>(ap + row * a.a_pitch + h * D + d, z);
+#pragma unroll
+        for (int j = 0; j < V; ++j) z[j] = dr_decay(rate, z[j] + bias[j]);
+        dr_store_v<V>(g_out + (row * H + h) * D + d, z);
+      }
+    }
+  }
+}
+
 // ------------------------------------------------------------------------------------------------ recurrence over rows
-// A warp holds 8 columns of S: lane = column group (4) x row group (8); a lane has 2 columns and the rows
+// A warp holds 4 CPT columns of S: lane = column group (4) x row group (8); a lane has CPT columns and the rows
 // {4 rg + 32 j + 0..3}. Both products with S are taken before u is known (o = (g S)^T q + u (k.q)), so a token costs one
-// round of shuffles. q, k, g, v of the next tokens are copied to shared memory while the current ones are processed.
+// round of shuffles. q, k, g, v of the next tokens are copied to shared memory while the current ones are processed. More columns
+// per lane mean fewer reads of q, k, g from shared memory (the bound of a full machine), fewer mean more warps (few requests).
 constexpr int DS_TOK = 8;  // tokens per copy
 
 __device__ __forceinline__ void ds_copy16(void* dst, const void* src) {
@@ -143,25 +302,33 @@ __device__ __forceinline__ float2 ds_mul2(float2 a, float2 b) {
   asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r.u) : "l"(x.u), "l"(y.u));
   return r.f;
 }
+// Row `src` of a [.., n] array into shared memory by one warp.
+__device__ __forceinline__ void ds_copy_row(float* dst, const float* src, int n, int lane, bool vec) {
+  if (vec) {
+    for (int d = lane * 4; d < n; d += 128) ds_copy16(dst + d, src + d);
+  } else {
+    for (int d = lane; d < n; d += 32) ds_copy4(dst + d, src + d);
+  }
+}
 
-// NR: rows per lane (multiple of 4; 8 NR >= D). Columns of a CTA: blockDim / 4.
+// NR: rows per lane (multiple of 4; 8 NR >= D). Columns of a CTA: 4 CPT per warp.
 template <int NR>
 struct DsSmem {
   static constexpr int W = 8 * NR;  // padded width of a key
   static __host__ __device__ int stage_floats(int cols, bool per_channel) { return DS_TOK * (W * (per_channel ? 3 : 2) + cols + 4); }
 };
 
-template <typename T, int NR>
+template <typename T, int NR, int CPT, bool PC>
 __global__ void __launch_bounds__(256)
 delta_scan_kernel(const __grid_constant__ DeltaIn a, const int4* __restrict__ segs, const float* __restrict__ q, const float* __restrict__ k,
                   const float* __restrict__ v, const float* __restrict__ g, const float* __restrict__ beta, const float* __restrict__ qk,
                   float* __restrict__ out) {
   constexpr int W = DsSmem<NR>::W;
   extern __shared__ __align__(16) float ds_smem[];
-  const int H = a.H, G = a.G, D = a.D, DV = a.DV, cols = blockDim.x / 4;
+  const int nwarp = blockDim.x / 32, cols = nwarp * 4 * CPT;
+  const int H = a.H, G = a.G, D = a.D, DV = a.DV;
   const int h = blockIdx.y, kh = h / (H / G), c0 = blockIdx.x * cols;
-  const bool pc = a.per_channel != 0;
-  const int stage = DsSmem<NR>::stage_floats(cols, pc);
+  const int stage = DsSmem<NR>::stage_floats(cols, PC);
   for (int i = threadIdx.x; i < 2 * stage; i += blockDim.x) ds_smem[i] = 0.f;  // padding of keys and columns stays zero
   __syncthreads();
   pdl_wait();
@@ -169,16 +336,16 @@ delta_scan_kernel(const __grid_constant__ DeltaIn a, const int4* __restrict__ se
   const int4 seg = segs[blockIdx.z];  // first row, tokens, first position, state slot
   const int n = seg.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rg = lane & 7, cg = lane >> 3;
-  const int col = warp * 8 + cg * 2;  // of this CTA
+  const int col = warp * 4 * CPT + cg * CPT;  // of this CTA
   const int ncol = min(cols, DV - c0);
   float* S_mem = a.state + (static_cast<long>(seg.w) * H + h) * D * DV + c0;
 
-  float2 S[2][NR / 2];
+  float2 S[CPT][NR / 2];
 #pragma unroll
   for (int j = 0; j < NR / 2; ++j) {
     const int r = rg * 4 + (j >> 1) * 32 + (j & 1) * 2;
 #pragma unroll
-    for (int c = 0; c < 2; ++c) {
+    for (int c = 0; c < CPT; ++c) {
       S[c][j] = make_float2(0.f, 0.f);
       if (seg.z > 0 && col + c < ncol) {
         if (r < D) S[c][j].x = S_mem[static_cast<long>(r) * DV + col + c];
@@ -188,46 +355,87 @@ delta_scan_kernel(const __grid_constant__ DeltaIn a, const int4* __restrict__ se
   }
 
   // stage layout: k [TOK][W], q [TOK][W], (g [TOK][W],) v [TOK][cols], beta, q.k, g, - [TOK][4]
+  constexpr int SQ = DS_TOK * W, SG = 2 * DS_TOK * W, SV = (PC ? 3 : 2) * DS_TOK * W;
+  const int SC = SV + DS_TOK * cols;
   const bool vec4 = D % 4 == 0, v4 = DV % 4 == 0;
   auto fetch = [&](int t0, int buf) {
     float* base = ds_smem + buf * stage;
-    float *sk = base, *sq = sk + DS_TOK * W, *sg = sq + DS_TOK * W, *sv = sg + (pc ? DS_TOK * W : 0), *sc = sv + DS_TOK * cols;
     const int cnt = min(DS_TOK, n - t0);
-    const long row = seg.x + t0;
-    if (vec4) {
-      const int w4 = D / 4;
-      for (int i = threadIdx.x; i < cnt * w4; i += blockDim.x) {
-        const int t = i / w4, d = (i - t * w4) * 4;
-        ds_copy16(sk + t * W + d, k + ((row + t) * G + kh) * D + d);
-        ds_copy16(sq + t * W + d, q + ((row + t) * G + kh) * D + d);
-        if (pc) ds_copy16(sg + t * W + d, g + ((row + t) * H + h) * D + d);
-      }
-    } else {
-      for (int i = threadIdx.x; i < cnt * D; i += blockDim.x) {
-        const int t = i / D, d = i - t * D;
-        ds_copy4(sk + t * W + d, k + ((row + t) * G + kh) * D + d);
-        ds_copy4(sq + t * W + d, q + ((row + t) * G + kh) * D + d);
-        if (pc) ds_copy4(sg + t * W + d, g + ((row + t) * H + h) * D + d);
-      }
-    }
-    if (v4) {
-      const int w4 = ncol / 4;
-      for (int i = threadIdx.x; i < cnt * w4; i += blockDim.x) {
-        const int t = i / w4, d = (i - t * w4) * 4;
-        ds_copy16(sv + t * cols + d, v + ((row + t) * H + h) * DV + c0 + d);
-      }
-    } else {
-      for (int i = threadIdx.x; i < cnt * ncol; i += blockDim.x) {
-        const int t = i / ncol, d = i - t * ncol;
-        ds_copy4(sv + t * cols + d, v + ((row + t) * H + h) * DV + c0 + d);
-      }
-    }
-    for (int t = threadIdx.x; t < cnt; t += blockDim.x) {
-      ds_copy4(sc + t * 4, beta + (row + t) * H + h);
-      ds_copy4(sc + t * 4 + 1, qk + (row + t) * G + kh);
-      if (!pc) ds_copy4(sc + t * 4 + 2, g + (row + t) * H + h);
+    for (int t = warp; t < cnt; t += nwarp) {
+      const long row = seg.x + t0 + t;
+      ds_copy_row(base + t * W, k + (row * G + kh) * D, D, lane, vec4);
+      ds_copy_row(base + SQ + t * W, q + (row * G + kh) * D, D, lane, vec4);
+      if (PC) ds_copy_row(base + SG + t * W, g + (row * H + h) * D, D, lane, vec4);
+      ds_copy_row(base + SV + t * cols, v + (row * H + h) * DV + c0, ncol, lane, v4);
+      if (lane == 0) ds_copy4(base + SC + t * 4, beta + row * H + h);
+      if (lane == 1) ds_copy4(base + SC + t * 4 + 1, qk + row * G + kh);
+      if (!PC && lane == 2) ds_copy4(base + SC + t * 4 + 2, g + row * H + h);
     }
     ds_commit();
+  };
+
+  const float* base = ds_smem;
+  float* orow = out + (static_cast<long>(seg.x) * H + h) * DV + c0;
+  auto token = [&](int t) {
+    const float4 scal = *reinterpret_cast<const float4*>(base + SC + t * 4);  // beta, q.k, decay of the head
+    // v of the column whose u this lane computes: rg & (CPT - 1)
+    const float v_own = base[SV + t * cols + col + (rg & (CPT - 1))];
+    float2 kr[NR / 2], dk[CPT], dq[CPT];
+#pragma unroll
+    for (int c = 0; c < CPT; ++c) dk[c] = dq[c] = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int j = 0; j < NR / 4; ++j) {
+      const int r = rg * 4 + j * 32;
+      const float4 k4 = *reinterpret_cast<const float4*>(base + t * W + r);
+      const float4 q4 = *reinterpret_cast<const float4*>(base + SQ + t * W + r);
+      const float4 g4 = PC ? *reinterpret_cast<const float4*>(base + SG + t * W + r) : make_float4(scal.z, scal.z, scal.z, scal.z);
+      kr[2 * j] = make_float2(k4.x, k4.y);
+      kr[2 * j + 1] = make_float2(k4.z, k4.w);
+#pragma unroll
+      for (int c = 0; c < CPT; ++c) {
+        S[c][2 * j] = ds_mul2(S[c][2 * j], make_float2(g4.x, g4.y));
+        S[c][2 * j + 1] = ds_mul2(S[c][2 * j + 1], make_float2(g4.z, g4.w));
+        dk[c] = ds_fma2(S[c][2 * j], kr[2 * j], dk[c]);
+        dq[c] = ds_fma2(S[c][2 * j], make_float2(q4.x, q4.y), dq[c]);
+        dk[c] = ds_fma2(S[c][2 * j + 1], kr[2 * j + 1], dk[c]);
+        dq[c] = ds_fma2(S[c][2 * j + 1], make_float2(q4.z, q4.w), dq[c]);
+      }
+    }
+    // Sums over the 8 row groups. In every round a lane keeps half of its sums and trades the other half: column bits first
+    // (lane bit b keeps the columns with that bit), then the product (key or query); a round without a choice just adds.
+    float x[2 * CPT];  // [product][column]
+#pragma unroll
+    for (int c = 0; c < CPT; ++c) {
+      x[c] = dk[c].x + dk[c].y;
+      x[CPT + c] = dq[c].x + dq[c].y;
+    }
+    int left = 2 * CPT;
+#pragma unroll
+    for (int b = 1; b < CPT; b <<= 1) {  // entries pair up as (2 i, 2 i + 1): the lowest column bit that is left
+      left /= 2;
+      const bool up = rg & b;
+#pragma unroll
+      for (int i = 0; i < CPT; ++i)
+        if (i < left) {
+          const float keep = up ? x[2 * i + 1] : x[2 * i], give = up ? x[2 * i] : x[2 * i + 1];
+          x[i] = keep + __shfl_xor_sync(0xffffffffu, give, b);
+        }
+    }
+    const bool up = rg & CPT;  // 0: key product, 1: query product
+    float y = (up ? x[1] : x[0]) + __shfl_xor_sync(0xffffffffu, up ? x[0] : x[1], CPT);
+#pragma unroll
+    for (int b = 2 * CPT; b < 8; b <<= 1) y += __shfl_xor_sync(0xffffffffu, y, b);
+    const float key_sum = __shfl_sync(0xffffffffu, y, (lane & ~7) | (rg & (CPT - 1)));
+    const float u_own = scal.x * (v_own - key_sum);
+    float u[CPT];
+#pragma unroll
+    for (int c = 0; c < CPT; ++c) u[c] = __shfl_sync(0xffffffffu, u_own, (lane & ~7) | c);
+#pragma unroll
+    for (int j = 0; j < NR / 2; ++j)
+#pragma unroll
+      for (int c = 0; c < CPT; ++c) S[c][j] = ds_fma2(kr[j], make_float2(u[c], u[c]), S[c][j]);
+    if (rg / CPT == 1 && col + (rg & (CPT - 1)) < ncol) orow[col + (rg & (CPT - 1))] = fmaf(u_own, scal.y, y);
+    orow += static_cast<long>(H) * DV;
   };
 
   const int chunks = (n + DS_TOK - 1) / DS_TOK;
@@ -240,54 +448,13 @@ delta_scan_kernel(const __grid_constant__ DeltaIn a, const int4* __restrict__ se
       ds_wait<0>();
     }
     __syncthreads();
-    const float* base = ds_smem + (ch & 1) * stage;
-    const float *sk = base, *sq = sk + DS_TOK * W, *sg = sq + DS_TOK * W, *sv = sg + (pc ? DS_TOK * W : 0), *sc = sv + DS_TOK * cols;
+    base = ds_smem + (ch & 1) * stage;
     const int cnt = min(DS_TOK, n - ch * DS_TOK);
-    for (int t = 0; t < cnt; ++t) {
-      const float4 scal = *reinterpret_cast<const float4*>(sc + t * 4);  // beta, q.k, decay of the head
-      const float2 vv = *reinterpret_cast<const float2*>(sv + t * cols + col);
-      float2 kr[NR / 2];
-      float2 dk[2], dq[2];
-      dk[0] = dk[1] = dq[0] = dq[1] = make_float2(0.f, 0.f);
-#pragma unroll
-      for (int j = 0; j < NR / 4; ++j) {
-        const int r = rg * 4 + j * 32;
-        const float4 k4 = *reinterpret_cast<const float4*>(sk + t * W + r);
-        const float4 q4 = *reinterpret_cast<const float4*>(sq + t * W + r);
-        const float4 g4 = pc ? *reinterpret_cast<const float4*>(sg + t * W + r) : make_float4(scal.z, scal.z, scal.z, scal.z);
-        kr[2 * j] = make_float2(k4.x, k4.y);
-        kr[2 * j + 1] = make_float2(k4.z, k4.w);
-#pragma unroll
-        for (int c = 0; c < 2; ++c) {
-          S[c][2 * j] = ds_mul2(S[c][2 * j], make_float2(g4.x, g4.y));
-          S[c][2 * j + 1] = ds_mul2(S[c][2 * j + 1], make_float2(g4.z, g4.w));
-          dk[c] = ds_fma2(S[c][2 * j], kr[2 * j], dk[c]);
-          dq[c] = ds_fma2(S[c][2 * j], make_float2(q4.x, q4.y), dq[c]);
-          dk[c] = ds_fma2(S[c][2 * j + 1], kr[2 * j + 1], dk[c]);
-          dq[c] = ds_fma2(S[c][2 * j + 1], make_float2(q4.z, q4.w), dq[c]);
-        }
-      }
-      // sums over the 8 row groups: first the two columns trade halves (lane parity picks the column it keeps) ...
-      float k0 = dk[0].x + dk[0].y, k1 = dk[1].x + dk[1].y, q0 = dq[0].x + dq[0].y, q1 = dq[1].x + dq[1].y;
-      const bool odd = rg & 1;
-      float kx = (odd ? k1 : k0) + __shfl_xor_sync(0xffffffffu, odd ? k0 : k1, 1);
-      float qx = (odd ? q1 : q0) + __shfl_xor_sync(0xffffffffu, odd ? q0 : q1, 1);
-      // ... then the two products do (bit 1 of the row group: 0 keeps the key's, 1 the query's)
-      const bool up = rg & 2;
-      float x = (up ? qx : kx) + __shfl_xor_sync(0xffffffffu, up ? kx : qx, 2);
-      x += __shfl_xor_sync(0xffffffffu, x, 4);
-      // lane rg has: column rg & 1 of the key's (rg & 2 == 0) or the query's product
-      const float sk_own = __shfl_sync(0xffffffffu, x, (lane & ~7) | (rg & 1));
-      const float u_own = scal.x * ((odd ? vv.y : vv.x) - sk_own);
-      const float u_other = __shfl_xor_sync(0xffffffffu, u_own, 1);
-      const float u0 = odd ? u_other : u_own, u1 = odd ? u_own : u_other;
-#pragma unroll
-      for (int j = 0; j < NR / 2; ++j) {
-        S[0][j] = ds_fma2(kr[j], make_float2(u0, u0), S[0][j]);
-        S[1][j] = ds_fma2(kr[j], make_float2(u1, u1), S[1][j]);
-      }
-      if ((rg & 6) == 2 && col + (rg & 1) < ncol)
-        out[((static_cast<long>(seg.x) + ch * DS_TOK + t) * H + h) * DV + c0 + col + (rg & 1)] = fmaf(u_own, scal.y, x);
+    if (cnt == DS_TOK) {
+#pragma unroll 2
+      for (int t = 0; t < DS_TOK; ++t) token(t);
+    } else {
+      for (int t = 0; t < cnt; ++t) token(t);
     }
     __syncthreads();
   }
@@ -296,7 +463,7 @@ delta_scan_kernel(const __grid_constant__ DeltaIn a, const int4* __restrict__ se
   for (int j = 0; j < NR / 2; ++j) {
     const int r = rg * 4 + (j >> 1) * 32 + (j & 1) * 2;
 #pragma unroll
-    for (int c = 0; c < 2; ++c)
+    for (int c = 0; c < CPT; ++c)
       if (col + c < ncol) {
         if (r < D) S_mem[static_cast<long>(r) * DV + col + c] = S[c][j].x;
         if (r + 1 < D) S_mem[static_cast<long>(r + 1) * DV + col + c] = S[c][j].y;
@@ -342,6 +509,45 @@ head_gate_kernel(const float* __restrict__ o, const T* __restrict__ z, const T* 
   for (int j = 0; j < DR_MAX / 32; ++j) {
     const int d = lane + 32 * j;
     if (d < DV) dr_store(out + t * out_pitch + h * DV + d, x[j] * r * dr_load(w + d) * dr_gate(dr_load(z + t * z_pitch + h * DV + d), sigmoid));
+  }
+}
+
+// The same with V adjacent columns per lane (DV <= 32 V).
+template <typename T, int V>
+__global__ void __launch_bounds__(128)
+head_gate_wide_kernel(const float* __restrict__ o, const T* __restrict__ z, const T* __restrict__ w, T* __restrict__ out, long pairs, int H,
+                      int DV, long z_pitch, long out_pitch, float eps, float scale, int sigmoid) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int lane = threadIdx.x & 31, d = lane * V;
+  const long stride = static_cast<long>(gridDim.x) * 4;
+  const bool on = d < DV;
+  float wt[V], x[V], gate[V];
+#pragma unroll
+  for (int i = 0; i < V; ++i) wt[i] = x[i] = gate[i] = 0.f;
+  if (on) dr_load_v<V>(w + d, wt);
+  for (long p = static_cast<long>(blockIdx.x) * 4 + (threadIdx.x >> 5); p < pairs; p += stride) {
+    const long t = p / H;
+    const int h = static_cast<int>(p - t * H);
+    float ss = 0.f;
+    if (on) {
+      dr_load_v<V>(o + p * DV + d, x);
+      dr_load_v<V>(z + t * z_pitch + h * DV + d, gate);
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) ss = fmaf(x[i], x[i], ss);
+    const float r = scale / sqrtf(warp_sum(ss) / DV + eps);
+    if (on) {
+      float y[V];
+#pragma unroll
+      for (int i = 0; i < V; ++i) {
+        float f;
+        if constexpr (sizeof(T) == 2) f = __fdividef(sigmoid ? 1.f : gate[i], 1.f + __expf(-gate[i]));
+        else f = dr_gate(gate[i], sigmoid);
+        y[i] = x[i] * r * wt[i] * f;
+      }
+      dr_store_v<V>(out + t * out_pitch + h * DV + d, y);
+    }
   }
 }
 
@@ -538,33 +744,71 @@ static int dr_check(int H, int G, int D, int DV, int taps) {
   return H <= 0 || G <= 0 || H % G != 0 || D <= 0 || DV <= 0 || D > DR_MAX || DV > DR_MAX || taps < 1 || taps > DR_MAX_TAPS;
 }
 
+template <typename... P>
+static bool dr_aligned(int bytes, P... p) {
+  return ((reinterpret_cast<uintptr_t>(p) | ... | uintptr_t(0)) % bytes) == 0;
+}
+
 template <typename T>
 static int launch_prep(const DeltaIn& a, int nruns, const int* runs, const int* segs, float* q, float* k, float* v, float* g, float* beta,
                        float* qk, cudaStream_t s) {
-  return (int)launch_pdl(delta_prep_kernel<T>, dim3(nruns, (a.G + 2 * a.H + 3) / 4), dim3(128), 0, s, a, reinterpret_cast<const int4*>(runs),
-                         reinterpret_cast<const int4*>(segs), q, k, v, g, beta, qk);
+  const dim3 grid(nruns, (a.G + 2 * a.H + 3) / 4);
+  const int widest = a.D > a.DV ? a.D : a.DV, V = widest <= 64 ? 2 : 4;
+  const bool wide = widest <= 32 * V && a.taps <= 4 && a.D % V == 0 && a.DV % V == 0 && a.pitch % V == 0 && a.a_pitch % V == 0 &&
+                    dr_aligned(V * static_cast<int>(sizeof(T)), a.q, a.k, a.v, a.ring, a.per_channel ? a.a : nullptr) &&
+                    dr_aligned(V * 4, q, k, v, g, a.dt_bias);
+  auto kern = !wide ? delta_prep_kernel<T> : V == 2 ? delta_prep_wide_kernel<T, 2> : delta_prep_wide_kernel<T, 4>;
+  return (int)launch_pdl(kern, grid, dim3(128), 0, s, a, reinterpret_cast<const int4*>(runs), reinterpret_cast<const int4*>(segs), q, k, v, g,
+                         beta, qk);
 }
 
-template <typename T, int NR>
-static int launch_scan(const DeltaIn& a, int nseg, const int* segs, const float* q, const float* k, const float* v, const float* g,
+template <typename T>
+static int launch_gate(const float* o, const T* z, const T* w, T* out, long pairs, int H, int DV, long z_pitch, long out_pitch, float eps,
+                       float scale, int sigmoid, cudaStream_t s) {
+  const int V = DV <= 64 ? 2 : 4;
+  const bool wide = DV <= 32 * V && DV % V == 0 && z_pitch % V == 0 && out_pitch % V == 0 &&
+                    dr_aligned(V * static_cast<int>(sizeof(T)), z, w, out) && dr_aligned(V * 4, o);
+  const long blocks = (pairs + 3) / 4, most = 148 * 16;
+  auto kern = !wide ? head_gate_kernel<T> : V == 2 ? head_gate_wide_kernel<T, 2> : head_gate_wide_kernel<T, 4>;
+  return (int)launch_pdl(kern, dim3(static_cast<unsigned>(wide && blocks > most ? most : blocks)), dim3(128), 0, s, o, z, w, out, pairs, H, DV,
+                         z_pitch, out_pitch, eps, scale, sigmoid);
+}
+
+template <typename T, int NR, int CPT, bool PC>
+static int launch_scan(const DeltaIn& a, int nseg, int warps, const int* segs, const float* q, const float* k, const float* v, const float* g,
                        const float* beta, const float* qk, float* out, cudaStream_t s) {
-  const int cols = a.DV > 32 ? 64 : a.DV > 16 ? 32 : 16;
-  const int bytes = 2 * DsSmem<NR>::stage_floats(cols, a.per_channel != 0) * 4;
-  auto kern = delta_scan_kernel<T, NR>;
-  if (cudaError_t e = ensure_dynamic_smem(reinterpret_cast<const void*>(kern), 2 * DsSmem<NR>::stage_floats(64, true) * 4); e != cudaSuccess)
+  const int cols = warps * 4 * CPT;
+  auto kern = delta_scan_kernel<T, NR, CPT, PC>;
+  if (cudaError_t e = ensure_dynamic_smem(reinterpret_cast<const void*>(kern), 2 * DsSmem<NR>::stage_floats(64, PC) * 4); e != cudaSuccess)
     return (int)e;
-  return (int)launch_pdl(kern, dim3((a.DV + cols - 1) / cols, a.H, nseg), dim3(cols * 4), bytes, s, a, reinterpret_cast<const int4*>(segs), q, k,
-                         v, g, beta, qk, out);
+  return (int)launch_pdl(kern, dim3((a.DV + cols - 1) / cols, a.H, nseg), dim3(warps * 32), 2 * DsSmem<NR>::stage_floats(cols, PC) * 4, s, a,
+                         reinterpret_cast<const int4*>(segs), q, k, v, g, beta, qk, out);
+}
+
+// CTAs of up to 64 columns. With enough of them to fill the machine a lane takes 4 columns, otherwise 2.
+template <typename T, int NR>
+static int scan_shape(const DeltaIn& a, int nseg, const int* segs, const float* q, const float* k, const float* v, const float* g,
+                      const float* beta, const float* qk, float* out, cudaStream_t s) {
+  const bool many = NR <= 16 && static_cast<long>(nseg) * a.H * ((a.DV + 63) / 64) > 148 * 2;
+#define SB_SCAN(CPT, PC) \
+  return launch_scan<T, NR, CPT, PC>(a, nseg, a.DV > 32 ? 16 / CPT : a.DV > 16 ? 8 / CPT : 4 / CPT, segs, q, k, v, g, beta, qk, out, s)
+  if constexpr (NR <= 16) {
+    if (many && a.per_channel) SB_SCAN(4, true);
+    if (many) SB_SCAN(4, false);
+  }
+  if (a.per_channel) SB_SCAN(2, true);
+  SB_SCAN(2, false);
+#undef SB_SCAN
 }
 
 template <typename T>
 static int scan_by_width(const DeltaIn& a, int nseg, const int* segs, const float* q, const float* k, const float* v, const float* g,
                          const float* beta, const float* qk, float* out, cudaStream_t s) {
-  if (a.D <= 32) return launch_scan<T, 4>(a, nseg, segs, q, k, v, g, beta, qk, out, s);
-  if (a.D <= 64) return launch_scan<T, 8>(a, nseg, segs, q, k, v, g, beta, qk, out, s);
-  if (a.D <= 96) return launch_scan<T, 12>(a, nseg, segs, q, k, v, g, beta, qk, out, s);
-  if (a.D <= 128) return launch_scan<T, 16>(a, nseg, segs, q, k, v, g, beta, qk, out, s);
-  return launch_scan<T, 32>(a, nseg, segs, q, k, v, g, beta, qk, out, s);
+  if (a.D <= 32) return scan_shape<T, 4>(a, nseg, segs, q, k, v, g, beta, qk, out, s);
+  if (a.D <= 64) return scan_shape<T, 8>(a, nseg, segs, q, k, v, g, beta, qk, out, s);
+  if (a.D <= 96) return scan_shape<T, 12>(a, nseg, segs, q, k, v, g, beta, qk, out, s);
+  if (a.D <= 128) return scan_shape<T, 16>(a, nseg, segs, q, k, v, g, beta, qk, out, s);
+  return scan_shape<T, 32>(a, nseg, segs, q, k, v, g, beta, qk, out, s);
 }
 
 template <typename T>
@@ -618,13 +862,9 @@ extern "C" int sb_head_gate(const float* o, const void* z, const void* w, void* 
   if (T == 0) return 0;
   if (H <= 0 || DV <= 0 || DV > sb::DR_MAX) return (int)cudaErrorInvalidValue;
   const long pairs = static_cast<long>(T) * H;
-  const dim3 grid(static_cast<unsigned>((pairs + 3) / 4));
   using bf16 = __nv_bfloat16;
-  if (f32)
-    return (int)sb::launch_pdl(sb::head_gate_kernel<float>, grid, dim3(128), 0, s, o, (const float*)z, (const float*)w, (float*)out, pairs, H, DV,
-                               z_pitch, out_pitch, eps, scale, sigmoid);
-  return (int)sb::launch_pdl(sb::head_gate_kernel<bf16>, grid, dim3(128), 0, s, o, (const bf16*)z, (const bf16*)w, (bf16*)out, pairs, H, DV,
-                             z_pitch, out_pitch, eps, scale, sigmoid);
+  if (f32) return sb::launch_gate<float>(o, (const float*)z, (const float*)w, (float*)out, pairs, H, DV, z_pitch, out_pitch, eps, scale, sigmoid, s);
+  return sb::launch_gate<bf16>(o, (const bf16*)z, (const bf16*)w, (bf16*)out, pairs, H, DV, z_pitch, out_pitch, eps, scale, sigmoid, s);
 }
 
 // One token per row: slot / active / pos [B]; rows that are not active leave every state alone and give zeros.
