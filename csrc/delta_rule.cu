@@ -280,7 +280,8 @@ delta_prep_wide_kernel(const __grid_constant__ DeltaIn a, const int4* __restrict
 // {4 rg + 32 j + 0..3}. Both products with S are taken before u is known (o = (g S)^T q + u (k.q)), so a token costs one
 // round of shuffles. q, k, g, v of the next tokens are copied to shared memory while the current ones are processed. More columns
 // per lane mean fewer reads of q, k, g from shared memory (the bound of a full machine), fewer mean more warps (few requests).
-constexpr int DS_TOK = 8;  // tokens per copy
+constexpr int DS_TOK = 8;     // tokens per copy
+constexpr int DS_STAGES = 4;  // copies in flight or in use: three chunks ahead cover the memory's latency
 
 __device__ __forceinline__ void ds_copy16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
@@ -329,7 +330,7 @@ delta_scan_kernel(const __grid_constant__ DeltaIn a, const int4* __restrict__ se
   const int H = a.H, G = a.G, D = a.D, DV = a.DV;
   const int h = blockIdx.y, kh = h / (H / G), c0 = blockIdx.x * cols;
   const int stage = DsSmem<NR>::stage_floats(cols, PC);
-  for (int i = threadIdx.x; i < 2 * stage; i += blockDim.x) ds_smem[i] = 0.f;  // padding of keys and columns stays zero
+  for (int i = threadIdx.x; i < DS_STAGES * stage; i += blockDim.x) ds_smem[i] = 0.f;  // padding of keys and columns stays zero
   __syncthreads();
   pdl_wait();
   pdl_launch_dependents();
@@ -439,16 +440,18 @@ delta_scan_kernel(const __grid_constant__ DeltaIn a, const int4* __restrict__ se
   };
 
   const int chunks = (n + DS_TOK - 1) / DS_TOK;
-  fetch(0, 0);
+#pragma unroll
+  for (int i = 0; i < DS_STAGES - 1; ++i) {
+    if (i < chunks) fetch(i * DS_TOK, i);
+    else ds_commit();
+  }
   for (int ch = 0; ch < chunks; ++ch) {
-    if (ch + 1 < chunks) {
-      fetch((ch + 1) * DS_TOK, (ch + 1) & 1);
-      ds_wait<1>();
-    } else {
-      ds_wait<0>();
-    }
-    __syncthreads();
-    base = ds_smem + (ch & 1) * stage;
+    ds_wait<DS_STAGES - 2>();
+    __syncthreads();  // this chunk has arrived for everyone, and everyone is done with the previous one
+    const int next = ch + DS_STAGES - 1;
+    if (next < chunks) fetch(next * DS_TOK, next % DS_STAGES);
+    else ds_commit();
+    base = ds_smem + (ch % DS_STAGES) * stage;
     const int cnt = min(DS_TOK, n - ch * DS_TOK);
     if (cnt == DS_TOK) {
 #pragma unroll 2
@@ -456,7 +459,6 @@ delta_scan_kernel(const __grid_constant__ DeltaIn a, const int4* __restrict__ se
     } else {
       for (int t = 0; t < cnt; ++t) token(t);
     }
-    __syncthreads();
   }
 
 #pragma unroll
@@ -779,9 +781,9 @@ static int launch_scan(const DeltaIn& a, int nseg, int warps, const int* segs, c
                        const float* beta, const float* qk, float* out, cudaStream_t s) {
   const int cols = warps * 4 * CPT;
   auto kern = delta_scan_kernel<T, NR, CPT, PC>;
-  if (cudaError_t e = ensure_dynamic_smem(reinterpret_cast<const void*>(kern), 2 * DsSmem<NR>::stage_floats(64, PC) * 4); e != cudaSuccess)
+  if (cudaError_t e = ensure_dynamic_smem(reinterpret_cast<const void*>(kern), DS_STAGES * DsSmem<NR>::stage_floats(64, PC) * 4); e != cudaSuccess)
     return (int)e;
-  return (int)launch_pdl(kern, dim3((a.DV + cols - 1) / cols, a.H, nseg), dim3(warps * 32), 2 * DsSmem<NR>::stage_floats(cols, PC) * 4, s, a,
+  return (int)launch_pdl(kern, dim3((a.DV + cols - 1) / cols, a.H, nseg), dim3(warps * 32), DS_STAGES * DsSmem<NR>::stage_floats(cols, PC) * 4, s, a,
                          reinterpret_cast<const int4*>(segs), q, k, v, g, beta, qk, out);
 }
 
