@@ -320,7 +320,7 @@ struct DsSmem {
 };
 
 template <typename T, int NR, int CPT, bool PC>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(CPT == 4 ? 128 : 256, CPT == 4 ? 4 : 1)
 delta_scan_kernel(const __grid_constant__ DeltaIn a, const int4* __restrict__ segs, const float* __restrict__ q, const float* __restrict__ k,
                   const float* __restrict__ v, const float* __restrict__ g, const float* __restrict__ beta, const float* __restrict__ qk,
                   float* __restrict__ out) {
@@ -379,11 +379,12 @@ delta_scan_kernel(const __grid_constant__ DeltaIn a, const int4* __restrict__ se
   float* orow = out + (static_cast<long>(seg.x) * H + h) * DV + c0;
   auto token = [&](int t) {
     const float4 scal = *reinterpret_cast<const float4*>(base + SC + t * 4);  // beta, q.k, decay of the head
-    // v of the column whose u this lane computes: rg & (CPT - 1)
-    const float v_own = base[SV + t * cols + col + (rg & (CPT - 1))];
-    float2 kr[NR / 2], dk[CPT], dq[CPT];
+    float vv[CPT];
+    dr_load_v<CPT>(base + SV + t * cols + col, vv);
+    float2 kr[NR / 2], dk[CPT], dq[CPT], dk2[CPT], dq2[CPT];
+    constexpr bool TWO = CPT == 2;  // two chains per sum where a lane has few columns
 #pragma unroll
-    for (int c = 0; c < CPT; ++c) dk[c] = dq[c] = make_float2(0.f, 0.f);
+    for (int c = 0; c < CPT; ++c) dk[c] = dq[c] = dk2[c] = dq2[c] = make_float2(0.f, 0.f);
 #pragma unroll
     for (int j = 0; j < NR / 4; ++j) {
       const int r = rg * 4 + j * 32;
@@ -398,44 +399,60 @@ delta_scan_kernel(const __grid_constant__ DeltaIn a, const int4* __restrict__ se
         S[c][2 * j + 1] = ds_mul2(S[c][2 * j + 1], make_float2(g4.z, g4.w));
         dk[c] = ds_fma2(S[c][2 * j], kr[2 * j], dk[c]);
         dq[c] = ds_fma2(S[c][2 * j], make_float2(q4.x, q4.y), dq[c]);
-        dk[c] = ds_fma2(S[c][2 * j + 1], kr[2 * j + 1], dk[c]);
-        dq[c] = ds_fma2(S[c][2 * j + 1], make_float2(q4.z, q4.w), dq[c]);
+        float2 &k_sum = TWO ? dk2[c] : dk[c], &q_sum = TWO ? dq2[c] : dq[c];
+        k_sum = ds_fma2(S[c][2 * j + 1], kr[2 * j + 1], k_sum);
+        q_sum = ds_fma2(S[c][2 * j + 1], make_float2(q4.z, q4.w), q_sum);
       }
     }
-    // Sums over the 8 row groups. In every round a lane keeps half of its sums and trades the other half: column bits first
-    // (lane bit b keeps the columns with that bit), then the product (key or query); a round without a choice just adds.
+    // Sums over the 8 row groups.
     float x[2 * CPT];  // [product][column]
 #pragma unroll
     for (int c = 0; c < CPT; ++c) {
-      x[c] = dk[c].x + dk[c].y;
-      x[CPT + c] = dq[c].x + dq[c].y;
+      x[c] = (dk[c].x + dk2[c].x) + (dk[c].y + dk2[c].y);
+      x[CPT + c] = (dq[c].x + dq2[c].x) + (dq[c].y + dq2[c].y);
     }
-    int left = 2 * CPT;
-#pragma unroll
-    for (int b = 1; b < CPT; b <<= 1) {  // entries pair up as (2 i, 2 i + 1): the lowest column bit that is left
-      left /= 2;
-      const bool up = rg & b;
-#pragma unroll
-      for (int i = 0; i < CPT; ++i)
-        if (i < left) {
-          const float keep = up ? x[2 * i + 1] : x[2 * i], give = up ? x[2 * i] : x[2 * i + 1];
-          x[i] = keep + __shfl_xor_sync(0xffffffffu, give, b);
-        }
-    }
-    const bool up = rg & CPT;  // 0: key product, 1: query product
-    float y = (up ? x[1] : x[0]) + __shfl_xor_sync(0xffffffffu, up ? x[0] : x[1], CPT);
-#pragma unroll
-    for (int b = 2 * CPT; b < 8; b <<= 1) y += __shfl_xor_sync(0xffffffffu, y, b);
-    const float key_sum = __shfl_sync(0xffffffffu, y, (lane & ~7) | (rg & (CPT - 1)));
-    const float u_own = scal.x * (v_own - key_sum);
     float u[CPT];
+    if constexpr (CPT == 2) {
+      // Few warps: the time of a token counts. Every lane adds up the key's sums completely, so that nothing has to travel back
+      // before the write; the query's follow behind it (lane bit 0 keeps the column it names).
 #pragma unroll
-    for (int c = 0; c < CPT; ++c) u[c] = __shfl_sync(0xffffffffu, u_own, (lane & ~7) | c);
+      for (int b = 1; b < 8; b <<= 1) {
+        x[0] += __shfl_xor_sync(0xffffffffu, x[0], b);
+        x[1] += __shfl_xor_sync(0xffffffffu, x[1], b);
+      }
+      u[0] = scal.x * (vv[0] - x[0]);
+      u[1] = scal.x * (vv[1] - x[1]);
+      const bool up = rg & 1;
+      float y = (up ? x[3] : x[2]) + __shfl_xor_sync(0xffffffffu, up ? x[2] : x[3], 1);
+      y += __shfl_xor_sync(0xffffffffu, y, 2);
+      y += __shfl_xor_sync(0xffffffffu, y, 4);
+      if (rg < 2 && col + rg < ncol) orow[col + rg] = fmaf(up ? u[1] : u[0], scal.y, y);
+    } else {
+      // Many warps: the number of shuffles counts. In every round a lane keeps half of its sums and trades the other half: by the
+      // two bits of the column, then by the product; u comes back by shuffles.
+      const bool b0 = rg & 1, b1 = rg & 2, b2 = rg & 4;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float keep = b0 ? x[2 * i + 1] : x[2 * i], give = b0 ? x[2 * i] : x[2 * i + 1];
+        x[i] = keep + __shfl_xor_sync(0xffffffffu, give, 1);
+      }
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const float keep = b1 ? x[2 * i + 1] : x[2 * i], give = b1 ? x[2 * i] : x[2 * i + 1];
+        x[i] = keep + __shfl_xor_sync(0xffffffffu, give, 2);
+      }
+      const float y = (b2 ? x[1] : x[0]) + __shfl_xor_sync(0xffffffffu, b2 ? x[0] : x[1], 4);
+      const float key_sum = __shfl_sync(0xffffffffu, y, lane & ~4);
+      const float v_own = b1 ? (b0 ? vv[3] : vv[2]) : (b0 ? vv[1] : vv[0]);
+      const float u_own = scal.x * (v_own - key_sum);
+#pragma unroll
+      for (int c = 0; c < CPT; ++c) u[c] = __shfl_sync(0xffffffffu, u_own, (lane & ~7) | c);
+      if (b2 && col + (rg & 3) < ncol) orow[col + (rg & 3)] = fmaf(u_own, scal.y, y);
+    }
 #pragma unroll
     for (int j = 0; j < NR / 2; ++j)
 #pragma unroll
       for (int c = 0; c < CPT; ++c) S[c][j] = ds_fma2(kr[j], make_float2(u[c], u[c]), S[c][j]);
-    if (rg / CPT == 1 && col + (rg & (CPT - 1)) < ncol) orow[col + (rg & (CPT - 1))] = fmaf(u_own, scal.y, y);
     orow += static_cast<long>(H) * DV;
   };
 
@@ -454,7 +471,7 @@ delta_scan_kernel(const __grid_constant__ DeltaIn a, const int4* __restrict__ se
     base = ds_smem + (ch % DS_STAGES) * stage;
     const int cnt = min(DS_TOK, n - ch * DS_TOK);
     if (cnt == DS_TOK) {
-#pragma unroll 2
+#pragma unroll(CPT == 2 ? 2 : 1)
       for (int t = 0; t < DS_TOK; ++t) token(t);
     } else {
       for (int t = 0; t < cnt; ++t) token(t);
@@ -783,17 +800,20 @@ static int launch_scan(const DeltaIn& a, int nseg, int warps, const int* segs, c
   auto kern = delta_scan_kernel<T, NR, CPT, PC>;
   if (cudaError_t e = ensure_dynamic_smem(reinterpret_cast<const void*>(kern), DS_STAGES * DsSmem<NR>::stage_floats(64, PC) * 4); e != cudaSuccess)
     return (int)e;
-  return (int)launch_pdl(kern, dim3((a.DV + cols - 1) / cols, a.H, nseg), dim3(warps * 32), DS_STAGES * DsSmem<NR>::stage_floats(cols, PC) * 4, s, a,
-                         reinterpret_cast<const int4*>(segs), q, k, v, g, beta, qk, out);
+  // A plain launch: CTAs that start while the previous kernel still holds most of the machine would pile up on the few SMs
+  // that are free, and stay there for the whole sequence.
+  kern<<<dim3((a.DV + cols - 1) / cols, a.H, nseg), warps * 32, DS_STAGES * DsSmem<NR>::stage_floats(cols, PC) * 4, s>>>(
+      a, reinterpret_cast<const int4*>(segs), q, k, v, g, beta, qk, out);
+  return (int)cudaGetLastError();
 }
 
 // CTAs of up to 64 columns. With enough of them to fill the machine a lane takes 4 columns, otherwise 2.
 template <typename T, int NR>
 static int scan_shape(const DeltaIn& a, int nseg, const int* segs, const float* q, const float* k, const float* v, const float* g,
                       const float* beta, const float* qk, float* out, cudaStream_t s) {
-  const bool many = NR <= 16 && static_cast<long>(nseg) * a.H * ((a.DV + 63) / 64) > 148 * 2;
-#define SB_SCAN(CPT, PC) \
-  return launch_scan<T, NR, CPT, PC>(a, nseg, a.DV > 32 ? 16 / CPT : a.DV > 16 ? 8 / CPT : 4 / CPT, segs, q, k, v, g, beta, qk, out, s)
+  const bool many = NR <= 16 && static_cast<long>(nseg) * a.H * ((a.DV + 63) / 64) > 148;
+  const int cols = a.DV > 32 ? 64 : a.DV > 16 ? 32 : 16;
+#define SB_SCAN(CPT, PC) return launch_scan<T, NR, CPT, PC>(a, nseg, cols / (4 * CPT), segs, q, k, v, g, beta, qk, out, s)
   if constexpr (NR <= 16) {
     if (many && a.per_channel) SB_SCAN(4, true);
     if (many) SB_SCAN(4, false);
