@@ -441,5 +441,28 @@ inline CUtensorMap make_tmap_2d(const void* base, CUtensorMapDataType dt, int el
                              std::to_string(box_rows) + "x" + std::to_string(box_cols));
   return m;
 }
+
+// 3-D bf16 tensor [d2, d1, d0] (d0 innermost, contiguous), pitches of d1 and d2 in elements, 128B swizzle; what lies outside
+// reads as zero.
+inline CUtensorMap make_tmap_3d(const void* base, uint64_t d0, uint64_t d1, uint64_t d2, uint64_t pitch1, uint64_t pitch2, uint32_t box0,
+                                uint32_t box1, uint32_t box2) {
+  CUtensorMap m;
+  cuuint64_t dims[3] = {d0, d1, d2};
+  cuuint64_t strides[2] = {pitch1 * 2, pitch2 * 2};
+  cuuint32_t box[3] = {box0, box1, box2};
+  cuuint32_t estr[3] = {1, 1, 1};
+  static thread_local bool ctx_bound = false;  // as in make_tmap_2d
+  if (!ctx_bound) {
+    int dev = 0;
+    if (cudaGetDevice(&dev) == cudaSuccess && cudaSetDevice(dev) == cudaSuccess) ctx_bound = true;
+  }
+  CUresult r = get_encode_tiled()(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr,
+                                  CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                                  CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  if (r != CUDA_SUCCESS)
+    throw std::runtime_error("cuTensorMapEncodeTiled (3-D) failed: " + std::to_string(int(r)) + " dims=" + std::to_string(d0) + "," +
+                             std::to_string(d1) + "," + std::to_string(d2) + " pitches=" + std::to_string(pitch1) + "," + std::to_string(pitch2));
+  return m;
+}
 }  // namespace sb
 #endif

@@ -23,7 +23,7 @@
 // block_table[b, i] = page id of the i-th page of request b. page_size must be 16, 32, 64 or 128.
 #include <type_traits>
 
-#include "common.cuh"
+#include "attn_combine.cuh"
 
 namespace sb {
 
@@ -57,15 +57,13 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return r;
 }
 
-// Windowed form (WIN): the query (the last token) sees the keys of its window and the first `keep_first` tokens, and scores
-// lose slopes[head] * distance. Only tiles with a visible key are visited: those of the kept tokens, then 128-key tiles from
-// the page that holds the window's first key. Head widths dk / dv may be smaller than D (the tensor maps read zeros past
-// them) and the group of query heads smaller than G (`group`; the surplus rows of Q are zero and never written out).
-// sinks: score of an extra softmax column without a value, per head; the output is multiplied by out_scale.
+// Windowed form (WIN): visibility and scores as attn_rule.cuh says. Only tiles with a visible key are visited: those of the kept
+// tokens, then 128-key tiles from the page that holds the first key of the window or chunk. Head widths dk / dv may be smaller
+// than D (the tensor maps read zeros past them) and the group of query heads smaller than G (`group`; the surplus rows of Q
+// are zero and never written out).
 struct DecWindow {
-  const float *slopes, *sinks;  // [Hq] or null
-  float out_scale;
-  int window, keep_first, group, dk, dv;
+  AttnRule rule;
+  int group, dk, dv;
 };
 struct DecFull {};
 
@@ -126,9 +124,9 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
   int t_begin, t_end, ntiles;
   int n_keep = 0, win_base = 0, tile0 = 0, low = 0;  // windowed: tiles of kept tokens, first key of the others, this split's first
   if constexpr (WIN) {
-    low = win.window >= len ? 0 : len - win.window;
+    low = rule_first_key(win.rule, len - 1);
     win_base = (low >> page_shift) << page_shift;
-    n_keep = min((min(win.keep_first, len) + DA_TILE - 1) / DA_TILE, (win_base + DA_TILE - 1) / DA_TILE);
+    n_keep = min((min(win.rule.keep_first, len) + DA_TILE - 1) / DA_TILE, (win_base + DA_TILE - 1) / DA_TILE);
     win_base = max(win_base, n_keep * DA_TILE);
     const int total = n_keep + (len > win_base ? (len - win_base + DA_TILE - 1) / DA_TILE : 0);
     const int per = (total + splits - 1) / splits;
@@ -269,7 +267,15 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
   if constexpr (WIN) {
 #pragma unroll
     for (int g = 0; g < G; ++g)
-      slope2[g] = (win.slopes != nullptr && g < win.group) ? win.slopes[kvh * win.group + g] * 1.4426950408889634f : 0.f;
+      slope2[g] = (win.rule.slopes != nullptr && g < win.group) ? win.rule.slopes[kvh * win.group + g] * 1.4426950408889634f : 0.f;
+  }
+  // capped scores: see cap_exp2
+  float cap2 = 0.f, cap_k = 0.f;
+  if constexpr (WIN) {
+    if (win.rule.softcap > 0.f) {
+      cap2 = win.rule.softcap * 1.4426950408889634f;
+      cap_k = 2.f * scale_log2 / win.rule.softcap;
+    }
   }
   const bool merges = tid < D;  // warp-uniform: D is 64 or 128
   // merge tile j (O^T is ready once bar_o completes phase j); its V buffer is then free for tile j + DA_STAGES
@@ -317,10 +323,22 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
       }
       if constexpr (WIN) {
         const int key = t0 + tid;
-        const bool see = tid < valid && (key >= low || key < win.keep_first);  // every visited tile has such a key
+        const bool see = tid < valid && (key >= low || key < win.rule.keep_first);  // every visited tile has such a key
         const float back = static_cast<float>(key - (len - 1));
 #pragma unroll
-        for (int g = 0; g < G; ++g) sc[g] = see ? fmaf(__uint_as_float(r[g]), scale_log2, slope2[g] * back) : -INFINITY;
+        for (int g = 0; g < G; ++g) sc[g] = __uint_as_float(r[g]) * scale_log2;
+        if (win.rule.softcap > 0.f) {
+#pragma unroll
+          for (int g = 0; g < G; ++g) sc[g] = fmaf(-2.f * cap2, fast_rcp(cap_exp2(__uint_as_float(r[g]), cap_k)), cap2);
+        }
+        if (win.rule.bias != nullptr && see) {
+          const float* row = win.rule.bias + static_cast<size_t>(min(len - 1 - key, win.rule.bias_rows - 1)) * Hq + kvh * win.group;
+#pragma unroll
+          for (int g = 0; g < G; ++g)
+            if (g < win.group) sc[g] = fmaf(row[g], 1.4426950408889634f, sc[g]);
+        }
+#pragma unroll
+        for (int g = 0; g < G; ++g) sc[g] = see ? fmaf(slope2[g], back, sc[g]) : -INFINITY;
       } else {
 #pragma unroll
         for (int g = 0; g < G; ++g) sc[g] = (tid < valid) ? __uint_as_float(r[g]) * scale_log2 : -INFINITY;
@@ -408,8 +426,8 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
         h = kvh * win.group + g;
         width = win.dv;
         if (splits == 1) {
-          if (win.sinks != nullptr) l_run += fast_exp2(fmaf(win.sinks[h], 1.4426950408889634f, -m_thr[g]));
-          gain = win.out_scale;
+          if (win.rule.sinks != nullptr) l_run += fast_exp2(fmaf(win.rule.sinks[h], 1.4426950408889634f, -m_thr[g]));
+          gain = win.rule.out_scale * rule_gate<__nv_bfloat16>(win.rule, b, h, min(tid, width - 1));
         }
       }
       if (splits == 1) {
@@ -439,49 +457,9 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
   if (warp == 0) tmem_dealloc(tmem_base, S::TMEM_COLS);
 }
 
-// out[b, h, :] = sum_s o_s exp(m_s - M) / sum_s l_s exp(m_s - M) over the splits of one (request, head).
-// dv: width of an output head (= D, or less where the kernel padded it). sinks / out_scale: as in DecWindow.
-__global__ void decode_attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                           __nv_bfloat16* __restrict__ out, int D, int dv, int splits, int out_stride, int Hq,
-                                           const float* __restrict__ sinks, float out_scale) {
-  pdl_wait();
-  pdl_launch_dependents();
-  const int bh = blockIdx.x, b = bh / Hq, h = bh % Hq;
-  const float* ml = part_ml + static_cast<size_t>(bh) * splits * 2;
-  float gm = -INFINITY;
-  for (int s = 0; s < splits; ++s) gm = fmaxf(gm, ml[2 * s]);
-  float gl = 0.f;
-  for (int s = 0; s < splits; ++s)
-    if (ml[2 * s] != -INFINITY) gl += ml[2 * s + 1] * __expf(ml[2 * s] - gm);
-  if (sinks != nullptr) gl += __expf(sinks[h] - gm);
-  const float inv = gl > 0.f ? out_scale / gl : 0.f;
-  for (int d = threadIdx.x; d < dv; d += blockDim.x) {
-    float o = 0.f;
-    for (int s = 0; s < splits; ++s)
-      if (ml[2 * s] != -INFINITY) o += part_o[(static_cast<size_t>(bh) * splits + s) * D + d] * __expf(ml[2 * s] - gm);
-    out[static_cast<size_t>(b) * out_stride + static_cast<size_t>(h) * dv + d] = __float2bfloat16(o * inv);
-  }
-}
-
 // [num_slots, Hkv, D] bf16 cache as a 3-D tensor map; box = one page of one head, 64 elements (128 B) wide.
 static CUtensorMap make_cache_tmap(const void* base, int num_slots, int Hkv, int D, int page_size) {
-  CUtensorMap m;
-  cuuint64_t dims[3] = {(cuuint64_t)D, (cuuint64_t)Hkv, (cuuint64_t)num_slots};
-  cuuint64_t strides[2] = {(cuuint64_t)D * 2, (cuuint64_t)Hkv * D * 2};
-  cuuint32_t box[3] = {64, 1, (cuuint32_t)page_size};
-  cuuint32_t estr[3] = {1, 1, 1};
-  static thread_local bool ctx_bound = false;  // the encoder needs the primary context current on this thread
-  if (!ctx_bound) {
-    int dev = 0;
-    if (cudaGetDevice(&dev) == cudaSuccess && cudaSetDevice(dev) == cudaSuccess) ctx_bound = true;
-  }
-  CUresult r = get_encode_tiled()(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr,
-                                  CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
-                                  CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  if (r != CUDA_SUCCESS)
-    throw std::runtime_error("cuTensorMapEncodeTiled (kv cache) failed: " + std::to_string(int(r)) + " slots=" +
-                             std::to_string(num_slots) + " Hkv=" + std::to_string(Hkv) + " D=" + std::to_string(D));
-  return m;
+  return make_tmap_3d(base, D, Hkv, num_slots, D, uint64_t(Hkv) * D, 64, 1, page_size);
 }
 
 template <int D, int G, typename Win = DecFull>
@@ -528,8 +506,8 @@ extern "C" int sb_paged_decode_tc(const void* q, const void* k_cache, const void
 #undef SB_DA
     if (rc != 0) return rc;
     if (splits > 1)
-      return (int)sb::launch_pdl(sb::decode_attn_combine_kernel, dim3(B * Hq), dim3(64), 0, s, part_o, part_ml, (bf16*)out, D,
-                                 D, splits, out_stride, Hq, static_cast<const float*>(nullptr), 1.f);
+      return (int)sb::launch_pdl(sb::attn_combine_kernel, dim3(B * Hq), dim3(64), 0, s, part_o, part_ml, (bf16*)out, D, D, splits,
+                                 out_stride, Hq, sb::plain_rule());
     return (int)cudaGetLastError();
   } catch (const std::exception& e) {
     sb::set_last_error(e.what());
@@ -541,13 +519,13 @@ extern "C" int sb_paged_decode_tc(const void* q, const void* k_cache, const void
 // pitch q_stride, out [B, Hq * DV]; part_o [B, Hq, splits, W] / part_ml [B, Hq, splits, 2] with W = 64 when both widths are at
 // most 64, else 128. Returns -1 for widths above 128 or no multiple of 8, groups above 16 heads, or a misaligned pointer.
 extern "C" int sb_paged_decode_window(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
-                                      const int* seq_lens, const float* slopes, const float* sinks, void* out, float* part_o, float* part_ml, int B,
-                                      int Hq, int Hkv, int DK, int DV, int page_size, int max_pages, int num_slots, int q_stride,
-                                      int out_stride, int splits, float scale, float out_scale, int window, int keep_first,
-                                      int* status, cudaStream_t s) {
+                                      const int* seq_lens, void* out, float* part_o, float* part_ml, int B, int Hq, int Hkv,
+                                      int DK, int DV, int page_size, int max_pages, int num_slots, int q_stride, int out_stride,
+                                      int splits, const void* attn_rule, int* status, cudaStream_t s) {
   using bf16 = __nv_bfloat16;
+  const sb::AttnRule* rule = (const sb::AttnRule*)attn_rule;
   if (B == 0) return 0;
-  if (Hkv <= 0 || Hq % Hkv != 0 || window < 1 || keep_first < 0 || splits < 1) return (int)cudaErrorInvalidValue;
+  if (Hkv <= 0 || Hq % Hkv != 0 || !rule_ok(rule) || splits < 1) return (int)cudaErrorInvalidValue;
   const int G = Hq / Hkv;
   if (G > 16 || DK <= 0 || DV <= 0 || DK > 128 || DV > 128 || DK % 8 || DV % 8) return -1;
   int page_shift = 0;
@@ -559,21 +537,21 @@ extern "C" int sb_paged_decode_window(const void* q, const void* k_cache, const 
   try {
     const CUtensorMap tk = sb::make_cache_tmap(k_cache, num_slots, Hkv, DK, page_size);
     const CUtensorMap tv = sb::make_cache_tmap(v_cache, num_slots, Hkv, DV, page_size);
-    const sb::DecWindow win{slopes, sinks, out_scale, window, keep_first, G, DK, DV};
+    const sb::DecWindow win{*rule, G, DK, DV};
     const dim3 grid(B, Hkv, splits);
     int rc = -1;
 #define SB_DW(WV, GV)                                                                                                       \
   if (rc == -1 && W == WV && G <= GV)                                                                                       \
     rc = sb::launch_decode_attn<WV, GV, sb::DecWindow>(grid, s, tk, tv, (const bf16*)q, block_table, seq_lens, (bf16*)out, part_o, \
                                                        part_ml, Hq, Hkv, page_size, page_shift, max_pages, q_stride, out_stride,   \
-                                                       splits, scale, status, win);
+                                                       splits, rule->scale, status, win);
     SB_DW(64, 1) SB_DW(64, 2) SB_DW(64, 4) SB_DW(64, 8) SB_DW(64, 16)
     SB_DW(128, 1) SB_DW(128, 2) SB_DW(128, 4) SB_DW(128, 8) SB_DW(128, 16)
 #undef SB_DW
     if (rc != 0) return rc;
     if (splits > 1)
-      return (int)sb::launch_pdl(sb::decode_attn_combine_kernel, dim3(B * Hq), dim3(64), 0, s, part_o, part_ml, (bf16*)out, W, DV,
-                                 splits, out_stride, Hq, sinks, out_scale);
+      return (int)sb::launch_pdl(sb::attn_combine_kernel, dim3(B * Hq), dim3(64), 0, s, part_o, part_ml, (bf16*)out, W, DV, splits,
+                                 out_stride, Hq, *rule);
     return (int)cudaGetLastError();
   } catch (const std::exception& e) {
     sb::set_last_error(e.what());

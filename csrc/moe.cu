@@ -87,11 +87,11 @@ moe_route_weight_grad_kernel(const __nv_bfloat16* __restrict__ rows, const int* 
 //   mode 1  weights = softmax over all experts, pick the k largest, no renormalisation
 //   mode 2  scores = sigmoid(logit); pick by score + bias (bias only steers the choice); weights = picked scores,
 //           divided by their sum when `renorm`
-// then weights *= scale. Ties go to the lower expert index. E <= 512.
+// then weights *= scale. Ties go to the lower expert index. E <= 512. `shift` [E] (or null) is added to the logits first.
 constexpr int TOPK_MAX_PER_LANE = 16;
 __global__ void __launch_bounds__(256)
-moe_topk_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int* __restrict__ idx, float* __restrict__ wts,
-                long T, int E, long ld, int k, int mode, int renorm, float scale) {
+moe_topk_kernel(const float* __restrict__ logits, const float* __restrict__ shift, const float* __restrict__ bias,
+                int* __restrict__ idx, float* __restrict__ wts, long T, int E, long ld, int k, int mode, int renorm, float scale) {
   const int lane = threadIdx.x & 31;
   for (long t = static_cast<long>(blockIdx.x) * 8 + (threadIdx.x >> 5); t < T; t += static_cast<long>(gridDim.x) * 8) {
     float raw[TOPK_MAX_PER_LANE], sel[TOPK_MAX_PER_LANE];
@@ -99,7 +99,7 @@ moe_topk_kernel(const float* __restrict__ logits, const float* __restrict__ bias
 #pragma unroll
     for (int i = 0; i < TOPK_MAX_PER_LANE; ++i) {
       const int e = lane + 32 * i;
-      raw[i] = e < E ? logits[t * ld + e] : -INFINITY;
+      raw[i] = e < E ? logits[t * ld + e] + (shift != nullptr ? shift[e] : 0.f) : -INFINITY;
       mx = fmaxf(mx, raw[i]);
     }
     mx = warp_max(mx);
@@ -305,12 +305,12 @@ extern "C" int sb_moe_route_weight_grad(const void* rows, const int* dest, const
 }
 
 // logits [T, E] fp32 (row pitch ld); bias [E] fp32 or null; idx [T, k] int32; weights [T, k] fp32. k <= 32.
-extern "C" int sb_moe_topk(const float* logits, const float* bias, int* idx, float* weights, long T, int E, long ld, int k, int mode,
-                           int renorm, float scale, cudaStream_t s) {
+extern "C" int sb_moe_topk(const float* logits, const float* shift, const float* bias, int* idx, float* weights, long T, int E, long ld,
+                           int k, int mode, int renorm, float scale, cudaStream_t s) {
   if (T == 0) return 0;
   if (E <= 0 || E > 32 * sb::TOPK_MAX_PER_LANE || k <= 0 || k > 32 || k > E || mode < 0 || mode > 2)
     return (int)cudaErrorInvalidValue;
-  sb::moe_topk_kernel<<<sb::moe_blocks(T), 256, 0, s>>>(logits, bias, idx, weights, T, E, ld, k, mode, renorm, scale);
+  sb::moe_topk_kernel<<<sb::moe_blocks(T), 256, 0, s>>>(logits, shift, bias, idx, weights, T, E, ld, k, mode, renorm, scale);
   return (int)cudaGetLastError();
 }
 

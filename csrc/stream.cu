@@ -4,7 +4,10 @@
 //                     and starts the stream; a second table can add a row chosen by (previous token, token).
 //   * sb_glu          activation of a feed-forward, gated or not (silu, tanh-gelu, squared relu)
 //   * sb_kv_scatter   new key / value rows into their cache slots, widths and element size free
-//   * sb_heads        per-head RMS norm and rotation of new queries and keys; keys and values into their cache slots
+//   * sb_heads        RMS norm (per head, or over all heads at once) and rotation of new queries and keys; keys and values into
+//                     their cache slots
+//   * sb_latent_place norms of a token's query and key/value latents, rotation of its shared key part, cache write
+//   * sb_latent_turn  rotation of the rotated part of latent queries, in place or beside absorbed queries
 // Element types are bf16 or fp32 throughout (fp32: the engine's full-precision mode); all arithmetic is fp32.
 #include "common.cuh"
 
@@ -63,6 +66,8 @@ struct StreamNorm {
   void* h;               // [T, H] normed input of the next sub-layer
   int k, y_rows, gate_ld, init, layer_norm, H;  // init: the stream starts here (res is written, not added to)
   float eps, w_off;      // w_off is added to every norm weight
+  const float* plus;     // [T, H] fp32 added to the sub-layer output (a mixer's, beside the experts), or null
+  float h_scale;         // factor of h
   // second embedding table: row (prev * mul_prev + token * mul_cur) mod pair_rows is added to the sub-layer output, row
   // pair_rows where there is no previous token (prev < 0)
   const void* pair;      // same type as y, or null
@@ -165,6 +170,12 @@ __global__ void __launch_bounds__(THREADS) stream_norm_kernel(const __grid_const
 #pragma unroll
         for (int i = 0; i < VEC; ++i) v[j][i] = 0.f;
       }
+      if (a.plus != nullptr) {
+        float e[VEC];
+        load_vec<float, VEC>(a.plus + row * H + off, e);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[j][i] += e[i];
+      }
       if (pair != nullptr) {
         float e[VEC];
         load_vec<TY, VEC>(pair + off, e);
@@ -196,6 +207,8 @@ __global__ void __launch_bounds__(THREADS) stream_norm_kernel(const __grid_const
 #pragma unroll
     for (int j = 0; j < MAXI; ++j) {
       const int c = threadIdx.x + j * THREADS;
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) o[j][i] *= a.h_scale;
       if (c < nvec) store_vec<TW, VEC>(h + row * H + static_cast<size_t>(c) * VEC, o[j]);
     }
   }
@@ -330,6 +343,169 @@ __global__ void __launch_bounds__(128) heads_kernel(const __grid_constant__ Head
   }
 }
 
+// The same with one norm over all query heads and one over all key heads (a weight per channel): one CTA per token, its rows
+// staged in shared memory as they came. sums: [T, 2] sums of squares of the whole projections (tensor-parallel ranks hold
+// parts of them) with q_all / k_all channels; null: computed here.
+struct HeadsAll {
+  Heads h;
+  const float* sums;
+  int q_all, k_all;
+};
+constexpr int HEADS_ALL_THREADS = 256;
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(HEADS_ALL_THREADS) heads_all_kernel(const __grid_constant__ HeadsAll p) {
+  const Heads& a = p.h;
+  extern __shared__ __align__(16) unsigned char raw_s[];
+  T* x = reinterpret_cast<T*>(raw_s);
+  __shared__ float scratch[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const long t = blockIdx.x;
+  const int nq = a.Hq * a.D, nk = a.Hkv * a.D, nv = a.Hkv * a.DV;
+  const T* q = reinterpret_cast<const T*>(a.q) + t * a.q_pitch;
+  const T* k = reinterpret_cast<const T*>(a.k) + t * a.k_pitch;
+  float sq = 0.f, sk = 0.f;
+  for (int c = threadIdx.x * VEC; c < nq + nk; c += HEADS_ALL_THREADS * VEC) {
+    float e[VEC];
+    load_vec<T, VEC>(c < nq ? q + c : k + (c - nq), e);
+    store_vec<T, VEC>(x + c, e);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) (c < nq ? sq : sk) += e[i] * e[i];
+  }
+  if (p.sums != nullptr) {
+    sq = p.sums[2 * t];
+    sk = p.sums[2 * t + 1];
+    __syncthreads();
+  } else {
+    sq = block_sum<HEADS_ALL_THREADS>(sq, scratch);
+    sk = block_sum<HEADS_ALL_THREADS>(sk, scratch);
+  }
+  const float rq = 1.f / sqrtf(sq / p.q_all + a.eps), rk = 1.f / sqrtf(sk / p.k_all + a.eps);
+  const int slot = a.slots[t];
+  const int half = a.dims / 2;
+  const float* cs = half > 0 ? a.table + static_cast<long>(a.positions[t]) * a.dims : nullptr;
+  T* q_out = reinterpret_cast<T*>(a.q) + t * a.q_pitch;
+  T* k_out = reinterpret_cast<T*>(a.k_cache) + static_cast<long>(slot < 0 ? 0 : slot) * nk;
+  for (int c = threadIdx.x * VEC; c < nq + nk; c += HEADS_ALL_THREADS * VEC) {
+    const bool is_q = c < nq;
+    if (!is_q && slot < 0) break;
+    const T* w = reinterpret_cast<const T*>(is_q ? a.q_norm : a.k_norm) + (is_q ? c : c - nq);
+    const float r = is_q ? rq : rk;
+    float y[VEC], g[VEC];
+    load_vec<T, VEC>(x + c, y);
+    load_vec<T, VEC>(w, g);
+    const int d0 = (is_q ? c : c - nq) % a.D;  // VEC divides D: a vector lies in one head
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+      y[i] *= r * g[i];
+      const int d = d0 + i;
+      if (d < a.dims) {
+        const int pair = a.interleaved ? d >> 1 : (d < half ? d : d - half);
+        const bool second = a.interleaved ? d & 1 : d >= half;
+        const int away = a.interleaved ? (d ^ 1) - d : (second ? -half : half);
+        const float other = to_f(x[c + i + away]) * r * to_f(w[i + away]);
+        y[i] = second ? fmaf(other, cs[half + pair], y[i] * cs[pair]) : fmaf(-other, cs[half + pair], y[i] * cs[pair]);
+      }
+    }
+    store_vec<T, VEC>(is_q ? q_out + c : k_out + (c - nq), y);
+  }
+  if (slot < 0) return;
+  const T* v = reinterpret_cast<const T*>(a.v) + t * a.v_pitch;
+  T* v_out = reinterpret_cast<T*>(a.v_cache) + static_cast<long>(slot) * nv;
+  for (int c = threadIdx.x * VEC; c < nv; c += HEADS_ALL_THREADS * VEC) {
+    float e[VEC];
+    load_vec<T, VEC>(v + c, e);
+    store_vec<T, VEC>(v_out + c, e);
+  }
+}
+
+template <typename T>
+static int launch_heads_all(const HeadsAll& p, int T_, bool vec, cudaStream_t s) {
+  const int bytes = (p.h.Hq + p.h.Hkv) * p.h.D * static_cast<int>(sizeof(T));
+  auto kern = vec ? heads_all_kernel<T, 8> : heads_all_kernel<T, 1>;
+  if (bytes > 200 * 1024) return (int)cudaErrorInvalidValue;
+  if (bytes > 40 * 1024)
+    if (cudaError_t e = ensure_dynamic_smem(reinterpret_cast<const void*>(kern), 200 * 1024); e != cudaSuccess) return (int)e;
+  return (int)launch_pdl(kern, dim3(T_), dim3(HEADS_ALL_THREADS), bytes, s, p);
+}
+
+// Latent attention, one CTA per token: the query latent dq [T, R1] is RMS normed into q_out; of dkv [T, R2 + dims] the first R2
+// are RMS normed and the last `dims` turned, both into cache row slots[t] (< 0: nowhere) of width R2 + dims.
+struct LatentPlace {
+  const void *dq, *dkv, *q_norm, *kv_norm;
+  const float* table;
+  const int *positions, *slots;
+  void *q_out, *cache;
+  int R1, R2, dims, interleaved;
+  long dq_pitch, dkv_pitch;
+  float eps;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(128) latent_place_kernel(const __grid_constant__ LatentPlace a) {
+  __shared__ float scratch[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const long t = blockIdx.x;
+  const T* dq = reinterpret_cast<const T*>(a.dq) + t * a.dq_pitch;
+  const T* dkv = reinterpret_cast<const T*>(a.dkv) + t * a.dkv_pitch;
+  float sq = 0.f, sk = 0.f;
+  for (int c = threadIdx.x; c < a.R1; c += 128) {
+    const float e = to_f(dq[c]);
+    sq = fmaf(e, e, sq);
+  }
+  for (int c = threadIdx.x; c < a.R2; c += 128) {
+    const float e = to_f(dkv[c]);
+    sk = fmaf(e, e, sk);
+  }
+  const float rq = 1.f / sqrtf(block_sum<128>(sq, scratch) / a.R1 + a.eps);
+  const float rk = 1.f / sqrtf(block_sum<128>(sk, scratch) / a.R2 + a.eps);
+  const T* wq = reinterpret_cast<const T*>(a.q_norm);
+  T* q_out = reinterpret_cast<T*>(a.q_out) + t * a.R1;
+  for (int c = threadIdx.x; c < a.R1; c += 128) q_out[c] = from_f<T>(to_f(dq[c]) * rq * to_f(wq[c]));
+  const int slot = a.slots[t];
+  if (slot < 0) return;
+  const T* wk = reinterpret_cast<const T*>(a.kv_norm);
+  T* out = reinterpret_cast<T*>(a.cache) + static_cast<long>(slot) * (a.R2 + a.dims);
+  const int half = a.dims / 2;
+  const float* cs = a.table + static_cast<long>(a.positions[t]) * a.dims;
+  for (int c = threadIdx.x; c < a.R2 + half; c += 128) {
+    if (c < a.R2) {
+      out[c] = from_f<T>(to_f(dkv[c]) * rk * to_f(wk[c]));
+      continue;
+    }
+    const int i = c - a.R2, d0 = a.R2 + (a.interleaved ? 2 * i : i), d1 = a.R2 + (a.interleaved ? 2 * i + 1 : i + half);
+    const float u = to_f(dkv[d0]), v = to_f(dkv[d1]), cosv = cs[i], sinv = cs[half + i];
+    out[d0] = from_f<T>(u * cosv - v * sinv);
+    out[d1] = from_f<T>(v * cosv + u * sinv);
+  }
+}
+
+// Rotated part of latent queries: the last `dims` coordinates of every head of q [T, H, D + dims] are turned and written to the
+// first `dims` coordinates behind dst [T, H, ...] (which may be the queries themselves). One thread per pair.
+template <typename T>
+__global__ void __launch_bounds__(256)
+latent_turn_kernel(const T* __restrict__ q, T* __restrict__ dst, const float* __restrict__ table, const int* __restrict__ positions,
+                   long pairs, int H, int D, int dims, int interleaved, long q_pitch, long q_head, long dst_pitch, long dst_head) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int half = dims / 2;
+  for (long n = static_cast<long>(blockIdx.x) * 256 + threadIdx.x; n < pairs; n += static_cast<long>(gridDim.x) * 256) {
+    const int i = static_cast<int>(n % half);
+    const long th = n / half;
+    const int h = static_cast<int>(th % H);
+    const long t = th / H;
+    const float* cs = table + static_cast<long>(positions[t]) * dims;
+    const int d0 = interleaved ? 2 * i : i, d1 = interleaved ? 2 * i + 1 : i + half;
+    const T* src = q + t * q_pitch + h * q_head + D;
+    T* out = dst + t * dst_pitch + h * dst_head;
+    const float u = to_f(src[d0]), v = to_f(src[d1]);
+    out[d0] = from_f<T>(u * cs[i] - v * cs[half + i]);
+    out[d1] = from_f<T>(v * cs[i] + u * cs[half + i]);
+  }
+}
+
 }  // namespace sb
 
 extern "C" int sb_heads(void* q, const void* k, const void* v, const void* q_norm, const void* k_norm, const float* table,
@@ -344,18 +520,58 @@ extern "C" int sb_heads(void* q, const void* k, const void* v, const void* q_nor
   return (int)sb::launch_pdl(sb::heads_kernel<__nv_bfloat16>, grid, dim3(128), 0, s, a);
 }
 
+// As sb_heads, with norms over all query heads and over all key heads (see HeadsAll).
+extern "C" int sb_heads_all(void* q, const void* k, const void* v, const void* q_norm, const void* k_norm, const float* table,
+                            const int* positions, const int* slots, void* k_cache, void* v_cache, int T, int Hq, int Hkv, int D, int DV,
+                            int dims, int interleaved, long q_pitch, long k_pitch, long v_pitch, const float* sums, int q_all, int k_all,
+                            float eps, int f32, cudaStream_t s) {
+  if (T == 0) return 0;
+  if (D <= 0 || DV <= 0 || dims < 0 || dims > D || dims % 2 || Hq <= 0 || Hkv <= 0 || q_norm == nullptr || k_norm == nullptr)
+    return (int)cudaErrorInvalidValue;
+  const sb::HeadsAll p{{q, k, v, q_norm, k_norm, table, positions, slots, k_cache, v_cache, Hq, Hkv, D, DV, dims, interleaved, q_pitch, k_pitch,
+                        v_pitch, eps}, sums, q_all, k_all};
+  bool vec = D % 8 == 0 && DV % 8 == 0 && q_pitch % 8 == 0 && k_pitch % 8 == 0 && v_pitch % 8 == 0;
+  for (const void* x : {static_cast<const void*>(q), k, v, q_norm, k_norm, static_cast<const void*>(k_cache), static_cast<const void*>(v_cache)})
+    vec = vec && (reinterpret_cast<uintptr_t>(x) & 15) == 0;
+  return f32 ? sb::launch_heads_all<float>(p, T, vec, s) : sb::launch_heads_all<__nv_bfloat16>(p, T, vec, s);
+}
+
+extern "C" int sb_latent_place(const void* dq, const void* dkv, const void* q_norm, const void* kv_norm, const float* table,
+                               const int* positions, const int* slots, void* q_out, void* cache, int T, int R1, int R2, int dims,
+                               int interleaved, long dq_pitch, long dkv_pitch, float eps, int f32, cudaStream_t s) {
+  if (T == 0) return 0;
+  if (R1 <= 0 || R2 <= 0 || dims <= 0 || dims % 2) return (int)cudaErrorInvalidValue;
+  const sb::LatentPlace a{dq, dkv, q_norm, kv_norm, table, positions, slots, q_out, cache, R1, R2, dims, interleaved, dq_pitch, dkv_pitch, eps};
+  if (f32) return (int)sb::launch_pdl(sb::latent_place_kernel<float>, dim3(T), dim3(128), 0, s, a);
+  return (int)sb::launch_pdl(sb::latent_place_kernel<__nv_bfloat16>, dim3(T), dim3(128), 0, s, a);
+}
+
+extern "C" int sb_latent_turn(const void* q, void* dst, const float* table, const int* positions, int T, int H, int D, int dims,
+                              int interleaved, long q_pitch, long q_head, long dst_pitch, long dst_head, int f32, cudaStream_t s) {
+  if (T == 0) return 0;
+  if (H <= 0 || D < 0 || dims <= 0 || dims % 2) return (int)cudaErrorInvalidValue;
+  const long pairs = static_cast<long>(T) * H * (dims / 2), want = (pairs + 255) / 256;
+  const dim3 grid(static_cast<unsigned>(want < 148 * 16 ? want : 148 * 16));
+  using bf16 = __nv_bfloat16;
+  if (f32)
+    return (int)sb::launch_pdl(sb::latent_turn_kernel<float>, grid, dim3(256), 0, s, (const float*)q, (float*)dst, table, positions, pairs, H,
+                               D, dims, interleaved, q_pitch, q_head, dst_pitch, dst_head);
+  return (int)sb::launch_pdl(sb::latent_turn_kernel<bf16>, grid, dim3(256), 0, s, (const bf16*)q, (bf16*)dst, table, positions, pairs, H, D,
+                             dims, interleaved, q_pitch, q_head, dst_pitch, dst_head);
+}
+
 // Types: y_f32 / w_f32 (norm weights and h) = 1 for fp32, 0 for bf16; fp32 weights need fp32 y. H <= 8192.
 extern "C" int sb_stream_norm(const void* y, int y_f32, const int* ids, int y_rows, const int* dest, const float* wts, int k,
                               const void* shared, const float* gate, int gate_ld, const void* post_w, float* res, int init,
                               const void* pre_w, void* h, int w_f32, int T, int H, float eps, float w_off, int layer_norm,
                               const void* pair, const int* pair_ids, const int* prev, long mul_prev, long mul_cur, int pair_rows,
-                              cudaStream_t s) {
+                              const float* plus, float h_scale, cudaStream_t s) {
   if (T == 0) return 0;
   if (H <= 0 || H > 8192 || (w_f32 && !y_f32) || (pair != nullptr && pair_rows <= 0)) return (int)cudaErrorInvalidValue;
   sb::StreamNorm a{y, ids, dest, wts, shared, gate, post_w, res, pre_w, h, k, y_rows, gate_ld, init, layer_norm, H, eps, w_off,
-                   pair, pair_ids, prev, mul_prev, mul_cur, pair_rows};
+                   plus, h_scale, pair, pair_ids, prev, mul_prev, mul_cur, pair_rows};
   bool vec = H % 8 == 0;
-  for (const void* p : {y, pair, shared, post_w, static_cast<const void*>(res), pre_w, static_cast<const void*>(h)})
+  for (const void* p : {y, pair, shared, post_w, static_cast<const void*>(plus), static_cast<const void*>(res), pre_w, static_cast<const void*>(h)})
     vec = vec && (reinterpret_cast<uintptr_t>(p) & 15) == 0;
   if (w_f32) return sb::launch_stream_norm<float, float>(a, T, vec, s);
   if (y_f32) return sb::launch_stream_norm<float, __nv_bfloat16>(a, T, vec, s);

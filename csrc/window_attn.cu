@@ -2,16 +2,16 @@
 // fp32 storage. It is the full-precision form of the tensor-core kernels (flash_window_sm100.cu for prompts,
 // decode_attn_sm100.cu for single tokens) and takes the shapes they do not cover.
 //
-// Query row t belongs to request row_req[t] (null: request t) and stands at position row_pos[t]; it sees the keys j <= pos
-// with pos - j < window or j < keep_first, and its scores are  scale * q.k - slope[head] * (pos - j).
-// sinks: score of an extra softmax column without a value, per head (null: none). The output is multiplied by out_scale.
-// Cache layout as everywhere: [num_slots, Hkv, D], slot = page * page_size + offset, pages from block_table[request].
-#include "common.cuh"
+// Query row t belongs to request row_req[t] (null: request t) and stands at position row_pos[t]; attn_rule.cuh says what it
+// sees and how its scores are made.
+// Cache layout as everywhere: [num_slots, Hkv, D], slot = page * page_size + offset, pages from block_table[request]; v_pitch:
+// elements between the value rows (a latent cache keeps one vector per token whose first DV elements are the value).
+#include "attn_rule.cuh"
 
 namespace sb {
 
 constexpr int WA_WARPS = 4;
-constexpr int WA_MAX_D = 512;
+constexpr int WA_MAX_D = 1024;
 constexpr int WA_ACC = WA_MAX_D / 32;
 
 __device__ __forceinline__ float wa_load(const float* p) { return *p; }
@@ -23,9 +23,8 @@ template <typename T>
 __global__ void __launch_bounds__(WA_WARPS * 32)
 window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                    const int* __restrict__ block_table, const int* __restrict__ row_req, const int* __restrict__ row_pos,
-                   const float* __restrict__ slopes, const float* __restrict__ sinks, T* __restrict__ out, int Hq, int Hkv, int D, int DV, int page_size,
-                   int max_pages, long q_stride, long out_stride, float scale, float out_scale, int window,
-                   int keep_first) {
+                   T* __restrict__ out, int Hq, int Hkv, int D, int DV, int page_size, int max_pages, long q_stride, long out_stride,
+                   long v_pitch, const AttnRule rule) {
   __shared__ float q_s[WA_WARPS][WA_MAX_D];
   pdl_wait();
   pdl_launch_dependents();
@@ -36,15 +35,15 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const
   const int kvh = h / (Hq / Hkv);
   const int pos = row_pos[t];
   const int* bt = block_table + static_cast<long>(row_req != nullptr ? row_req[t] : t) * max_pages;
-  const float slope = slopes != nullptr ? slopes[h] : 0.f;
+  const float slope = rule.slopes != nullptr ? rule.slopes[h] : 0.f;
   for (int d = lane; d < D; d += 32) q_s[warp][d] = wa_load(q + t * q_stride + static_cast<long>(h) * D + d);
   __syncwarp();
 
   float m = -INFINITY, l = 0.f, acc[WA_ACC];
 #pragma unroll
   for (int i = 0; i < WA_ACC; ++i) acc[i] = 0.f;
-  const int lo = window > pos ? 0 : pos - window + 1;  // first key of the window
-  const int kept = min(keep_first, lo);                // kept keys in front of it
+  const int lo = rule_first_key(rule, pos);  // first key of the window
+  const int kept = min(rule.keep_first, lo);  // kept keys in front of it
   const int nkeys = kept + (pos - lo + 1);
   for (int n0 = 0; n0 < nkeys; n0 += 32) {
     const int n = n0 + lane;
@@ -56,7 +55,10 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const
       const T* kr = k_cache + (slot * Hkv + kvh) * D;
       float dot = 0.f;
       for (int d = 0; d < D; ++d) dot = fmaf(q_s[warp][d], wa_load(kr + d), dot);
-      s = dot * scale - slope * static_cast<float>(pos - key);
+      s = dot * rule.scale;
+      if (rule.softcap > 0.f) s = rule.softcap * tanhf(s / rule.softcap);
+      if (rule.bias != nullptr) s += rule.bias[static_cast<long>(min(pos - key, rule.bias_rows - 1)) * Hq + h];
+      s -= slope * static_cast<float>(pos - key);
     }
     const float nm = fmaxf(m, warp_max(s));
     const float p = n < nkeys ? expf(s - nm) : 0.f;
@@ -69,35 +71,39 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const
     for (int j = 0; j < cnt; ++j) {
       const float pj = __shfl_sync(0xffffffffu, p, j);
       const long sj = __shfl_sync(0xffffffffu, slot, j);
-      const T* vr = v_cache + (sj * Hkv + kvh) * DV;
+      const T* vr = v_cache + (sj * Hkv + kvh) * v_pitch;
 #pragma unroll
       for (int i = 0; i < WA_ACC; ++i)
         if (lane + 32 * i < DV) acc[i] = fmaf(pj, wa_load(vr + lane + 32 * i), acc[i]);
     }
   }
-  if (sinks != nullptr) l += expf(sinks[h] - m);
-  const float inv = out_scale / l;  // a row always sees its own key: l > 0
+  if (rule.sinks != nullptr) l += expf(rule.sinks[h] - m);
+  const float inv = rule.out_scale / l;  // a row always sees its own key: l > 0
+  const T* gate = reinterpret_cast<const T*>(rule.gate) + (rule.gate != nullptr ? t * rule.gate_pitch + static_cast<long>(h) * rule.gate_width : 0);
 #pragma unroll
-  for (int i = 0; i < WA_ACC; ++i)
-    if (lane + 32 * i < DV) wa_store(out + t * out_stride + static_cast<long>(h) * DV + lane + 32 * i, acc[i] * inv);
+  for (int i = 0; i < WA_ACC; ++i) {
+    const int d = lane + 32 * i;
+    if (d >= DV) continue;
+    const float g = rule.gate != nullptr ? sigmoid_f(wa_load(gate + (rule.gate_width > 1 ? d : 0))) : 1.f;
+    wa_store(out + t * out_stride + static_cast<long>(h) * DV + d, acc[i] * inv * g);
+  }
 }
 
 }  // namespace sb
 
 extern "C" int sb_window_attn(const void* q, const void* k_cache, const void* v_cache, const int* block_table, const int* row_req,
-                              const int* row_pos, const float* slopes, const float* sinks, void* out, int T, int Hq, int Hkv, int D, int DV,
-                              int page_size, int max_pages, long q_stride, long out_stride, float scale, float out_scale,
-                              int window, int keep_first, int f32, cudaStream_t s) {
+                              const int* row_pos, void* out, int T, int Hq, int Hkv, int D, int DV, int page_size, int max_pages,
+                              long q_stride, long out_stride, long v_pitch, const void* rule, int f32, cudaStream_t s) {
   if (T == 0) return 0;
-  if (Hkv <= 0 || Hq % Hkv != 0 || D <= 0 || DV <= 0 || D > sb::WA_MAX_D || DV > sb::WA_MAX_D || window < 1 || keep_first < 0)
-    return (int)cudaErrorInvalidValue;
+  const sb::AttnRule* r = (const sb::AttnRule*)rule;
+  if (Hkv <= 0 || Hq % Hkv != 0 || D <= 0 || DV <= 0 || D > sb::WA_MAX_D || DV > sb::WA_MAX_D || !rule_ok(r)) return (int)cudaErrorInvalidValue;
   const dim3 grid(T, (Hq + sb::WA_WARPS - 1) / sb::WA_WARPS);
   using bf16 = __nv_bfloat16;
   if (f32)
     return (int)sb::launch_pdl(sb::window_attn_kernel<float>, grid, dim3(sb::WA_WARPS * 32), 0, s, (const float*)q, (const float*)k_cache,
-                               (const float*)v_cache, block_table, row_req, row_pos, slopes, sinks, (float*)out, Hq, Hkv, D, DV, page_size,
-                               max_pages, q_stride, out_stride, scale, out_scale, window, keep_first);
+                               (const float*)v_cache, block_table, row_req, row_pos, (float*)out, Hq, Hkv, D, DV, page_size, max_pages,
+                               q_stride, out_stride, v_pitch, *r);
   return (int)sb::launch_pdl(sb::window_attn_kernel<bf16>, grid, dim3(sb::WA_WARPS * 32), 0, s, (const bf16*)q, (const bf16*)k_cache,
-                             (const bf16*)v_cache, block_table, row_req, row_pos, slopes, sinks, (bf16*)out, Hq, Hkv, D, DV, page_size,
-                             max_pages, q_stride, out_stride, scale, out_scale, window, keep_first);
+                             (const bf16*)v_cache, block_table, row_req, row_pos, (bf16*)out, Hq, Hkv, D, DV, page_size, max_pages, q_stride,
+                             out_stride, v_pitch, *r);
 }

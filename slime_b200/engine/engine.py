@@ -122,7 +122,7 @@ class Engine:
         c, out = self.cfg, []
         for L in self.weights.layers + self.weights.draft:
             if L["kind"] == "specified":
-                out += [(a.kv_heads // self.weights.tp, a.dim, a.vdim) for a in cached_mixers(L)]
+                out += [a.cache_geometry(self.weights.tp) for a in cached_mixers(L)]
             elif not cached_mixers(L):
                 continue
             elif L["kind"] == "mla":

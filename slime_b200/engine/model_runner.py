@@ -21,8 +21,8 @@ from slime_b200.engine.kv_cache import PagedKVCache
 from slime_b200.engine.projections import LayerProjections
 from slime_b200.engine.state_cache import RecurrentStates
 from slime_b200.models.config import ModelConfig
-from slime_b200.models.layer_spec import AttentionSpec, DeltaSpec
-from slime_b200.ops import delta, stream
+from slime_b200.models.layer_spec import AttentionSpec, DeltaSpec, LatentSpec
+from slime_b200.ops import delta, latent, stream, window_attention
 
 logger = logging.getLogger(__name__)
 
@@ -36,11 +36,11 @@ _MIMO_DRAFT_RE = re.compile(r"^model\.mtp_layers\.(\d+)\.(.+)$")
 KV_KINDS = ("attention", "mla")  # layer kinds that keep keys and values in the paged cache
 
 
-def cached_mixers(L) -> list[AttentionSpec | None]:
+def cached_mixers(L) -> list[AttentionSpec | LatentSpec | None]:
     """What layer ``L`` keeps keys and values for: the attention mixers of a specified layer, one unnamed entry of another
     attention layer, nothing for a recurrent one."""
     if L["kind"] == "specified":
-        return [m for _, m, _ in L["spec"].branches() if isinstance(m, AttentionSpec)]
+        return [m for _, m, _ in L["spec"].branches() if not isinstance(m, DeltaSpec)]
     return [None] if L["kind"] in KV_KINDS else []
 
 
@@ -90,6 +90,7 @@ class EngineWeights:
         self.embed = e(self.vocab_local, h)
         self.lm_head = self.embed if cfg.tie_word_embeddings else e(self.vocab_local, h)
         self.final_norm = e(h)
+        self.embed_norm = e(h) if cfg.embed_norm else None
         self.bigram = e(cfg.bigram["buckets"] + 1, h) if cfg.bigram else None  # replicated over tensor-parallel ranks
         self._specified_tensors = None
         self.layers = []
@@ -187,22 +188,37 @@ class EngineWeights:
         if self.cfg.padded_vocab_size % tp:
             raise ValueError(f"a vocabulary of {self.cfg.padded_vocab_size} does not divide over {tp} tensor-parallel ranks")
         lay = LayerProjections(spec, tp)
-        attention_only = all(isinstance(x, AttentionSpec) for _, x, _ in spec.branches())
+        attention_only = not any(isinstance(x, DeltaSpec) for _, x, _ in spec.branches())
         L = {"kind": "specified", "spec": spec, "proj": lay}
         L.update({_NORMS[n]: e(h) for n in spec.norms(self.cfg.post_self_attn_layernorm)})
         # block-scaled fp8 covers plain attention projections; what enters a recurrence keeps its precision
         L["in"] = mat(lay.in_rows, h, parts=[r for r, _ in lay.ins.values() if r]) if attention_only else e(lay.in_rows, h)
         L["out"] = mat(h, lay.out_cols) if attention_only and len(lay.outs) == 1 else e(h, lay.out_cols)
-        f32 = lambda n: torch.zeros(n, dtype=torch.float32, device=self.device)  # noqa: E731
+        if lay.biased:
+            L["in_bias"] = e(lay.in_rows)
+        f32 = lambda *n: torch.zeros(*n, dtype=torch.float32, device=self.device)  # noqa: E731
         for p, x, _ in spec.branches():
+            if isinstance(x, LatentSpec):
+                n = x.heads // tp
+                L.update({p + "dq.norm": e(x.q_rank), p + "dkv.norm": e(x.kv_rank), p + "up_q": mat(n * (x.dim + x.rot_dim), x.q_rank),
+                          p + "up_kv": e(n * (x.dim + x.vdim), x.kv_rank)})  # fmt: skip
+                continue
             if isinstance(x, DeltaSpec):
                 L.update({p + "conv": e(x.channels // tp, x.conv), p + "A_log": f32(x.heads // tp), p + "dt_bias": f32(x.decays // tp),
                           p + "norm": e(x.vdim)})  # fmt: skip
                 if p in lay.low:
                     L[p + "low"] = e(lay.low[p][2], lay.low[p][1])
-            elif x.qk_norm:
-                L.update({p + "q.norm": e(x.dim), p + "k.norm": e(x.dim)})
-        if m is None or spec.parallel_ff:
+                continue
+            if x.qk_norm:
+                whole = x.norm_over == "projection"  # sharded like the projections
+                nq, nk = x.norm_widths()
+                L.update({p + "q.norm": e(nq // tp if whole else nq), p + "k.norm": e(nk // tp if whole else nk)})
+            if x.learned_bias is not None:
+                # the table as it is stored, and spread over distances: [distance, head], the last row for everything beyond
+                rows = x.learned_bias.by_distance()
+                L.update({p + "rel": e(x.learned_bias.rows, x.heads // tp), p + "rel_rows": torch.tensor(rows, device=self.device),
+                          p + "bias": f32(len(rows), x.heads // tp)})  # fmt: skip
+        if m is None or (spec.parallel_ff and m.experts is None):
             return L
         up = 2 if m.gated else 1
         if m.experts is None:
@@ -211,12 +227,14 @@ class EngineWeights:
             f = m.ff // tp
             L.update(gate_up=mat(up * f, h, parts=(f,)), down=mat(h, f))
             return L
-        if m.experts % self.ep or m.shared_ff % tp:
+        if m.experts % self.ep or (m.shared_ff % tp and not spec.parallel_ff):
             raise ValueError(f"{m.experts} experts / a shared expert of width {m.shared_ff} do not divide over {tp} ranks")
         el, fs = m.experts // self.ep, m.shared_ff // tp
         L.update(first_expert=0 if self.ep == 1 else self.rank * el, router=e(-(-(m.experts + 1) // 8) * 8, h),
                  w13=mat(el, up * m.ff, h, parts=(m.ff,)), w2=mat(el, h, m.ff))  # fmt: skip
-        if m.shared_ff:
+        if m.router_bias:
+            L["router_shift"] = f32(m.experts)
+        if m.shared_ff and not spec.parallel_ff:
             L.update(shared_gate_up=mat(up * fs, h, parts=(fs,)), shared_down=mat(h, fs))
         return L
 
@@ -224,20 +242,26 @@ class EngineWeights:
         """Checkpoint tensors (name -> full shape) of a model with ``layer_specs``."""
         if self._specified_tensors is None:
             h, v = self.cfg.hidden_size, self.cfg.vocab_size
-            out = {"embed": (v, h), "head": (v, h), "final.norm": (h,)}
+            out = {"embed": (v, h), "final.norm": (h,)}
+            if not self.cfg.tie_word_embeddings:
+                out["head"] = (v, h)
+            if self.cfg.embed_norm:
+                out["embed.norm"] = (h,)
             if self.cfg.bigram:
                 out["bigram"] = (self.cfg.bigram["buckets"] + 1, h)
             for i, s in enumerate(self.cfg.layer_specs):
                 m, p = s.mlp, f"l{i}."
                 out.update({p + n: (h,) for n in s.norms(self.cfg.post_self_attn_layernorm)})
                 out.update({p + n: shape for n, shape in LayerProjections(s).tensors(h).items()})
-                if m is None or s.parallel_ff:
+                if m is None or (s.parallel_ff and m.experts is None):
                     continue
                 stems = {p + "mlp": m.ff}
                 if m.experts is not None:
                     stems = {f"{p}mlp.e{e}": m.ff for e in range(m.experts)}
                     out[p + "mlp.router"] = (m.experts, h)
-                    if m.shared_ff:
+                    if m.router_bias:
+                        out[p + "mlp.router.b"] = (m.experts,)
+                    if m.shared_ff and not s.parallel_ff:
                         stems[p + "mlp.shared"] = m.shared_ff
                     if m.shared_gate:
                         out[p + "mlp.shared.sg"] = (1, h)
@@ -262,12 +286,28 @@ class EngineWeights:
             else:
                 self._put(L["out"], 0, h, 1, t, raw, scale=False)
             return True
+        if sub.endswith(".b") and sub[:-2] in lay.biased:
+            r0, rows = lay.ins[sub[:-2]]
+            L["in_bias"][r0 : r0 + rows].copy_(self._rows(t, rows))
+            return True
         for p, (_, _, _, parts) in lay.low.items():
             if sub in parts:
                 r0, rows, c0, cols = parts[sub]
                 L[p + "low"][r0 : r0 + rows, c0 : c0 + cols].copy_(self._rows(t, rows))
                 return True
         for p, m, _ in L["spec"].branches():
+            if isinstance(m, LatentSpec):
+                n = m.heads // self.tp
+                if sub in (p + "dq.norm", p + "dkv.norm"):
+                    L[sub].copy_(t)
+                elif sub == p + "uq":
+                    self._put(L[p + "up_q"], 0, n * (m.dim + m.rot_dim), 0, t, raw, scale=False)
+                elif sub in (p + "uk", p + "uv"):
+                    r0, rows = (0, n * m.dim) if sub == p + "uk" else (n * m.dim, n * m.vdim)
+                    L[p + "up_kv"][r0 : r0 + rows].copy_(self._rows(t, rows))
+                else:
+                    continue
+                return True
             if sub in (p + "q.conv", p + "k.conv", p + "v.conv"):
                 g, v = m.kv_heads // self.tp * m.dim, m.heads // self.tp * m.vdim
                 r0, rows = {"q": (0, g), "k": (g, g), "v": (2 * g, v)}[sub[len(p)]]
@@ -276,10 +316,18 @@ class EngineWeights:
             if sub in (p + "A_log", p + "dt_bias"):
                 L[sub].copy_(self._rows(raw, L[sub].numel()))
                 return True
+            if sub == p + "rel":
+                L[sub].copy_(t[:, self.rank * L[sub].shape[1] : (self.rank + 1) * L[sub].shape[1]])
+                self._spread_bias(L, p)
+                return True
             if sub in (p + "norm", p + "q.norm", p + "k.norm"):
-                L[sub].copy_(t)
+                L[sub].copy_(self._rows(t, L[sub].numel()) if L[sub].numel() != t.numel() else t)
                 return True
         return False
+
+    def _spread_bias(self, L, p: str):
+        """The learned distance bias by distance, from its table by bucket (in place: captured graphs keep its address)."""
+        L[p + "bias"].copy_(L[p + "rel"].float().index_select(0, L[p + "rel_rows"]))
 
     def _load_specified(self, L, sub: str, t, raw) -> bool:
         """One tensor of a specified layer, addressed by its name behind ``l<i>.`` (one of ``specified_tensors``)."""
@@ -297,6 +345,9 @@ class EngineWeights:
         else:
             if sub == "mlp.router":
                 L["router"][: m.experts].copy_(t)
+                return True
+            if sub == "mlp.router.b":
+                L["router_shift"].copy_(raw)
                 return True
             if sub == "mlp.shared.sg":
                 L["router"][m.experts].copy_(t.view(-1))
@@ -345,11 +396,13 @@ class EngineWeights:
         yield self.final_norm
         if self.bigram is not None:
             yield self.bigram
+        if self.embed_norm is not None:
+            yield self.embed_norm
         if self.vision is not None:
             yield from self.vision.parameters()
         for L in self.layers + self.draft:
             for v in L.values():
-                if isinstance(v, torch.Tensor):
+                if isinstance(v, torch.Tensor) and v.is_floating_point():
                     yield v
                 elif isinstance(v, Fp8Weight):  # a quantised matrix: its bytes and its scales
                     yield from v.tensors()
@@ -373,6 +426,9 @@ class EngineWeights:
                     self.layers[int(m.group(1))], m.group(2), t.to(self.device, self.dtype, non_blocking=True), t)
             if name == "bigram":
                 self.bigram.copy_(t.to(self.device, self.dtype))
+                return True
+            if name == "embed.norm":
+                self.embed_norm.copy_(t.to(self.device, self.dtype))
                 return True
             name = _LAYERED_TOP.get(name, name)
         if name.startswith("model.visual."):  # the image encoder keeps the checkpoint's parameter names
@@ -595,6 +651,10 @@ class EngineWeights:
             t.fill_(1.0 - self.cfg.norm_offset)
         for L in self.layers:
             for k, t in L.items():
+                if k in ("in_bias", "router_shift"):
+                    t.zero_()
+                if k.endswith("rel_rows"):
+                    self._spread_bias(L, k[: -len("rel_rows")])
                 if k.endswith("A_log"):  # the decay parameter of the delta rule must start in its valid range
                     t.copy_(torch.empty_like(t).uniform_(1e-3, 16.0, generator=g).log())
         for L in self.layers + self.draft:
@@ -670,12 +730,17 @@ class ModelRunner:
         self.slopes, self.sinks, self.rotary = [], [], {}
         for L in weights.layers if self.layered else ():
             for a in cached_mixers(L):
-                n, sl = a.heads // weights.tp, a.slopes()
                 f32 = lambda x: torch.tensor(x, dtype=torch.float32, device=self.device)  # noqa: E731
+                if a.rot is not None and a.rot.dims and a.rot not in self.rotary:
+                    self.rotary[a.rot] = stream.rotary_table(max_context + 1, a.rot.dims, a.rot.base, self.device,
+                                                             frequencies=a.rot.frequencies(), gain=a.rot.gain())  # fmt: skip
+                if isinstance(a, LatentSpec):
+                    self.slopes.append(None)
+                    self.sinks.append(None)
+                    continue
+                n, sl = a.heads // weights.tp, a.slopes()
                 self.slopes.append(None if sl is None else f32(sl[weights.rank * n : (weights.rank + 1) * n]))
                 self.sinks.append(None if a.sink is None else f32([a.sink] * n))
-                if a.rot is not None and a.rot.dims and a.rot not in self.rotary:
-                    self.rotary[a.rot] = stream.rotary_table(max_context + 1, a.rot.dims, a.rot.base, self.device)
         self.stream_hook = None  # called with (layer, fp32 residual stream) after every specified layer (eager passes only)
         self.scale = 1.0 / math.sqrt(cfg.head_dim)
         if cfg.multi_latent_attention:
@@ -984,10 +1049,11 @@ class ModelRunner:
         return recur
 
     # ------------------------------------------------------------ specified layers (models/layer_spec.py)
-    def _specified_layers(self, ids, prev, positions, slots, attend, recur):
+    def _specified_layers(self, ids, prev, positions, slots, attend, attend_latent, recur):
         """All layers of a model with ``layer_specs`` over the tokens ``ids`` (``prev``: the tokens in front of them, -1 at a
-        sequence's start; read by models with a bigram table) -> the final norm's output. ``attend(slab, spec, q, factor, out)`` runs an
-        attention mixer once its keys and values are in the cache, ``recur`` (``_extend_recurrence``) a recurrent one: the
+        sequence's start; read by models with a bigram table) -> the final norm's output. ``attend(slab, spec, q, form, out)`` runs an
+        attention mixer once its keys and values are in the cache, ``attend_latent(slab, latent, q, gate, out)`` a latent one,
+        ``recur`` (``_extend_recurrence``) a recurrent one: the
         only parts that differ between a prefill pass and a decode step. The residual stream is fp32; between two
         sub-layers there is one fused launch."""
         cfg, w = self.cfg, self.w
@@ -1001,26 +1067,30 @@ class ModelRunner:
             x = self._tp_reduce(stream.stream_norm(w.embed, None, None, eps, ids=ids - w.rank * w.vocab_local)[1])
             if pair is not None:
                 x = x + pair.table[pair.rows()].float()
-            h, res = stream.stream_norm(x, None, first, eps, **norm)
+            h, res = stream.stream_norm(x, None, first, eps, post_w=w.embed_norm, **norm)
         else:
-            h, res = stream.stream_norm(w.embed, None, first, eps, ids=ids, pair=pair, **norm)
+            h, res = stream.stream_norm(w.embed, None, first, eps, ids=ids, pair=pair, post_w=w.embed_norm, **norm)
         for li, L in enumerate(w.layers):
-            spec = L["spec"]
-            y = self._tp_reduce(_linear(self._specified_mixers(L, li, h, positions, slots, attend, recur), L["out"], out_dtype=f32))
-            after = w.layers[li + 1]["ln1"] if li + 1 < len(w.layers) else w.final_norm
+            spec, last = L["spec"], li + 1 == len(w.layers)
+            after, gain = (w.final_norm, cfg.logit_scale) if last else (w.layers[li + 1]["ln1"], 1.0)
             behind = spec.mlp is not None and not spec.parallel_ff
-            h, _ = stream.stream_norm(y, res, L["ln2"] if behind else after, eps, post_w=L.get("post_attn_ln"), **norm)
+            y = _linear(self._specified_mixers(L, li, h, positions, slots, attend, attend_latent, recur), L["out"], out_dtype=f32)
+            if spec.parallel_ff and spec.mlp is not None and spec.mlp.experts is not None:
+                y = self._specified_experts(L, spec.mlp, h, y)
+            else:
+                y = self._tp_reduce(y)
+            h, _ = stream.stream_norm(y, res, L["ln2"] if behind else after, eps, post_w=L.get("post_attn_ln"), gain=1.0 if behind else gain, **norm)
             if behind:
-                h, _ = stream.stream_norm(self._specified_mlp(L, spec.mlp, h), res, after, eps, post_w=L.get("post_mlp_ln"), **norm)
+                h, _ = stream.stream_norm(self._specified_mlp(L, spec.mlp, h), res, after, eps, post_w=L.get("post_mlp_ln"), gain=gain, **norm)
             if self.stream_hook is not None:
                 self.stream_hook(li, res)
         return h
 
-    def _specified_mixers(self, L, li, h, positions, slots, attend, recur):
+    def _specified_mixers(self, L, li, h, positions, slots, attend, attend_latent, recur):
         """What goes into a layer's output projection: the heads of its mixers, scaled, and the hidden units of a feed-forward
         beside them, side by side as in ``LayerProjections.outs``."""
         spec, lay, T = L["spec"], L["proj"], h.shape[0]
-        x = _linear(h, L["in"])
+        x = _linear(h, L["in"], bias=L.get("in_bias"))
         cols = lambda name: x[:, lay.ins[name][0] : sum(lay.ins[name])]  # noqa: E731
         y = (torch.zeros if lay.padded(lay.outs) else torch.empty)(T, lay.out_cols, dtype=h.dtype, device=h.device)
         slab, number = self.kv_of[li], self.state_of[li]
@@ -1028,10 +1098,27 @@ class ModelRunner:
             c0, n = lay.outs[p + "o"]
             out = y[:, c0 : c0 + n]
             if isinstance(m, AttentionSpec):
-                q = stream.place_heads(cols(p + "q"), cols(p + "k"), cols(p + "v"), slots, self.kv.k[slab], self.kv.v[slab],
+                q, k, sums = cols(p + "q"), cols(p + "k"), None
+                if m.qk_norm and m.norm_over == "projection" and self.w.tp > 1:
+                    sums = (self._tp_reduce(stream.head_sums(q, k)), m.norm_widths())
+                q = stream.place_heads(q, k, cols(p + ("k" if m.tied_values else "v")), slots, self.kv.k[slab], self.kv.v[slab],
                                        q_norm=L.get(p + "q.norm"), k_norm=L.get(p + "k.norm"), eps=self.cfg.norm_epsilon,
-                                       table=self.rotary.get(m.rot), positions=positions, interleaved=m.rot is None or m.rot.interleaved)  # fmt: skip
-                attend(slab, m, q, factor, out)
+                                       table=self.rotary.get(m.rot), positions=positions, interleaved=m.rot is None or m.rot.interleaved,
+                                       sums=sums)  # fmt: skip
+                form = dict(out_scale=factor, chunk=m.chunk, softcap=m.softcap, bias=L.get(p + "bias"), gate=cols(p + "g") if m.gate else None)
+                attend(slab, m, q, form, out)
+                slab += 1
+                continue
+            if isinstance(m, LatentSpec):
+                heads, table = m.heads // self.w.tp, self.rotary[m.rot]
+                c = latent.latent_place(cols(p + "dq"), cols(p + "dkv"), L[p + "dq.norm"], L[p + "dkv.norm"], self.cfg.norm_epsilon, table,
+                                        positions, slots, self.kv.k[slab], m.rot.interleaved)  # fmt: skip
+                q = _linear(c, L[p + "up_q"]).view(T, heads, m.dim + m.rot_dim)
+                gate = cols(p + "g").unflatten(1, (heads, m.vdim)) if m.gate else None
+                sizes = latent.Latent(heads, m.dim, m.vdim, m.kv_rank, m.scale, L[p + "up_q"], L[p + "up_kv"], table, m.rot.interleaved)
+                attend_latent(slab, sizes, q, gate, out.unflatten(1, (heads, m.vdim)))
+                if factor != 1.0:
+                    out.mul_(factor)
                 slab += 1
                 continue
             a, z = (cols(p + s) if p + s in lay.ins else None for s in "ag")
@@ -1045,39 +1132,49 @@ class ModelRunner:
             inputs = delta.DeltaInputs(cols(p + "q"), cols(p + "k"), cols(p + "v"), a, cols(p + "b"), L[p + "conv"], L[p + "A_log"], L[p + "dt_bias"])
             recur(number, inputs, z, L[p + "norm"], m.gate, factor, out)
             number += 1
-        if spec.parallel_ff and spec.mlp is not None:
-            m, (c0, n) = spec.mlp, lay.outs["mlp.down"]
-            r0 = lay.ins["mlp.gate" if m.gated else "mlp.up"][0]
+        if lay.ff is not None:
+            m, (c0, n), r0 = spec.mlp, lay.outs[spec.joint_ff[0] + ".down"], lay.ff[0]
             stream.feed_forward_act(x[:, r0 : r0 + (2 * n if m.gated else n)], m.act, m.gated, out=y[:, c0 : c0 + n])
         return y
 
     def _specified_mlp(self, L, m, h):
-        """Feed-forward of a specified layer: fp32 output, or for experts the unfinished sum the next norm completes."""
+        """Feed-forward behind the mixer of a specified layer: fp32 output, or for experts the unfinished sum the next norm completes."""
         w, f32 = self.w, torch.float32
         if m.experts is None:
             act = stream.feed_forward_act(_linear(h, L["gate_up"]), m.act, m.gated)
             return self._tp_reduce(_linear(act, L["down"], out_dtype=f32))
+        out = self._expert_rows(L, m, h)
+        if m.shared_ff:
+            out.shared = _linear(stream.feed_forward_act(_linear(h, L["shared_gate_up"]), m.act, m.gated), L["shared_down"])
+        if w.ep > 1:  # this rank's experts and its part of the shared one travel in one reduction
+            return self._tp_reduce(stream.combine(out))
+        if w.tp > 1 and out.shared is not None:
+            out.shared = self._tp_reduce(out.shared)
+        return out
+
+    def _specified_experts(self, L, m, h, y):
+        """Experts beside a mixer: the unfinished sum of both, ``y`` being this rank's part of the mixer's output (and of the shared
+        expert's)."""
+        out = self._expert_rows(L, m, h)
+        out.base = y if self.w.ep > 1 else self._tp_reduce(y)
+        return self._tp_reduce(stream.combine(out)) if self.w.ep > 1 else out
+
+    def _expert_rows(self, L, m, h) -> stream.ExpertSum:
+        """Routing and the experts' products."""
+        f32 = torch.float32
         from slime_b200.ops import grouped
 
         # bf16 products are exact in fp32, so the tensor-core product is a 32-bit router too; the CUDA-core kernel is the
         # faster one for a handful of tokens
         big = h.is_cuda and h.dtype == torch.bfloat16 and h.shape[0] >= 256
         logits = ops.gemm(h, L["router"], out_dtype=f32, splitk=1) if big else ops.router_gemm(h, L["router"])
-        probs, idx = grouped.route_topk(logits[:, : m.experts], m.top, score=m.score, renorm=m.renorm, raw_index=True)
+        probs, idx = grouped.route_topk(logits[:, : m.experts], m.top, score=m.score, renorm=m.renorm, raw_index=True, shift=L.get("router_shift"))
         if self.record_routed:
             pad = self.cfg.moe_router_topk - m.top
             self._routed.append(torch.nn.functional.pad(idx.to(torch.int32), (0, pad)) if pad else idx.to(torch.int32))
         lay = grouped.DeviceLayout(idx, L["w13"].shape[0], L["first_expert"])
         rows = _grouped_linear(stream.feed_forward_act(_grouped_linear(lay.pad(h), L["w13"], lay), m.act, m.gated), L["w2"], lay)
-        out = stream.ExpertSum(rows, lay.slot_dest, probs)
-        if m.shared_ff:
-            out.shared = _linear(stream.feed_forward_act(_linear(h, L["shared_gate_up"]), m.act, m.gated), L["shared_down"])
-            out.gate = logits[:, m.experts] if m.shared_gate else None
-        if w.ep > 1:  # this rank's experts and its part of the shared one travel in one reduction
-            return self._tp_reduce(stream.combine(out))
-        if w.tp > 1 and out.shared is not None:
-            out.shared = self._tp_reduce(out.shared)
-        return out
+        return stream.ExpertSum(rows, lay.slot_dest, probs, gate=logits[:, m.experts] if m.shared_gate else None)
 
     def _post_norm(self, x, w):
         """GLM-4 sandwich norm: the sub-layer's output is normalised before it joins the residual stream."""
@@ -1102,13 +1199,14 @@ class ModelRunner:
         """
         cfg, w, d = self.cfg, self.w, self.cfg.head_dim
         if self.layered:
-            from slime_b200.ops import window_attention
-
-            def attend(n, a, q, factor, out):
+            def attend(n, a, q, form, out):
                 return window_attention.window_extend(q, self.kv.k[n], self.kv.v[n], extend, a.scale, a.window, a.keep_first, self.slopes[n],
-                                                      self.sinks[n], factor, out)  # fmt: skip
+                                                      self.sinks[n], out=out, **form)  # fmt: skip
 
-            h = self._specified_layers(ids, prev, positions, slots, attend, self._extend_recurrence(extend))
+            def attend_latent(n, sizes, q, gate, out):
+                return latent.latent_extend(sizes, q, self.kv.k[n], extend, gate, out)
+
+            h = self._specified_layers(ids, prev, positions, slots, attend, attend_latent, self._extend_recurrence(extend))
             h = h if last_rows is None else h.index_select(0, last_rows)
             return self._gather_logits(ops.gemm(h, w.lm_head, out_dtype=torch.float32))
         x = ops.embedding(ids, w.embed, w.rank * w.vocab_local)
@@ -1301,14 +1399,15 @@ class ModelRunner:
         """Embedding to final norm for one token per slot."""
         cfg, w, d, ps = self.cfg, self.w, self.cfg.head_dim, self.kv.page_size
         if self.layered:
-            from slime_b200.ops import window_attention
-
-            def attend(i, a, q, factor, out):
+            def attend(i, a, q, form, out):
                 return window_attention.window_decode(q, self.kv.k[i], self.kv.v[i], bt, seq_lens, pos, ps, a.scale, a.window, a.keep_first,
-                                                      self.slopes[i], self.max_context, self.sinks[i], factor, out)  # fmt: skip
+                                                      self.slopes[i], self.max_context, self.sinks[i], out=out, **form)  # fmt: skip
+
+            def attend_latent(i, sizes, q, gate, out):
+                return latent.latent_decode(sizes, q, self.kv.k[i], bt, pos, ps, self.max_context, gate, out)
 
             prev = self._dev_state["prev_eff"][:n] if cfg.bigram else None
-            return self._specified_layers(ids, prev, pos, slots, attend, self._step_recurrence(n, pos))
+            return self._specified_layers(ids, prev, pos, slots, attend, attend_latent, self._step_recurrence(n, pos))
         recur = self._step_recurrence(n, pos)  # (a state's position counts tokens, whatever the rotary position is)
         if self.rope_delta is not None:
             pos = pos + self.rope_delta[:n]  # rotary position of a request that carries images

@@ -6,12 +6,15 @@ mixers' heads, the feed-forward's hidden units). So a layer costs two large prod
 sum over mixers and feed-forward is the second one's inner product, and one all-reduce covers it. Two-factor projections
 share a third, block-diagonal matrix ``low`` that reads a column range of the first product.
 
+Latent attention's down-projections are rows of ``in``; the expansions of its latents stay matrices of their own
+(``up_q``, ``up_kv``). A mixture beside the mixer contributes its shared expert to ``in`` and ``out`` as a dense feed-forward does.
+
 Every range starts at a multiple of 8 (16 bytes in bf16); what is in between is zero in the matrices.
 """
 
 from __future__ import annotations
 
-from slime_b200.models.layer_spec import AttentionSpec, DeltaSpec, LayerSpec
+from slime_b200.models.layer_spec import DeltaSpec, LatentSpec, LayerSpec
 
 
 def up8(n: int) -> int:
@@ -20,7 +23,8 @@ def up8(n: int) -> int:
 
 class LayerProjections:
     """``ins[name] = (first row, rows)`` and ``outs[name] = (first column, columns)`` of this rank's part of checkpoint tensor
-    ``name`` (behind ``l<i>.``); ``whole``: names that every rank holds completely. ``low[prefix]``: the second factors of mixer
+    ``name`` (behind ``l<i>.``); ``whole``: names that every rank holds completely; ``biased``: names with a bias (tensor
+    ``<name>.b``). ``ff``: (first row, width per rank) of the dense feed-forward in ``in``, or None. ``low[prefix]``: the second factors of mixer
     ``prefix``: (first column in the first product, inner width, rows, {name: (first row, rows, first column, columns)})."""
 
     def __init__(self, spec: LayerSpec, tp: int = 1):
@@ -29,29 +33,49 @@ class LayerProjections:
         self.outs: dict[str, tuple[int, int]] = {}
         self.low: dict[str, tuple[int, int, int, dict]] = {}
         self.whole: set[str] = set()
+        self.biased: set[str] = set()
+        self.ff: tuple[int, int] | None = None
         self.in_rows = self.out_cols = 0
         for p, m, _ in spec.branches():
             if m.heads % tp or m.kv_heads % tp:
                 raise ValueError(f"{m.heads} and {m.kv_heads} heads do not divide over {tp} tensor-parallel ranks")
             h, g = m.heads // tp, m.kv_heads // tp
-            self._in(p + "q", (h if isinstance(m, AttentionSpec) else g) * m.dim)
-            self._in(p + "k", g * m.dim)
-            self._in(p + "v", (g if isinstance(m, AttentionSpec) else h) * m.vdim)
-            if isinstance(m, DeltaSpec):
+            if isinstance(m, LatentSpec):
+                self._in(p + "dq", m.q_rank)
+                self._in(p + "dkv", m.cached)
+                self.whole |= {p + "dq", p + "dkv"}
+                self._gate(p, m)
+            elif isinstance(m, DeltaSpec):
+                self._in(p + "q", g * m.dim)
+                self._in(p + "k", g * m.dim)
+                self._in(p + "v", h * m.vdim)
                 self._delta(p, m, h)
+            else:
+                self._in(p + "q", h * m.dim)
+                self._in(p + "k", g * m.dim)
+                if not m.tied_values:
+                    self._in(p + "v", g * m.vdim)
+                if m.qk_bias:
+                    self.biased |= {p + "q", p + "k"}
+                self._gate(p, m)
             self._out(p + "o", h * m.vdim)
-        m = spec.mlp
-        if m is not None and spec.parallel_ff:
-            if m.ff % tp:
-                raise ValueError(f"a feed-forward of width {m.ff} does not divide over {tp} tensor-parallel ranks")
-            f = m.ff // tp
-            if m.gated:  # gate and up rows without a gap: the activation reads them as one range
-                self.ins["mlp.gate"] = (self.in_rows, f)
-                self.ins["mlp.up"] = (self.in_rows + f, f)
+        if spec.joint_ff is not None:
+            stem, width = spec.joint_ff
+            if width % tp:
+                raise ValueError(f"a feed-forward of width {width} does not divide over {tp} tensor-parallel ranks")
+            f = width // tp
+            self.ff = (self.in_rows, f)
+            if spec.mlp.gated:  # gate and up rows without a gap: the activation reads them as one range
+                self.ins[stem + ".gate"] = (self.in_rows, f)
+                self.ins[stem + ".up"] = (self.in_rows + f, f)
                 self.in_rows += up8(2 * f)
             else:
-                self._in("mlp.up", f)
-            self._out("mlp.down", f)
+                self._in(stem + ".up", f)
+            self._out(stem + ".down", f)
+
+    def _gate(self, p: str, m):
+        if m.gate is not None:
+            self._in(p + "g", m.gate_rows // self.tp)
 
     def _in(self, name: str, rows: int):
         self.ins[name] = (self.in_rows, rows)
@@ -88,11 +112,20 @@ class LayerProjections:
         out.update({n: (width, cols) for n, (_, cols) in self.outs.items()})
         for _, _, _, parts in self.low.values():
             out.update({n: (rows, cols) for n, (_, rows, _, cols) in parts.items()})
+        out.update({n + ".b": (self.ins[n][1],) for n in self.biased})
         for p, m, _ in self.spec.branches():
             if isinstance(m, DeltaSpec):
                 g, h = m.kv_heads * m.dim, m.heads * m.vdim
                 out.update({p + "q.conv": (g, m.conv), p + "k.conv": (g, m.conv), p + "v.conv": (h, m.conv), p + "A_log": (m.heads,),
                             p + "dt_bias": (m.decays,), p + "norm": (m.vdim,)})  # fmt: skip
-            elif m.qk_norm:
-                out.update({p + "q.norm": (m.dim,), p + "k.norm": (m.dim,)})
+                continue
+            if isinstance(m, LatentSpec):
+                out.update({p + "dq.norm": (m.q_rank,), p + "dkv.norm": (m.kv_rank,), p + "uq": (m.heads * (m.dim + m.rot_dim), m.q_rank),
+                            p + "uk": (m.heads * m.dim, m.kv_rank), p + "uv": (m.heads * m.vdim, m.kv_rank)})  # fmt: skip
+                continue
+            if m.qk_norm:
+                nq, nk = m.norm_widths()
+                out.update({p + "q.norm": (nq,), p + "k.norm": (nk,)})
+            if m.learned_bias is not None:
+                out[p + "rel"] = (m.learned_bias.rows, m.heads)
         return out

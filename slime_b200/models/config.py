@@ -99,6 +99,8 @@ class ModelConfig:
     # second embedding table (models with layer_specs): row (previous token * mul_prev + token * mul_cur) mod buckets is added,
     # row ``buckets`` for a sequence's first token
     bigram: dict | None = None
+    embed_norm: bool = False  # the embedding passes a norm with a weight of its own (models with layer_specs)
+    logit_scale: float = 1.0  # factor of the logits (models with layer_specs)
     # multi-token prediction (draft head)
     mtp_num_layers: int | None = None
     model_arch: str = "qwen2"
@@ -112,8 +114,8 @@ class ModelConfig:
             self.padded_vocab_size = self.vocab_size
         if self.layer_specs is not None:
             self.layer_specs = [LayerSpec.of(x) for x in self.layer_specs]
-        elif self.norm_kind != "rms" or self.norm_offset or self.bigram:
-            raise ValueError("norm_kind, norm_offset and bigram are available to models with layer_specs only")
+        elif self.norm_kind != "rms" or self.norm_offset or self.bigram or self.embed_norm or self.logit_scale != 1.0:
+            raise ValueError("norm_kind, norm_offset, bigram, embed_norm and logit_scale are available to models with layer_specs only")
 
     @property
     def head_dim(self) -> int:
@@ -186,6 +188,7 @@ class ModelConfig:
         total += self.vocab_size * h * (1 if self.tie_word_embeddings else 2) + h
         if self.bigram:
             total += (self.bigram["buckets"] + 1) * h
+        total += h if self.embed_norm else 0
         if self.vision:
             v = self.vision
             d, inter, big = v["hidden_size"], v["intermediate_size"], v["hidden_size"] * v.get("spatial_merge_size", 2) ** 2

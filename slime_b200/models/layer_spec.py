@@ -5,37 +5,110 @@ widths, window or feed-forward carries a list of ``LayerSpec`` instead (``ModelC
 hold the largest value of each size, for code that only budgets memory. The specs are mechanism parameters, not a model:
 any architecture whose layers are built from these pieces can use them.
 
-A layer is a mixer (``AttentionSpec``, ``DeltaSpec``, or two of them side by side: ``ParallelSpec``) and a feed-forward, one
-after the other with a residual sum each, or both reading one normed input (``LayerSpec.parallel_ff``).
+A layer is a mixer (``AttentionSpec``, ``LatentSpec``, ``DeltaSpec``, or two of them side by side: ``ParallelSpec``) and a
+feed-forward, one after the other with a residual sum each, or both reading one normed input (``LayerSpec.parallel_ff``).
 """
 
 from __future__ import annotations
 
 import dataclasses
+import math
 from dataclasses import dataclass
+
+
+@dataclass(frozen=True)
+class YarnSpec:
+    """Stretching of a rotation to ``factor`` times the ``original`` context: frequencies that turn more than ``fast`` times in it
+    stay, those that turn less than ``slow`` times are divided by ``factor``, a linear ramp over the pair numbers between."""
+
+    factor: float
+    original: int
+    fast: float
+    slow: float
+
+    def gain(self) -> float:
+        """Factor of every cosine and sine."""
+        return 0.1 * math.log(self.factor) + 1.0
+
+    def stretched(self, dims: int, base: float) -> list[float]:
+        """Share (0 to 1) of each pair's frequency that is divided by ``factor``."""
+        pair = lambda turns: dims * math.log(self.original / (2 * math.pi * turns)) / (2 * math.log(base))  # noqa: E731
+        lo, hi = max(math.floor(pair(self.fast)), 0), min(math.ceil(pair(self.slow)), dims - 1)
+        return [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(dims // 2)]
 
 
 @dataclass(frozen=True)
 class RotarySpec:
     """Rotation of the first ``dims`` coordinates of a query / key head by ``position * base^(-2i / dims)`` for pair i;
-    ``interleaved``: pair i is (2i, 2i + 1), otherwise (i, i + dims / 2)."""
+    ``interleaved``: pair i is (2i, 2i + 1), otherwise (i, i + dims / 2). ``scaling``: the frequencies are stretched."""
 
     dims: int
     base: float
     interleaved: bool = True
+    scaling: YarnSpec | None = None
 
     def __post_init__(self):
+        if isinstance(self.scaling, dict):
+            object.__setattr__(self, "scaling", YarnSpec(**self.scaling))
         if self.dims < 0 or self.dims % 2:
             raise ValueError(f"a rotation of {self.dims} coordinates: they come in pairs")
+
+    def frequencies(self) -> list[float]:
+        """Angle per position of every pair."""
+        f = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+        if self.scaling is None:
+            return f
+        return [x / self.scaling.factor * r + x * (1.0 - r) for x, r in zip(f, self.scaling.stretched(self.dims, self.base))]
+
+    def gain(self) -> float:
+        return 1.0 if self.scaling is None else self.scaling.gain()
+
+
+@dataclass(frozen=True)
+class DistanceBiasSpec:
+    """Learned number per (distance bucket, query head) that is added to a score: ``rows`` buckets, the first half one distance
+    each, the others growing geometrically up to distance ``far``; the last one takes everything beyond."""
+
+    rows: int
+    far: int
+
+    def __post_init__(self):
+        if self.rows < 2 or self.far <= self.rows // 2:
+            raise ValueError(f"{self.rows} distance buckets up to distance {self.far}: the last must lie beyond half their number")
+
+    def bucket(self, n: int) -> int:
+        half = self.rows // 2
+        if n < half:
+            return n
+        x = math.log(n / half) / math.log(self.far / half) * (self.rows - half)
+        # a distance that is exactly a bucket's first one must not fall below it by the logarithm's rounding
+        return min(self.rows - 1, half + (round(x) if abs(x - round(x)) < 1e-9 else math.floor(x)))
+
+    def by_distance(self) -> list[int]:
+        """Bucket of the distances 0, 1, ...; from the last entry on it is the last bucket."""
+        out = [0]
+        while out[-1] < self.rows - 1:
+            out.append(self.bucket(len(out)))
+        return out
+
+
+GATES = (None, "head", "channel")  # sigmoid gate of a mixer's output: one number per head, or one per output channel
+
+
+def _gate_rows(gate: str | None, heads: int, vdim: int) -> int:
+    return 0 if gate is None else heads * (vdim if gate == "channel" else 1)
 
 
 @dataclass(frozen=True)
 class AttentionSpec:
     """Grouped-query attention. ``window``: a query at position i sees keys j with i - j < window (None:
-    all earlier ones) and, whatever the distance, the first ``keep_first`` tokens of the sequence. ``distance_bias``
-    "geometric": head h of H subtracts ``2^(-8 (h + 1) / H) * (i - j)`` from its scores. ``qk_norm``: RMS norm of every query
-    and key head (one weight each, shared by the heads) before the rotation ``rot``. ``sink``: score of an extra column of
-    the softmax that has no value (None: no such column)."""
+    all earlier ones) and, whatever the distance, the first ``keep_first`` tokens of the sequence; ``chunk``: only keys of its
+    own block of that many positions. ``softcap``: scores pass ``c tanh(score / c)``. ``distance_bias``
+    "geometric": head h of H subtracts ``2^(-8 (h + 1) / H) * (i - j)`` from its scores; a ``DistanceBiasSpec``: a learned number
+    is added. ``qk_norm``: RMS norm of every query and key head (one weight each, shared by the heads) before the rotation
+    ``rot``; with ``norm_over`` "projection" of all heads at once, a weight per channel. ``qk_bias``: the query and key
+    projections have biases. ``tied_values``: the values are the keys as projected, before norm and rotation. ``gate``: see
+    ``GATES``. ``sink``: score of an extra column of the softmax that has no value (None: no such column)."""
 
     heads: int
     kv_heads: int
@@ -44,31 +117,113 @@ class AttentionSpec:
     scale: float
     window: int | None = None
     keep_first: int = 0
-    distance_bias: str | None = None
+    distance_bias: str | DistanceBiasSpec | None = None
     qk_norm: bool = False
     rot: RotarySpec | None = None
     sink: float | None = None
+    chunk: int | None = None
+    softcap: float | None = None
+    norm_over: str = "head"
+    qk_bias: bool = False
+    tied_values: bool = False
+    gate: str | None = None
 
     def __post_init__(self):
         if isinstance(self.rot, dict):
             object.__setattr__(self, "rot", RotarySpec(**self.rot))
+        if isinstance(self.distance_bias, dict):
+            object.__setattr__(self, "distance_bias", DistanceBiasSpec(**self.distance_bias))
         if self.rot is not None and self.rot.dims > self.dim:
             raise ValueError(f"a rotation of {self.rot.dims} coordinates in a head of {self.dim}")
         if self.heads % self.kv_heads:
             raise ValueError(f"{self.heads} query heads do not divide over {self.kv_heads} key/value heads")
         if self.window is not None and self.window < 1:
             raise ValueError(f"attention window of {self.window} tokens: a query must at least see itself")
-        if self.distance_bias not in (None, "geometric"):
+        if self.chunk is not None and self.chunk < 1:
+            raise ValueError(f"attention chunks of {self.chunk} tokens")
+        if self.softcap is not None and not self.softcap > 0:
+            raise ValueError(f"scores capped at {self.softcap}")
+        if self.distance_bias not in (None, "geometric") and self.learned_bias is None:
             raise ValueError(f"unknown distance bias {self.distance_bias!r}")
+        if self.distance_bias == "geometric" and self.softcap is not None:
+            raise ValueError("a distance penalty and capped scores in one mixer")
+        if self.norm_over not in ("head", "projection") or self.gate not in GATES:
+            raise ValueError(f"unknown norm {self.norm_over!r} or gate {self.gate!r}")
+        if self.tied_values and self.vdim != self.dim:
+            raise ValueError(f"keys of width {self.dim} cannot be the values of width {self.vdim}")
+
+    @property
+    def learned_bias(self) -> DistanceBiasSpec | None:
+        return self.distance_bias if isinstance(self.distance_bias, DistanceBiasSpec) else None
+
+    @property
+    def gate_rows(self) -> int:
+        return _gate_rows(self.gate, self.heads, self.vdim)
+
+    def cache_geometry(self, tp: int = 1) -> tuple[int, int, int]:
+        """(heads, key width, value width) of what one token leaves in the cache."""
+        return self.kv_heads // tp, self.dim, self.vdim
+
+    def norm_widths(self) -> tuple[int, int]:
+        """Weights of the query norm and of the key norm."""
+        return (self.dim, self.dim) if self.norm_over == "head" else (self.heads * self.dim, self.kv_heads * self.dim)
 
     def slopes(self) -> list[float] | None:
         """Distance-penalty factor of every query head (None: no penalty)."""
-        if self.distance_bias is None:
+        if self.distance_bias != "geometric":
             return None
         return [2.0 ** (-8.0 * (h + 1) / self.heads) for h in range(self.heads)]
 
     def params(self, width: int) -> int:
-        return width * (self.heads + self.kv_heads) * (self.dim + self.vdim) + (2 * self.dim if self.qk_norm else 0)
+        n = width * (self.heads * (self.dim + self.vdim) + self.kv_heads * (self.dim + (0 if self.tied_values else self.vdim)) + self.gate_rows)
+        n += sum(self.norm_widths()) if self.qk_norm else 0
+        n += (self.heads + self.kv_heads) * self.dim if self.qk_bias else 0
+        return n + (self.learned_bias.rows * self.heads if self.learned_bias else 0)
+
+
+@dataclass(frozen=True)
+class LatentSpec:
+    """Latent attention: queries come from a normed latent of width ``q_rank``, keys and values of all heads from one of width
+    ``kv_rank``, and a rotated key part of ``rot_dim`` coordinates is shared by the heads; the latent and that part are what the
+    cache keeps of a token. Per head ``dim`` unrotated and ``rot_dim`` rotated query / key coordinates and ``vdim`` values.
+    ``rot`` turns the rotated part only."""
+
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    q_rank: int
+    kv_rank: int
+    scale: float
+    rot: RotarySpec
+    gate: str | None = None
+
+    def __post_init__(self):
+        if isinstance(self.rot, dict):
+            object.__setattr__(self, "rot", RotarySpec(**self.rot))
+        if self.rot.dims != self.rot_dim:
+            raise ValueError(f"a rotation of {self.rot.dims} coordinates of a rotated part of {self.rot_dim}")
+        if self.gate not in (None, "channel"):
+            raise ValueError(f"latent attention has no gate {self.gate!r}")
+
+    @property
+    def kv_heads(self) -> int:
+        return self.heads  # every head expands keys and values of its own
+
+    @property
+    def cached(self) -> int:
+        return self.kv_rank + self.rot_dim
+
+    @property
+    def gate_rows(self) -> int:
+        return _gate_rows(self.gate, self.heads, self.vdim)
+
+    def cache_geometry(self, tp: int = 1) -> tuple[int, int, int]:
+        return 1, self.cached, 0
+
+    def params(self, width: int) -> int:
+        n = width * (self.q_rank + self.cached + self.gate_rows + self.heads * self.vdim) + self.q_rank + self.kv_rank
+        return n + self.heads * ((self.dim + self.rot_dim) * self.q_rank + (self.dim + self.vdim) * self.kv_rank)
 
 
 @dataclass(frozen=True)
@@ -117,8 +272,8 @@ class DeltaSpec:
 class ParallelSpec:
     """Two mixers that read the same input; the result is ``left_scale * left + right_scale * right``."""
 
-    left: AttentionSpec | DeltaSpec
-    right: AttentionSpec | DeltaSpec
+    left: AttentionSpec | LatentSpec | DeltaSpec
+    right: AttentionSpec | LatentSpec | DeltaSpec
     left_scale: float = 1.0
     right_scale: float = 1.0
 
@@ -131,7 +286,7 @@ def _mixer_of(x):
         return x
     if "left" in x:
         return ParallelSpec(**{**x, "left": _mixer_of(x["left"]), "right": _mixer_of(x["right"])})
-    return DeltaSpec(**x) if "conv" in x else AttentionSpec(**x)
+    return DeltaSpec(**x) if "conv" in x else LatentSpec(**x) if "kv_rank" in x else AttentionSpec(**x)
 
 
 @dataclass(frozen=True)
@@ -139,7 +294,7 @@ class FeedForwardSpec:
     """Dense (``experts`` None) or mixture-of-experts feed-forward. ``gated``: ``down(act(gate x) * up x)``, otherwise
     ``down(act(up x))``; with experts the same form is every expert's. ``score`` / ``renorm``: router scores over all
     experts, kept as they are or divided by the sum of the chosen ones. ``shared_ff`` > 0: an expert of that width runs
-    for every token, scaled by a sigmoid gate of its own when ``shared_gate``."""
+    for every token, scaled by a sigmoid gate of its own when ``shared_gate``. ``router_bias``: added to the router's logits."""
 
     ff: int
     act: str
@@ -150,6 +305,7 @@ class FeedForwardSpec:
     renorm: bool = False
     shared_ff: int = 0
     shared_gate: bool = False
+    router_bias: bool = False
 
     def __post_init__(self):
         if self.act not in ("silu", "gelu_tanh", "relu2"):
@@ -161,7 +317,7 @@ class FeedForwardSpec:
         mats = 3 if self.gated else 2
         if self.experts is None:
             return mats * width * self.ff
-        n = self.experts * (mats * width * self.ff + width)
+        n = self.experts * (mats * width * self.ff + width + (1 if self.router_bias else 0))
         if self.shared_ff:
             n += mats * width * self.shared_ff + (width if self.shared_gate else 0)
         return n
@@ -169,13 +325,25 @@ class FeedForwardSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: AttentionSpec | DeltaSpec | ParallelSpec
+    mixer: AttentionSpec | LatentSpec | DeltaSpec | ParallelSpec
     mlp: FeedForwardSpec | None = None  # None: the layer is its mixer only
     parallel_ff: bool = False  # mixer and feed-forward read the same normed input and join the stream in one sum
 
     def __post_init__(self):
-        if self.parallel_ff and self.mlp is not None and self.mlp.experts is not None:
-            raise ValueError("a feed-forward beside the mixer is dense: experts have no form of it")
+        m = self.mlp
+        if self.parallel_ff and m is not None and m.experts is not None and m.shared_gate:
+            raise ValueError("the shared expert of a mixture beside the mixer has no gate: its output is summed with the mixer's")
+
+    @property
+    def joint_ff(self) -> tuple[str, int] | None:
+        """(stem of its tensors, width) of the dense feed-forward that is computed together with the mixer: the whole one, or the
+        shared expert of a mixture."""
+        m = self.mlp
+        if not self.parallel_ff or m is None:
+            return None
+        if m.experts is None:
+            return "mlp", m.ff
+        return ("mlp.shared", m.shared_ff) if m.shared_ff else None
 
     @classmethod
     def of(cls, x) -> "LayerSpec":
@@ -189,7 +357,7 @@ class LayerSpec:
     def to_dict(self) -> dict:
         return dataclasses.asdict(self)
 
-    def branches(self) -> list[tuple[str, AttentionSpec | DeltaSpec, float]]:
+    def branches(self) -> list[tuple[str, AttentionSpec | LatentSpec | DeltaSpec, float]]:
         """(prefix of its tensors behind ``l<i>.``, mixer, factor of its output) of every mixer of the layer."""
         m = self.mixer
         if isinstance(m, ParallelSpec):
@@ -272,13 +440,14 @@ def pefolix_json(cfg) -> dict:
 # gate, both through two-factor projections), a bigram table added to the embedding.
 
 
-def _inner_width(shapes: dict | None, name: str, m: dict, key: str) -> int:
-    """Inner width of a two-factor projection: the checkpoint's tensor says it, or ``key`` of the mixer's description."""
+def _rows_of(shapes: dict | None, name: str, m: dict, key: str) -> int:
+    """Rows of a tensor that config.json need not state (the inner width of a two-factor projection, distance buckets): the
+    checkpoint's tensor says it, or ``key`` of the mixer's description."""
     if shapes and name in shapes:
         return int(shapes[name][0])
     if key in m:
         return int(m[key])
-    raise ValueError(f"the inner width of {name} is not in config.json: give the checkpoint's tensor shapes, or {key!r} in the mixer")
+    raise ValueError(f"the inner width of {name} (its rows) is not in config.json: give the checkpoint's tensor shapes, or {key!r} in the mixer")
 
 
 def ledazen_config(c: dict, shapes: dict | None = None) -> dict:
@@ -294,8 +463,8 @@ def ledazen_config(c: dict, shapes: dict | None = None) -> dict:
             rot = RotarySpec(a["rot"]["dims"], float(a["rot"]["base"])) if a.get("rot") else None
             left = AttentionSpec(*sizes(a), float(a["scale"]), qk_norm=True, rot=rot, sink=0.0)
             p = f"l{i}.mix.right."
-            right = DeltaSpec(*sizes(d), d["conv"], "channel", "sigmoid", _inner_width(shapes, p + "a1", d, "decay_rank"),
-                              _inner_width(shapes, p + "g1", d, "gate_rank"))  # fmt: skip
+            right = DeltaSpec(*sizes(d), d["conv"], "channel", "sigmoid", _rows_of(shapes, p + "a1", d, "decay_rank"),
+                              _rows_of(shapes, p + "g1", d, "gate_rank"))  # fmt: skip
             mixer = ParallelSpec(left, right, float(m["left_scale"]), float(m["right_scale"]))
         else:
             raise ValueError(f"layer {i}: a Ledazen model has no mixer of type {layer['type']!r}")
@@ -327,5 +496,75 @@ def ledazen_json(cfg) -> dict:
                 vocab=cfg.vocab_size, width=cfg.hidden_size)  # fmt: skip
 
 
+# ------------------------------------------------------------------------------------------------- Zetizen
+# Fixed by the design: one layer norm per layer whose output mixer and feed-forward both read, a normed embedding that is also
+# the output matrix; three mixers: attention with a learned distance bias and capped scores, chunked attention with stretched
+# rotation of halves, keys as values and a gate per head, latent attention with a gate per channel; norms over whole query and
+# key projections; gated silu experts weighted by a softmax over the chosen logits, a shared one beside them.
+
+
+def _yarn_of(r: dict) -> RotarySpec:
+    s = r.get("scaling")
+    return RotarySpec(r["dims"], float(r["base"]), False, None if s is None else YarnSpec(float(s["factor"]), s["original"], float(s["fast"]), float(s["slow"])))
+
+
+def zetizen_config(c: dict, shapes: dict | None = None) -> dict:
+    """``config.json`` of a Zetizen model (and the shapes of its tensors by name) -> ``ModelConfig`` arguments."""
+    specs = []
+    for i, layer in enumerate(c["layers"]):
+        m, f = layer["mixer"], layer.get("mlp")
+        if layer["type"] == "latent_attention":
+            mixer = LatentSpec(m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["q_rank"], m["kv_rank"], float(m["scale"]), _yarn_of(m["rot"]), "channel")
+        elif layer["type"] in ("attention", "attention_2"):
+            sizes = (m["heads"], m["kv_heads"], m["dim"], m["vdim"], float(m["scale"]))
+            both = dict(softcap=float(m["softcap"]), qk_norm=True, norm_over="projection")
+            if layer["type"] == "attention":
+                rows = _rows_of(shapes, f"l{i}.mix.rel", m, "bias_rows")
+                mixer = AttentionSpec(*sizes, distance_bias=DistanceBiasSpec(rows, m["bias_max"]), **both)
+            else:
+                mixer = AttentionSpec(*sizes, rot=_yarn_of(m["rot"]), chunk=m["mask"]["size"], qk_bias=True, tied_values=True, gate="head", **both)
+        else:
+            raise ValueError(f"layer {i}: a Zetizen model has no mixer of type {layer['type']!r}")
+        if f is not None and f["kind"] != "moe":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
+        mlp = None
+        if f is not None:
+            shared = f.get("shared")
+            mlp = FeedForwardSpec(f["expert"]["ff"], "silu", experts=f["router"]["experts"], top=f["router"]["top"], renorm=True,
+                                  shared_ff=shared["ff"] if shared else 0, router_bias=True)  # fmt: skip
+        specs.append(LayerSpec(mixer, mlp, parallel_ff=True))
+    return dict(flat_sizes(specs), layer_specs=specs, hidden_size=c["width"], vocab_size=c["vocab"], norm_epsilon=c["norm"]["eps"],
+                norm_kind="layer", embed_norm=True, logit_scale=float(c["logit_scale"]), tie_word_embeddings=True, model_arch="Zetizen")  # fmt: skip
+
+
+def zetizen_json(cfg) -> dict:
+    """The ``config.json`` of a Zetizen ``ModelConfig`` (inverse of ``zetizen_config``; carries the number of distance buckets too)."""
+
+    def rot(r: RotarySpec) -> dict:
+        return dict(dims=r.dims, base=r.base, **({"scaling": dataclasses.asdict(r.scaling)} if r.scaling else {}))
+
+    layers = []
+    for s in cfg.layer_specs:
+        a, f = s.mixer, s.mlp
+        if isinstance(a, LatentSpec):
+            kind, mixer = "latent_attention", dict(heads=a.heads, dim=a.dim, rot_dim=a.rot_dim, vdim=a.vdim, q_rank=a.q_rank, kv_rank=a.kv_rank,
+                                                   scale=a.scale, rot=rot(a.rot))  # fmt: skip
+        else:
+            mixer = dict(heads=a.heads, kv_heads=a.kv_heads, dim=a.dim, vdim=a.vdim, scale=a.scale, softcap=a.softcap)
+            if a.learned_bias is not None:
+                kind, mixer = "attention", dict(mixer, bias_max=a.learned_bias.far, bias_rows=a.learned_bias.rows)
+            else:
+                kind, mixer = "attention_2", dict(mixer, mask=dict(size=a.chunk), rot=rot(a.rot))
+        mlp = None
+        if f is not None:
+            mlp = dict(kind="moe", expert=dict(ff=f.ff), router=dict(experts=f.experts, top=f.top))
+            if f.shared_ff:
+                mlp["shared"] = dict(ff=f.shared_ff)
+        layers.append(dict(type=kind, mixer=mixer, mlp=mlp))
+    return dict(architecture="Zetizen", layers=layers, logit_scale=cfg.logit_scale, norm=dict(eps=cfg.norm_epsilon), vocab=cfg.vocab_size,
+                width=cfg.hidden_size)  # fmt: skip
+
+
 # ``config.json`` files that name their design in "architecture": name -> (reader(config, tensor shapes or None), writer)
-LAYERED_ARCHITECTURES = {"Pefolix": (pefolix_config, pefolix_json), "Ledazen": (ledazen_config, ledazen_json)}
+LAYERED_ARCHITECTURES = {"Pefolix": (pefolix_config, pefolix_json), "Ledazen": (ledazen_config, ledazen_json),
+                         "Zetizen": (zetizen_config, zetizen_json)}  # fmt: skip

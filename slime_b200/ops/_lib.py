@@ -34,16 +34,23 @@ _SIGS = {
     "sb_dp_reduce_shard": [P, I, I, I, L, L, P, P, P, P, P],
     "sb_dp_adam_bcast": [P, P, P, P, P, I, I, I, L, L, F, F, F, F, F, F, F, F, F, P, I, P],
     "sb_group_fp8_quant_1x128": [P, P, P, P, I, I, L, L, I, P],
-    "sb_moe_topk": [P, P, P, P, L, I, L, I, I, I, F, P],
+    "sb_moe_topk": [P, P, P, P, P, L, I, L, I, I, I, F, P],
     "sb_moe_layout": [P, P, P, I, I, I, I, P],
-    "sb_stream_norm": [P, I, P, I, P, P, I, P, P, I, P, P, I, P, P, I, I, I, F, F, I, P, P, P, L, L, I, P],
+    "sb_stream_norm": [P, I, P, I, P, P, I, P, P, I, P, P, I, P, P, I, I, I, F, F, I, P, P, P, L, L, I, P, F, P],
     "sb_glu": [P, P, P, L, I, L, L, I, I, P],
     "sb_heads": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, L, L, L, F, I, P],
+    "sb_heads_all": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, L, L, L, P, I, I, F, I, P],
+    "sb_latent_place": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, L, L, F, I, P],
+    "sb_latent_turn": [P, P, P, P, I, I, I, I, I, L, L, L, L, I, P],
+    "sb_latent_attn": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P, P, P],
+    "sb_flash_latent": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, L, L, L, L, L, P, P, P],
+    "sb_head_gemm": [P, P, P, P, I, I, I, I, I, L, L, L, L, L, L, L, L, P, P],
+    "sb_gemm_simt_heads": [P, P, P, P, I, I, I, I, I, L, L, L, L, L, L, L, L, I, P],
     "sb_kv_scatter": [P, P, P, P, P, I, I, I, L, L, P],
     "sb_gemm_simt": [P, P, P, P, P, I, I, I, L, L, L, I, I, P],
-    "sb_window_attn": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, L, L, F, F, I, I, I, P],
-    "sb_flash_window": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, L, L, F, F, I, I, P, P],
-    "sb_paged_decode_window": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, F, I, I, P, P],
+    "sb_window_attn": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, L, L, L, P, I, P],
+    "sb_flash_window": [P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, L, L, P, P, P],
+    "sb_paged_decode_window": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, P, P, P],
     "sb_delta_prep": [P, P, P, P, P, L, L, L, P, P, P, P, P, P, I, P, P, P, P, P, P, I, I, I, I, I, I, I, P],
     "sb_delta_scan": [P, P, P, L, P, P, P, I, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P],
     "sb_delta_step": [P, P, P, P, P, L, L, L, P, P, P, P, P, P, P, P, P, P, P, L, L, F, F, I, I, I, I, I, I, I, I, I, P],

@@ -27,13 +27,14 @@ P = _lib.ptr
 
 
 def route_topk(logits: torch.Tensor, k: int, *, score: str = "softmax", pre_softmax: bool = False, renorm: bool = True,
-               bias: torch.Tensor | None = None, scale: float | None = None, raw_index: bool = False):
+               bias: torch.Tensor | None = None, scale: float | None = None, raw_index: bool = False, shift: torch.Tensor | None = None):
     """Router logits [T, E] (fp32) -> ``(weights [T, k] fp32, indices [T, k] int64)`` in one kernel (``raw_index``: the
     kernel's own int32 indices on CUDA, which is what ``DeviceLayout`` reads).
 
     ``score="softmax"`` with ``renorm`` and not ``pre_softmax``: softmax over the k picked logits; with ``pre_softmax``
     or ``renorm=False``: full softmax, pick k, keep the probabilities. ``score="sigmoid"``: sigmoid scores, ``bias``
     steers the choice only, weights are the picked scores (normalised when ``renorm``). ``scale`` multiplies the result.
+    ``shift`` [E] is added to the logits before all this.
     """
     T, E = logits.shape
     mode = 2 if score == "sigmoid" else (1 if (pre_softmax or not renorm) else 0)
@@ -43,10 +44,11 @@ def route_topk(logits: torch.Tensor, k: int, *, score: str = "softmax", pre_soft
         idx = torch.empty(T, k, dtype=torch.int32, device=lg.device)
         w = torch.empty(T, k, dtype=torch.float32, device=lg.device)
         b = None if bias is None else bias.float().contiguous()
-        rc = _lib.lib().sb_moe_topk(P(lg), P(b), P(idx), P(w), T, E, lg.stride(0), k, mode, int(renorm), float(scale or 1.0), _lib.stream())
+        shift = None if shift is None else shift.float().contiguous()
+        rc = _lib.lib().sb_moe_topk(P(lg), P(shift), P(b), P(idx), P(w), T, E, lg.stride(0), k, mode, int(renorm), float(scale or 1.0), _lib.stream())
         _lib.check(rc, "sb_moe_topk")
         return w, idx if raw_index else idx.long()
-    lg = logits.float()
+    lg = logits.float() if shift is None else logits.float() + shift.float()
     if mode == 2:
         scores = torch.sigmoid(lg)
         idx = torch.topk(scores + bias.float() if bias is not None else scores, k, dim=-1).indices

@@ -19,13 +19,15 @@ ACTS = {"silu": 0, "gelu_tanh": 1, "relu2": 2}
 @dataclasses.dataclass
 class ExpertSum:
     """Unfinished output of a mixture-of-experts feed-forward: token t is ``sum_j weights[t, j] * rows[dest[t * k + j]]``
-    (``dest`` < 0: no row here) ``+ sigmoid(gate[t]) * shared[t]``. ``gate``: a column of the router's logits, or None."""
+    (``dest`` < 0: no row here) ``+ sigmoid(gate[t]) * shared[t] + base[t]``. ``gate``: a column of the router's logits, or None;
+    ``base``: fp32 output of what runs beside the experts, or None."""
 
     rows: torch.Tensor
     dest: torch.Tensor
     weights: torch.Tensor
     shared: torch.Tensor | None = None
     gate: torch.Tensor | None = None
+    base: torch.Tensor | None = None
 
     def tokens(self) -> int:
         return self.weights.shape[0]
@@ -64,10 +66,11 @@ def _combine(e: ExpertSum) -> torch.Tensor:
     if e.shared is not None:
         s = e.shared.float()
         y += s if e.gate is None else torch.sigmoid(e.gate.float())[:, None] * s
-    return y
+    return y if e.base is None else y + e.base
 
 
-def stream_norm(y, res, pre_w, eps, *, kind="rms", post_w=None, ids=None, offset=0.0, pair: PairTable | None = None):
+def stream_norm(y, res, pre_w, eps, *, kind="rms", post_w=None, ids=None, offset=0.0, pair: PairTable | None = None,
+                gain=1.0):  # fmt: skip
     """``res (+)= norm(y) * post_w`` and return ``norm(res) * pre_w``, in one launch.
 
     ``y``: sub-layer output [T, H], an ``ExpertSum``, or an embedding table when ``ids`` [T] is given (ids outside the table give
@@ -75,7 +78,7 @@ def stream_norm(y, res, pre_w, eps, *, kind="rms", post_w=None, ids=None, offset
     updated in place; None starts the stream (a new tensor is returned as second value). ``post_w`` None: no norm of the
     sub-layer's output; ``pre_w`` None: nothing but the stream is wanted (the first value is None). ``kind``: "rms" or
     "layer" (mean removed, no bias); ``offset`` is added to the norm weights in fp32. ``pair``: rows of a second table added to
-    ``y``. Norms, sums and the stream are fp32 whatever the element types."""
+    ``y``. ``gain``: factor of the returned norm. Norms, sums and the stream are fp32 whatever the element types."""
     moe = y if isinstance(y, ExpertSum) else None
     src = moe.rows if moe is not None else y
     T = moe.tokens() if moe is not None else (ids.numel() if ids is not None else y.shape[0])
@@ -98,13 +101,13 @@ def stream_norm(y, res, pre_w, eps, *, kind="rms", post_w=None, ids=None, offset
             res = v.clone()
         else:
             res.add_(v)
-        return (None if pre_w is None else _norm(res, pre_w, eps, kind, offset).to(w_dtype)), res
+        return (None if pre_w is None else (_norm(res, pre_w, eps, kind, offset) * gain).to(w_dtype)), res
     src = src.contiguous()
     if init:
         res = torch.empty(T, H, dtype=torch.float32, device=src.device)
     assert res.dtype == torch.float32 and res.is_contiguous() and src.dtype in (torch.bfloat16, torch.float32)
     h = torch.empty(T, H, dtype=w_dtype, device=src.device) if pre_w is not None else None
-    dest = wts = shared = gate = None
+    dest = wts = shared = gate = base = None
     k = 1
     if moe is not None:
         k = moe.weights.shape[1]
@@ -114,6 +117,8 @@ def stream_norm(y, res, pre_w, eps, *, kind="rms", post_w=None, ids=None, offset
         assert shared is None or shared.dtype == src.dtype
         gate = moe.gate if shared is not None else None
         assert gate is None or gate.dtype == torch.float32
+        base = moe.base
+        assert base is None or (base.dtype == torch.float32 and base.is_contiguous() and base.shape == (T, H))
     ids32 = None if ids is None else ids.to(torch.int32).contiguous()
     if pair is not None:
         assert pair.table.is_contiguous() and pair.table.dtype == src.dtype and pair.table.shape[1] == H
@@ -123,7 +128,7 @@ def stream_norm(y, res, pre_w, eps, *, kind="rms", post_w=None, ids=None, offset
         gate.stride(0) if gate is not None else 0, P(post_w), P(res), int(init), P(pre_w), P(h), int(w_dtype == torch.float32),
         T, H, float(eps), float(offset), int(kind == "layer"), P(pair.table) if pair else None, P(pair.ids) if pair else None,
         P(pair.prev) if pair else None, pair.mul_prev if pair else 0, pair.mul_cur if pair else 0, pair.table.shape[0] - 1 if pair else 0,
-        _lib.stream(),
+        P(base), float(gain), _lib.stream(),
     )  # fmt: skip
     _lib.check(rc, "sb_stream_norm")
     return h, res
@@ -157,11 +162,14 @@ def feed_forward_act(x: torch.Tensor, act: str, gated: bool, out: torch.Tensor |
     return out
 
 
-def rotary_table(positions: int, dims: int, base: float, device=None) -> torch.Tensor:
-    """fp32 ``[positions, dims]`` = cos | sin of ``p * base^(-2i / dims)`` for the dims / 2 pairs i (computed in fp64)."""
+def rotary_table(positions: int, dims: int, base: float, device=None, *, frequencies: list[float] | None = None, gain: float = 1.0) -> torch.Tensor:
+    """fp32 ``[positions, dims]`` = cos | sin of ``p * base^(-2i / dims)`` for the dims / 2 pairs i (computed in fp64); ``frequencies``:
+    those instead; ``gain`` multiplies the table."""
     f = base ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)
+    if frequencies is not None:
+        f = torch.tensor(frequencies, dtype=torch.float64)
     angle = torch.arange(positions, dtype=torch.float64)[:, None] * f
-    return torch.cat([angle.cos(), angle.sin()], 1).float().to(device)
+    return (torch.cat([angle.cos(), angle.sin()], 1) * gain).float().to(device)
 
 
 def _turn(x, table, positions, interleaved):
@@ -176,13 +184,16 @@ def _turn(x, table, positions, interleaved):
     return out
 
 
-def place_heads(q, k, v, slots, k_cache, v_cache, *, q_norm=None, k_norm=None, eps=0.0, table=None, positions=None, interleaved=True):
-    """New queries ``q`` [T, Hq * D], keys [T, Hkv * D] and values [T, Hkv * DV] (column ranges of a projection are fine): RMS norm
-    per query / key head (``q_norm`` / ``k_norm`` [D]; None: none), rotation by ``table`` (``rotary_table``; None: none) at
-    ``positions``. Queries are changed in place and returned [T, Hq, D]; keys and values go to cache slot ``slots[t]`` (< 0:
-    nowhere)."""
+def place_heads(q, k, v, slots, k_cache, v_cache, *, q_norm=None, k_norm=None, eps=0.0, table=None, positions=None, interleaved=True,
+                sums=None):  # fmt: skip
+    """New queries ``q`` [T, Hq * D], keys [T, Hkv * D] and values [T, Hkv * DV] (column ranges of a projection are fine; values may be
+    the keys): RMS norm (``q_norm`` / ``k_norm`` [D]: per query / key head; [Hq * D] / [Hkv * D]: over all heads at once; None: none),
+    rotation by ``table`` (``rotary_table``; None: none) at ``positions``. Queries are changed in place and returned [T, Hq, D]; keys
+    and values go to cache slot ``slots[t]`` (< 0: nowhere). ``sums``: for a norm over all heads of which this rank has a part,
+    ([T, 2] sums of squares of the whole projections, their widths)."""
     T, (Hkv, D), DV = q.shape[0], k_cache.shape[1:], v_cache.shape[2]
     Hq = q.shape[1] // D
+    over_all = q_norm is not None and q_norm.numel() == Hq * D and k_norm.numel() == Hkv * D and (Hq > 1 or Hkv > 1 or sums is not None)
     _checks.index_range("place_heads", "slots", slots, upper=k_cache.shape[0], lower=-(1 << 31))
     if table is not None:
         _checks.index_range("place_heads", "positions", positions, upper=table.shape[0])
@@ -191,20 +202,34 @@ def place_heads(q, k, v, slots, k_cache, v_cache, *, q_norm=None, k_norm=None, e
         return q.unflatten(1, (Hq, D))
     if not q.is_cuda:
         out = []
-        for x, w in ((q, q_norm), (k, k_norm)):
-            y = x.unflatten(1, (-1, D)).float()
-            y = y if w is None else _norm(y, w, eps, "rms")
-            out.append((y if table is None else _turn(y, table, positions, interleaved)).flatten(1).to(x.dtype))
+        for i, (x, w) in enumerate(((q, q_norm), (k, k_norm))):
+            if over_all and sums is not None:
+                x = (x.float() * torch.rsqrt(sums[0][:, i : i + 1] / sums[1][i] + eps) * w.float()).unflatten(1, (-1, D))
+            elif over_all:
+                x = _norm(x.float(), w, eps, "rms").unflatten(1, (-1, D))
+            else:
+                x = x.unflatten(1, (-1, D)).float()
+                x = x if w is None else _norm(x, w, eps, "rms")
+            out.append((x if table is None else _turn(x, table, positions, interleaved)).flatten(1).to(q.dtype))
         q.copy_(out[0])
         kv_scatter(out[1], v, slots, k_cache, v_cache)
         return q.unflatten(1, (Hq, D))
     assert q.stride(1) == k.stride(1) == v.stride(1) == 1 and q.dtype == k.dtype == v.dtype == k_cache.dtype == v_cache.dtype
     assert k_cache.is_contiguous() and v_cache.is_contiguous() and (q_norm is None or q_norm.dtype == k_norm.dtype == q.dtype)
-    rc = _lib.lib().sb_heads(P(q), P(k), P(v), P(q_norm), P(k_norm), P(table), P(positions), P(slots), P(k_cache), P(v_cache), T, Hq, Hkv, D, DV,
-                             0 if table is None else table.shape[1], int(interleaved), q.stride(0), k.stride(0), v.stride(0), float(eps),
-                             int(q.dtype == torch.float32), _lib.stream())  # fmt: skip
-    _lib.check(rc, "sb_heads")
+    head = (P(q), P(k), P(v), P(q_norm), P(k_norm), P(table), P(positions), P(slots), P(k_cache), P(v_cache), T, Hq, Hkv, D, DV,
+            0 if table is None else table.shape[1], int(interleaved), q.stride(0), k.stride(0), v.stride(0))  # fmt: skip
+    f32 = int(q.dtype == torch.float32)
+    if over_all:
+        part, widths = sums if sums is not None else (None, (Hq * D, Hkv * D))
+        _lib.check(_lib.lib().sb_heads_all(*head, P(part), *widths, float(eps), f32, _lib.stream()), "sb_heads_all")
+    else:
+        _lib.check(_lib.lib().sb_heads(*head, float(eps), f32, _lib.stream()), "sb_heads")
     return q.unflatten(1, (Hq, D))
+
+
+def head_sums(q, k) -> torch.Tensor:
+    """[T, 2] fp32 sums of squares of query and key rows (a rank's part of them)."""
+    return torch.stack([q.float().square().sum(-1), k.float().square().sum(-1)], 1)
 
 
 def kv_scatter(k, v, slots, k_cache, v_cache):

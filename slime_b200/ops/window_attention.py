@@ -1,8 +1,11 @@
-"""Windowed attention over the paged KV cache, for prompts (``window_extend``) and single tokens (``window_decode``).
+"""Attention over the paged KV cache, for prompts (``window_extend``) and single tokens (``window_decode``).
 
-A query at position i sees key j when ``j <= i`` and (``i - j < window`` or ``j < keep_first``); its score is
-``scale * q.k - slope[head] * (i - j)`` (``slopes`` None: no distance term). ``sinks`` [Hq]: score of an extra softmax column
-without a value (None: no such column); ``out_scale`` multiplies the output, ``out`` may be a column range of a wider matrix. Keys and values are read from the cache only,
+A query at position i sees key j when ``j <= i`` and (``j`` is in its window, ``i - j < window``, and in its chunk, ``j // chunk ==
+i // chunk``; or ``j < keep_first``). Its score is ``scale * q.k``, capped to ``softcap * tanh(score / softcap)``, plus
+``bias[i - j, head]`` (``bias`` [N, Hq] fp32 by distance, the last row for everything beyond), minus ``slope[head] * (i - j)``; None:
+no such term. ``sinks`` [Hq]: score of an extra softmax column
+without a value (None: no such column). The output is multiplied by ``out_scale`` and by ``sigmoid(gate)`` (``gate``: [T, Hq] logits, or
+[T, Hq * DV]); ``out`` may be a column range of a wider matrix. Keys and values are read from the cache only,
 so a prompt's later portions, portions of several requests and single tokens beside them are one launch.
 
 Dispatch on CUDA: bf16 with head widths that are multiples of 8 up to 128 run on the tensor cores
@@ -12,6 +15,7 @@ Dispatch on CUDA: bf16 with head widths that are multiples of 8 up to 128 run on
 
 from __future__ import annotations
 
+import ctypes
 import dataclasses
 
 import numpy as np
@@ -43,6 +47,7 @@ class ExtendBatch:
     counts: list[int]
     page_size: int
     state_slots: list[int] | None = None
+    pages: list[list[int]] | None = None  # the same as block_table, on the host
     _tiles: dict = dataclasses.field(default_factory=dict)
 
     @classmethod
@@ -56,34 +61,83 @@ class ExtendBatch:
         req = np.repeat(np.arange(len(pages)), counts)
         pos = np.concatenate([np.arange(s, s + n) for s, n in zip(starts, counts)])
         return cls(up(table), up(req), up(pos), [int(s) for s in starts], [int(n) for n in counts], page_size,
-                   state_slots)
+                   state_slots, pages)
 
-    def tiles(self, tokens: int) -> torch.Tensor:
-        """[n, 4] int32 (first row, tokens, first position, request) of query tiles of at most ``tokens`` tokens."""
-        if tokens not in self._tiles:
-            rows, row = [], 0
-            for r, (s, n) in enumerate(zip(self.starts, self.counts)):
-                off = np.arange(0, n, tokens)
-                rows.append(np.stack([row + off, np.minimum(tokens, n - off), s + off, np.full_like(off, r)], 1))
-                row += n
-            host = torch.from_numpy(np.concatenate(rows).astype(np.int32))
+    def tiles(self, tokens: int, requests: tuple[int, ...] | None = None) -> torch.Tensor:
+        """[n, 4] int32 (first row, tokens, first position, request) of query tiles of at most ``tokens`` tokens (of some requests
+        only)."""
+
+        def make():
+            rows, first = [], np.concatenate([[0], np.cumsum(self.counts)])
+            for r in range(len(self.counts)) if requests is None else requests:
+                off = np.arange(0, self.counts[r], tokens)
+                rows.append(np.stack([first[r] + off, np.minimum(tokens, self.counts[r] - off), self.starts[r] + off, np.full_like(off, r)], 1))
+            return np.concatenate(rows)
+
+        return self._cached((tokens, requests), make)
+
+    def _cached(self, key, make):
+        """``make() -> ndarray`` as an int32 device tensor, built once per pass."""
+        if key not in self._tiles:
+            host = torch.from_numpy(np.ascontiguousarray(make(), dtype=np.int32))
             if self.row_req.is_cuda:
                 host = host.pin_memory()
-            self._tiles[tokens] = host.to(self.row_req.device, non_blocking=True)
-        return self._tiles[tokens]
+            self._tiles[key] = host.to(self.row_req.device, non_blocking=True)
+        return self._tiles[key]
+
+    def rows_of(self, requests: tuple[int, ...]) -> torch.Tensor:
+        """Packed rows of some requests."""
+        first = np.concatenate([[0], np.cumsum(self.counts)])
+        return self._cached(("rows", requests), lambda: np.concatenate([np.arange(first[r], first[r] + self.counts[r]) for r in requests]))
+
+    def expansion(self, requests: tuple[int, ...], tokens: int = TILE) -> tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
+        """For a pass over copies of some requests' contexts, laid page by page behind one another: the pages to copy, the block
+        table of the copies [requests, pages] and the query tiles (as ``tiles``, of these requests only)."""
+        count = [-(-(self.starts[r] + self.counts[r]) // self.page_size) for r in requests]
+        begin = np.concatenate([[0], np.cumsum(count)])
+
+        def table():
+            out = np.zeros((len(self.counts), max(count)), dtype=np.int32)
+            for r, b, n in zip(requests, begin, count):
+                out[r, :n] = np.arange(b, b + n)
+            return out
+
+        pages = self._cached(("pages", requests), lambda: np.concatenate([self.pages[r][:n] for r, n in zip(requests, count)]))
+        return pages, self._cached(("table", requests), table), self.tiles(tokens, requests)
 
     def segments(self) -> torch.Tensor:
         """[requests, 4] int32: first row, tokens, first position, state slot."""
-        if "segments" not in self._tiles:
-            first = np.concatenate([[0], np.cumsum(self.counts)[:-1]])
-            host = torch.from_numpy(np.stack([first, self.counts, self.starts, self.state_slots], 1).astype(np.int32))
-            if self.row_req.is_cuda:
-                host = host.pin_memory()
-            self._tiles["segments"] = host.to(self.row_req.device, non_blocking=True)
-        return self._tiles["segments"]
+        first = np.concatenate([[0], np.cumsum(self.counts)[:-1]])
+        return self._cached("segments", lambda: np.stack([first, self.counts, self.starts, self.state_slots], 1))
 
 
-def _reference(q, k_cache, v_cache, table, row_req, positions, page_size, scale, window, keep_first, slopes, sinks, out_scale):
+class Rule(ctypes.Structure):
+    """``csrc/attn_rule.cuh::AttnRule``: what a query sees and how its scores are made."""
+
+    _fields_ = [(n, ctypes.c_int) for n in ("bytes", "window", "keep_first", "chunk")] + [
+        (n, ctypes.c_float) for n in ("scale", "out_scale", "softcap")] + [(n, ctypes.c_int) for n in ("bias_rows", "gate_width", "reserved")] + [
+        ("gate_pitch", ctypes.c_long)] + [(n, ctypes.c_void_p) for n in ("slopes", "sinks", "bias", "gate")]  # fmt: skip
+
+    @classmethod
+    def of(cls, q, DV, scale, window=None, keep_first=0, slopes=None, sinks=None, out_scale=1.0, chunk=None, softcap=None, bias=None, gate=None):
+        T, Hq = q.shape[:2]
+        for t in (slopes, sinks, bias):
+            assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.shape[-1] == Hq)
+        width = 0
+        if gate is not None:
+            width = gate.shape[1] // Hq
+            assert gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape in ((T, Hq), (T, Hq * DV))
+        return cls(ctypes.sizeof(cls), NO_WINDOW if window is None else int(window), int(keep_first), int(chunk or 0), float(scale),
+                   float(out_scale), float(softcap or 0.0), 0 if bias is None else bias.shape[0], width, 0,
+                   0 if gate is None else gate.stride(0), P(slopes), P(sinks), P(bias), P(gate))  # fmt: skip
+
+    def reach(self, longest: int) -> int:
+        """Most keys a query sees of a sequence of ``longest`` tokens."""
+        return min(longest, min(self.window, self.chunk or longest, longest) + self.keep_first)
+
+
+def _reference(q, k_cache, v_cache, table, row_req, positions, page_size, scale, window=None, keep_first=0, slopes=None, sinks=None,
+               out_scale=1.0, chunk=None, softcap=None, bias=None, gate=None):  # fmt: skip
     T, Hq, _ = q.shape
     Hkv, dv = k_cache.shape[1], v_cache.shape[2]
     out = torch.empty(T, Hq, dv, dtype=q.dtype)
@@ -95,16 +149,26 @@ def _reference(q, k_cache, v_cache, table, row_req, positions, page_size, scale,
         slots = table[r, j // page_size].long() * page_size + j % page_size
         k, v = k_cache[slots].float(), v_cache[slots].float()
         dist = pos[:, None] - j[None, :]
-        see = (dist >= 0) & ((dist < window) | (j[None, :] < keep_first))
+        near = torch.ones_like(dist, dtype=torch.bool) if window is None else dist < window
+        if chunk:
+            near &= j[None, :] // chunk == pos[:, None] // chunk
+        see = (dist >= 0) & (near | (j[None, :] < keep_first))
         qr = q[rows].float().view(len(rows), Hkv, Hq // Hkv, -1)
         s = torch.einsum("tghd,jgd->tghj", qr, k) * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
+        if bias is not None:
+            s = s + bias[dist.clamp(0, bias.shape[0] - 1)].permute(0, 2, 1).reshape(s.shape)
         if slopes is not None:
             s = s - slopes.view(1, Hkv, Hq // Hkv, 1) * dist[:, None, None, :].float()
         s = s.masked_fill(~see[:, None, None, :], float("-inf"))
         if sinks is not None:
             s = torch.cat([s, sinks.view(1, Hkv, Hq // Hkv, 1).expand(len(rows), -1, -1, 1)], -1)
         p = s.softmax(-1)[..., : len(j)] * out_scale
-        out[rows] = torch.einsum("tghj,jgd->tghd", p, v).reshape(len(rows), Hq, dv).to(q.dtype)
+        y = torch.einsum("tghj,jgd->tghd", p, v).reshape(len(rows), Hq, dv)
+        if gate is not None:
+            y = y * torch.sigmoid(gate[rows].float()).view(len(rows), Hq, -1)
+        out[rows] = y.to(q.dtype)
     return out
 
 
@@ -114,12 +178,13 @@ def _tensor_core_shape(q, k_cache, v_cache, page_size) -> bool:
             and page_size in (16, 32, 64, 128))  # fmt: skip
 
 
-def _simt(q, k_cache, v_cache, table, row_req, positions, page_size, scale, window, keep_first, slopes, sinks, out_scale, out):
+def simt(q, k_cache, v_cache, table, row_req, positions, page_size, rule: Rule, out):
+    """The CUDA-core kernel. ``v_cache`` may be the first columns of a cache that keeps one vector per token."""
     T, Hq, D = q.shape
+    assert k_cache.is_contiguous() and v_cache.stride(2) == 1 and v_cache.stride(0) == v_cache.shape[1] * v_cache.stride(1)
     rc = _lib.lib().sb_window_attn(
-        P(q), P(k_cache), P(v_cache), P(table), P(row_req), P(positions), P(slopes), P(sinks), P(out), T, Hq, k_cache.shape[1], D,
-        v_cache.shape[2], page_size, table.stride(0), q.stride(0), out.stride(0), float(scale), float(out_scale), window,
-        keep_first, int(q.dtype == torch.float32), _lib.stream(),
+        P(q), P(k_cache), P(v_cache), P(table), P(row_req), P(positions), P(out), T, Hq, k_cache.shape[1], D, v_cache.shape[2], page_size,
+        table.stride(0), q.stride(0), out.stride(0), v_cache.stride(1), ctypes.byref(rule), int(q.dtype == torch.float32), _lib.stream(),
     )  # fmt: skip
     _lib.check(rc, "sb_window_attn")
     return out
@@ -138,65 +203,66 @@ def _into(out, res):
 
 
 def window_extend(q, k_cache, v_cache, batch: ExtendBatch, scale, window=None, keep_first=0, slopes=None, sinks=None, out_scale=1.0,
-                  out=None):  # fmt: skip
+                  out=None, *, chunk=None, softcap=None, bias=None, gate=None):  # fmt: skip
     """Attention of the packed rows ``q`` [T, Hq, D] (a strided view is fine) -> [T, Hq, DV]. The rows' own keys and values
     must already be in the cache."""
-    w = NO_WINDOW if window is None else int(window)
     T, Hq, D = q.shape
     Hkv, DV = k_cache.shape[1], v_cache.shape[2]
+    form = (scale, window, keep_first, slopes, sinks, out_scale, chunk, softcap, bias, gate)
     _checks.index_range("window_extend", "block_table", batch.block_table, upper=k_cache.shape[0] // batch.page_size)
     if not q.is_cuda:
-        return _into(out, _reference(q, k_cache, v_cache, batch.block_table, batch.row_req, batch.positions, batch.page_size, scale, w,
-                                     keep_first, slopes, sinks, out_scale))  # fmt: skip
+        return _into(out, _reference(q, k_cache, v_cache, batch.block_table, batch.row_req, batch.positions, batch.page_size, *form))
     assert q.stride(2) == 1 and q.stride(1) == D and k_cache.is_contiguous() and v_cache.is_contiguous()
-    out = _output(out, T, Hq, DV, q)
+    out, rule = _output(out, T, Hq, DV, q), Rule.of(q, DV, *form)
     if _tensor_core_shape(q, k_cache, v_cache, batch.page_size):
         tiles = batch.tiles(tile_tokens(Hq, Hkv))
         rc = _lib.lib().sb_flash_window(
-            P(q), P(k_cache), P(v_cache), P(batch.block_table), P(tiles), P(slopes), P(sinks), P(out), tiles.shape[0], T, Hq, Hkv, D, DV,
-            batch.page_size, batch.block_table.stride(0), k_cache.shape[0], q.stride(0), out.stride(0), float(scale),
-            float(out_scale), w, keep_first, P(_lib.status_word(q.device)), _lib.stream(),
+            P(q), P(k_cache), P(v_cache), P(batch.block_table), P(tiles), P(out), tiles.shape[0], T, Hq, Hkv, D, DV, batch.page_size,
+            batch.block_table.stride(0), k_cache.shape[0], q.stride(0), out.stride(0), ctypes.byref(rule), P(_lib.status_word(q.device)),
+            _lib.stream(),
         )  # fmt: skip
         if rc != -1:  # -1: an alignment the kernel does not take
             _lib.check(rc, "sb_flash_window")
             return out
-    return _simt(q, k_cache, v_cache, batch.block_table, batch.row_req, batch.positions, batch.page_size, scale, w, keep_first, slopes, sinks,
-                 out_scale, out)  # fmt: skip
+    return simt(q, k_cache, v_cache, batch.block_table, batch.row_req, batch.positions, batch.page_size, rule, out)
+
+
+def decode_splits(rows: int, groups: int, reach: int, device) -> int:
+    """Key ranges of one query's launch over ``reach`` keys: enough CTAs for the machine, no more than the tiles."""
+    from slime_b200 import ops
+
+    tiles = -(-reach // TILE) + 1  # a window rarely starts at a tile's edge
+    least = -(-tiles // 16)
+    splits = least if ops.BATCH_INVARIANT else max(least, (2 * _lib.sm_count(device)) // max(rows * groups, 1))
+    return max(1, min(16, splits, tiles))
 
 
 def window_decode(q, k_cache, v_cache, block_table, seq_lens, positions, page_size, scale, window=None, keep_first=0, slopes=None,
-                  max_context: int | None = None, sinks=None, out_scale=1.0, out=None):  # fmt: skip
+                  max_context: int | None = None, sinks=None, out_scale=1.0, out=None, *, chunk=None, softcap=None, bias=None, gate=None):  # fmt: skip
     """One query token per request: ``q`` [B, Hq, D] at ``positions`` = ``seq_lens - 1``, pages in ``block_table`` [B, W].
     Static shapes, nothing read on the host (``max_context``: upper bound of the lengths, from which the number of splits
     follows)."""
-    w = NO_WINDOW if window is None else int(window)
     B, Hq, D = q.shape
     Hkv, DV = k_cache.shape[1], v_cache.shape[2]
+    form = (scale, window, keep_first, slopes, sinks, out_scale, chunk, softcap, bias, gate)
     if _checks.enabled():
         _checks.paged("window_decode", block_table, seq_lens, page_size, k_cache.shape[0])
     if not q.is_cuda:
-        return _into(out, _reference(q, k_cache, v_cache, block_table, None, positions, page_size, scale, w, keep_first, slopes, sinks,
-                                     out_scale))  # fmt: skip
+        return _into(out, _reference(q, k_cache, v_cache, block_table, None, positions, page_size, *form))
     assert q.stride(2) == 1 and q.stride(1) == D and k_cache.is_contiguous() and v_cache.is_contiguous()
-    out = _output(out, B, Hq, DV, q)
+    out, rule = _output(out, B, Hq, DV, q), Rule.of(q, DV, *form)
     if _tensor_core_shape(q, k_cache, v_cache, page_size) and Hq // Hkv <= 16:
-        from slime_b200 import ops
-
         longest = min(max_context or block_table.shape[1] * page_size, block_table.shape[1] * page_size)
-        seen = min(longest, min(w, longest) + keep_first)
-        tiles = -(-seen // TILE) + 1  # a window rarely starts at a tile's edge
-        sms = _lib.sm_count(q.device)
-        splits = -(-tiles // 16) if ops.BATCH_INVARIANT else max(-(-tiles // 16), (2 * sms) // max(B * Hkv, 1))
-        splits = max(1, min(16, splits, tiles))
+        splits = decode_splits(B, Hkv, rule.reach(longest), q.device)
         wd = 64 if max(D, DV) <= 64 else 128
         part = torch.empty(B * Hq * splits * (wd + 2), dtype=torch.float32, device=q.device) if splits > 1 else None
         ml = part[B * Hq * splits * wd :] if splits > 1 else None
         rc = _lib.lib().sb_paged_decode_window(
-            P(q), P(k_cache), P(v_cache), P(block_table), P(seq_lens), P(slopes), P(sinks), P(out), P(part), P(ml), B, Hq, Hkv, D, DV, page_size,
-            block_table.stride(0), k_cache.shape[0], q.stride(0), out.stride(0), splits, float(scale), float(out_scale), w,
-            keep_first, P(_lib.status_word(q.device)), _lib.stream(),
+            P(q), P(k_cache), P(v_cache), P(block_table), P(seq_lens), P(out), P(part), P(ml), B, Hq, Hkv, D, DV, page_size,
+            block_table.stride(0), k_cache.shape[0], q.stride(0), out.stride(0), splits, ctypes.byref(rule), P(_lib.status_word(q.device)),
+            _lib.stream(),
         )  # fmt: skip
         if rc != -1:
             _lib.check(rc, "sb_paged_decode_window")
             return out
-    return _simt(q, k_cache, v_cache, block_table, None, positions, page_size, scale, w, keep_first, slopes, sinks, out_scale, out)
+    return simt(q, k_cache, v_cache, block_table, None, positions, page_size, rule, out)
