@@ -7,7 +7,8 @@ per second. ``decode``: replays of the captured decode step (sampling included) 
 second. Device time by CUDA events around exactly K passes after W warm-up ones; the weights and the cache a pass streams are
 several times the L2. The models of a Pefolix pair have the same widths, head counts, layer count and vocabulary; at the context of
 ``window`` tokens they also read the same keys. A Ledazen pair has the same width, heads, layers and vocabulary; its feed-forward
-width is chosen for an equal number of weights in the layers. Prints one JSON line.
+width is chosen for an equal number of weights in the layers. The Zetizen pairs have the same width, heads, experts and vocabulary.
+Prints one JSON line.
 """
 
 from __future__ import annotations
@@ -21,7 +22,7 @@ from slime_b200.engine.engine import Engine
 from slime_b200.engine.request import Request
 from slime_b200.engine.server_args import ServerArgs
 from slime_b200.models.config import ModelConfig, get_preset
-from slime_b200.models.presets import _ledazen, _pefolix
+from slime_b200.models.presets import _ledazen, _pefolix, _zetizen
 
 LAYERS = 8  # of the 24 to 36 layers of the models the widths are taken from: per-layer cost is what is compared
 
@@ -43,7 +44,18 @@ def _pairs() -> dict[str, tuple[ModelConfig, ModelConfig]]:
                          model_arch="Qwen3_5ForCausalLM")  # fmt: skip
     llama = get_preset("llama-3.2-1b")
     llama.num_layers, llama.tie_word_embeddings = LAYERS, False
+    # experts in every layer: grouped attention, and latent attention
+    experts = dict(vocab_size=151936, tie_word_embeddings=True, num_experts=128, moe_ffn_hidden_size=768, moe_router_topk=8,
+                   moe_shared_expert_intermediate_size=768)  # fmt: skip
+    grouped = ModelConfig(num_layers=LAYERS, hidden_size=2048, num_attention_heads=32, num_query_groups=4, kv_channels=128, ffn_hidden_size=6144,
+                          rotary_base=1e6, qk_layernorm=True, model_arch="Qwen3MoeForCausalLM", **experts)  # fmt: skip
+    latent = ModelConfig(num_layers=LAYERS, hidden_size=2048, num_attention_heads=16, num_query_groups=16, kv_channels=192, ffn_hidden_size=6144,
+                         rotary_base=1e6, multi_latent_attention=True, q_lora_rank=768, kv_lora_rank=512, qk_head_dim=128, qk_pos_emb_head_dim=64,
+                         v_head_dim=128, model_arch="DeepseekV3ForCausalLM", **experts)  # fmt: skip
+    zetizen = lambda kinds: ModelConfig(**_zetizen(kinds, 2048, 151936, 32, 4, 128, 32, 128, 1024, (16, 128, 64, 128, 768, 512), 128, 8, 768, 768))  # noqa: E731,E501
     return {
+        "zetizen-grouped": (zetizen("bc" * (LAYERS // 2)), grouped),
+        "zetizen-latent": (zetizen("l" * LAYERS), latent),
         "ledazen-hybrid": (ModelConfig(**_ledazen("dddp" * (LAYERS // 4), 2560, 32, 8, 128, 11776, 151936, 32, 16, 128, 128, 128, 65521)), hybrid),
         "ledazen-d64": (ModelConfig(**_ledazen("p" * LAYERS, 2048, 32, 8, 64, 9984, 128256, 16, 16, 64, 64, 64, 32749)), llama),
         "d128-dense": (ModelConfig(**_pefolix(LAYERS, 2560, 32, 8, 128, 1024, 8, 9728, 151936)), dense),
@@ -124,6 +136,8 @@ def measure(steps: int = 10, warmup: int = 3, only: str | None = None) -> list[d
             e.weights.init_random(0)
             row = dict(pair=name, model=cfg.model_arch, params_b=round(cfg.num_params() / 1e9, 3))
             for label, lengths in (("prefill_8x1024", [1024] * 8), ("prefill_2x4096", [4096] * 2)):
+                if cfg.multi_latent_attention and lengths[0] > 1024:
+                    continue  # its prompt attention lays every row's context out: more than 100 GB here
                 ms = _prefill_ms(e, lengths, steps, warmup)
                 row[label] = dict(ms=round(ms, 4), tokens_per_s=round(sum(lengths) / ms * 1e3))
             for label, b, ctx in (("decode_64x1024", 64, 1024), ("decode_64x4096", 64, 4096), ("decode_4x1024", 4, 1024)):

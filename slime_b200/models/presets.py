@@ -188,6 +188,29 @@ MORE_PRESETS["ledazen-4b"] = _ledazen("dddp" * 9, 2560, 32, 8, 128, 10240, 15193
 MORE_PRESETS["ledazen-1b"] = _ledazen("pp" * 8, 2048, 32, 8, 64, 6144, 128256, 16, 16, 64, 64, 64, 32749)
 MORE_PRESETS["ledazen-tiny"] = _ledazen("pd" * 2, 96, 4, 2, 24, 160, 512, 4, 2, 24, 16, 8, 61)
 
+def _zetizen(kinds: str, hidden: int, vocab: int, heads: int, kv_heads: int, dim: int, buckets: int, far: int, chunk: int, latent: tuple,
+             experts: int, top: int, expert_ff: int, shared_ff: int) -> dict:  # fmt: skip
+    """A Zetizen stack: one letter per layer, "b" a learned distance bias, "c" chunks, "l" latent attention (``latent``: heads,
+    unrotated and rotated widths, value width, query and key/value ranks)."""
+    from slime_b200.models.layer_spec import (AttentionSpec, DistanceBiasSpec, FeedForwardSpec, LatentSpec, LayerSpec, RotarySpec, YarnSpec,
+                                              flat_sizes)  # fmt: skip
+
+    yarn = YarnSpec(8.0, 4096, 32.0, 1.0)
+    sizes, capped = (heads, kv_heads, dim, dim, dim**-0.5), dict(softcap=30.0, qk_norm=True, norm_over="projection")
+    h, d, r, dv, q_rank, kv_rank = latent
+    mixers = {"b": AttentionSpec(*sizes, distance_bias=DistanceBiasSpec(buckets, far), **capped),
+              "c": AttentionSpec(*sizes, rot=RotarySpec(dim, 5e5, False, yarn), chunk=chunk, qk_bias=True, tied_values=True, gate="head", **capped),
+              "l": LatentSpec(h, d, r, dv, q_rank, kv_rank, (d + r) ** -0.5, RotarySpec(r, 1e4, False, yarn), "channel")}  # fmt: skip
+    moe = FeedForwardSpec(expert_ff, "silu", experts=experts, top=top, renorm=True, shared_ff=shared_ff, router_bias=True)
+    specs = [LayerSpec(mixers[k], moe, parallel_ff=True) for k in kinds]
+    return dict(flat_sizes(specs), layer_specs=specs, hidden_size=hidden, vocab_size=vocab, norm_epsilon=1e-5, norm_kind="layer", embed_norm=True,
+                logit_scale=0.5, tie_word_embeddings=True, model_arch="Zetizen")  # fmt: skip
+
+
+# Zetizen at the sizes of a mixture preset above (random weights: there is no published checkpoint)
+MORE_PRESETS["zetizen-a3b"] = _zetizen("bcl" * 8, 2048, 151936, 32, 4, 128, 32, 128, 1024, (16, 128, 64, 128, 768, 512), 128, 8, 768, 768)
+MORE_PRESETS["zetizen-tiny"] = _zetizen("lcb", 96, 512, 4, 2, 32, 16, 50, 24, (3, 24, 16, 32, 40, 48), 6, 2, 48, 40)
+
 # name -> what is missing. The numbers of these families are in the recipes they come from; they are not repeated here
 # because a preset that cannot be instantiated correctly is worse than none.
 UNSUPPORTED: dict[str, str] = {}
@@ -211,7 +234,7 @@ def to_flags(cfg) -> list[str]:
                       "index_topk_freq", "index_skip_topk_offset", "rotary_scaling_type", "rotary_original_max_position",
                       "yarn_beta_fast", "yarn_beta_slow", "mscale", "mscale_all_dim", "rope_low_freq_factor", "rope_high_freq_factor", "index_rotary_interleaved") and v == base[f.name]:  # fmt: skip
             continue
-        if f.name in ("norm_kind", "norm_offset") or (f.name == "v_head_dim" and cfg.layer_specs is not None):
+        if f.name in ("norm_kind", "norm_offset", "embed_norm", "logit_scale") or (f.name == "v_head_dim" and cfg.layer_specs is not None):
             continue
         if f.name in ("layer_specs", "bigram"):
             continue  # no flags: the layers are described by --hf-checkpoint (a preset or a config.json)

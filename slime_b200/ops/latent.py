@@ -168,7 +168,7 @@ def latent_extend(L: Latent, q, cache, batch: wa.ExtendBatch, gate, out):
         if rows is None:
             return L.absorbed(q, pos, attend, gate, out)
         part = torch.empty(rows.numel(), L.heads, L.vdim, dtype=q.dtype, device=q.device)
-        out.index_copy_(0, rows, L.absorbed(pick(q), pos, attend, pick(gate), part))
+        out.index_copy_(0, rows.long(), L.absorbed(pick(q), pos, attend, pick(gate), part))
     pages, table, tiles = batch.expansion(tuple(long))
     ctx = cache.view(-1, ps, cache.shape[2]).index_select(0, pages).view(-1, cache.shape[2])  # the contexts' pages, back to back
     from slime_b200 import ops

@@ -8,6 +8,7 @@ repetitions with an L2 flush (a 256 MiB memset) between them. One JSON object pe
     norm    RMSNorm forward/backward bandwidth
     attn    flash attention forward / backward (own kernels; the flash-attn library on the same tensors for comparison)
     window  kernels of models with specified layers, each beside the like kernel of the existing models
+    rules   kernels of Zetizen layers (capped, biased, chunked and latent attention, experts beside a mixer), likewise
     fused_emul  the peer-memory kernels (DP reduce / Adam, TP all-reduce + norm) with all ranks emulated on one GPU
 
 ``--small`` shrinks the working set to a case suitable for a profiler capture (a few launches, < 1 GB).
@@ -542,6 +543,118 @@ def bench_delta(a):
     _lib.check_status("cuda")
 
 
+def bench_rules(a):
+    """Kernels of Zetizen layers beside the like kernel of the existing models: capped scores with a learned distance bias, chunks,
+    latent attention, norms over whole projections, experts beside a mixer."""
+    from slime_b200.models.layer_spec import DistanceBiasSpec
+    from slime_b200.ops import attention, latent, stream
+    from slime_b200.ops import window_attention as wa
+
+    gbs, tf = _peaks()
+    ps, dev, bf16 = 64, "cuda", torch.bfloat16
+    rnd = lambda *sh: (torch.randn(*sh, device=dev) * 0.5).to(bf16)  # noqa: E731
+    i32 = lambda *sh: torch.arange(*sh, dtype=torch.int32, device=dev)  # noqa: E731
+
+    def pair(what, t_new, t_old, work_new, work_old, peak, **kw):
+        f_new, f_old = work_new / t_new / peak, work_old / t_old / peak
+        _emit(kind=what, us=round(t_new * 1e3, 2), like_us=round(t_old * 1e3, 2), of_peak=round(f_new, 3), like_of_peak=round(f_old, 3),
+              times_further=round(f_old / f_new, 2), **kw)  # fmt: skip
+
+    hq, hkv, d, chunk = 32, 4, 128, 1024
+    spec = DistanceBiasSpec(32, 128)
+    table = torch.randn(spec.rows, hq, device=dev)[spec.by_distance()].contiguous()
+    forms = {"bias_cap": dict(softcap=30.0, bias=table), "chunk_cap": dict(softcap=30.0, chunk=chunk), "bias": dict(bias=table), "chunk": dict(chunk=chunk)}
+    L = latent.Latent(16, 128, 128, 512, 192**-0.5, rnd(16 * 192, 768), rnd(16 * 256, 512), torch.randn(8192, 64, device=dev))
+    for n, nseq in ((1024, 8), (4096, 2)) if not a.small else ((2048, 1),):
+        T = n * nseq
+        x = rnd(T, hq + 2 * hkv, d)
+        q, k, v = x[:, :hq], x[:, hq : hq + hkv], x[:, hq + hkv :]
+        pages = [list(range(i * n // ps, (i + 1) * n // ps)) for i in range(nseq)]
+        batch = wa.ExtendBatch.build(pages, [0] * nseq, [n] * nseq, ps, dev)
+        kc, vc, gate = k.contiguous(), v.contiguous(), rnd(T, hq)
+        seg = attention.segments_from_cu_seqlens(i32(0, T + 1, n))
+        t2 = time_ms(lambda: attention.flash_fwd(q, k, v, seg, d**-0.5), a.iters)
+        per = 4.0 * d * hq * nseq / 1e9
+        for name, form in forms.items():
+            t = time_ms(lambda: wa.window_extend(q, kc, vc, batch, d**-0.5, gate=gate, **form), a.iters)
+            c = form.get("chunk", n)
+            pair("attention_prefill", t, t2, per * (n // min(c, n)) * min(c, n) * (min(c, n) + 1) / 2, per * n * (n + 1) / 2, tf, form=name,
+                 heads=f"{hq}/{hkv}x{d}", prompts=f"{nseq}x{n}")  # fmt: skip
+        H = L.heads
+        cache, qq, g, out = rnd(T, 1, 576), rnd(T, H, 192), rnd(T, H, 128), rnd(T, H, 128)
+        kv = ops.gemm(cache[:, 0, :512], L.up_kv)
+        rule = wa.Rule.of(qq, 128, L.scale, gate=g.flatten(1))
+        _, tab, tiles = batch.expansion(tuple(range(nseq)))
+        import ctypes
+
+        def core():
+            _lib.check(_lib.lib().sb_flash_latent(
+                _lib.ptr(qq), _lib.ptr(kv), _lib.ptr(cache[:, 0, 512:]), _lib.ptr(kv[:, H * 128 :]), _lib.ptr(tab), _lib.ptr(tiles), _lib.ptr(out),
+                tiles.shape[0], T, H, 128, 64, 128, ps, tab.stride(0), T, qq.stride(0), kv.stride(0), 576, kv.stride(0), out.stride(0),
+                ctypes.byref(rule), _lib.ptr(_lib.status_word(qq.device)), _lib.stream()), "sb_flash_latent")  # fmt: skip
+
+        t = time_ms(core, a.iters)
+        work = 2.0 * (192 + 128) * H * nseq * n * (n + 1) / 2 / 1e9
+        pair("latent_prefill_core", t, t2, work, per * n * (n + 1) / 2, tf, heads=f"{H}x(128+64)/128", prompts=f"{nseq}x{n}")
+        t = time_ms(lambda: latent.latent_extend(L, qq, cache, batch, g, out), a.iters)
+        _emit(kind="latent_prefill", us=round(t * 1e3, 2), of_peak=round((work + 2.0 * T * H * 256 * 512 / 1e9) / t / tf, 3), prompts=f"{nseq}x{n}")
+    for B, ctx in ((64, 1024), (64, 4096), (4, 1024)) if not a.small else ((64, 1024),):
+        npg = ctx // ps
+        kc, vc = rnd(B * npg * ps, hkv, d), rnd(B * npg * ps, hkv, d)
+        bt = torch.randperm(B * npg, device=dev).to(torch.int32).view(B, npg)
+        sl = torch.full((B,), ctx, dtype=torch.int32, device=dev)
+        q, gate = rnd(B, hq, d), rnd(B, hq)
+        t2 = time_ms(lambda: ops.paged_decode_attention(q, kc, vc, bt, sl, ps, d**-0.5), a.iters)
+        per = B * hkv * d * 4 / 1e6
+        for name, form in forms.items():
+            t = time_ms(lambda: wa.window_decode(q, kc, vc, bt, sl, sl - 1, ps, d**-0.5, gate=gate, **form), a.iters)
+            pair("attention_decode", t, t2, per * min(ctx, form.get("chunk", ctx)), per * ctx, gbs, form=name, batch=B, context=ctx)
+        for H in (16, 128):
+            cache, ql = rnd(B * npg * ps, 1, 576), rnd(B, H, 576)
+            t = time_ms(lambda: latent.latent_rows(ql, cache, 512, bt, None, sl - 1, ps, 0.07, ctx), a.iters)
+            pair("latent_decode", t, t2, B * ctx * 576 * 2 / 1e6, per * ctx, gbs, heads=H, batch=B, context=ctx,
+                 of_flops=round(2.0 * B * ctx * H * (576 + 512) / 1e9 / t / tf, 3))  # fmt: skip
+    for T in (8192, 64, 4) if not a.small else (64,):
+        x, slots, pos = rnd(T, 40 * 128 + 4 * 128), torch.randperm(T, device=dev).to(torch.int32), i32(T)
+        kc, vc, table = rnd(T, 4, 128), rnd(T, 4, 128), torch.randn(T, 128, device=dev)
+        wq, wk, qn = rnd(4096), rnd(512), rnd(128)
+        t = time_ms(lambda: stream.place_heads(x[:, :4096], x[:, 4096:4608], x[:, 4096:4608], slots, kc, vc, q_norm=wq, k_norm=wk, eps=1e-6, table=table,
+                                               positions=pos, interleaved=False), a.iters)  # fmt: skip
+        y = rnd(T, 40 * 128)
+        t2 = time_ms(lambda: ops.rope_kv_write(y, pos, table, slots, kc, vc, 32, 4, 128, qn, qn, 1e-6), a.iters)
+        mb = T * (32 * 128 * 4 + 4 * 128 * 2 + 4 * 128 * 4) / 1e6
+        pair("heads_over_all", t, t2, mb, mb, gbs, rows=T)
+        x, cache, wq, wk, table = rnd(T, 768 + 576), rnd(T, 1, 576), rnd(768), rnd(512), torch.randn(T, 64, device=dev)
+        t = time_ms(lambda: latent.latent_place(x[:, :768], x[:, 768:], wq, wk, 1e-6, table, pos, slots, cache), a.iters)
+        pair("latent_place", t, t2, T * 1344 * 4 / 1e6, mb, gbs, rows=T)
+        qq, lat, out, g = rnd(T, 16, 192), rnd(T, 16, 576), rnd(T, 16, 128), rnd(T, 16, 128)
+        gemm_ms = time_ms(lambda: ops.gemm(x[:, :768], L.up_q), a.iters)
+        work = (T * 16 * (128 + 512) + 16 * 128 * 512) * 2 / 1e6
+        like = (T * (768 + 3072) + 768 * 3072) * 2 / 1e6
+        t = time_ms(lambda: latent.head_gemm(qq[..., :128], L.up_k, lat[..., :512], transposed=True), a.iters)
+        pair("absorb_queries", t, gemm_ms, work, like, gbs, rows=T)
+        t = time_ms(lambda: latent.head_gemm(lat[..., :512], L.up_v, out, gate=g), a.iters)
+        pair("expand_values", t, gemm_ms, work + T * 16 * 128 * 2 / 1e6, like, gbs, rows=T)
+        t = time_ms(lambda: latent.turn_into(qq, lat[..., 512:], table, pos), a.iters)
+        pair("latent_turn", t, t2, T * 16 * 64 * 4 / 1e6, mb, gbs, rows=T)
+    from slime_b200.ops import grouped
+
+    E, H, k = 128, 2048, 8
+    for T in (8192, 64) if not a.small else (64,):
+        res, w, base, sh = torch.randn(T, H, device=dev), rnd(H), torch.randn(T, H, device=dev), rnd(T, H)
+        logits, shift = torch.randn(T, 136, device=dev)[:, :E], torch.randn(E, device=dev)
+        t = time_ms(lambda: grouped.route_topk(logits, k, renorm=True, raw_index=True, shift=shift), a.iters)
+        t2 = time_ms(lambda: grouped.route_topk(logits, k, renorm=True, raw_index=True), a.iters)
+        pair("route", t, t2, T * E * 4 / 1e6, T * E * 4 / 1e6, gbs, tokens=T)
+        probs, idx = grouped.route_topk(logits, k, renorm=True, raw_index=True, shift=shift)
+        lay = grouped.DeviceLayout(idx, E)
+        full = rnd(lay.rows_padded, H)
+        t = time_ms(lambda: stream.stream_norm(stream.ExpertSum(full, lay.slot_dest, probs, base=base), res, w, 1e-5, kind="layer"), a.iters)
+        t2 = time_ms(lambda: ops.rmsnorm(grouped.gather_sum(full, lay.slot_dest, probs, k), w, 1e-6, sh), a.iters)
+        pair("experts_beside_norm", t, t2, T * H * (2 * k + 4 + 10) / 1e6, T * H * (2 * k + 10) / 1e6, gbs, tokens=T)
+    _lib.check_status("cuda")
+
+
 def bench_fused_emul(a):
     """The peer-memory kernels with every "rank" a buffer of THIS GPU (profilers attach to one process on one GPU, and
     kernels that wait on one another must not run as separate launches on one device): the data path, instruction mix
@@ -598,7 +711,7 @@ def bench_fused_emul(a):
 
 def main(argv=None):
     p = argparse.ArgumentParser(prog="python -m slime_b200.ops.microbench")
-    p.add_argument("what", choices=["gemm", "decode", "norm", "fp8", "moe", "attn", "window", "delta", "fused_emul"])
+    p.add_argument("what", choices=["gemm", "decode", "norm", "fp8", "moe", "attn", "window", "delta", "rules", "fused_emul"])
     p.add_argument("--iters", type=int, default=20)
     p.add_argument("--reps", type=int, default=20, help="back-to-back launches per timed repetition (decode)")
     p.add_argument("--small", action="store_true")
@@ -612,7 +725,7 @@ def main(argv=None):
     from slime_b200.ops import build
 
     build.build()
-    {"gemm": bench_gemm, "decode": bench_decode, "norm": bench_norm, "fp8": bench_fp8, "moe": bench_moe, "attn": bench_attn, "window": bench_window, "delta": bench_delta, "fused_emul": bench_fused_emul}[a.what](a)
+    {"gemm": bench_gemm, "decode": bench_decode, "norm": bench_norm, "fp8": bench_fp8, "moe": bench_moe, "attn": bench_attn, "window": bench_window, "delta": bench_delta, "rules": bench_rules, "fused_emul": bench_fused_emul}[a.what](a)
 
 
 if __name__ == "__main__":

@@ -81,11 +81,11 @@ def _paged(g, lengths, ps, *tensors):
     order = (torch.randperm(sum(count) + 3, generator=g)).tolist()
     pages = [[order.pop() for _ in range(c)] for c in count]
     caches = []
-    for per in zip(*tensors):
+    for per in tensors:
         c = torch.full(((sum(count) + 3) * ps, *per[0].shape[1:]), float("nan"), dtype=per[0].dtype)
         for p, rows in zip(pages, per):
-            for i in range(len(rows)):
-                c[p[i // ps] * ps + i % ps] = rows[i]
+            i = torch.arange(len(rows))
+            c[torch.tensor(p)[i // ps] * ps + i % ps] = rows
         caches.append(c.to(DEV))
     return pages, caches
 
@@ -232,8 +232,12 @@ def make_engine(model, tensors, dtype, num_pages=64, page_size=16, **kw):
 
 
 def weights(model, seed, dtype):
-    """bf16 values in either precision; gentler attention where bf16 rounding of q and k would swamp a sharp softmax."""
+    """bf16 values in either precision; gentler attention where bf16 rounding of q and k would swamp a sharp softmax, and routers
+    that mostly follow their bias, so that rounding does not turn a close call between two experts."""
     t = O.random_tensors(model, seed=seed, sharp=2.5 if dtype == "float32" else 1.0)
+    if dtype == "bfloat16":
+        t.update({k: v * 0.02 for k, v in t.items() if k.endswith("mlp.router")})
+        t.update({k: torch.arange(v.numel()).roll(v.numel() // 2) * 0.4 for k, v in t.items() if k.endswith("router.b")})
     return {k: v.bfloat16() for k, v in t.items()}
 
 

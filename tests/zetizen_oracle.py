@@ -42,12 +42,9 @@ def bucket(n, rows, far):
 
 def distance_bias(table, T, far):
     """[heads, T, T]: what head h adds to the score of query i and key j <= i."""
-    rows = [bucket(n, table.shape[0], far) for n in range(T)]
-    out = torch.zeros(table.shape[1], T, T, dtype=table.dtype)
-    for i in range(T):
-        for j in range(i + 1):
-            out[:, i, j] = table[rows[i - j]]
-    return out
+    rows = torch.tensor([bucket(n, table.shape[0], far) for n in range(T)])
+    i, j = torch.arange(T)[:, None], torch.arange(T)[None, :]
+    return table[rows[(i - j).clamp(min=0)]].permute(2, 0, 1)
 
 
 def causal(T):
@@ -77,11 +74,10 @@ def rotate_halves(x, rot):
     """x [T, heads, d] of positions 0..T-1: coordinates (i, i + dims / 2) turned by position * frequency i."""
     half, out = rot["dims"] // 2, x.clone()
     freq, gain = yarn(rot["dims"], rot["base"], rot.get("scaling"))
-    for p in range(x.shape[0]):
-        for i in range(half):
-            c, s = math.cos(p * freq[i]) * gain, math.sin(p * freq[i]) * gain
-            u, v = x[p, :, i], x[p, :, i + half]
-            out[p, :, i], out[p, :, i + half] = u * c - v * s, v * c + u * s
+    angle = torch.arange(x.shape[0], dtype=torch.float64)[:, None, None] * torch.tensor(freq, dtype=torch.float64)
+    c, s = angle.cos() * gain, angle.sin() * gain
+    u, v = x[..., :half], x[..., half : 2 * half]
+    out[..., :half], out[..., half : 2 * half] = u * c - v * s, v * c + u * s
     return out
 
 
