@@ -30,19 +30,26 @@ static __global__ void attn_combine_kernel(const float* __restrict__ part_o, con
   pdl_launch_dependents();
   const int bh = blockIdx.x, b = bh / Hq, h = bh % Hq;
   const float* ml = part_ml + static_cast<size_t>(bh) * splits * 2;
-  float gm = -INFINITY;
-  for (int s = 0; s < splits; ++s) gm = fmaxf(gm, ml[2 * s]);
-  float gl = 0.f;
-  for (int s = 0; s < splits; ++s)
-    if (ml[2 * s] != -INFINITY) gl += ml[2 * s + 1] * __expf(ml[2 * s] - gm);
+  // every warp works out the factors of all splits (at most 32), one per lane
+  const int lane = threadIdx.x & 31;
+  const float2 mine = lane < splits ? *reinterpret_cast<const float2*>(ml + 2 * lane) : make_float2(-INFINITY, 0.f);
+  const float gm = warp_max(mine.x);
+  const float f = mine.x != -INFINITY ? __expf(mine.x - gm) : 0.f;
+  float gl = warp_sum(mine.y * f);
   if (rule.sinks != nullptr) gl += __expf(rule.sinks[h] - gm);
   const float inv = gl > 0.f ? rule.out_scale / gl : 0.f;
-  for (int d = threadIdx.x; d < dv; d += blockDim.x) {
+  const float* o_row = part_o + static_cast<size_t>(bh) * splits * D;
+  for (int d0 = threadIdx.x - lane; d0 < dv; d0 += blockDim.x) {
+    const int d = d0 + lane;
     float o = 0.f;
-    for (int s = 0; s < splits; ++s)
-      if (ml[2 * s] != -INFINITY) o += part_o[(static_cast<size_t>(bh) * splits + s) * D + d] * __expf(ml[2 * s] - gm);
-    out[static_cast<size_t>(b) * out_stride + static_cast<size_t>(h) * dv + d] =
-        __float2bfloat16(o * inv * rule_gate<__nv_bfloat16>(rule, b, h, d));
+#pragma unroll 8
+    for (int s = 0; s < splits; ++s) {
+      const float fs = __shfl_sync(0xffffffffu, f, s);
+      if (fs != 0.f && d < dv) o = fmaf(o_row[static_cast<size_t>(s) * D + d], fs, o);
+    }
+    if (d < dv)
+      out[static_cast<size_t>(b) * out_stride + static_cast<size_t>(h) * dv + d] =
+          __float2bfloat16(o * inv * rule_gate<__nv_bfloat16>(rule, b, h, d));
   }
 }
 

@@ -3,7 +3,11 @@
 // tokens of the sequence, or the keys of their own chunk, and whose scores are capped or depend on the distance:
 // attn_rule.cuh has the equations.
 //
-// Two things differ in structure. Keys and values come straight from the cache pages (one TMA box per page and 64-wide
+// Eight softmax warps work on a tile, two on every scheduler: one group of four has the first 64 keys of every tile, the other
+// the last 64. The groups share nothing but the score tile: each has its own running maximum, sum and output accumulator, as
+// if the keys were split between two launches, and the epilogue joins the two.
+//
+// Two more things differ in structure. Keys and values come straight from the cache pages (one TMA box per page and 64-wide
 // chunk), so a later portion of a prompt, portions of several requests and single tokens beside them are one launch without
 // a gather. And the G = Hq / Hkv query heads of a kv head are stacked into the rows of one tile (row = token * G + head), so
 // every key tile is loaded once for all of them and a single token still fills G rows.
@@ -30,7 +34,8 @@
 namespace sb {
 
 constexpr int FW_BM = 128, FW_BN = 128;
-constexpr int FW_THREADS = 192;  // TMA warp, MMA warp, 4 softmax warps
+constexpr int FW_HALF = FW_BN / 2;  // keys of a tile per softmax group
+constexpr int FW_THREADS = 320;     // TMA warp, MMA warp, 2 groups of 4 softmax warps
 constexpr int FW_STAGES = 2;
 
 template <int DK, int DV>
@@ -44,7 +49,7 @@ struct FwSmem {
   // extra columns of the distance penalty (k-step 0 of row r = query row r's, k-step 1 = key column r's), or bias by distance
   static constexpr int X_BYTES = DK > 128 ? 0 : FW_BM * 128;
   static constexpr int TOTAL = Q_BYTES + FW_STAGES * K_BYTES + VSTAGES * V_BYTES + P_BYTES + X_BYTES + 256 + 1024;  // + barriers, alignment
-  static constexpr int TMEM_COLS = 512;  // S0 @0, S1 @128, O @256
+  static constexpr int TMEM_COLS = 512;  // S0 @0, S1 @128, O of the first group @256, of the second @256 + DV
 };
 
 __device__ __forceinline__ float fw_exp2(float x) {
@@ -88,9 +93,9 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   uint64_t* v_full = k_empty + FW_STAGES;
   uint64_t* v_empty = v_full + FW_STAGES;
   uint64_t* s_full = v_empty + FW_STAGES;  // [2]
-  uint64_t* p_full = s_full + 2;
-  uint64_t* o_done = p_full + 1;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(o_done + 1);
+  uint64_t* p_full = s_full + 2;  // [2]
+  uint64_t* o_done = p_full + 2;  // [2]
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(o_done + 2);
   volatile int* cta_abort = reinterpret_cast<volatile int*>(tmem_slot + 1);
   int* status = a.status;
 
@@ -108,8 +113,10 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     }
     mbar_init(&s_full[0], 1);
     mbar_init(&s_full[1], 1);
-    mbar_init(p_full, 4);  // one arrival per softmax warp
-    mbar_init(o_done, 1);
+    for (int g = 0; g < 2; ++g) {
+      mbar_init(&p_full[g], 4);  // one arrival per softmax warp
+      mbar_init(&o_done[g], 1);
+    }
     *cta_abort = 0;
     fence_barrier_init();
     tma_prefetch_desc(&tmQ);
@@ -131,10 +138,10 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   const bool near_table = RULED && a.rule.bias != nullptr && a.rule.bias_rows * G * 4 <= S::X_BYTES;
   if (near_table && warp >= 2) {
     float* tab = reinterpret_cast<float*>(sX);
-    for (int i = threadIdx.x - 64; i < a.rule.bias_rows * G; i += 128)
+    for (int i = threadIdx.x - 64; i < a.rule.bias_rows * G; i += 256)
       tab[i] = a.rule.bias[static_cast<size_t>(i / G) * a.Hq + kvh * G + i % G] * 1.4426950408889634f;
   }
-  if (!RULED && S::X_BYTES > 0 && a.rule.slopes != nullptr && warp >= 2) {
+  if (!RULED && S::X_BYTES > 0 && a.rule.slopes != nullptr && warp >= 2 && warp < 6) {
     const int r = threadIdx.x - 64;
     const float f = r < bq * G ? a.rule.slopes[kvh * G + r % G] / a.rule.scale : 0.f;
     const __nv_bfloat16 hi = __float2bfloat16(f);
@@ -249,24 +256,28 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           tc_fence_after();
           issue_s(j + 1);
         }
-        ok = mbar_wait(p_full, j & 1, cta_abort, status, ERR_WAIT_TMEM_EMPTY) &&
-             mbar_wait(&v_full[j % S::VSTAGES], (j / S::VSTAGES) & 1, cta_abort, status, ERR_WAIT_FULL);
+        ok = mbar_wait(&v_full[j % S::VSTAGES], (j / S::VSTAGES) & 1, cta_abort, status, ERR_WAIT_FULL);
         if (!ok) break;
-        tc_fence_after();
         const uint32_t v_addr = smem_u32(sV + (j % S::VSTAGES) * S::V_BYTES);
 #pragma unroll
-        for (int k = 0; k < FW_BN / 16; ++k) {
-          const uint64_t da = make_smem_desc(p_addr + (k >> 2) * (FW_BM * 128) + (k & 3) * 32, 16, 1024, UMMA_SWIZZLE_128B);
-          const uint64_t db = make_smem_desc(v_addr + k * 2048, FW_BN * 128, 1024, UMMA_SWIZZLE_128B);
-          umma_f16(tmem_base + 2 * FW_BN, da, db, idesc_o, (j != 0 || k != 0) ? 1u : 0u);
+        for (int g = 0; g < 2; ++g) {
+          ok = ok && mbar_wait(&p_full[g], j & 1, cta_abort, status, ERR_WAIT_TMEM_EMPTY);
+          if (!ok) break;
+          tc_fence_after();
+#pragma unroll
+          for (int k = 0; k < FW_HALF / 16; ++k) {
+            const uint64_t da = make_smem_desc(p_addr + g * (FW_BM * 128) + k * 32, 16, 1024, UMMA_SWIZZLE_128B);
+            const uint64_t db = make_smem_desc(v_addr + (g * (FW_HALF / 16) + k) * 2048, FW_BN * 128, 1024, UMMA_SWIZZLE_128B);
+            umma_f16(tmem_base + 2 * FW_BN + g * DV, da, db, idesc_o, (j != 0 || k != 0) ? 1u : 0u);
+          }
+          if (g == 1) umma_commit(&v_empty[j % S::VSTAGES]);
+          umma_commit(&o_done[g]);
         }
-        umma_commit(&v_empty[j % S::VSTAGES]);
-        umma_commit(o_done);
       }
     }
   } else {
     // -------------------------------------------------------------------- softmax + epilogue
-    const int quarter = warp & 3;
+    const int quarter = warp & 3, half = warp >= 6;
     const int row = quarter * 32 + lane;  // row of the tile = TMEM lane = token * G + head
     const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(quarter * 32) << 16);
     const float c_log2 = a.rule.scale * 1.4426950408889634f;
@@ -290,23 +301,23 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
       tc_fence_after();
-      const uint32_t s_addr = lane_addr + (j & 1) * FW_BN;
-      const int key0 = key0_of(j);
-      // every row sees the whole tile: no element tests (rows past the tile's tokens never do: their scores are garbage)
-      const bool masked = key0 + FW_BN - 1 > p0 || key0 < low_last || ntok < bq || row >= bq * G;
+      const uint32_t s_addr = lane_addr + (j & 1) * FW_BN + half * FW_HALF;
+      const int tile0 = key0_of(j), key0 = tile0 + half * FW_HALF;  // of the tile, of this group's part
+      // every row sees the whole part: no element tests (rows past the tile's tokens never do: their scores are garbage)
+      const bool masked = key0 + FW_HALF - 1 > p0 || key0 < low_last || ntok < bq || row >= bq * G;
       // bit i of vis[w]: column 32 w + i is visible: c <= up and (c >= dn or c < kp)
       const int up = valid ? pos - key0 : -1, dn = low - key0, kp = a.rule.keep_first - key0;
-      uint32_t vis[FW_BN / 32];
+      uint32_t vis[FW_HALF / 32];
 #pragma unroll
-      for (int w = 0; w < FW_BN / 32; ++w)
+      for (int w = 0; w < FW_HALF / 32; ++w)
         vis[w] = fw_below(up + 1 - 32 * w) & (~fw_below(dn - 32 * w) | fw_below(kp - 32 * w));
-      const float rowb = slope2 * static_cast<float>(key0 - pos);
+      const float rowb = slope2 * static_cast<float>(tile0 - pos);
       float mx = -INFINITY;  // plain: of the raw products, as scale > 0 and rowb is the same for the whole row
-      float sv[RULED ? FW_BN : 1];
+      float sv[RULED ? FW_HALF : 1];
       if constexpr (RULED) {
-        const bool uniform = a.rule.bias == nullptr || p0 - (key0 + FW_BN - 1) >= far;
+        const bool uniform = a.rule.bias == nullptr || p0 - (key0 + FW_HALF - 1) >= far;
 #pragma unroll
-        for (int c4 = 0; c4 < FW_BN / 32; ++c4) {
+        for (int c4 = 0; c4 < FW_HALF / 32; ++c4) {
           uint32_t r[32];
           tmem_ld_32x32(s_addr + c4 * 32, r);
           tmem_ld_wait();
@@ -341,7 +352,7 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         }
       } else {
   #pragma unroll
-        for (int c4 = 0; c4 < FW_BN / 32; ++c4) {
+        for (int c4 = 0; c4 < FW_HALF / 32; ++c4) {
           uint32_t r[32];
           tmem_ld_32x32(s_addr + c4 * 32, r);
           tmem_ld_wait();
@@ -362,10 +373,10 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       else raise = __any_sync(0xffffffffu, m_run == -INFINITY ? m_new > -INFINITY : m_new > m_run + 8.f);
       const float m_use = raise ? m_new : m_run;
       const float m_sub = m_use == -INFINITY ? 0.f : m_use;
-      uint32_t pk[FW_BN / 2];
+      uint32_t pk[FW_HALF / 2];
       float lsum = 0.f;
 #pragma unroll
-      for (int c4 = 0; c4 < FW_BN / 32; ++c4) {
+      for (int c4 = 0; c4 < FW_HALF / 32; ++c4) {
         if constexpr (RULED) {
 #pragma unroll
           for (int i = 0; i < 32; i += 2) {
@@ -392,7 +403,7 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         }
       }
       if (j > 0) {  // the previous product has finished: P may be overwritten and O corrected
-        ok = mbar_wait(o_done, (j - 1) & 1, cta_abort, status, ERR_WAIT_TMEM_FULL);
+        ok = mbar_wait(&o_done[half], (j - 1) & 1, cta_abort, status, ERR_WAIT_TMEM_FULL);
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) break;
         tc_fence_after();
@@ -402,11 +413,11 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 #pragma unroll
           for (int c4 = 0; c4 < DV / 32; ++c4) {
             uint32_t r[32];
-            tmem_ld_32x32(lane_addr + 2 * FW_BN + c4 * 32, r);
+            tmem_ld_32x32(lane_addr + 2 * FW_BN + half * DV + c4 * 32, r);
             tmem_ld_wait();
 #pragma unroll
             for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) * f);
-            tmem_st_32x32(lane_addr + 2 * FW_BN + c4 * 32, r);
+            tmem_st_32x32(lane_addr + 2 * FW_BN + half * DV + c4 * 32, r);
           }
           tmem_st_wait();
           m_run = m_use;
@@ -414,23 +425,23 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       }
       l_run += lsum;
       {
-        uint8_t* prow = sP + row * 128;
+        uint8_t* prow = sP + half * (FW_BM * 128) + row * 128;
         const int sw = row & 7;
 #pragma unroll
-        for (int i = 0; i < FW_BN / 8; ++i)
-          *reinterpret_cast<uint4*>(prow + (i >> 3) * (FW_BM * 128) + (((i & 7) ^ sw) << 4)) =
+        for (int i = 0; i < FW_HALF / 8; ++i)
+          *reinterpret_cast<uint4*>(prow + ((i ^ sw) << 4)) =
               make_uint4(pk[4 * i], pk[4 * i + 1], pk[4 * i + 2], pk[4 * i + 3]);
       }
-      const int nvalid = hi - key0;  // keys of this tile that exist
-      if (nvalid < FW_BN) {
+      const int nvalid = hi - key0;  // keys of this part that exist
+      if (nvalid < FW_HALF) {
         // Value rows past the end hold whatever the page or an older tile left there, or were never written; their p is 0,
         // but 0 x NaN would poison O. Every thread observes the copy's barrier before it overwrites a row.
         const int st = j % S::VSTAGES;
         ok = mbar_wait(&v_full[st], (j / S::VSTAGES) & 1, cta_abort, status, ERR_WAIT_FULL);
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) break;
-        if (row >= nvalid) {
-          uint8_t* vrow = sV + st * S::V_BYTES + row * 128;
+        if (row < FW_HALF && row >= nvalid) {
+          uint8_t* vrow = sV + st * S::V_BYTES + (half * FW_HALF + row) * 128;
 #pragma unroll
           for (int c = 0; c < S::VCH; ++c)
 #pragma unroll
@@ -440,18 +451,24 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       fence_proxy_async();
       tc_fence_before();
       __syncwarp();
-      if (lane == 0) mbar_arrive(p_full);
+      if (lane == 0) mbar_arrive(&p_full[half]);
     }
-    // ---- epilogue: O / l -> bf16 -> staged through shared memory (the P buffer) -> rows of `out`
+    // ---- epilogue: both groups' O, joined, / l -> bf16 -> staged through shared memory (the P buffer) -> rows of `out`. Each group
+    // does half of the columns. The queries are no longer needed: their buffer carries the maxima and sums across.
     constexpr int CH = DV / 8;  // 16-byte chunks per output row
-    if (ok) {
-      ok = mbar_wait(o_done, (n_kv - 1) & 1, cta_abort, status, ERR_WAIT_TMEM_FULL);
-      ok = __all_sync(0xffffffffu, ok);
-    }
+    float2* ml = reinterpret_cast<float2*>(sQ);
+    for (int g = 0; g < 2 && ok; ++g) ok = mbar_wait(&o_done[g], (n_kv - 1) & 1, cta_abort, status, ERR_WAIT_TMEM_FULL);
+    ok = __all_sync(0xffffffffu, ok);
+    if (ok) ml[half * FW_BM + row] = make_float2(m_run, l_run);
+    asm volatile("bar.sync 1, 256;" ::: "memory");  // all softmax warps, also when a wait has expired
     if (ok) {
       tc_fence_after();
-      if (valid && a.rule.sinks != nullptr) l_run += fw_exp2(fmaf(a.rule.sinks[head], 1.4426950408889634f, -m_run));
-      float inv = l_run > 0.f ? a.rule.out_scale / l_run : 0.f;
+      const float2 other = ml[(half ^ 1) * FW_BM + row];
+      const float m = fmaxf(m_run, other.x);
+      const float mine = m_run == -INFINITY ? 0.f : fw_exp2(m_run - m), theirs = other.x == -INFINITY ? 0.f : fw_exp2(other.x - m);
+      float l = l_run * mine + other.y * theirs;
+      if (valid && a.rule.sinks != nullptr) l += fw_exp2(fmaf(a.rule.sinks[head], 1.4426950408889634f, -m));
+      float inv = l > 0.f ? a.rule.out_scale / l : 0.f;
       const __nv_bfloat16* gate = nullptr;  // of this row; one number for the head is part of inv
       if (valid && a.rule.gate != nullptr) {
         gate = reinterpret_cast<const __nv_bfloat16*>(a.rule.gate) + static_cast<size_t>(row0 + tok) * a.rule.gate_pitch +
@@ -461,12 +478,18 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           gate = nullptr;
         }
       }
+      const float f0 = inv * (half == 0 ? mine : theirs), f1 = inv * (half == 0 ? theirs : mine);
       uint8_t* orow = sP + row * (DV * 2);
 #pragma unroll
-      for (int c4 = 0; c4 < DV / 32; ++c4) {
-        uint32_t r[32];
+      for (int c = 0; c < DV / 64; ++c) {
+        const int c4 = half * (DV / 64) + c;
+        uint32_t r[32], r1[32];
         tmem_ld_32x32(lane_addr + 2 * FW_BN + c4 * 32, r);
+        tmem_ld_32x32(lane_addr + 2 * FW_BN + DV + c4 * 32, r1);
         tmem_ld_wait();
+        // a group that has seen nothing has multiplied by zeros only: its O is 0
+#pragma unroll
+        for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(fmaf(__uint_as_float(r[i]), f0, __uint_as_float(r1[i]) * f1));
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           const int ch = c4 * 4 + i;
@@ -481,17 +504,17 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
             }
           }
           *reinterpret_cast<uint4*>(orow + ((ch ^ (row & (CH - 1))) << 4)) =
-              make_uint4(pack_bf16x2(__uint_as_float(r[8 * i]) * inv, __uint_as_float(r[8 * i + 1]) * inv),
-                         pack_bf16x2(__uint_as_float(r[8 * i + 2]) * inv, __uint_as_float(r[8 * i + 3]) * inv),
-                         pack_bf16x2(__uint_as_float(r[8 * i + 4]) * inv, __uint_as_float(r[8 * i + 5]) * inv),
-                         pack_bf16x2(__uint_as_float(r[8 * i + 6]) * inv, __uint_as_float(r[8 * i + 7]) * inv));
+              make_uint4(pack_bf16x2(__uint_as_float(r[8 * i]), __uint_as_float(r[8 * i + 1])),
+                         pack_bf16x2(__uint_as_float(r[8 * i + 2]), __uint_as_float(r[8 * i + 3])),
+                         pack_bf16x2(__uint_as_float(r[8 * i + 4]), __uint_as_float(r[8 * i + 5])),
+                         pack_bf16x2(__uint_as_float(r[8 * i + 6]), __uint_as_float(r[8 * i + 7])));
         }
       }
     }
-    asm volatile("bar.sync 1, 128;" ::: "memory");  // the four softmax warps, also when a wait has expired
+    asm volatile("bar.sync 1, 256;" ::: "memory");
     if (ok && *cta_abort == 0) {
       const int t = threadIdx.x - 64, ch_used = a.dv / 8, rows_used = ntok * G;
-      for (int idx = t; idx < rows_used * ch_used; idx += 128) {
+      for (int idx = t; idx < rows_used * ch_used; idx += 256) {
         const int rr = idx / ch_used, ch = idx - rr * ch_used;
         const int tk = rr / G, hd = kvh * G + rr - tk * G;
         *reinterpret_cast<uint4*>(a.out + static_cast<size_t>(row0 + tk) * a.out_stride + hd * a.dv + ch * 8) =

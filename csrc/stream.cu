@@ -448,28 +448,39 @@ __global__ void __launch_bounds__(128) latent_place_kernel(const __grid_constant
   pdl_wait();
   pdl_launch_dependents();
   const long t = blockIdx.x;
+  const int slot = a.slots[t];
+  const float* cs = a.table + static_cast<long>(a.positions[t]) * a.dims;
   const T* dq = reinterpret_cast<const T*>(a.dq) + t * a.dq_pitch;
   const T* dkv = reinterpret_cast<const T*>(a.dkv) + t * a.dkv_pitch;
   float sq = 0.f, sk = 0.f;
+#pragma unroll 4
   for (int c = threadIdx.x; c < a.R1; c += 128) {
     const float e = to_f(dq[c]);
     sq = fmaf(e, e, sq);
   }
+#pragma unroll 4
   for (int c = threadIdx.x; c < a.R2; c += 128) {
     const float e = to_f(dkv[c]);
     sk = fmaf(e, e, sk);
   }
-  const float rq = 1.f / sqrtf(block_sum<128>(sq, scratch) / a.R1 + a.eps);
-  const float rk = 1.f / sqrtf(block_sum<128>(sk, scratch) / a.R2 + a.eps);
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if ((threadIdx.x & 31) == 0) {
+    scratch[threadIdx.x >> 5] = sq;
+    scratch[4 + (threadIdx.x >> 5)] = sk;
+  }
+  __syncthreads();
+  const float rq = 1.f / sqrtf((scratch[0] + scratch[1] + scratch[2] + scratch[3]) / a.R1 + a.eps);
+  const float rk = 1.f / sqrtf((scratch[4] + scratch[5] + scratch[6] + scratch[7]) / a.R2 + a.eps);
   const T* wq = reinterpret_cast<const T*>(a.q_norm);
   T* q_out = reinterpret_cast<T*>(a.q_out) + t * a.R1;
+#pragma unroll 4
   for (int c = threadIdx.x; c < a.R1; c += 128) q_out[c] = from_f<T>(to_f(dq[c]) * rq * to_f(wq[c]));
-  const int slot = a.slots[t];
   if (slot < 0) return;
   const T* wk = reinterpret_cast<const T*>(a.kv_norm);
   T* out = reinterpret_cast<T*>(a.cache) + static_cast<long>(slot) * (a.R2 + a.dims);
   const int half = a.dims / 2;
-  const float* cs = a.table + static_cast<long>(a.positions[t]) * a.dims;
+#pragma unroll 4
   for (int c = threadIdx.x; c < a.R2 + half; c += 128) {
     if (c < a.R2) {
       out[c] = from_f<T>(to_f(dkv[c]) * rk * to_f(wk[c]));

@@ -517,7 +517,7 @@ def zetizen_config(c: dict, shapes: dict | None = None) -> dict:
             mixer = LatentSpec(m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["q_rank"], m["kv_rank"], float(m["scale"]), _yarn_of(m["rot"]), "channel")
         elif layer["type"] in ("attention", "attention_2"):
             sizes = (m["heads"], m["kv_heads"], m["dim"], m["vdim"], float(m["scale"]))
-            both = dict(softcap=float(m["softcap"]), qk_norm=True, norm_over="projection")
+            both = dict(softcap=float(m["softcap"]) if m.get("softcap") else None, qk_norm=True, norm_over="projection")
             if layer["type"] == "attention":
                 rows = _rows_of(shapes, f"l{i}.mix.rel", m, "bias_rows")
                 mixer = AttentionSpec(*sizes, distance_bias=DistanceBiasSpec(rows, m["bias_max"]), **both)

@@ -93,9 +93,10 @@ def latent_rows(q, cache, R2, block_table, row_req, positions, page_size, scale,
     if q.dtype == torch.bfloat16:
         longest = min(max_context, block_table.shape[1] * page_size)
         heads = 16 if H <= 16 else 32
-        splits = wa.decode_splits(T, -(-H // heads), longest, q.device)
-        part = torch.empty(T * H * splits * (R2 + 2), dtype=torch.float32, device=q.device) if splits > 1 else None
-        ml = part[T * H * splits * R2 :] if splits > 1 else None
+        splits = wa.decode_splits(T, -(-H // heads), longest, q.device, resident=1, tile=64, limit=32)
+        n = T * H * splits  # partial (maximum, sum) pairs come first: they are read as pairs
+        ml = torch.empty(n * (R2 + 2), dtype=torch.float32, device=q.device) if splits > 1 else None
+        part = ml[2 * n :] if splits > 1 else None
         rule = wa.Rule.of(q, R2, scale)
         rc = _lib.lib().sb_latent_attn(P(q), P(cache), P(block_table), P(row_req), P(positions), P(out), P(part), P(ml), T, H, R2, W, page_size,
                                        block_table.stride(0), cache.shape[0], heads, splits, ctypes.byref(rule), P(_lib.status_word(q.device)),

@@ -227,14 +227,18 @@ def window_extend(q, k_cache, v_cache, batch: ExtendBatch, scale, window=None, k
     return simt(q, k_cache, v_cache, batch.block_table, batch.row_req, batch.positions, batch.page_size, rule, out)
 
 
-def decode_splits(rows: int, groups: int, reach: int, device) -> int:
-    """Key ranges of one query's launch over ``reach`` keys: enough CTAs for the machine, no more than the tiles."""
+def decode_splits(rows: int, groups: int, reach: int, device, resident: int = 2, tile: int = TILE, limit: int = 16) -> int:
+    """Key ranges of one query's launch over ``reach`` keys in tiles of ``tile``: enough CTAs for the machine (``resident`` on an SM), no
+    more than the tiles or ``limit``."""
     from slime_b200 import ops
 
-    tiles = -(-reach // TILE) + 1  # a window rarely starts at a tile's edge
-    least = -(-tiles // 16)
-    splits = least if ops.BATCH_INVARIANT else max(least, (2 * _lib.sm_count(device)) // max(rows * groups, 1))
-    return max(1, min(16, splits, tiles))
+    tiles = -(-reach // tile) + 1  # a window rarely starts at a tile's edge
+    most = -(-tiles // 16)  # ranges of 16 tiles: what a launch that must not look at the batch takes
+    if ops.BATCH_INVARIANT:
+        splits = most
+    else:  # a CTA that has an SM to itself walks a longer range rather than wait for a second turn
+        splits = max(most if resident > 1 else 1, (resident * _lib.sm_count(device)) // max(rows * groups, 1))
+    return max(1, min(limit, splits, tiles))
 
 
 def window_decode(q, k_cache, v_cache, block_table, seq_lens, positions, page_size, scale, window=None, keep_first=0, slopes=None,

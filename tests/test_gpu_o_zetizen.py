@@ -134,7 +134,7 @@ def test_capped_biased_and_chunked_attention(kernels, H, G, D, DV, ps, kind, dty
 
 
 LATENTS = [(6, 64, 32, 48, 96, 64), (16, 128, 64, 128, 512, 64), (40, 32, 16, 64, 192, 16), (3, 24, 8, 40, 320, 32), (3, 10, 6, 14, 22, 16),
-           (128, 128, 64, 128, 512, 64), (2, 160, 64, 32, 64, 128), (20, 64, 64, 64, 64, 64)]  # fmt: skip
+           (128, 128, 64, 128, 512, 64), (2, 160, 64, 32, 64, 128), (20, 64, 64, 64, 64, 64), (5, 16, 6, 8, 34, 16)]  # fmt: skip
 
 
 @pytest.mark.parametrize("H,D,r,DV,R,ps", LATENTS)
