@@ -53,4 +53,35 @@ static __global__ void attn_combine_kernel(const float* __restrict__ part_o, con
   }
 }
 
+// The same for pairs of heads (AttnRule::pair): one CTA of 128 threads per (request, output head), dv <= 128.
+static __global__ void __launch_bounds__(128)
+attn_pair_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, __nv_bfloat16* __restrict__ out, int D, int dv,
+                         int splits, int out_stride, int Hout, const AttnRule rule) {
+  __shared__ float scratch[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int b = blockIdx.x / Hout, h = blockIdx.x % Hout, lane = threadIdx.x & 31, d = threadIdx.x;
+  float a[2];
+#pragma unroll
+  for (int m = 0; m < 2; ++m) {
+    const size_t bh = (static_cast<size_t>(b) * Hout + h) * 2 + m;
+    const float* ml = part_ml + bh * splits * 2;
+    const float2 mine = lane < splits ? *reinterpret_cast<const float2*>(ml + 2 * lane) : make_float2(-INFINITY, 0.f);
+    const float gm = warp_max(mine.x);
+    const float f = mine.x != -INFINITY ? __expf(mine.x - gm) : 0.f;
+    const float gl = warp_sum(mine.y * f);
+    const float* o_row = part_o + bh * splits * D;
+    float o = 0.f;
+#pragma unroll 8
+    for (int s = 0; s < splits; ++s) {
+      const float fs = __shfl_sync(0xffffffffu, f, s);
+      if (fs != 0.f && d < dv) o = fmaf(o_row[static_cast<size_t>(s) * D + d], fs, o);
+    }
+    a[m] = gl > 0.f ? o / gl : 0.f;
+  }
+  const float x = d < dv ? fmaf(-rule.pair[0], a[1], a[0]) : 0.f;
+  const float r = rule.pair_gain / sqrtf(block_sum<128>(x * x, scratch) / dv + rule.pair_eps);
+  if (d < dv) out[static_cast<size_t>(b) * out_stride + static_cast<size_t>(h) * dv + d] = __float2bfloat16(x * r);
+}
+
 }  // namespace sb

@@ -4,6 +4,9 @@
 //   query at position i sees key j  iff  j <= i  and  (j >= max(i - window + 1, chunk * floor(i / chunk))  or  j < keep_first)
 //   s = scale * q.k;   s = softcap * tanh(s / softcap);   s += bias[i - j][head];   s -= slopes[head] * (i - j)
 //   output = out_scale * sigmoid(gate) * softmax(s, sinks[head]) v
+//
+// Pairs (differential attention): query heads 2 i and 2 i + 1 are two attentions a1, a2 over the same values, and output head i is
+//   d / rms(d) * pair_gain  with  d = a1 - pair[0] * a2  and  rms(d) = sqrt(mean(d^2) + pair_eps)
 #pragma once
 
 #include "common.cuh"
@@ -18,12 +21,15 @@ struct AttnRule {
   float softcap;          // 0: scores are not capped
   int bias_rows;          // distances from bias_rows - 1 on share the last row
   int gate_width;         // gate columns of a head: 1, or the value width
-  int reserved;
+  float pair_gain;
   long gate_pitch;        // elements between rows of gate
+  float pair_eps;
+  int reserved;
   const float* slopes;    // [Hq] or null
   const float* sinks;     // [Hq] score of an extra softmax column that has no value, or null
   const float* bias;      // [bias_rows, Hq] or null
   const void* gate;       // logits, rows as q and type of q, column head * gate_width (+ channel), or null
+  const float* pair;      // one number, or null: every query head has an output of its own
 };
 
 __device__ __forceinline__ int rule_first_key(const AttnRule& r, int pos) {
@@ -50,5 +56,9 @@ __device__ __forceinline__ float fast_rcp(float x) {
 
 static inline bool rule_ok(const sb::AttnRule* r) {
   return r != nullptr && r->bytes == static_cast<int>(sizeof(sb::AttnRule)) && r->window >= 1 && r->keep_first >= 0 && r->chunk >= 0 &&
-         r->softcap >= 0.f && r->scale > 0.f && (r->bias == nullptr || r->bias_rows >= 1) && (r->gate == nullptr || r->gate_width >= 1);
+         r->softcap >= 0.f && r->scale > 0.f && (r->bias == nullptr || r->bias_rows >= 1) && (r->gate == nullptr || r->gate_width >= 1) &&
+         (r->pair == nullptr || (r->gate == nullptr && r->sinks == nullptr && r->bias == nullptr && r->slopes == nullptr && r->softcap == 0.f));
 }
+
+// Pairs need the two heads of each to share their keys' head.
+static inline bool rule_pairs_ok(const sb::AttnRule* r, int group) { return r->pair == nullptr || group % 2 == 0; }

@@ -415,8 +415,41 @@ decode_attn_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constan
     if (lane == 0) red_l[warp][g] = ws;
   }
   const bool all_ok = __syncthreads_and(ok) && (*cta_abort == 0);
+  // ---- pairs of heads, one key range: the difference of the two, over its root mean square
+  if constexpr (WIN) {
+    if (win.rule.pair != nullptr && splits == 1) {
+      float x[G / 2 > 0 ? G / 2 : 1];
+#pragma unroll
+      for (int i = 0; i < G / 2; ++i) {
+        float o[2];
+#pragma unroll
+        for (int m = 0; m < 2; ++m) {
+          const float l = red_l[0][2 * i + m] + red_l[1][2 * i + m] + red_l[2][2 * i + m] + red_l[3][2 * i + m];
+          o[m] = l > 0.f ? acc[2 * i + m] / l : 0.f;
+        }
+        x[i] = merges && tid < win.dv ? fmaf(-win.rule.pair[0], o[1], o[0]) : 0.f;
+      }
+      __syncthreads();  // everyone has read the denominators
+#pragma unroll
+      for (int i = 0; i < G / 2; ++i) {
+        const float ss = warp_sum(x[i] * x[i]);
+        if (lane == 0) red_l[warp][i] = ss;
+      }
+      __syncthreads();
+      if (all_ok && tid < win.dv)
+#pragma unroll
+        for (int i = 0; i < G / 2; ++i) {
+          if (2 * i >= win.group) break;
+          const float ss = red_l[0][i] + red_l[1][i] + red_l[2][i] + red_l[3][i];
+          const float r = win.rule.pair_gain / sqrtf(ss / win.dv + win.rule.pair_eps);
+          out[static_cast<size_t>(b) * out_stride + static_cast<size_t>(kvh * (win.group / 2) + i) * win.dv + tid] = __float2bfloat16(x[i] * r);
+        }
+    }
+  }
   // ---- output: thread d writes dim d of each head (consecutive threads -> consecutive addresses)
-  if (all_ok && merges) {
+  bool plain = all_ok && merges;
+  if constexpr (WIN) plain = plain && (win.rule.pair == nullptr || splits > 1);
+  if (plain) {
 #pragma unroll
     for (int g = 0; g < G; ++g) {
       float l_run = red_l[0][g] + red_l[1][g] + red_l[2][g] + red_l[3][g], gain = 1.f;
@@ -528,6 +561,7 @@ extern "C" int sb_paged_decode_window(const void* q, const void* k_cache, const 
   if (Hkv <= 0 || Hq % Hkv != 0 || !rule_ok(rule) || splits < 1) return (int)cudaErrorInvalidValue;
   const int G = Hq / Hkv;
   if (G > 16 || DK <= 0 || DV <= 0 || DK > 128 || DV > 128 || DK % 8 || DV % 8) return -1;
+  if (!rule_pairs_ok(rule, G)) return (int)cudaErrorInvalidValue;
   int page_shift = 0;
   while ((1 << page_shift) < page_size) ++page_shift;
   if ((1 << page_shift) != page_size || page_size < 16 || page_size > 128) return -1;
@@ -549,6 +583,9 @@ extern "C" int sb_paged_decode_window(const void* q, const void* k_cache, const 
     SB_DW(128, 1) SB_DW(128, 2) SB_DW(128, 4) SB_DW(128, 8) SB_DW(128, 16)
 #undef SB_DW
     if (rc != 0) return rc;
+    if (splits > 1 && rule->pair != nullptr)
+      return (int)sb::launch_pdl(sb::attn_pair_combine_kernel, dim3(B * (Hq / 2)), dim3(128), 0, s, part_o, part_ml, (bf16*)out, W, DV, splits,
+                                 out_stride, Hq / 2, *rule);
     if (splits > 1)
       return (int)sb::launch_pdl(sb::attn_combine_kernel, dim3(B * Hq), dim3(64), 0, s, part_o, part_ml, (bf16*)out, W, DV, splits,
                                  out_stride, Hq, *rule);

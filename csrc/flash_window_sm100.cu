@@ -29,10 +29,13 @@
 //
 // Keys may come in two parts (latent attention): the first `kchunks` 64-wide chunks from one tensor per head, the others from
 // a second one that all heads share, and queries likewise. Keys wider than 128 leave room for one value stage only.
+// Pairs of heads (FORM 2): the two attentions of an output head are adjacent rows of the tile, so adjacent lanes exchange their columns
+// in the epilogue; the two groups of warps, which have half of the columns each, exchange the sum of squares.
 #include "attn_rule.cuh"
 
 namespace sb {
 
+enum : int { FW_PLAIN = 0, FW_RULED = 1, FW_PAIR = 2 };
 constexpr int FW_BM = 128, FW_BN = 128;
 constexpr int FW_HALF = FW_BN / 2;  // keys of a tile per softmax group
 constexpr int FW_THREADS = 320;     // TMA warp, MMA warp, 2 groups of 4 softmax warps
@@ -74,12 +77,13 @@ struct FwArgs {
   AttnRule rule;
 };
 
-template <int DK, int DV, bool RULED>
+template <int DK, int DV, int FORM>
 __global__ void __launch_bounds__(FW_THREADS, 1)
 flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                     const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmQ2,
                     const __grid_constant__ CUtensorMap tmK2, const __grid_constant__ FwArgs a) {
   using S = FwSmem<DK, DV>;
+  constexpr bool RULED = FORM == FW_RULED, PAIR = FORM == FW_PAIR;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sQ = smem;
@@ -479,6 +483,38 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         }
       }
       const float f0 = inv * (half == 0 ? mine : theirs), f1 = inv * (half == 0 ? theirs : mine);
+      if constexpr (PAIR) {
+        float x[DV / 2], ss = 0.f;  // columns half * DV / 2 ...
+#pragma unroll
+        for (int c = 0; c < DV / 64; ++c) {
+          uint32_t r[32], r1[32];
+          tmem_ld_32x32(lane_addr + 2 * FW_BN + half * (DV / 2) + c * 32, r);
+          tmem_ld_32x32(lane_addr + 2 * FW_BN + DV + half * (DV / 2) + c * 32, r1);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            const float o = fmaf(__uint_as_float(r[i]), f0, __uint_as_float(r1[i]) * f1);
+            const float y = fmaf(-a.rule.pair[0], __shfl_xor_sync(0xffffffffu, o, 1), o);  // (of even rows)
+            x[c * 32 + i] = y;
+            ss = fmaf(y, y, ss);
+          }
+        }
+        float* sums = reinterpret_cast<float*>(ml + 2 * FW_BM);
+        sums[half * FW_BM + row] = ss;
+        asm volatile("bar.sync 2, 256;" ::: "memory");
+        const float r = a.rule.pair_gain / sqrtf((ss + sums[(half ^ 1) * FW_BM + row]) / a.dv + a.rule.pair_eps);
+        if (!(row & 1)) {
+          const int rr = row >> 1;
+          uint8_t* orow = sP + rr * (DV * 2);
+#pragma unroll
+          for (int i = 0; i < DV / 16; ++i) {
+            const int ch = half * (DV / 16) + i;
+            *reinterpret_cast<uint4*>(orow + ((ch ^ (rr & (CH - 1))) << 4)) =
+                make_uint4(pack_bf16x2(x[8 * i] * r, x[8 * i + 1] * r), pack_bf16x2(x[8 * i + 2] * r, x[8 * i + 3] * r),
+                           pack_bf16x2(x[8 * i + 4] * r, x[8 * i + 5] * r), pack_bf16x2(x[8 * i + 6] * r, x[8 * i + 7] * r));
+          }
+        }
+      } else {
       uint8_t* orow = sP + row * (DV * 2);
 #pragma unroll
       for (int c = 0; c < DV / 64; ++c) {
@@ -510,9 +546,13 @@ flash_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
                          pack_bf16x2(__uint_as_float(r[8 * i + 6]), __uint_as_float(r[8 * i + 7])));
         }
       }
+      }
+    } else if constexpr (PAIR) {
+      asm volatile("bar.sync 2, 256;" ::: "memory");  // the exchange of sums, also when a wait has expired
     }
     asm volatile("bar.sync 1, 256;" ::: "memory");
     if (ok && *cta_abort == 0) {
+      const int G = PAIR ? a.G / 2 : a.G;  // output heads of this kv head
       const int t = threadIdx.x - 64, ch_used = a.dv / 8, rows_used = ntok * G;
       for (int idx = t; idx < rows_used * ch_used; idx += 256) {
         const int rr = idx / ch_used, ch = idx - rr * ch_used;
@@ -548,14 +588,18 @@ template <int DK, int DV>
 static int launch_flash_window(dim3 grid, const FwMaps& m, const FwArgs& a, cudaStream_t s) {
   constexpr int bytes = FwSmem<DK, DV>::TOTAL;
   const bool ruled = a.rule.softcap > 0.f || a.rule.bias != nullptr;
-  auto kern = ruled ? flash_window_kernel<DK, DV, true> : flash_window_kernel<DK, DV, false>;
+  auto kern = ruled ? flash_window_kernel<DK, DV, FW_RULED> : flash_window_kernel<DK, DV, FW_PLAIN>;
+  if (a.rule.pair != nullptr) {
+    if constexpr (DK > 128) return -1;
+    else kern = flash_window_kernel<DK, DV, FW_PAIR>;
+  }
   if (cudaError_t e = ensure_dynamic_smem(reinterpret_cast<const void*>(kern), bytes); e != cudaSuccess) return (int)e;
   return (int)launch_pdl(kern, grid, dim3(FW_THREADS), bytes, s, m.q, m.k, m.v, m.q2, m.k2, a);
 }
 
 // What both entry points check: groups, page size, alignment of everything the kernel moves in 16-byte pieces.
 static bool fw_takes(const AttnRule& r, int G, int DV, int page_size, int* shift, long q_stride, long out_stride, uintptr_t pointers) {
-  if (G > FW_BM || DV <= 0 || DV > 128 || DV % 8) return false;
+  if (G > FW_BM || DV <= 0 || DV > 128 || DV % 8 || !rule_pairs_ok(&r, G)) return false;
   if (r.slopes != nullptr && (r.softcap > 0.f || r.bias != nullptr)) return false;
   *shift = 0;
   while ((1 << *shift) < page_size) ++*shift;
@@ -568,7 +612,7 @@ static bool fw_takes(const AttnRule& r, int G, int DV, int page_size, int* shift
 
 // q [T, Hq, D] bf16 (heads adjacent, row pitch q_stride), caches [num_slots, Hkv, D] and [num_slots, Hkv, DV] contiguous;
 // block_table rows of max_pages ints; tiles: ntiles x int4 as described above with at most 128 / (Hq / Hkv) tokens each;
-// out [T, Hq * DV] with row pitch out_stride; attn_rule: AttnRule. D, DV multiples of 8 up to 128.
+// out [T, Hq * DV] (pairs: half as many heads) with row pitch out_stride; attn_rule: AttnRule. D, DV multiples of 8 up to 128.
 // Returns 0, a cudaError_t value, or -1 when the shape or an alignment is outside what the kernel takes.
 extern "C" int sb_flash_window(const void* q, const void* k_cache, const void* v_cache, const int* block_table, const int* tiles,
                                void* out, int ntiles, int T, int Hq, int Hkv, int D, int DV, int page_size, int max_pages,

@@ -88,10 +88,13 @@ moe_route_weight_grad_kernel(const __nv_bfloat16* __restrict__ rows, const int* 
 //   mode 2  scores = sigmoid(logit); pick by score + bias (bias only steers the choice); weights = picked scores,
 //           divided by their sum when `renorm`
 // then weights *= scale. Ties go to the lower expert index. E <= 512. `shift` [E] (or null) is added to the logits first.
+// mode 2 with groups > 1: the experts form that many equal groups of neighbours (at most 32); a group's value is the sum of its two
+// largest choices (score + bias), and only experts of the `keep` best groups can be chosen. Ties go to the lower group.
 constexpr int TOPK_MAX_PER_LANE = 16;
 __global__ void __launch_bounds__(256)
 moe_topk_kernel(const float* __restrict__ logits, const float* __restrict__ shift, const float* __restrict__ bias,
-                int* __restrict__ idx, float* __restrict__ wts, long T, int E, long ld, int k, int mode, int renorm, float scale) {
+                int* __restrict__ idx, float* __restrict__ wts, long T, int E, long ld, int k, int mode, int renorm, float scale, int groups,
+                int keep) {
   const int lane = threadIdx.x & 31;
   for (long t = static_cast<long>(blockIdx.x) * 8 + (threadIdx.x >> 5); t < T; t += static_cast<long>(gridDim.x) * 8) {
     float raw[TOPK_MAX_PER_LANE], sel[TOPK_MAX_PER_LANE];
@@ -119,6 +122,49 @@ moe_topk_kernel(const float* __restrict__ logits, const float* __restrict__ shif
         sel[i] = raw[i] + (bias != nullptr ? bias[e] : 0.f);
       } else {
         sel[i] = raw[i];
+      }
+    }
+    if (groups > 1) {
+      const int per = E / groups;
+      float value = -INFINITY;  // lane g: of group g
+      for (int g = 0; g < groups; ++g) {
+        float hi = -INFINITY, lo = -INFINITY;  // the two largest
+#pragma unroll
+        for (int i = 0; i < TOPK_MAX_PER_LANE; ++i) {
+          const int e = lane + 32 * i;
+          if (e >= g * per && e < (g + 1) * per) {
+            lo = fmaxf(lo, fminf(hi, sel[i]));
+            hi = fmaxf(hi, sel[i]);
+          }
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+          const float h2 = __shfl_xor_sync(0xffffffffu, hi, o), l2 = __shfl_xor_sync(0xffffffffu, lo, o);
+          lo = fmaxf(fminf(hi, h2), fmaxf(lo, l2));
+          hi = fmaxf(hi, h2);
+        }
+        if (lane == g) value = per > 1 ? hi + lo : hi;
+      }
+      unsigned open = 0;  // groups that stay eligible
+      for (int r = 0; r < keep; ++r) {
+        float best = value;
+        int which = lane;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+          const float v2 = __shfl_xor_sync(0xffffffffu, best, o);
+          const int w2 = __shfl_xor_sync(0xffffffffu, which, o);
+          if (v2 > best || (v2 == best && w2 < which)) {
+            best = v2;
+            which = w2;
+          }
+        }
+        open |= 1u << which;
+        if (lane == which) value = -INFINITY;
+      }
+#pragma unroll
+      for (int i = 0; i < TOPK_MAX_PER_LANE; ++i) {
+        const int e = lane + 32 * i;
+        if (e < E && !(open >> (e / per) & 1)) sel[i] = -INFINITY;
       }
     }
     float picked_w = 0.f;  // lane j < k ends up holding the weight of the j-th pick
@@ -306,11 +352,13 @@ extern "C" int sb_moe_route_weight_grad(const void* rows, const int* dest, const
 
 // logits [T, E] fp32 (row pitch ld); bias [E] fp32 or null; idx [T, k] int32; weights [T, k] fp32. k <= 32.
 extern "C" int sb_moe_topk(const float* logits, const float* shift, const float* bias, int* idx, float* weights, long T, int E, long ld,
-                           int k, int mode, int renorm, float scale, cudaStream_t s) {
+                           int k, int mode, int renorm, float scale, int groups, int keep, cudaStream_t s) {
   if (T == 0) return 0;
+  if (groups > 1 && (mode != 2 || groups > 32 || E % groups || keep < 1 || keep > groups || k > keep * (E / groups)))
+    return (int)cudaErrorInvalidValue;
   if (E <= 0 || E > 32 * sb::TOPK_MAX_PER_LANE || k <= 0 || k > 32 || k > E || mode < 0 || mode > 2)
     return (int)cudaErrorInvalidValue;
-  sb::moe_topk_kernel<<<sb::moe_blocks(T), 256, 0, s>>>(logits, shift, bias, idx, weights, T, E, ld, k, mode, renorm, scale);
+  sb::moe_topk_kernel<<<sb::moe_blocks(T), 256, 0, s>>>(logits, shift, bias, idx, weights, T, E, ld, k, mode, renorm, scale, groups, keep);
   return (int)cudaGetLastError();
 }
 

@@ -2,10 +2,13 @@
 //   * sb_stream_norm  one launch between two sub-layers: (mixture-of-experts combine, gated shared expert,) post-norm,
 //                     residual add in fp32, pre-norm of the next sub-layer. With `ids` it gathers embedding rows instead
 //                     and starts the stream; a second table can add a row chosen by (previous token, token).
+//                     Norms treat a row as a whole or in equal parts; without a pre-norm the next sub-layer gets the stream itself.
 //   * sb_glu          activation of a feed-forward, gated or not (silu, tanh-gelu, squared relu)
+//   * sb_poly_norm    activation a N(z) + b N(z^2) + c N(z^3) + e of whole rows, N dividing by the root mean square
+//   * sb_softcap      c tanh(x / c), in place
 //   * sb_kv_scatter   new key / value rows into their cache slots, widths and element size free
 //   * sb_heads        RMS norm (per head, or over all heads at once) and rotation of new queries and keys; keys and values into
-//                     their cache slots
+//                     their cache slots; queries of differential attention spread over key pairs
 //   * sb_latent_place norms of a token's query and key/value latents, rotation of its shared key part, cache write
 //   * sb_latent_turn  rotation of the rotated part of latent queries, in place or beside absorbed queries
 // Element types are bf16 or fp32 throughout (fp32: the engine's full-precision mode); all arithmetic is fp32.
@@ -63,11 +66,12 @@ struct StreamNorm {
   const void* post_w;    // norm of the sub-layer output, or null
   float* res;            // [T, H] residual stream, updated in place
   const void* pre_w;     // norm of the next sub-layer's input, or null
-  void* h;               // [T, H] normed input of the next sub-layer
+  void* h;               // [T, H] normed input of the next sub-layer (the stream itself without pre_w), or null
   int k, y_rows, gate_ld, init, layer_norm, H;  // init: the stream starts here (res is written, not added to)
   float eps, w_off;      // w_off is added to every norm weight
   const float* plus;     // [T, H] fp32 added to the sub-layer output (a mixer's, beside the experts), or null
   float h_scale;         // factor of h
+  int groups;            // equal parts of a row with a norm of their own
   // second embedding table: row (prev * mul_prev + token * mul_cur) mod pair_rows is added to the sub-layer output, row
   // pair_rows where there is no previous token (prev < 0)
   const void* pair;      // same type as y, or null
@@ -75,6 +79,46 @@ struct StreamNorm {
   long mul_prev, mul_cur;
   int pair_rows;
 };
+
+constexpr int STREAM_MAX_H = 8192;
+
+// The same with an RMS norm of its own for each of `groups` parts: sums of squares by vector in shared memory, a warp per part. A vector
+// lies in one part.
+template <typename TW, int VEC, int MAXI, int THREADS>
+__device__ __forceinline__ void row_norm_parts(float (&v)[MAXI][VEC], const TW* w, int H, int nvec, float eps, float w_off, int groups,
+                                               float* part, float (&o)[MAXI][VEC]) {
+  __syncthreads();  // an earlier use of `part`
+#pragma unroll
+  for (int j = 0; j < MAXI; ++j) {
+    const int c = threadIdx.x + j * THREADS;
+    if (c < nvec) {
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) ss = fmaf(v[j][i], v[j][i], ss);
+      part[c] = ss;
+    }
+  }
+  __syncthreads();
+  const int per = nvec / groups, lane = threadIdx.x & 31;
+  for (int g = threadIdx.x >> 5; g < groups; g += THREADS / 32) {
+    float ss = 0.f;
+    for (int c = lane; c < per; c += 32) ss += part[g * per + c];
+    ss = warp_sum(ss);
+    if (lane == 0) part[g * per] = 1.f / sqrtf(ss / (H / groups) + eps);
+  }
+  __syncthreads();
+#pragma unroll
+  for (int j = 0; j < MAXI; ++j) {
+    const int c = threadIdx.x + j * THREADS;
+    if (c < nvec) {
+      const float rstd = part[c / per * per];
+      float g[VEC];
+      load_vec<TW, VEC>(w + static_cast<size_t>(c) * VEC, g);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) o[j][i] = v[j][i] * rstd * (g[i] + w_off);
+    }
+  }
+}
 
 // v <- norm(v) * w over the row held by the CTA (thread t holds vectors t, t + THREADS, ...).
 template <typename TW, int VEC, int MAXI, int THREADS>
@@ -112,10 +156,10 @@ __device__ __forceinline__ void row_norm(float (&v)[MAXI][VEC], const TW* w, int
   }
 }
 
-template <typename TY, typename TW, int VEC, int THREADS>
+template <typename TY, typename TW, int VEC, int THREADS, bool PARTS>
 __global__ void __launch_bounds__(THREADS) stream_norm_kernel(const __grid_constant__ StreamNorm a) {
   constexpr int MAXI = 32 / VEC;
-  __shared__ float scratch[32];
+  __shared__ float scratch[PARTS ? STREAM_MAX_H / VEC : 32];
   pdl_wait();  // inputs come from the previous kernel in the stream
   pdl_launch_dependents();
   const size_t row = blockIdx.x;
@@ -184,8 +228,10 @@ __global__ void __launch_bounds__(THREADS) stream_norm_kernel(const __grid_const
       }
     }
   }
-  if (a.post_w != nullptr)
-    row_norm<TW, VEC, MAXI, THREADS>(v, reinterpret_cast<const TW*>(a.post_w), H, nvec, a.eps, a.w_off, a.layer_norm, scratch, v);
+  if (a.post_w != nullptr) {
+    if constexpr (PARTS) row_norm_parts<TW, VEC, MAXI, THREADS>(v, reinterpret_cast<const TW*>(a.post_w), H, nvec, a.eps, a.w_off, a.groups, scratch, v);
+    else row_norm<TW, VEC, MAXI, THREADS>(v, reinterpret_cast<const TW*>(a.post_w), H, nvec, a.eps, a.w_off, a.layer_norm, scratch, v);
+  }
 #pragma unroll
   for (int j = 0; j < MAXI; ++j) {
     const int c = threadIdx.x + j * THREADS;
@@ -200,9 +246,18 @@ __global__ void __launch_bounds__(THREADS) stream_norm_kernel(const __grid_const
       store_vec<float, VEC>(rp, v[j]);
     }
   }
-  if (a.pre_w != nullptr) {
+  if (a.h != nullptr) {
     float o[MAXI][VEC];
-    row_norm<TW, VEC, MAXI, THREADS>(v, reinterpret_cast<const TW*>(a.pre_w), H, nvec, a.eps, a.w_off, a.layer_norm, scratch, o);
+    if (a.pre_w == nullptr) {
+#pragma unroll
+      for (int j = 0; j < MAXI; ++j)
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) o[j][i] = v[j][i];
+    } else if constexpr (PARTS) {
+      row_norm_parts<TW, VEC, MAXI, THREADS>(v, reinterpret_cast<const TW*>(a.pre_w), H, nvec, a.eps, a.w_off, a.groups, scratch, o);
+    } else {
+      row_norm<TW, VEC, MAXI, THREADS>(v, reinterpret_cast<const TW*>(a.pre_w), H, nvec, a.eps, a.w_off, a.layer_norm, scratch, o);
+    }
     TW* h = reinterpret_cast<TW*>(a.h);
 #pragma unroll
     for (int j = 0; j < MAXI; ++j) {
@@ -214,12 +269,17 @@ __global__ void __launch_bounds__(THREADS) stream_norm_kernel(const __grid_const
   }
 }
 
+template <typename TY, typename TW, bool PARTS>
+static int launch_stream_norm_form(const StreamNorm& a, int T, bool vec, cudaStream_t s) {
+  if (vec && a.H <= 1024)
+    return (int)launch_pdl(stream_norm_kernel<TY, TW, 8, 128, PARTS>, dim3(T), dim3(128), 0, s, a);
+  if (vec) return (int)launch_pdl(stream_norm_kernel<TY, TW, 8, 256, PARTS>, dim3(T), dim3(256), 0, s, a);
+  return (int)launch_pdl(stream_norm_kernel<TY, TW, 1, 256, PARTS>, dim3(T), dim3(256), 0, s, a);
+}
 template <typename TY, typename TW>
 static int launch_stream_norm(const StreamNorm& a, int T, bool vec, cudaStream_t s) {
-  if (vec && a.H <= 1024)
-    return (int)launch_pdl(stream_norm_kernel<TY, TW, 8, 128>, dim3(T), dim3(128), 0, s, a);
-  if (vec) return (int)launch_pdl(stream_norm_kernel<TY, TW, 8, 256>, dim3(T), dim3(256), 0, s, a);
-  return (int)launch_pdl(stream_norm_kernel<TY, TW, 1, 256>, dim3(T), dim3(256), 0, s, a);
+  if (a.groups > 1) return launch_stream_norm_form<TY, TW, true>(a, T, vec && a.H / a.groups % 8 == 0, s);
+  return launch_stream_norm_form<TY, TW, false>(a, T, vec, s);
 }
 
 enum : int { ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_RELU2 = 2 };
@@ -256,6 +316,80 @@ glu_kernel(const T* __restrict__ in, const T* __restrict__ up, T* __restrict__ o
   }
 }
 
+// Rows of F hidden units: a N(z) + b N(z^2) + c N(z^3) + e with N(x) = x / sqrt(mean(x^2) + eps) and (a, b, c, e) = coef. One CTA per row;
+// the second sweep finds the row in the caches. sums: [T, 3] sums of z^2, z^4, z^6 over the whole row of `all` units (tensor-parallel
+// ranks hold parts of it); null: computed here.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+poly_norm_kernel(const T* __restrict__ in, T* __restrict__ out, const float* __restrict__ coef, const float* __restrict__ sums, int F, int all,
+                 long in_pitch, long out_pitch, float eps) {
+  constexpr int KEEP = VEC == 8 ? 4 : 8;  // vectors a thread keeps between the sweeps
+  __shared__ float scratch[32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const long t = blockIdx.x;
+  const T* x = in + t * in_pitch;
+  T* y = out + t * out_pitch;
+  const int n = F / VEC;
+  float keep[KEEP][VEC], s2 = 0.f, s4 = 0.f, s6 = 0.f;
+  auto add = [&](const float (&z)[VEC]) {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+      const float p2 = z[i] * z[i], p4 = p2 * p2;
+      s2 += p2;
+      s4 += p4;
+      s6 = fmaf(p4, p2, s6);
+    }
+  };
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int c = threadIdx.x + j * 256;
+    if (c < n) {
+      load_vec<T, VEC>(x + static_cast<long>(c) * VEC, keep[j]);
+      if (sums == nullptr) add(keep[j]);
+    }
+  }
+  if (sums == nullptr) {
+    for (int c = threadIdx.x + KEEP * 256; c < n; c += 256) {
+      float z[VEC];
+      load_vec<T, VEC>(x + static_cast<long>(c) * VEC, z);
+      add(z);
+    }
+    s2 = block_sum<256>(s2, scratch);
+    s4 = block_sum<256>(s4, scratch);
+    s6 = block_sum<256>(s6, scratch);
+  } else {
+    s2 = sums[3 * t];
+    s4 = sums[3 * t + 1];
+    s6 = sums[3 * t + 2];
+  }
+  const float a = coef[0] / sqrtf(s2 / all + eps), b = coef[1] / sqrtf(s4 / all + eps), c3 = coef[2] / sqrtf(s6 / all + eps), e = coef[3];
+  auto put = [&](int c, float (&z)[VEC]) {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) z[i] = fmaf(z[i], fmaf(z[i], fmaf(z[i], c3, b), a), e);
+    store_vec<T, VEC>(y + static_cast<long>(c) * VEC, z);
+  };
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int c = threadIdx.x + j * 256;
+    if (c < n) put(c, keep[j]);
+  }
+  for (int c = threadIdx.x + KEEP * 256; c < n; c += 256) {
+    float z[VEC];
+    load_vec<T, VEC>(x + static_cast<long>(c) * VEC, z);
+    put(c, z);
+  }
+}
+
+// x <- cap tanh(x / cap) over a row of n floats per y-block, rows `pitch` apart
+__global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, long n, long pitch, float cap) {
+  pdl_wait();
+  pdl_launch_dependents();
+  float* row = x + static_cast<long>(blockIdx.y) * pitch;
+  const float inv = 1.f / cap;
+  for (long i = static_cast<long>(blockIdx.x) * 256 + threadIdx.x; i < n; i += static_cast<long>(gridDim.x) * 256) row[i] = cap * tanhf(row[i] * inv);
+}
+
 // One CTA per token: `kb` bytes of its key row and `vb` bytes of its value row to cache slot slots[t] (< 0: skipped).
 template <typename U>
 __global__ void __launch_bounds__(128)
@@ -279,16 +413,18 @@ kv_scatter_kernel(const char* __restrict__ k, const char* __restrict__ v, const 
 // New queries, keys and values of one attention layer. One warp per (token, head): query heads first, then key heads, then value
 // heads. Query and key heads: RMS norm over D times q_norm / k_norm (null: none), then the first `dims` coordinates turned by
 // the position's angles (table [positions, dims] = cos | sin of the dims / 2 pairs; pair i is (2i, 2i + 1) when interleaved,
-// else (i, i + dims / 2)). Queries are written back in place, keys and values to cache slot slots[t] (< 0: nowhere).
+// else (i, i + dims / 2)). Queries go to q_out (which may be q), keys and values to cache slot slots[t] (< 0: nowhere).
+// maps = 2: query heads 2 i and 2 i + 1 meet the first and the second D coordinates of a key of 2 D: head h is written as a row of
+// 2 D, zero in the other half; key heads 2 g and 2 g + 1 are the halves of one key. Hkv = Hv = 0: queries only.
 struct Heads {
-  void *q;
-  const void *k, *v;
+  const void *q, *k, *v;
+  void* q_out;
   const void *q_norm, *k_norm;
   const float* table;
   const int *positions, *slots;
   void *k_cache, *v_cache;
-  int Hq, Hkv, D, DV, dims, interleaved;
-  long q_pitch, k_pitch, v_pitch;
+  int Hq, Hkv, Hv, D, DV, dims, interleaved, maps;
+  long q_pitch, k_pitch, v_pitch, q_out_pitch;
   float eps;
 };
 constexpr int HEADS_MAX_D = 512;
@@ -299,14 +435,14 @@ __global__ void __launch_bounds__(128) heads_kernel(const __grid_constant__ Head
   pdl_wait();
   pdl_launch_dependents();
   const int lane = threadIdx.x & 31, vec = blockIdx.y * 4 + (threadIdx.x >> 5);
-  if (vec >= a.Hq + 2 * a.Hkv) return;
+  if (vec >= a.Hq + a.Hkv + a.Hv) return;
   const long t = blockIdx.x;
   const int slot = a.slots[t];
   if (vec >= a.Hq + a.Hkv) {
     const int h = vec - a.Hq - a.Hkv;
     if (slot < 0) return;
     const T* src = reinterpret_cast<const T*>(a.v) + t * a.v_pitch + static_cast<long>(h) * a.DV;
-    T* dst = reinterpret_cast<T*>(a.v_cache) + (static_cast<long>(slot) * a.Hkv + h) * a.DV;
+    T* dst = reinterpret_cast<T*>(a.v_cache) + (static_cast<long>(slot) * a.Hv + h) * a.DV;
     for (int d = lane; d < a.DV; d += 32) dst[d] = src[d];
     return;
   }
@@ -326,9 +462,14 @@ __global__ void __launch_bounds__(128) heads_kernel(const __grid_constant__ Head
     for (int d = lane; d < a.D; d += 32) x[d] *= r * to_f(w[d]);
   }
   __syncwarp();
-  T* dst = is_q ? reinterpret_cast<T*>(a.q) + t * a.q_pitch + static_cast<long>(h) * a.D
+  T* dst = is_q ? reinterpret_cast<T*>(a.q_out) + t * a.q_out_pitch + static_cast<long>(h) * a.maps * a.D
                 : reinterpret_cast<T*>(a.k_cache) + (static_cast<long>(slot < 0 ? 0 : slot) * a.Hkv + h) * a.D;
   if (!is_q && slot < 0) return;
+  if (is_q && a.maps == 2) {
+    T* zero = h & 1 ? dst : dst + a.D;
+    dst += h & 1 ? a.D : 0;
+    for (int d = lane; d < a.D; d += 32) zero[d] = from_f<T>(0.f);
+  }
   const int half = a.dims / 2;
   const float* cs = half > 0 ? a.table + static_cast<long>(a.positions[t]) * a.dims : nullptr;
   for (int d = lane; d < a.D; d += 32) {
@@ -385,7 +526,7 @@ __global__ void __launch_bounds__(HEADS_ALL_THREADS) heads_all_kernel(const __gr
   const int slot = a.slots[t];
   const int half = a.dims / 2;
   const float* cs = half > 0 ? a.table + static_cast<long>(a.positions[t]) * a.dims : nullptr;
-  T* q_out = reinterpret_cast<T*>(a.q) + t * a.q_pitch;
+  T* q_out = reinterpret_cast<T*>(a.q_out) + t * a.q_pitch;
   T* k_out = reinterpret_cast<T*>(a.k_cache) + static_cast<long>(slot < 0 ? 0 : slot) * nk;
   for (int c = threadIdx.x * VEC; c < nq + nk; c += HEADS_ALL_THREADS * VEC) {
     const bool is_q = c < nq;
@@ -519,14 +660,18 @@ latent_turn_kernel(const T* __restrict__ q, T* __restrict__ dst, const float* __
 
 }  // namespace sb
 
-extern "C" int sb_heads(void* q, const void* k, const void* v, const void* q_norm, const void* k_norm, const float* table,
-                        const int* positions, const int* slots, void* k_cache, void* v_cache, int T, int Hq, int Hkv, int D, int DV,
-                        int dims, int interleaved, long q_pitch, long k_pitch, long v_pitch, float eps, int f32, cudaStream_t s) {
+// q_out (row pitch q_out_pitch): where the queries go; maps 1, or 2 for pairs (see Heads).
+extern "C" int sb_heads(const void* q, const void* k, const void* v, void* q_out, const void* q_norm, const void* k_norm, const float* table,
+                        const int* positions, const int* slots, void* k_cache, void* v_cache, int T, int Hq, int Hkv, int Hv, int D, int DV,
+                        int dims, int interleaved, int maps, long q_pitch, long k_pitch, long v_pitch, long q_out_pitch, float eps, int f32,
+                        cudaStream_t s) {
   if (T == 0) return 0;
-  if (D <= 0 || D > sb::HEADS_MAX_D || DV <= 0 || dims < 0 || dims > D || dims % 2 || Hq <= 0 || Hkv <= 0) return (int)cudaErrorInvalidValue;
-  const sb::Heads a{q, k, v, q_norm, k_norm, table, positions, slots, k_cache, v_cache, Hq, Hkv, D, DV, dims, interleaved, q_pitch, k_pitch,
-                    v_pitch, eps};
-  const dim3 grid(T, (Hq + 2 * Hkv + 3) / 4);
+  if (D <= 0 || D > sb::HEADS_MAX_D || DV <= 0 || dims < 0 || dims > D || dims % 2 || Hq <= 0 || Hkv < 0 || Hv < 0 || (maps != 1 && maps != 2) ||
+      (maps == 2 && (Hq % 2 || q == q_out)))
+    return (int)cudaErrorInvalidValue;
+  const sb::Heads a{q, k, v, q_out, q_norm, k_norm, table, positions, slots, k_cache, v_cache, Hq, Hkv, Hv, D, DV, dims, interleaved, maps,
+                    q_pitch, k_pitch, v_pitch, q_out_pitch, eps};
+  const dim3 grid(T, (Hq + Hkv + Hv + 3) / 4);
   if (f32) return (int)sb::launch_pdl(sb::heads_kernel<float>, grid, dim3(128), 0, s, a);
   return (int)sb::launch_pdl(sb::heads_kernel<__nv_bfloat16>, grid, dim3(128), 0, s, a);
 }
@@ -539,8 +684,8 @@ extern "C" int sb_heads_all(void* q, const void* k, const void* v, const void* q
   if (T == 0) return 0;
   if (D <= 0 || DV <= 0 || dims < 0 || dims > D || dims % 2 || Hq <= 0 || Hkv <= 0 || q_norm == nullptr || k_norm == nullptr)
     return (int)cudaErrorInvalidValue;
-  const sb::HeadsAll p{{q, k, v, q_norm, k_norm, table, positions, slots, k_cache, v_cache, Hq, Hkv, D, DV, dims, interleaved, q_pitch, k_pitch,
-                        v_pitch, eps}, sums, q_all, k_all};
+  const sb::HeadsAll p{{q, k, v, q, q_norm, k_norm, table, positions, slots, k_cache, v_cache, Hq, Hkv, Hkv, D, DV, dims, interleaved, 1, q_pitch,
+                        k_pitch, v_pitch, q_pitch, eps}, sums, q_all, k_all};
   bool vec = D % 8 == 0 && DV % 8 == 0 && q_pitch % 8 == 0 && k_pitch % 8 == 0 && v_pitch % 8 == 0;
   for (const void* x : {static_cast<const void*>(q), k, v, q_norm, k_norm, static_cast<const void*>(k_cache), static_cast<const void*>(v_cache)})
     vec = vec && (reinterpret_cast<uintptr_t>(x) & 15) == 0;
@@ -571,16 +716,18 @@ extern "C" int sb_latent_turn(const void* q, void* dst, const float* table, cons
                              dims, interleaved, q_pitch, q_head, dst_pitch, dst_head);
 }
 
-// Types: y_f32 / w_f32 (norm weights and h) = 1 for fp32, 0 for bf16; fp32 weights need fp32 y. H <= 8192.
+// Types: y_f32 / w_f32 (norm weights and h) = 1 for fp32, 0 for bf16; fp32 weights need fp32 y. H <= 8192. groups: parts of a row
+// with an RMS norm of their own.
 extern "C" int sb_stream_norm(const void* y, int y_f32, const int* ids, int y_rows, const int* dest, const float* wts, int k,
                               const void* shared, const float* gate, int gate_ld, const void* post_w, float* res, int init,
                               const void* pre_w, void* h, int w_f32, int T, int H, float eps, float w_off, int layer_norm,
                               const void* pair, const int* pair_ids, const int* prev, long mul_prev, long mul_cur, int pair_rows,
-                              const float* plus, float h_scale, cudaStream_t s) {
+                              const float* plus, float h_scale, int groups, cudaStream_t s) {
   if (T == 0) return 0;
-  if (H <= 0 || H > 8192 || (w_f32 && !y_f32) || (pair != nullptr && pair_rows <= 0)) return (int)cudaErrorInvalidValue;
+  if (groups < 1 || H % groups || (groups > 1 && layer_norm) || (pre_w != nullptr && h == nullptr)) return (int)cudaErrorInvalidValue;
+  if (H <= 0 || H > sb::STREAM_MAX_H || (w_f32 && !y_f32) || (pair != nullptr && pair_rows <= 0)) return (int)cudaErrorInvalidValue;
   sb::StreamNorm a{y, ids, dest, wts, shared, gate, post_w, res, pre_w, h, k, y_rows, gate_ld, init, layer_norm, H, eps, w_off,
-                   plus, h_scale, pair, pair_ids, prev, mul_prev, mul_cur, pair_rows};
+                   plus, h_scale, groups, pair, pair_ids, prev, mul_prev, mul_cur, pair_rows};
   bool vec = H % 8 == 0;
   for (const void* p : {y, pair, shared, post_w, static_cast<const void*>(plus), static_cast<const void*>(res), pre_w, static_cast<const void*>(h)})
     vec = vec && (reinterpret_cast<uintptr_t>(p) & 15) == 0;
@@ -606,6 +753,30 @@ extern "C" int sb_glu(const void* in, const void* up, void* out, long rows, int 
   if (vec) SB_GLU(bf16, 8);
   SB_GLU(bf16, 1);
 #undef SB_GLU
+}
+
+// in, out [T, F] (row pitches in_pitch, out_pitch); coef [4] fp32; sums [T, 3] or null, of rows of `all` units.
+extern "C" int sb_poly_norm(const void* in, void* out, const float* coef, const float* sums, int T, int F, int all, long in_pitch,
+                            long out_pitch, float eps, int f32, cudaStream_t s) {
+  if (T == 0) return 0;
+  if (F <= 0 || all < F) return (int)cudaErrorInvalidValue;
+  const bool vec = F % 8 == 0 && ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(out)) & 15) == 0 && in_pitch % 8 == 0 && out_pitch % 8 == 0;
+  using bf16 = __nv_bfloat16;
+#define SB_POLY(T_, V) \
+  return (int)sb::launch_pdl(sb::poly_norm_kernel<T_, V>, dim3(T), dim3(256), 0, s, (const T_*)in, (T_*)out, coef, sums, F, all, in_pitch, out_pitch, eps)
+  if (f32 && vec) SB_POLY(float, 8);
+  if (f32) SB_POLY(float, 1);
+  if (vec) SB_POLY(bf16, 8);
+  SB_POLY(bf16, 1);
+#undef SB_POLY
+}
+
+// rows x n floats, rows `pitch` apart; rows <= 65535
+extern "C" int sb_softcap(float* x, int rows, long n, long pitch, float cap, cudaStream_t s) {
+  if (rows == 0 || n == 0) return 0;
+  if (!(cap > 0.f) || rows > 65535) return (int)cudaErrorInvalidValue;
+  const long want = (n + 1023) / 1024;
+  return (int)sb::launch_pdl(sb::softcap_kernel, dim3(static_cast<unsigned>(want < 148 * 8 ? want : 148 * 8), rows), dim3(256), 0, s, x, n, pitch, cap);
 }
 
 // Row widths and pitches in bytes.

@@ -6,6 +6,7 @@
 // sees and how its scores are made.
 // Cache layout as everywhere: [num_slots, Hkv, D], slot = page * page_size + offset, pages from block_table[request]; v_pitch:
 // elements between the value rows (a latent cache keeps one vector per token whose first DV elements are the value).
+// Pairs of heads: a warp has one output head and computes its two attentions one after the other.
 #include "attn_rule.cuh"
 
 namespace sb {
@@ -19,7 +20,7 @@ __device__ __forceinline__ float wa_load(const __nv_bfloat16* p) { return __bflo
 __device__ __forceinline__ void wa_store(float* p, float v) { *p = v; }
 __device__ __forceinline__ void wa_store(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
 
-template <typename T>
+template <typename T, bool PAIR>
 __global__ void __launch_bounds__(WA_WARPS * 32)
 window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                    const int* __restrict__ block_table, const int* __restrict__ row_req, const int* __restrict__ row_pos,
@@ -30,12 +31,17 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const
   pdl_launch_dependents();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long t = blockIdx.x;
-  const int h = blockIdx.y * WA_WARPS + warp;
-  if (h >= Hq) return;
+  const int out_head = blockIdx.y * WA_WARPS + warp;
+  if (out_head >= (PAIR ? Hq / 2 : Hq)) return;
+  float first[PAIR ? WA_ACC : 1];  // the first attention of a pair
+#pragma unroll
+  for (int map = 0; map < (PAIR ? 2 : 1); ++map) {
+  const int h = PAIR ? 2 * out_head + map : out_head;
   const int kvh = h / (Hq / Hkv);
   const int pos = row_pos[t];
   const int* bt = block_table + static_cast<long>(row_req != nullptr ? row_req[t] : t) * max_pages;
   const float slope = rule.slopes != nullptr ? rule.slopes[h] : 0.f;
+  __syncwarp();
   for (int d = lane; d < D; d += 32) q_s[warp][d] = wa_load(q + t * q_stride + static_cast<long>(h) * D + d);
   __syncwarp();
 
@@ -77,6 +83,25 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const
         if (lane + 32 * i < DV) acc[i] = fmaf(pj, wa_load(vr + lane + 32 * i), acc[i]);
     }
   }
+  if constexpr (PAIR) {
+    const float norm = 1.f / l;
+    if (map == 0) {
+#pragma unroll
+      for (int i = 0; i < WA_ACC; ++i) first[i] = acc[i] * norm;
+      continue;
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < WA_ACC; ++i) {
+      first[i] = lane + 32 * i < DV ? fmaf(-rule.pair[0], acc[i] * norm, first[i]) : 0.f;
+      ss = fmaf(first[i], first[i], ss);
+    }
+    const float r = rule.pair_gain / sqrtf(warp_sum(ss) / DV + rule.pair_eps);
+#pragma unroll
+    for (int i = 0; i < WA_ACC; ++i)
+      if (lane + 32 * i < DV) wa_store(out + t * out_stride + static_cast<long>(out_head) * DV + lane + 32 * i, first[i] * r);
+    return;
+  }
   if (rule.sinks != nullptr) l += expf(rule.sinks[h] - m);
   const float inv = rule.out_scale / l;  // a row always sees its own key: l > 0
   const T* gate = reinterpret_cast<const T*>(rule.gate) + (rule.gate != nullptr ? t * rule.gate_pitch + static_cast<long>(h) * rule.gate_width : 0);
@@ -87,6 +112,7 @@ window_attn_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const
     const float g = rule.gate != nullptr ? sigmoid_f(wa_load(gate + (rule.gate_width > 1 ? d : 0))) : 1.f;
     wa_store(out + t * out_stride + static_cast<long>(h) * DV + d, acc[i] * inv * g);
   }
+  }
 }
 
 }  // namespace sb
@@ -96,14 +122,17 @@ extern "C" int sb_window_attn(const void* q, const void* k_cache, const void* v_
                               long q_stride, long out_stride, long v_pitch, const void* rule, int f32, cudaStream_t s) {
   if (T == 0) return 0;
   const sb::AttnRule* r = (const sb::AttnRule*)rule;
-  if (Hkv <= 0 || Hq % Hkv != 0 || D <= 0 || DV <= 0 || D > sb::WA_MAX_D || DV > sb::WA_MAX_D || !rule_ok(r)) return (int)cudaErrorInvalidValue;
-  const dim3 grid(T, (Hq + sb::WA_WARPS - 1) / sb::WA_WARPS);
+  if (Hkv <= 0 || Hq % Hkv != 0 || D <= 0 || DV <= 0 || D > sb::WA_MAX_D || DV > sb::WA_MAX_D || !rule_ok(r) || !rule_pairs_ok(r, Hq / Hkv))
+    return (int)cudaErrorInvalidValue;
+  const int heads = r->pair != nullptr ? Hq / 2 : Hq;
+  const dim3 grid(T, (heads + sb::WA_WARPS - 1) / sb::WA_WARPS);
   using bf16 = __nv_bfloat16;
+  const bool pair = r->pair != nullptr;
   if (f32)
-    return (int)sb::launch_pdl(sb::window_attn_kernel<float>, grid, dim3(sb::WA_WARPS * 32), 0, s, (const float*)q, (const float*)k_cache,
+    return (int)sb::launch_pdl(pair ? sb::window_attn_kernel<float, true> : sb::window_attn_kernel<float, false>, grid, dim3(sb::WA_WARPS * 32), 0, s, (const float*)q, (const float*)k_cache,
                                (const float*)v_cache, block_table, row_req, row_pos, (float*)out, Hq, Hkv, D, DV, page_size, max_pages,
                                q_stride, out_stride, v_pitch, *r);
-  return (int)sb::launch_pdl(sb::window_attn_kernel<bf16>, grid, dim3(sb::WA_WARPS * 32), 0, s, (const bf16*)q, (const bf16*)k_cache,
+  return (int)sb::launch_pdl(pair ? sb::window_attn_kernel<bf16, true> : sb::window_attn_kernel<bf16, false>, grid, dim3(sb::WA_WARPS * 32), 0, s, (const bf16*)q, (const bf16*)k_cache,
                              (const bf16*)v_cache, block_table, row_req, row_pos, (bf16*)out, Hq, Hkv, D, DV, page_size, max_pages, q_stride,
                              out_stride, v_pitch, *r);
 }

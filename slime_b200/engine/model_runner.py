@@ -19,10 +19,10 @@ import torch
 from slime_b200 import ops
 from slime_b200.engine.kv_cache import PagedKVCache
 from slime_b200.engine.projections import LayerProjections
-from slime_b200.engine.state_cache import RecurrentStates
+from slime_b200.engine.state_cache import RecurrentStates, StateShape
 from slime_b200.models.config import ModelConfig
-from slime_b200.models.layer_spec import AttentionSpec, DeltaSpec, LatentSpec
-from slime_b200.ops import delta, latent, stream, window_attention
+from slime_b200.models.layer_spec import RECURRENT, AttentionSpec, DeltaSpec, LatentSpec, MatrixMemorySpec, StateSpaceSpec
+from slime_b200.ops import delta, latent, linear_scan, stream, window_attention
 
 logger = logging.getLogger(__name__)
 
@@ -30,6 +30,7 @@ _LAYER_RE = re.compile(r"^model\.layers\.(\d+)\.(.+)$")
 _LAYERED_RE = re.compile(r"^l(\d+)\.(.+)$")  # designs described layer by layer (models/layer_spec.py)
 _LAYERED_TOP = {"embed": "model.embed_tokens.weight", "head": "lm_head.weight", "final.norm": "model.norm.weight"}
 _NORMS = {"norm1": "ln1", "norm1b": "post_attn_ln", "norm2": "ln2", "norm2b": "post_mlp_ln"}  # of a specified layer
+_OUTPUT_NORMS = {"norm1": "post_attn_ln", "norm2": "post_mlp_ln"}  # where sub-layers read the stream itself
 _MIMO_DRAFT_RE = re.compile(r"^model\.mtp_layers\.(\d+)\.(.+)$")
 
 
@@ -37,10 +38,10 @@ KV_KINDS = ("attention", "mla")  # layer kinds that keep keys and values in the 
 
 
 def cached_mixers(L) -> list[AttentionSpec | LatentSpec | None]:
-    """What layer ``L`` keeps keys and values for: the attention mixers of a specified layer, one unnamed entry of another
-    attention layer, nothing for a recurrent one."""
+    """What layer ``L`` keeps keys and values for: the attention mixers of a specified layer (but not those that use another
+    layer's), one unnamed entry of another attention layer, nothing for a recurrent one."""
     if L["kind"] == "specified":
-        return [m for _, m, _ in L["spec"].branches() if not isinstance(m, DeltaSpec)]
+        return [m for _, m, _ in L["spec"].branches() if not isinstance(m, RECURRENT) and getattr(m, "kv_from", None) is None]
     return [None] if L["kind"] in KV_KINDS else []
 
 
@@ -188,14 +189,16 @@ class EngineWeights:
         if self.cfg.padded_vocab_size % tp:
             raise ValueError(f"a vocabulary of {self.cfg.padded_vocab_size} does not divide over {tp} tensor-parallel ranks")
         lay = LayerProjections(spec, tp)
-        attention_only = not any(isinstance(x, DeltaSpec) for _, x, _ in spec.branches())
+        attention_only = not any(isinstance(x, RECURRENT) for _, x, _ in spec.branches())
         L = {"kind": "specified", "spec": spec, "proj": lay}
-        L.update({_NORMS[n]: e(h) for n in spec.norms(self.cfg.post_self_attn_layernorm)})
+        L.update({self._norm_keys[n]: e(h) for n in self.cfg.spec_norms(spec)})
         # block-scaled fp8 covers plain attention projections; what enters a recurrence keeps its precision
         L["in"] = mat(lay.in_rows, h, parts=[r for r, _ in lay.ins.values() if r]) if attention_only else e(lay.in_rows, h)
         L["out"] = mat(h, lay.out_cols) if attention_only and len(lay.outs) == 1 else e(h, lay.out_cols)
         if lay.biased:
             L["in_bias"] = e(lay.in_rows)
+        if lay.out_biased:
+            L["out_bias"] = e(h)
         f32 = lambda *n: torch.zeros(*n, dtype=torch.float32, device=self.device)  # noqa: E731
         for p, x, _ in spec.branches():
             if isinstance(x, LatentSpec):
@@ -209,10 +212,23 @@ class EngineWeights:
                 if p in lay.low:
                     L[p + "low"] = e(lay.low[p][2], lay.low[p][1])
                 continue
+            if isinstance(x, StateSpaceSpec):
+                if x.norm_groups % tp:
+                    raise ValueError(f"{x.norm_groups} normed parts do not divide over {tp} tensor-parallel ranks")
+                L.update({p + "conv": e(x.channels // tp, x.conv), p + "conv.b": e(x.channels // tp), p + "norm": e(x.heads * x.vdim // tp)})
+                L.update({p + n: f32(x.heads // tp) for n in ("A_log", "dt_bias", "D")})
+                continue
+            if isinstance(x, MatrixMemorySpec):
+                L.update({p + "i.b": f32(x.heads // tp), p + "f.b": f32(x.heads // tp), p + "norm": e(x.heads * x.vdim // tp)})
+                continue
             if x.qk_norm:
                 whole = x.norm_over == "projection"  # sharded like the projections
                 nq, nk = x.norm_widths()
-                L.update({p + "q.norm": e(nq // tp if whole else nq), p + "k.norm": e(nk // tp if whole else nk)})
+                L[p + "q.norm"] = e(nq // tp if whole else nq)
+                if x.kv_from is None:
+                    L[p + "k.norm"] = e(nk // tp if whole else nk)
+            if x.diff is not None:  # the vectors as stored, and the factor of the second attention they give
+                L.update({p + "pair_rows": f32(4, x.dim), p + "pair": f32(1)})
             if x.learned_bias is not None:
                 # the table as it is stored, and spread over distances: [distance, head], the last row for everything beyond
                 rows = x.learned_bias.by_distance()
@@ -226,6 +242,8 @@ class EngineWeights:
                 raise ValueError(f"a feed-forward of width {m.ff} does not divide over {tp} tensor-parallel ranks")
             f = m.ff // tp
             L.update(gate_up=mat(up * f, h, parts=(f,)), down=mat(h, f))
+            if m.act == "poly_norm":
+                L["act_coef"] = f32(4)
             return L
         if m.experts % self.ep or (m.shared_ff % tp and not spec.parallel_ff):
             raise ValueError(f"{m.experts} experts / a shared expert of width {m.shared_ff} do not divide over {tp} ranks")
@@ -251,7 +269,7 @@ class EngineWeights:
                 out["bigram"] = (self.cfg.bigram["buckets"] + 1, h)
             for i, s in enumerate(self.cfg.layer_specs):
                 m, p = s.mlp, f"l{i}."
-                out.update({p + n: (h,) for n in s.norms(self.cfg.post_self_attn_layernorm)})
+                out.update({p + n: (h,) for n in self.cfg.spec_norms(s)})
                 out.update({p + n: shape for n, shape in LayerProjections(s).tensors(h).items()})
                 if m is None or (s.parallel_ff and m.experts is None):
                     continue
@@ -265,6 +283,8 @@ class EngineWeights:
                         stems[p + "mlp.shared"] = m.shared_ff
                     if m.shared_gate:
                         out[p + "mlp.shared.sg"] = (1, h)
+                if m.act == "poly_norm":
+                    out[p + "mlp.act"] = (4,)
                 for stem, f in stems.items():
                     out.update({stem + ".up": (f, h), stem + ".down": (h, f)})
                     if m.gated:
@@ -278,6 +298,15 @@ class EngineWeights:
         if sub in lay.ins:
             r0, rows = lay.ins[sub]
             self._put(L["in"], r0, rows, None if sub in lay.whole else 0, t, raw, scale=False)
+            return True
+        if sub in lay.split:  # several projections in one tensor
+            parts = lay.split[sub]
+            for (name, _), part in zip(parts, t.split([rows for _, rows in parts])):
+                self._put(L["in"], *lay.ins[name], 0, part, part, scale=False)
+            return True
+        if sub.endswith(".b") and sub[:-2] in lay.out_biased:
+            if self.rank == 0:  # the ranks' outputs are summed
+                L["out_bias"].copy_(t)
             return True
         if sub in lay.outs:
             c0, cols = lay.outs[sub]
@@ -308,6 +337,18 @@ class EngineWeights:
                 else:
                     continue
                 return True
+            if isinstance(m, StateSpaceSpec) and sub in (p + "conv", p + "conv.b"):
+                v, g = m.heads * m.vdim, m.groups * m.dim
+                L[sub].copy_(torch.cat([self._rows(part, n // self.tp) for part, n in zip(t.split([v, g, g]), (v, g, g))]))
+                return True
+            if isinstance(m, (StateSpaceSpec, MatrixMemorySpec)) and sub in L and sub.startswith(p):
+                L[sub].copy_(self._rows(raw, L[sub].numel()))
+                return True
+            vectors = [p + n for n in ("lq1", "lk1", "lq2", "lk2")]
+            if p + "pair" in L and sub in vectors:
+                L[p + "pair_rows"][vectors.index(sub)].copy_(raw)
+                self._weigh_pair(L, p, m)
+                return True
             if sub in (p + "q.conv", p + "k.conv", p + "v.conv"):
                 g, v = m.kv_heads // self.tp * m.dim, m.heads // self.tp * m.vdim
                 r0, rows = {"q": (0, g), "k": (g, g), "v": (2 * g, v)}[sub[len(p)]]
@@ -329,17 +370,29 @@ class EngineWeights:
         """The learned distance bias by distance, from its table by bucket (in place: captured graphs keep its address)."""
         L[p + "bias"].copy_(L[p + "rel"].float().index_select(0, L[p + "rel_rows"]))
 
+    def _weigh_pair(self, L, p: str, m: AttentionSpec):
+        """Factor of the second attention of a pair, from its vectors (in place: captured graphs keep its address)."""
+        q1, k1, q2, k2 = L[p + "pair_rows"]
+        L[p + "pair"].copy_(torch.exp((q1 * k1).sum()) - torch.exp((q2 * k2).sum()) + m.diff)
+
+    @property
+    def _norm_keys(self) -> dict[str, str]:
+        return _NORMS if self.cfg.pre_norm else _OUTPUT_NORMS
+
     def _load_specified(self, L, sub: str, t, raw) -> bool:
         """One tensor of a specified layer, addressed by its name behind ``l<i>.`` (one of ``specified_tensors``)."""
         spec, h, tp = L["spec"], self.cfg.hidden_size, self.tp
         m = spec.mlp
-        if sub in _NORMS:
-            L[_NORMS[sub]].copy_(t)
+        if sub in self._norm_keys:
+            L[self._norm_keys[sub]].copy_(t)
             return True
         if self._load_mixer(L, sub, t, raw):
             return True
         table = {}
         if m.experts is None:
+            if sub == "mlp.act":
+                L["act_coef"].copy_(raw)
+                return True
             f = m.ff // tp
             table = {"mlp.gate": ("gate_up", 0, f, 0), "mlp.up": ("gate_up", f if m.gated else 0, f, 0), "mlp.down": ("down", 0, h, 1)}
         else:
@@ -370,14 +423,17 @@ class EngineWeights:
         self._put(L[key], r0, rows, cut, t, raw, scale=False)
         return True
 
-    def state_geometry(self) -> list[tuple[int, int, int, int, int]]:
-        """(heads, key width, value width, convolution channels, taps) of this rank's recurrent mixers, in layer order."""
+    def state_geometry(self) -> list[StateShape]:
+        """Shapes of the states of this rank's recurrent mixers, in layer order."""
         c, out = self.cfg, []
         for L in self.layers:
             if L["kind"] == "gdn":
-                out.append((c.linear_num_value_heads, c.linear_key_head_dim, c.linear_value_head_dim, L["gdn_conv"].shape[0], L["gdn_conv"].shape[1]))
-            if L["kind"] == "specified":
-                out += [(m.heads // self.tp, m.dim, m.vdim, m.channels // self.tp, m.conv) for _, m, _ in L["spec"].branches() if isinstance(m, DeltaSpec)]
+                out.append(StateShape(c.linear_num_value_heads, c.linear_key_head_dim, c.linear_value_head_dim, *L["gdn_conv"].shape))
+            for _, m, _ in L["spec"].branches() if L["kind"] == "specified" else ():
+                if isinstance(m, MatrixMemorySpec):
+                    out.append(StateShape(m.heads // self.tp, m.dim, m.vdim, normalised=True))
+                elif isinstance(m, RECURRENT):
+                    out.append(StateShape(m.heads // self.tp, m.dim, m.vdim, m.channels // self.tp, m.conv))
         return out
 
     def num_bytes(self) -> int:
@@ -651,8 +707,11 @@ class EngineWeights:
             t.fill_(1.0 - self.cfg.norm_offset)
         for L in self.layers:
             for k, t in L.items():
-                if k in ("in_bias", "router_shift"):
+                if k in ("in_bias", "out_bias", "router_shift"):
                     t.zero_()
+                if k.endswith("pair_rows"):
+                    p = k[: -len("pair_rows")]
+                    self._weigh_pair(L, p, next(m for q, m, _ in L["spec"].branches() if q == p))
                 if k.endswith("rel_rows"):
                     self._spread_bias(L, k[: -len("rel_rows")])
                 if k.endswith("A_log"):  # the decay parameter of the delta rule must start in its valid range
@@ -713,7 +772,7 @@ class ModelRunner:
         self.kv_of, self.state_of, n_attn, n_state = [], [], 0, 0  # per layer: number of its first slab / state
         for L in weights.layers + weights.draft:  # a draft head's layer number is num_layers + depth
             n = len(cached_mixers(L))
-            r = len(L["spec"].branches()) - n if L["kind"] == "specified" else int(L["kind"] == "gdn")
+            r = sum(isinstance(m, RECURRENT) for _, m, _ in L["spec"].branches()) if L["kind"] == "specified" else int(L["kind"] == "gdn")
             self.kv_of.append(n_attn if n else None)
             self.state_of.append(n_state if r else None)
             n_attn, n_state = n_attn + n, n_state + r
@@ -726,21 +785,21 @@ class ModelRunner:
         self._mrope_axes = None
         rot = int(cfg.head_dim * cfg.rotary_percent) // 2 * 2
         self.rope = None if self.layered else ops.rope_table(cfg, max_context + 1, rot, self.device)
-        # specified attention mixers, by slab: this rank's distance-penalty factors, scores of the column without a value
-        self.slopes, self.sinks, self.rotary = [], [], {}
-        for L in weights.layers if self.layered else ():
-            for a in cached_mixers(L):
+        # specified attention mixers, by layer and prefix: this rank's distance-penalty factors, scores of the column without a value
+        self.slopes, self.sinks, self.rotary = {}, {}, {}
+        for li, L in enumerate(weights.layers if self.layered else ()):
+            for p, a, _ in L["spec"].branches():
+                if isinstance(a, RECURRENT):
+                    continue
                 f32 = lambda x: torch.tensor(x, dtype=torch.float32, device=self.device)  # noqa: E731
                 if a.rot is not None and a.rot.dims and a.rot not in self.rotary:
                     self.rotary[a.rot] = stream.rotary_table(max_context + 1, a.rot.dims, a.rot.base, self.device,
                                                              frequencies=a.rot.frequencies(), gain=a.rot.gain())  # fmt: skip
                 if isinstance(a, LatentSpec):
-                    self.slopes.append(None)
-                    self.sinks.append(None)
                     continue
                 n, sl = a.heads // weights.tp, a.slopes()
-                self.slopes.append(None if sl is None else f32(sl[weights.rank * n : (weights.rank + 1) * n]))
-                self.sinks.append(None if a.sink is None else f32([a.sink] * n))
+                self.slopes[li, p] = None if sl is None else f32(sl[weights.rank * n : (weights.rank + 1) * n])
+                self.sinks[li, p] = None if a.sink is None else f32([a.sink] * n)
         self.stream_hook = None  # called with (layer, fp32 residual stream) after every specified layer (eager passes only)
         self.scale = 1.0 / math.sqrt(cfg.head_dim)
         if cfg.multi_latent_attention:
@@ -820,16 +879,8 @@ class ModelRunner:
         from slime_b200.ops import grouped
 
         if cfg.moe_router_num_groups and cfg.moe_router_group_topk and cfg.moe_router_num_groups > 1:
-            # group-limited routing (sigmoid scores): no kernel for it; a handful of small device ops, capturable
-            from slime_b200.models.moe import group_limited
-
-            scores = torch.sigmoid(logits.float())
-            sel = scores + L["router_bias"] if L.get("router_bias") is not None else scores
-            idx = torch.topk(group_limited(sel, cfg.moe_router_num_groups, cfg.moe_router_group_topk), cfg.moe_router_topk, dim=-1).indices
-            probs = scores.gather(-1, idx)
-            if cfg.norm_topk_prob:
-                probs = probs / (probs.sum(-1, keepdim=True) + 1e-20)
-            return probs * (cfg.moe_router_topk_scaling_factor or 1.0), idx
+            return grouped.route_topk(logits, cfg.moe_router_topk, score="sigmoid", renorm=cfg.norm_topk_prob, bias=L.get("router_bias"),
+                                      scale=cfg.moe_router_topk_scaling_factor, groups=(cfg.moe_router_num_groups, cfg.moe_router_group_topk))  # fmt: skip
         return grouped.route_topk(logits, cfg.moe_router_topk, score=cfg.moe_router_score_function,
                                   pre_softmax=cfg.moe_router_pre_softmax, renorm=cfg.norm_topk_prob,
                                   bias=L.get("router_bias"), scale=cfg.moe_router_topk_scaling_factor)  # fmt: skip
@@ -1027,39 +1078,30 @@ class ModelRunner:
         mixed, z, b, a = self._gdn_project(L, x)
         q, k, v = mixed.contiguous().split([hk * dk, hk * dk, hv * dv], dim=-1)
         inputs = delta.DeltaInputs(q, k, v, a, b, L["gdn_conv"], L["gdn_A_log"], L["gdn_dt_bias"])
-        return ops.gemm(recur(self.state_of[li], inputs, z.reshape(T, -1), L["gdn_norm"], "silu", 1.0, None), L["gdn_out"])
+        return ops.gemm(recur(self.state_of[li], inputs.gated(z.reshape(T, -1), L["gdn_norm"], "silu", cfg.norm_epsilon), None), L["gdn_out"])
 
     def _extend_recurrence(self, extend):
-        """``recur(state number, inputs, gate, norm weight, gate activation, output factor, output view or None)`` of an extend pass."""
-
-        def recur(n, inputs, z, w, act, scale, out):
-            o = delta.delta_extend(inputs, self.states.state[n], self.states.ring[n], extend)
-            return delta.head_gate(o, z, w, act, self.cfg.norm_epsilon, scale, out)
-
-        return recur
+        """``recur(state number, mixer, output view or None)`` of an extend pass; ``mixer``: ``ops.delta.DeltaMixer`` or one of
+        ``ops.linear_scan``."""
+        return lambda n, mixer, out: mixer.extend(self.states.of[n], extend, out)
 
     def _step_recurrence(self, n_rows: int, positions):
         """The same of a decode step: idle rows touch no state."""
         slots, active = self._static["state_slot"][:n_rows], self._static["active"][:n_rows]
-
-        def recur(n, inputs, z, w, act, scale, out):
-            return delta.delta_step(inputs, self.states.state[n], self.states.ring[n], slots, active, positions, z, w, act,
-                                    self.cfg.norm_epsilon, scale, out)  # fmt: skip
-
-        return recur
+        return lambda n, mixer, out: mixer.step(self.states.of[n], slots, active, positions, out)
 
     # ------------------------------------------------------------ specified layers (models/layer_spec.py)
     def _specified_layers(self, ids, prev, positions, slots, attend, attend_latent, recur):
         """All layers of a model with ``layer_specs`` over the tokens ``ids`` (``prev``: the tokens in front of them, -1 at a
         sequence's start; read by models with a bigram table) -> the final norm's output. ``attend(slab, spec, q, form, out)`` runs an
-        attention mixer once its keys and values are in the cache, ``attend_latent(slab, latent, q, gate, out)`` a latent one,
+        attention mixer once the keys and values of cache slab ``slab`` are there, ``attend_latent(slab, latent, q, gate, out)`` a latent one,
         ``recur`` (``_extend_recurrence``) a recurrent one: the
         only parts that differ between a prefill pass and a decode step. The residual stream is fp32; between two
-        sub-layers there is one fused launch."""
+        sub-layers there is one fused launch (which hands on the stream itself where a model has no norms of inputs)."""
         cfg, w = self.cfg, self.w
-        norm = dict(kind=cfg.norm_kind, offset=cfg.norm_offset)
+        norm = dict(kind=cfg.norm_kind, offset=cfg.norm_offset, groups=cfg.norm_groups, emit=w.dtype)
         f32, eps = torch.float32, cfg.norm_epsilon
-        first = w.layers[0]["ln1"]
+        first = w.layers[0].get("ln1")
         pair = None
         if cfg.bigram:
             pair = stream.PairTable(w.bigram, ids.to(torch.int32), prev, cfg.bigram["mul_prev"], cfg.bigram["mul_cur"])
@@ -1072,14 +1114,14 @@ class ModelRunner:
             h, res = stream.stream_norm(w.embed, None, first, eps, ids=ids, pair=pair, post_w=w.embed_norm, **norm)
         for li, L in enumerate(w.layers):
             spec, last = L["spec"], li + 1 == len(w.layers)
-            after, gain = (w.final_norm, cfg.logit_scale) if last else (w.layers[li + 1]["ln1"], 1.0)
+            after, gain = (w.final_norm, cfg.logit_scale) if last else (w.layers[li + 1].get("ln1"), 1.0)
             behind = spec.mlp is not None and not spec.parallel_ff
-            y = _linear(self._specified_mixers(L, li, h, positions, slots, attend, attend_latent, recur), L["out"], out_dtype=f32)
+            y = _linear(self._specified_mixers(L, li, h, positions, slots, attend, attend_latent, recur), L["out"], bias=L.get("out_bias"), out_dtype=f32)
             if spec.parallel_ff and spec.mlp is not None and spec.mlp.experts is not None:
                 y = self._specified_experts(L, spec.mlp, h, y)
             else:
                 y = self._tp_reduce(y)
-            h, _ = stream.stream_norm(y, res, L["ln2"] if behind else after, eps, post_w=L.get("post_attn_ln"), gain=1.0 if behind else gain, **norm)
+            h, _ = stream.stream_norm(y, res, L.get("ln2") if behind else after, eps, post_w=L.get("post_attn_ln"), gain=1.0 if behind else gain, **norm)
             if behind:
                 h, _ = stream.stream_norm(self._specified_mlp(L, spec.mlp, h), res, after, eps, post_w=L.get("post_mlp_ln"), gain=gain, **norm)
             if self.stream_hook is not None:
@@ -1093,25 +1135,32 @@ class ModelRunner:
         x = _linear(h, L["in"], bias=L.get("in_bias"))
         cols = lambda name: x[:, lay.ins[name][0] : sum(lay.ins[name])]  # noqa: E731
         y = (torch.zeros if lay.padded(lay.outs) else torch.empty)(T, lay.out_cols, dtype=h.dtype, device=h.device)
-        slab, number = self.kv_of[li], self.state_of[li]
+        slab, number, eps = self.kv_of[li], self.state_of[li], self.cfg.norm_epsilon
         for p, m, factor in spec.branches():
             c0, n = lay.outs[p + "o"]
             out = y[:, c0 : c0 + n]
             if isinstance(m, AttentionSpec):
-                q, k, sums = cols(p + "q"), cols(p + "k"), None
+                own = m.kv_from is None
+                at = slab if own else self.kv_of[m.kv_from]  # where its keys and values are
+                slab = slab + 1 if own else slab
+                q, k, v, sums = cols(p + "q"), None, None, None
+                if own:
+                    k = cols(p + "k")
+                    v = k if m.tied_values else cols(p + "v")
                 if m.qk_norm and m.norm_over == "projection" and self.w.tp > 1:
                     sums = (self._tp_reduce(stream.head_sums(q, k)), m.norm_widths())
-                q = stream.place_heads(q, k, cols(p + ("k" if m.tied_values else "v")), slots, self.kv.k[slab], self.kv.v[slab],
-                                       q_norm=L.get(p + "q.norm"), k_norm=L.get(p + "k.norm"), eps=self.cfg.norm_epsilon,
-                                       table=self.rotary.get(m.rot), positions=positions, interleaved=m.rot is None or m.rot.interleaved,
-                                       sums=sums)  # fmt: skip
-                form = dict(out_scale=factor, chunk=m.chunk, softcap=m.softcap, bias=L.get(p + "bias"), gate=cols(p + "g") if m.gate else None)
-                attend(slab, m, q, form, out)
-                slab += 1
+                q = stream.place_heads(q, k, v, slots, self.kv.k[at], self.kv.v[at], q_norm=L.get(p + "q.norm"), k_norm=L.get(p + "k.norm"),
+                                       eps=eps, table=self.rotary.get(m.rot), positions=positions, interleaved=m.rot is None or m.rot.interleaved,
+                                       sums=sums, maps=m.maps)  # fmt: skip
+                form = dict(slopes=self.slopes[li, p], sinks=self.sinks[li, p], out_scale=factor, chunk=m.chunk, softcap=m.softcap,
+                            bias=L.get(p + "bias"), gate=cols(p + "g") if m.gate else None)  # fmt: skip
+                if m.diff is not None:
+                    form["pair"] = window_attention.Pair(L[p + "pair"], factor * (1.0 - m.diff), eps)
+                attend(at, m, q, form, out)
                 continue
             if isinstance(m, LatentSpec):
                 heads, table = m.heads // self.w.tp, self.rotary[m.rot]
-                c = latent.latent_place(cols(p + "dq"), cols(p + "dkv"), L[p + "dq.norm"], L[p + "dkv.norm"], self.cfg.norm_epsilon, table,
+                c = latent.latent_place(cols(p + "dq"), cols(p + "dkv"), L[p + "dq.norm"], L[p + "dkv.norm"], eps, table,
                                         positions, slots, self.kv.k[slab], m.rot.interleaved)  # fmt: skip
                 q = _linear(c, L[p + "up_q"]).view(T, heads, m.dim + m.rot_dim)
                 gate = cols(p + "g").unflatten(1, (heads, m.vdim)) if m.gate else None
@@ -1120,6 +1169,17 @@ class ModelRunner:
                 if factor != 1.0:
                     out.mul_(factor)
                 slab += 1
+                continue
+            if isinstance(m, StateSpaceSpec):
+                mixer = linear_scan.StateSpace(*(cols(p + n) for n in ("z", "x", "B", "C", "dt")), L[p + "conv"], L[p + "conv.b"], L[p + "A_log"],
+                                               L[p + "dt_bias"], L[p + "D"], L[p + "norm"], m.norm_groups // self.w.tp, eps, factor)  # fmt: skip
+                recur(number, mixer, out)
+                number += 1
+                continue
+            if isinstance(m, MatrixMemorySpec):
+                recur(number, linear_scan.MatrixMemory(*(cols(p + n) for n in "qkvifg"), L[p + "i.b"], L[p + "f.b"], L[p + "norm"], m.gate_cap, eps,
+                                                       factor), out)  # fmt: skip
+                number += 1
                 continue
             a, z = (cols(p + s) if p + s in lay.ins else None for s in "ag")
             if p in lay.low:
@@ -1130,7 +1190,7 @@ class ModelRunner:
                 if p + "g2" in parts:
                     z = second[:, parts[p + "g2"][0] : sum(parts[p + "g2"][:2])]
             inputs = delta.DeltaInputs(cols(p + "q"), cols(p + "k"), cols(p + "v"), a, cols(p + "b"), L[p + "conv"], L[p + "A_log"], L[p + "dt_bias"])
-            recur(number, inputs, z, L[p + "norm"], m.gate, factor, out)
+            recur(number, inputs.gated(z, L[p + "norm"], m.gate, eps, factor), out)
             number += 1
         if lay.ff is not None:
             m, (c0, n), r0 = spec.mlp, lay.outs[spec.joint_ff[0] + ".down"], lay.ff[0]
@@ -1141,7 +1201,12 @@ class ModelRunner:
         """Feed-forward behind the mixer of a specified layer: fp32 output, or for experts the unfinished sum the next norm completes."""
         w, f32 = self.w, torch.float32
         if m.experts is None:
-            act = stream.feed_forward_act(_linear(h, L["gate_up"]), m.act, m.gated)
+            act = _linear(h, L["gate_up"])
+            if m.act == "poly_norm":
+                sums = self._tp_reduce(stream.poly_sums(act)) if w.tp > 1 else None
+                act = stream.poly_norm(act, L["act_coef"], self.cfg.norm_epsilon, sums, m.ff)
+            else:
+                act = stream.feed_forward_act(act, m.act, m.gated)
             return self._tp_reduce(_linear(act, L["down"], out_dtype=f32))
         out = self._expert_rows(L, m, h)
         if m.shared_ff:
@@ -1168,7 +1233,8 @@ class ModelRunner:
         # faster one for a handful of tokens
         big = h.is_cuda and h.dtype == torch.bfloat16 and h.shape[0] >= 256
         logits = ops.gemm(h, L["router"], out_dtype=f32, splitk=1) if big else ops.router_gemm(h, L["router"])
-        probs, idx = grouped.route_topk(logits[:, : m.experts], m.top, score=m.score, renorm=m.renorm, raw_index=True, shift=L.get("router_shift"))
+        probs, idx = grouped.route_topk(logits[:, : m.experts], m.top, score=m.score, renorm=m.renorm, raw_index=True, shift=L.get("router_shift"),
+                                        groups=(m.expert_groups, m.keep_groups))  # fmt: skip
         if self.record_routed:
             pad = self.cfg.moe_router_topk - m.top
             self._routed.append(torch.nn.functional.pad(idx.to(torch.int32), (0, pad)) if pad else idx.to(torch.int32))
@@ -1200,15 +1266,14 @@ class ModelRunner:
         cfg, w, d = self.cfg, self.w, self.cfg.head_dim
         if self.layered:
             def attend(n, a, q, form, out):
-                return window_attention.window_extend(q, self.kv.k[n], self.kv.v[n], extend, a.scale, a.window, a.keep_first, self.slopes[n],
-                                                      self.sinks[n], out=out, **form)  # fmt: skip
+                return window_attention.window_extend(q, self.kv.k[n], self.kv.v[n], extend, a.scale, a.window, a.keep_first, out=out, **form)
 
             def attend_latent(n, sizes, q, gate, out):
                 return latent.latent_extend(sizes, q, self.kv.k[n], extend, gate, out)
 
             h = self._specified_layers(ids, prev, positions, slots, attend, attend_latent, self._extend_recurrence(extend))
             h = h if last_rows is None else h.index_select(0, last_rows)
-            return self._gather_logits(ops.gemm(h, w.lm_head, out_dtype=torch.float32))
+            return self.logits_of(h)
         x = ops.embedding(ids, w.embed, w.rank * w.vocab_local)
         x = self._tp_reduce(x) if w.tp > 1 else x
         deepstack = []
@@ -1298,7 +1363,8 @@ class ModelRunner:
 
     def logits_of(self, normed):
         """Output head over already normalised rows -> fp32 logits over the whole vocabulary."""
-        return self._gather_logits(ops.gemm(normed, self.w.lm_head, out_dtype=torch.float32))
+        logits = ops.gemm(normed, self.w.lm_head, out_dtype=torch.float32)
+        return self._gather_logits(stream.softcap_(logits, self.cfg.logit_softcap) if self.cfg.logit_softcap else logits)
 
     # ---------------------------------------------------------------------- decode
     # Per-slot decode state is device-owned (ids / pos / out_pos): the token sampled in step t is the
@@ -1377,7 +1443,7 @@ class ModelRunner:
         else:
             self._prepare_reference(n)
         h = self._decode_layers(n, ids, pos, slots, bt, seq_lens)
-        logits = self._gather_logits(ops.gemm(h, w.lm_head, out_dtype=torch.float32))
+        logits = self.logits_of(h)
         tok, lp, kept_ids, kept_cnt = ops.sample(
             logits, st["temperature"][:n], st["top_k"][:n] if filtered else None, st["top_p"][:n] if filtered else None,
             st["min_p"][:n] if filtered else None, st["seeds"][:n], ds["out_pos"][:n], kept_cap,
@@ -1401,7 +1467,7 @@ class ModelRunner:
         if self.layered:
             def attend(i, a, q, form, out):
                 return window_attention.window_decode(q, self.kv.k[i], self.kv.v[i], bt, seq_lens, pos, ps, a.scale, a.window, a.keep_first,
-                                                      self.slopes[i], self.max_context, self.sinks[i], out=out, **form)  # fmt: skip
+                                                      max_context=self.max_context, out=out, **form)  # fmt: skip
 
             def attend_latent(i, sizes, q, gate, out):
                 return latent.latent_decode(sizes, q, self.kv.k[i], bt, pos, ps, self.max_context, gate, out)

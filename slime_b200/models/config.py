@@ -11,7 +11,7 @@ import json
 import os
 from dataclasses import dataclass
 
-from slime_b200.models.layer_spec import LAYERED_ARCHITECTURES, LayerSpec
+from slime_b200.models.layer_spec import LAYERED_ARCHITECTURES, AttentionSpec, LayerSpec
 
 VISION_FIELDS = ("vision", "image_token_id", "video_token_id", "mrope_section", "mrope_interleaved")
 
@@ -101,6 +101,9 @@ class ModelConfig:
     bigram: dict | None = None
     embed_norm: bool = False  # the embedding passes a norm with a weight of its own (models with layer_specs)
     logit_scale: float = 1.0  # factor of the logits (models with layer_specs)
+    logit_softcap: float | None = None  # logits pass c tanh(logit / c) (models with layer_specs)
+    norm_groups: int = 1  # equal parts of a row that the stream's norms treat on their own (models with layer_specs)
+    pre_norm: bool = True  # False: sub-layers read the stream itself, only their outputs are normed (models with layer_specs)
     # multi-token prediction (draft head)
     mtp_num_layers: int | None = None
     model_arch: str = "qwen2"
@@ -114,8 +117,24 @@ class ModelConfig:
             self.padded_vocab_size = self.vocab_size
         if self.layer_specs is not None:
             self.layer_specs = [LayerSpec.of(x) for x in self.layer_specs]
-        elif self.norm_kind != "rms" or self.norm_offset or self.bigram or self.embed_norm or self.logit_scale != 1.0:
-            raise ValueError("norm_kind, norm_offset, bigram, embed_norm and logit_scale are available to models with layer_specs only")
+            self._check_shared_keys()
+            if self.norm_groups < 1 or self.hidden_size % self.norm_groups:
+                raise ValueError(f"a width of {self.hidden_size} does not divide into {self.norm_groups} normed parts")
+        elif (self.norm_kind != "rms" or self.norm_offset or self.bigram or self.embed_norm or self.logit_scale != 1.0 or self.logit_softcap
+              or self.norm_groups != 1 or not self.pre_norm):  # fmt: skip
+            raise ValueError("norm_kind, norm_offset, norm_groups, pre_norm, bigram, embed_norm, logit_scale and logit_softcap are available to "
+                             "models with layer_specs only")
+
+    def _check_shared_keys(self):
+        """A layer without keys and values of its own names an earlier attention layer that has some of its geometry."""
+        for i, s in enumerate(self.layer_specs):
+            for _, m, _ in s.branches():
+                j = getattr(m, "kv_from", None)
+                if j is None:
+                    continue
+                src = self.layer_specs[j].mixer if 0 <= j < i else None
+                if not isinstance(src, AttentionSpec) or src.kv_from is not None or src.cache_geometry() != m.cache_geometry() or src.rot != m.rot:
+                    raise ValueError(f"layer {i} cannot use the keys and values of layer {j}")
 
     @property
     def head_dim(self) -> int:
@@ -133,6 +152,11 @@ class ModelConfig:
         if isinstance(f, (list, tuple)):
             return bool(f[min(layer, len(f) - 1)])  # draft depths (layer >= num_layers) follow the last layer
         return layer % f == 0
+
+    def spec_norms(self, spec: LayerSpec) -> list[str]:
+        """Names of a specified layer's norms; a norm stands in front of its sub-layer (``norm1``, ``norm2``), behind it (the same with a "b"),
+        or, without ``pre_norm``, behind it under the plain name."""
+        return spec.norms(self.pre_norm and self.post_self_attn_layernorm)
 
     def mixer(self, layer: int) -> str:
         """Token mixer of a layer: ``attention`` (the fused kernel path), ``general_attention`` (attention variants
@@ -176,7 +200,7 @@ class ModelConfig:
         for i in range(self.num_layers):
             if self.layer_specs is not None:
                 spec = self.layer_specs[i]
-                total += self.mixer_params(i) + len(spec.norms(self.post_self_attn_layernorm)) * h + (spec.mlp.params(h) if spec.mlp else 0)
+                total += self.mixer_params(i) + len(self.spec_norms(spec)) * h + (spec.mlp.params(h) if spec.mlp else 0)
                 continue
             total += self.mixer_params(i) + 2 * h
             if self.is_moe_layer(i):

@@ -5,8 +5,9 @@ widths, window or feed-forward carries a list of ``LayerSpec`` instead (``ModelC
 hold the largest value of each size, for code that only budgets memory. The specs are mechanism parameters, not a model:
 any architecture whose layers are built from these pieces can use them.
 
-A layer is a mixer (``AttentionSpec``, ``LatentSpec``, ``DeltaSpec``, or two of them side by side: ``ParallelSpec``) and a
-feed-forward, one after the other with a residual sum each, or both reading one normed input (``LayerSpec.parallel_ff``).
+A layer is a mixer (``AttentionSpec``, ``LatentSpec``, ``DeltaSpec``, ``StateSpaceSpec``, ``MatrixMemorySpec``, or two of them side by side:
+``ParallelSpec``) and a feed-forward, one after the other with a residual sum each, or both reading one normed input
+(``LayerSpec.parallel_ff``).
 """
 
 from __future__ import annotations
@@ -107,8 +108,13 @@ class AttentionSpec:
     "geometric": head h of H subtracts ``2^(-8 (h + 1) / H) * (i - j)`` from its scores; a ``DistanceBiasSpec``: a learned number
     is added. ``qk_norm``: RMS norm of every query and key head (one weight each, shared by the heads) before the rotation
     ``rot``; with ``norm_over`` "projection" of all heads at once, a weight per channel. ``qk_bias``: the query and key
-    projections have biases. ``tied_values``: the values are the keys as projected, before norm and rotation. ``gate``: see
-    ``GATES``. ``sink``: score of an extra column of the softmax that has no value (None: no such column)."""
+    projections have biases, ``vo_bias``: the value and output projections have. ``tied_values``: the values are the keys as projected,
+    before norm and rotation. ``gate``: see ``GATES``. ``sink``: score of an extra column of the softmax that has no value (None: no
+    such column).
+
+    ``diff``: every head is the difference of two attentions over the same values, ``o = a1 - w a2`` with a learned w per layer that
+    starts out near ``diff``, over its root mean square and times ``1 - diff``; ``dim`` is then the width of each of the two query /
+    key halves of a head. ``kv_from``: the keys and values are those that layer ``kv_from`` left in the cache."""
 
     heads: int
     kv_heads: int
@@ -127,6 +133,9 @@ class AttentionSpec:
     qk_bias: bool = False
     tied_values: bool = False
     gate: str | None = None
+    vo_bias: bool = False
+    diff: float | None = None
+    kv_from: int | None = None
 
     def __post_init__(self):
         if isinstance(self.rot, dict):
@@ -151,6 +160,11 @@ class AttentionSpec:
             raise ValueError(f"unknown norm {self.norm_over!r} or gate {self.gate!r}")
         if self.tied_values and self.vdim != self.dim:
             raise ValueError(f"keys of width {self.dim} cannot be the values of width {self.vdim}")
+        if self.diff is not None and (self.distance_bias is not None or self.sink is not None or self.gate is not None or self.tied_values
+                                      or (self.qk_norm and self.norm_over != "head")):  # fmt: skip
+            raise ValueError("a difference of two attentions has no distance bias, sink, gate, tied values or norm over all heads")
+        if self.kv_from is not None and (self.tied_values or self.kv_from < 0):
+            raise ValueError("keys and values of another layer cannot be tied")
 
     @property
     def learned_bias(self) -> DistanceBiasSpec | None:
@@ -162,7 +176,12 @@ class AttentionSpec:
 
     def cache_geometry(self, tp: int = 1) -> tuple[int, int, int]:
         """(heads, key width, value width) of what one token leaves in the cache."""
-        return self.kv_heads // tp, self.dim, self.vdim
+        return self.kv_heads // tp, self.maps * self.dim, self.vdim
+
+    @property
+    def maps(self) -> int:
+        """Attentions per head."""
+        return 1 if self.diff is None else 2
 
     def norm_widths(self) -> tuple[int, int]:
         """Weights of the query norm and of the key norm."""
@@ -175,9 +194,13 @@ class AttentionSpec:
         return [2.0 ** (-8.0 * (h + 1) / self.heads) for h in range(self.heads)]
 
     def params(self, width: int) -> int:
-        n = width * (self.heads * (self.dim + self.vdim) + self.kv_heads * (self.dim + (0 if self.tied_values else self.vdim)) + self.gate_rows)
-        n += sum(self.norm_widths()) if self.qk_norm else 0
-        n += (self.heads + self.kv_heads) * self.dim if self.qk_bias else 0
+        own, dim = (0 if self.kv_from is not None else self.kv_heads), self.maps * self.dim
+        values = 0 if self.tied_values else own * self.vdim
+        n = width * (self.heads * (dim + self.vdim) + own * dim + values + self.gate_rows)
+        n += sum(self.norm_widths()[: 2 if own else 1]) if self.qk_norm else 0
+        n += (self.heads + own) * dim if self.qk_bias else 0
+        n += values + width if self.vo_bias else 0
+        n += 4 * self.dim if self.diff is not None else 0
         return n + (self.learned_bias.rows * self.heads if self.learned_bias else 0)
 
 
@@ -269,13 +292,81 @@ class DeltaSpec:
 
 
 @dataclass(frozen=True)
+class StateSpaceSpec:
+    """State-space duality (Mamba-2). Per head a state S [dim, vdim] follows ``S <- exp(-exp(A_log) dt) S + dt B x^T``, ``y = S^T C + D x`` with
+    ``dt = softplus(projection + dt_bias)``; B and C belong to groups of heads; x, B and C come from a causal convolution (with bias)
+    over ``conv`` tokens per channel and silu. The heads' outputs times silu of a gate are RMS normed in ``norm_groups`` equal parts."""
+
+    heads: int
+    groups: int
+    dim: int
+    vdim: int
+    conv: int
+    norm_groups: int = 1
+
+    def __post_init__(self):
+        if self.groups < 1 or self.heads % self.groups:
+            raise ValueError(f"{self.heads} heads do not divide over {self.groups} groups")
+        if self.conv < 1:
+            raise ValueError(f"a convolution over {self.conv} tokens")
+        if self.norm_groups < 1 or (self.heads * self.vdim) % self.norm_groups:
+            raise ValueError(f"{self.heads} x {self.vdim} channels do not divide into {self.norm_groups} normed parts")
+
+    @property
+    def kv_heads(self) -> int:
+        return self.groups
+
+    @property
+    def channels(self) -> int:
+        """Channels that pass the convolution: x, B, C."""
+        return self.heads * self.vdim + 2 * self.groups * self.dim
+
+    def params(self, width: int) -> int:
+        inner = self.heads * self.vdim
+        return width * (2 * inner + self.channels + self.heads) + self.channels * (self.conv + 1) + 3 * self.heads + inner
+
+
+@dataclass(frozen=True)
+class MatrixMemorySpec:
+    """Matrix memory with exponential gates (the mLSTM of xLSTM). Per head a state S [dim, vdim] and a normaliser n [dim] follow, with log
+    gates i and f capped softly at ``gate_cap`` and a running maximum m that keeps the exponentials in range,
+    ``S <- exp(f + m' - m) S + exp(i - m) k v^T`` (n alike), ``o = S^T q / (max(|n q|, exp(-m)) + 1e-6)``. The output is RMS normed per head
+    with a weight per channel and multiplied by a sigmoid gate."""
+
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+    def __post_init__(self):
+        if not self.gate_cap > 0:
+            raise ValueError(f"gates capped at {self.gate_cap}")
+
+    @property
+    def kv_heads(self) -> int:
+        return self.heads
+
+    def params(self, width: int) -> int:
+        inner = self.heads * self.vdim
+        return width * (2 * self.heads * self.dim + 3 * inner + 2 * self.heads) + inner + 2 * self.heads
+
+
+RECURRENT = (DeltaSpec, StateSpaceSpec, MatrixMemorySpec)  # mixers that keep a state per request instead of keys and values
+Mixer = AttentionSpec | LatentSpec | DeltaSpec | StateSpaceSpec | MatrixMemorySpec
+
+
+@dataclass(frozen=True)
 class ParallelSpec:
     """Two mixers that read the same input; the result is ``left_scale * left + right_scale * right``."""
 
-    left: AttentionSpec | LatentSpec | DeltaSpec
-    right: AttentionSpec | LatentSpec | DeltaSpec
+    left: Mixer
+    right: Mixer
     left_scale: float = 1.0
     right_scale: float = 1.0
+
+    def __post_init__(self):
+        if any(getattr(m, "vo_bias", False) or getattr(m, "kv_from", None) is not None for m in (self.left, self.right)):
+            raise ValueError("mixers side by side have neither output biases nor another layer's keys and values")
 
     def params(self, width: int) -> int:
         return self.left.params(width) + self.right.params(width)
@@ -286,7 +377,8 @@ def _mixer_of(x):
         return x
     if "left" in x:
         return ParallelSpec(**{**x, "left": _mixer_of(x["left"]), "right": _mixer_of(x["right"])})
-    return DeltaSpec(**x) if "conv" in x else LatentSpec(**x) if "kv_rank" in x else AttentionSpec(**x)
+    kinds = (("norm_groups", StateSpaceSpec), ("gate_cap", MatrixMemorySpec), ("conv", DeltaSpec), ("kv_rank", LatentSpec))
+    return next((kind for key, kind in kinds if key in x), AttentionSpec)(**x)
 
 
 @dataclass(frozen=True)
@@ -294,7 +386,10 @@ class FeedForwardSpec:
     """Dense (``experts`` None) or mixture-of-experts feed-forward. ``gated``: ``down(act(gate x) * up x)``, otherwise
     ``down(act(up x))``; with experts the same form is every expert's. ``score`` / ``renorm``: router scores over all
     experts, kept as they are or divided by the sum of the chosen ones. ``shared_ff`` > 0: an expert of that width runs
-    for every token, scaled by a sigmoid gate of its own when ``shared_gate``. ``router_bias``: added to the router's logits."""
+    for every token, scaled by a sigmoid gate of its own when ``shared_gate``. ``router_bias``: added to the router's logits.
+    ``score`` "softmax" or "sigmoid". ``expert_groups`` > 1: the experts form that many groups of neighbours, a group's score is the sum of
+    its two best ones, and only experts of the ``keep_groups`` best groups can be chosen. ``act`` "poly_norm": ``a N(z) + b N(z^2) + c N(z^3)
+    + e`` of the row's hidden units with learned numbers, N dividing a row by its root mean square."""
 
     ff: int
     act: str
@@ -306,17 +401,29 @@ class FeedForwardSpec:
     shared_ff: int = 0
     shared_gate: bool = False
     router_bias: bool = False
+    expert_groups: int = 1
+    keep_groups: int = 1
 
     def __post_init__(self):
-        if self.act not in ("silu", "gelu_tanh", "relu2"):
+        if self.act not in ("silu", "gelu_tanh", "relu2", "poly_norm"):
             raise ValueError(f"unknown activation {self.act!r}")
+        if self.act == "poly_norm" and (self.gated or self.experts is not None):
+            raise ValueError("a normed polynomial is the activation of dense, ungated feed-forwards")
+        if self.score not in ("softmax", "sigmoid"):
+            raise ValueError(f"unknown router score {self.score!r}")
+        if self.expert_groups != 1 or self.keep_groups != 1:
+            per, rest = divmod(self.experts or 0, self.expert_groups)
+            if rest or not 1 <= self.keep_groups <= self.expert_groups or self.top > self.keep_groups * per:
+                raise ValueError(f"{self.top} of {self.experts} experts in the best {self.keep_groups} of {self.expert_groups} groups")
+            if self.score != "sigmoid":
+                raise ValueError("groups of experts are compared by sigmoid scores")
         if self.experts is not None and not 1 <= self.top <= self.experts:
             raise ValueError(f"{self.top} of {self.experts} experts per token")
 
     def params(self, width: int) -> int:
         mats = 3 if self.gated else 2
         if self.experts is None:
-            return mats * width * self.ff
+            return mats * width * self.ff + (4 if self.act == "poly_norm" else 0)
         n = self.experts * (mats * width * self.ff + width + (1 if self.router_bias else 0))
         if self.shared_ff:
             n += mats * width * self.shared_ff + (width if self.shared_gate else 0)
@@ -325,7 +432,7 @@ class FeedForwardSpec:
 
 @dataclass(frozen=True)
 class LayerSpec:
-    mixer: AttentionSpec | LatentSpec | DeltaSpec | ParallelSpec
+    mixer: Mixer | ParallelSpec
     mlp: FeedForwardSpec | None = None  # None: the layer is its mixer only
     parallel_ff: bool = False  # mixer and feed-forward read the same normed input and join the stream in one sum
 
@@ -333,6 +440,8 @@ class LayerSpec:
         m = self.mlp
         if self.parallel_ff and m is not None and m.experts is not None and m.shared_gate:
             raise ValueError("the shared expert of a mixture beside the mixer has no gate: its output is summed with the mixer's")
+        if self.parallel_ff and m is not None and m.act == "poly_norm":
+            raise ValueError("a normed polynomial is the activation of a feed-forward behind its mixer")
 
     @property
     def joint_ff(self) -> tuple[str, int] | None:
@@ -357,7 +466,7 @@ class LayerSpec:
     def to_dict(self) -> dict:
         return dataclasses.asdict(self)
 
-    def branches(self) -> list[tuple[str, AttentionSpec | LatentSpec | DeltaSpec, float]]:
+    def branches(self) -> list[tuple[str, Mixer, float]]:
         """(prefix of its tensors behind ``l<i>.``, mixer, factor of its output) of every mixer of the layer."""
         m = self.mixer
         if isinstance(m, ParallelSpec):
@@ -365,7 +474,7 @@ class LayerSpec:
         return [("mix.", m, 1.0)]
 
     def norms(self, post: bool) -> list[str]:
-        """Names of the layer's norms (``post``: every sub-layer's output has one too)."""
+        """Names of the layer's norms: one per sub-layer, or with ``post`` two (of its input, and with a "b" of its output)."""
         subs = ["norm1"] if self.mlp is None or self.parallel_ff else ["norm1", "norm2"]
         return [n + x for n in subs for x in (("", "b") if post else ("",))]
 
@@ -565,6 +674,72 @@ def zetizen_json(cfg) -> dict:
                 width=cfg.hidden_size)  # fmt: skip
 
 
+# ------------------------------------------------------------------------------------------------- Pebodra
+# Fixed by the design: a norm (RMS, in parts) on every sub-layer's output and none on its input; three mixers: windowed
+# differential attention with biases and norms of query and key halves, whose keys and values another layer may share;
+# Mamba-2; mLSTM; dense feed-forwards with a normed polynomial, gated silu experts weighted by the sigmoid of their logits.
+
+
+def pebodra_config(c: dict, shapes: dict | None = None) -> dict:
+    """``config.json`` of a Pebodra model -> ``ModelConfig`` arguments."""
+    specs = []
+    for i, layer in enumerate(c["layers"]):
+        m, f = layer["mixer"], layer.get("mlp")
+        if layer["type"] == "attention":
+            rot, mask = m.get("rot"), m.get("mask") or {}
+            mixer = AttentionSpec(m["heads"], m["kv_heads"], m["dim"], m["vdim"], float(m["scale"]), mask.get("size"), qk_norm=True,
+                                  rot=RotarySpec(rot["dims"], float(rot["base"]), False) if rot else None, qk_bias=True, vo_bias=True,
+                                  diff=float(m["diff"]), kv_from=m.get("kv_from"))  # fmt: skip
+        elif layer["type"] == "mamba2":
+            mixer = StateSpaceSpec(m["heads"], m["groups"], m["state"], m["vdim"], m["conv"], m["norm_groups"])
+        elif layer["type"] == "mlstm":
+            mixer = MatrixMemorySpec(m["heads"], m["dim"], m["vdim"], float(m["gate_cap"]))
+        else:
+            raise ValueError(f"layer {i}: a Pebodra model has no mixer of type {layer['type']!r}")
+        mlp = None
+        if f is not None and f["kind"] == "dense":
+            mlp = FeedForwardSpec(f["ff"], "poly_norm", gated=False)
+        elif f is not None and f["kind"] == "moe":
+            r = f["router"]
+            g = r.get("groups") or dict(count=1, keep=1)
+            mlp = FeedForwardSpec(f["expert"]["ff"], "silu", experts=r["experts"], top=r["top"], score="sigmoid", expert_groups=g["count"],
+                                  keep_groups=g["keep"])  # fmt: skip
+        elif f is not None:
+            raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
+        specs.append(LayerSpec(mixer, mlp))
+    return dict(flat_sizes(specs), layer_specs=specs, hidden_size=c["width"], vocab_size=c["vocab"], norm_epsilon=c["norm"]["eps"],
+                norm_groups=c["norm"].get("groups") or 1, pre_norm=False, post_self_attn_layernorm=True, post_mlp_layernorm=True,
+                logit_softcap=float(c["logit_softcap"]) if c.get("logit_softcap") else None, tie_word_embeddings=False,
+                model_arch="Pebodra")  # fmt: skip
+
+
+def pebodra_json(cfg) -> dict:
+    """The ``config.json`` of a Pebodra ``ModelConfig`` (inverse of ``pebodra_config``)."""
+    layers = []
+    for s in cfg.layer_specs:
+        a, f = s.mixer, s.mlp
+        if isinstance(a, StateSpaceSpec):
+            kind, mixer = "mamba2", dict(heads=a.heads, groups=a.groups, state=a.dim, vdim=a.vdim, conv=a.conv, norm_groups=a.norm_groups)
+        elif isinstance(a, MatrixMemorySpec):
+            kind, mixer = "mlstm", dict(heads=a.heads, dim=a.dim, vdim=a.vdim, gate_cap=a.gate_cap)
+        else:
+            kind, mixer = "attention", dict(heads=a.heads, kv_heads=a.kv_heads, dim=a.dim, vdim=a.vdim, scale=a.scale, diff=a.diff)
+            if a.window is not None:
+                mixer["mask"] = dict(size=a.window)
+            if a.rot is not None:
+                mixer["rot"] = dict(dims=a.rot.dims, base=a.rot.base)
+            if a.kv_from is not None:
+                mixer["kv_from"] = a.kv_from
+        mlp = None
+        if f is not None and f.experts is None:
+            mlp = dict(kind="dense", ff=f.ff)
+        elif f is not None:
+            mlp = dict(kind="moe", expert=dict(ff=f.ff), router=dict(experts=f.experts, top=f.top, groups=dict(count=f.expert_groups, keep=f.keep_groups)))
+        layers.append(dict(type=kind, mixer=mixer, mlp=mlp))
+    return dict(architecture="Pebodra", layers=layers, logit_softcap=cfg.logit_softcap, norm=dict(eps=cfg.norm_epsilon, groups=cfg.norm_groups),
+                vocab=cfg.vocab_size, width=cfg.hidden_size)  # fmt: skip
+
+
 # ``config.json`` files that name their design in "architecture": name -> (reader(config, tensor shapes or None), writer)
 LAYERED_ARCHITECTURES = {"Pefolix": (pefolix_config, pefolix_json), "Ledazen": (ledazen_config, ledazen_json),
-                         "Zetizen": (zetizen_config, zetizen_json)}  # fmt: skip
+                         "Zetizen": (zetizen_config, zetizen_json), "Pebodra": (pebodra_config, pebodra_json)}  # fmt: skip

@@ -234,7 +234,7 @@ def to_flags(cfg) -> list[str]:
                       "index_topk_freq", "index_skip_topk_offset", "rotary_scaling_type", "rotary_original_max_position",
                       "yarn_beta_fast", "yarn_beta_slow", "mscale", "mscale_all_dim", "rope_low_freq_factor", "rope_high_freq_factor", "index_rotary_interleaved") and v == base[f.name]:  # fmt: skip
             continue
-        if f.name in ("norm_kind", "norm_offset", "embed_norm", "logit_scale") or (f.name == "v_head_dim" and cfg.layer_specs is not None):
+        if f.name in ("norm_kind", "norm_offset", "embed_norm", "logit_scale", "logit_softcap", "norm_groups", "pre_norm") or (f.name == "v_head_dim" and cfg.layer_specs is not None):
             continue
         if f.name in ("layer_specs", "bigram"):
             continue  # no flags: the layers are described by --hf-checkpoint (a preset or a config.json)

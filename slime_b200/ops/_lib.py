@@ -34,11 +34,13 @@ _SIGS = {
     "sb_dp_reduce_shard": [P, I, I, I, L, L, P, P, P, P, P],
     "sb_dp_adam_bcast": [P, P, P, P, P, I, I, I, L, L, F, F, F, F, F, F, F, F, F, P, I, P],
     "sb_group_fp8_quant_1x128": [P, P, P, P, I, I, L, L, I, P],
-    "sb_moe_topk": [P, P, P, P, P, L, I, L, I, I, I, F, P],
+    "sb_moe_topk": [P, P, P, P, P, L, I, L, I, I, I, F, I, I, P],
     "sb_moe_layout": [P, P, P, I, I, I, I, P],
-    "sb_stream_norm": [P, I, P, I, P, P, I, P, P, I, P, P, I, P, P, I, I, I, F, F, I, P, P, P, L, L, I, P, F, P],
+    "sb_stream_norm": [P, I, P, I, P, P, I, P, P, I, P, P, I, P, P, I, I, I, F, F, I, P, P, P, L, L, I, P, F, I, P],
+    "sb_poly_norm": [P, P, P, P, I, I, I, L, L, F, I, P],
+    "sb_softcap": [P, I, L, L, F, P],
     "sb_glu": [P, P, P, L, I, L, L, I, I, P],
-    "sb_heads": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, L, L, L, F, I, P],
+    "sb_heads": [P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, L, L, L, L, F, I, P],
     "sb_heads_all": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, L, L, L, P, I, I, F, I, P],
     "sb_latent_place": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, L, L, F, I, P],
     "sb_latent_turn": [P, P, P, P, I, I, I, I, I, L, L, L, L, I, P],
@@ -55,6 +57,12 @@ _SIGS = {
     "sb_delta_scan": [P, P, P, L, P, P, P, I, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P],
     "sb_delta_step": [P, P, P, P, P, L, L, L, P, P, P, P, P, P, P, P, P, P, P, L, L, F, F, I, I, I, I, I, I, I, I, I, P],
     "sb_head_gate": [P, P, P, P, I, I, I, L, L, F, F, I, I, P],
+    "sb_ssd_prep": [P, P, P, P, L, P, P, P, P, P, P, P, I, P, P, P, P, I, I, I, I, I, I, P],
+    "sb_memory_prep": [P, P, P, P, P, L, P, P, P, P, I, I, P, P, P, P, I, I, I, F, I, P],
+    "sb_linear_scan": [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, P, P, P, P, L, I, I, I, I, I, P],
+    "sb_ssd_step": [P, P, P, P, L, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, P],
+    "sb_memory_step": [P, P, P, P, P, L, P, P, P, P, P, P, P, P, P, P, I, I, I, I, F, I, P],
+    "sb_part_gate": [P, P, P, P, P, I, I, I, L, L, F, F, I, I, I, P],
     "sb_moe_scatter_rows": [P, P, P, L, I, I, P],
     "sb_moe_gather_sum": [P, P, P, P, L, I, I, I, P],
     "sb_moe_route_weight_grad": [P, P, P, P, L, I, I, P],

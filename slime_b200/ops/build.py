@@ -52,7 +52,7 @@ def sources() -> list[str]:
 
 # Parts of the library that can be built on their own (``ensure``): a process that only serves layered models has no use for
 # the training, fp8 and multi-GPU kernels, and a fresh checkout should not wait for them.
-GROUPS = {"serve": ("gemm_sm100", "gemm_simt", "stream", "delta_rule", "window_attn", "flash_window_sm100", "latent_sm100", "decode_attn_sm100", "paged_attn", "moe",
+GROUPS = {"serve": ("gemm_sm100", "gemm_simt", "stream", "delta_rule", "linear_scan", "window_attn", "flash_window_sm100", "latent_sm100", "decode_attn_sm100", "paged_attn", "moe",
                     "quant", "elementwise", "sampling")}  # fmt: skip
 
 

@@ -40,6 +40,9 @@ class DeltaInputs:
     A_log: torch.Tensor
     dt_bias: torch.Tensor
 
+    def gated(self, z, w, act: str, eps: float, scale: float = 1.0) -> "DeltaMixer":
+        return DeltaMixer(self, z, w, act, eps, scale)
+
     def sizes(self, state):
         """(H, G, D, DV, taps, per_channel)"""
         H, D, DV = state.shape[1:]
@@ -165,3 +168,22 @@ def delta_step(x: DeltaInputs, state, ring, slots, active, positions, z, w, act:
                                   int(x.q.dtype == torch.float32), _lib.stream())  # fmt: skip
     _lib.check(rc, "sb_delta_step")
     return out
+
+
+@dataclasses.dataclass
+class DeltaMixer:
+    """The rule with the norm and gate of its output (``head_gate``), as the engine runs recurrent mixers: ``extend`` over the packed rows of a
+    pass, ``step`` over the decode rows, both on the slots of a ``SlotState``."""
+
+    inputs: DeltaInputs
+    z: torch.Tensor
+    w: torch.Tensor
+    act: str
+    eps: float
+    scale: float = 1.0
+
+    def extend(self, s, batch, out=None):
+        return head_gate(delta_extend(self.inputs, s.state, s.ring, batch), self.z, self.w, self.act, self.eps, self.scale, out)
+
+    def step(self, s, slots, active, positions, out=None):
+        return delta_step(self.inputs, s.state, s.ring, slots, active, positions, self.z, self.w, self.act, self.eps, self.scale, out)

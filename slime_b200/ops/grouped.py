@@ -27,31 +27,41 @@ P = _lib.ptr
 
 
 def route_topk(logits: torch.Tensor, k: int, *, score: str = "softmax", pre_softmax: bool = False, renorm: bool = True,
-               bias: torch.Tensor | None = None, scale: float | None = None, raw_index: bool = False, shift: torch.Tensor | None = None):
+               bias: torch.Tensor | None = None, scale: float | None = None, raw_index: bool = False, shift: torch.Tensor | None = None,
+               groups: tuple[int, int] | None = None):  # fmt: skip
     """Router logits [T, E] (fp32) -> ``(weights [T, k] fp32, indices [T, k] int64)`` in one kernel (``raw_index``: the
     kernel's own int32 indices on CUDA, which is what ``DeviceLayout`` reads).
 
     ``score="softmax"`` with ``renorm`` and not ``pre_softmax``: softmax over the k picked logits; with ``pre_softmax``
     or ``renorm=False``: full softmax, pick k, keep the probabilities. ``score="sigmoid"``: sigmoid scores, ``bias``
     steers the choice only, weights are the picked scores (normalised when ``renorm``). ``scale`` multiplies the result.
-    ``shift`` [E] is added to the logits before all this.
+    ``shift`` [E] is added to the logits before all this. ``groups`` = (number, kept), with sigmoid scores: the experts form equal
+    groups of neighbours, of which only those with the largest sum of two best choices can be chosen from.
     """
     T, E = logits.shape
     mode = 2 if score == "sigmoid" else (1 if (pre_softmax or not renorm) else 0)
-    if logits.is_cuda and E <= 512 and k <= 32:
+    n_groups, kept = groups or (1, 1)
+    assert n_groups == 1 or mode == 2, "groups of experts are compared by sigmoid scores"
+    if logits.is_cuda and E <= 512 and k <= 32 and n_groups <= 32:
         lg = logits.float()  # a column range of wider rows is fine
         lg = lg if lg.stride(1) == 1 else lg.contiguous()
         idx = torch.empty(T, k, dtype=torch.int32, device=lg.device)
         w = torch.empty(T, k, dtype=torch.float32, device=lg.device)
         b = None if bias is None else bias.float().contiguous()
         shift = None if shift is None else shift.float().contiguous()
-        rc = _lib.lib().sb_moe_topk(P(lg), P(shift), P(b), P(idx), P(w), T, E, lg.stride(0), k, mode, int(renorm), float(scale or 1.0), _lib.stream())
+        rc = _lib.lib().sb_moe_topk(P(lg), P(shift), P(b), P(idx), P(w), T, E, lg.stride(0), k, mode, int(renorm), float(scale or 1.0),
+                                    n_groups, kept, _lib.stream())  # fmt: skip
         _lib.check(rc, "sb_moe_topk")
         return w, idx if raw_index else idx.long()
     lg = logits.float() if shift is None else logits.float() + shift.float()
     if mode == 2:
         scores = torch.sigmoid(lg)
-        idx = torch.topk(scores + bias.float() if bias is not None else scores, k, dim=-1).indices
+        choice = scores + bias.float() if bias is not None else scores
+        if n_groups > 1:
+            from slime_b200.models.moe import group_limited
+
+            choice = group_limited(choice, n_groups, kept)
+        idx = torch.topk(choice, k, dim=-1).indices
         w = scores.gather(-1, idx)
         if renorm:
             w = w / (w.sum(-1, keepdim=True) + 1e-20)

@@ -1,5 +1,5 @@
 """Ops around an fp32 residual stream (``csrc/stream.cu``): the fused step between two sub-layers of a decoder that
-normalises before and after each of them, feed-forward activations, and cache writes of any width.
+normalises before each of them, behind it, or both, feed-forward activations, and cache writes of any width.
 
 CUDA tensors run the kernels; CPU tensors run the definitions in this file.
 """
@@ -50,7 +50,10 @@ class PairTable:
         return torch.where(self.prev >= 0, r, torch.full_like(r, n))
 
 
-def _norm(v, w, eps, kind, offset=0.0):
+def _norm(v, w, eps, kind, offset=0.0, groups=1):
+    if groups > 1:
+        p = v.unflatten(-1, (groups, -1))
+        return (p * torch.rsqrt(p.pow(2).mean(-1, keepdim=True) + eps)).flatten(-2) * (w.float() + offset)
     mean = v.mean(-1, keepdim=True) if kind == "layer" else 0.0
     d = v - mean
     return d * torch.rsqrt(d.pow(2).mean(-1, keepdim=True) + eps) * (w.float() + offset)
@@ -70,15 +73,15 @@ def _combine(e: ExpertSum) -> torch.Tensor:
 
 
 def stream_norm(y, res, pre_w, eps, *, kind="rms", post_w=None, ids=None, offset=0.0, pair: PairTable | None = None,
-                gain=1.0):  # fmt: skip
+                gain=1.0, groups=1, emit: torch.dtype | None = None):  # fmt: skip
     """``res (+)= norm(y) * post_w`` and return ``norm(res) * pre_w``, in one launch.
 
     ``y``: sub-layer output [T, H], an ``ExpertSum``, or an embedding table when ``ids`` [T] is given (ids outside the table give
     zero rows: other ranks' part of a sharded vocabulary). ``res``: fp32 [T, H],
     updated in place; None starts the stream (a new tensor is returned as second value). ``post_w`` None: no norm of the
-    sub-layer's output; ``pre_w`` None: nothing but the stream is wanted (the first value is None). ``kind``: "rms" or
-    "layer" (mean removed, no bias); ``offset`` is added to the norm weights in fp32. ``pair``: rows of a second table added to
-    ``y``. ``gain``: factor of the returned norm. Norms, sums and the stream are fp32 whatever the element types."""
+    sub-layer's output; ``pre_w`` None: nothing but the stream is wanted (the first value is None), or with ``emit`` the stream itself in
+    that type. ``kind``: "rms" or "layer" (mean removed, no bias); ``groups``: equal parts of a row with an RMS norm of their own; ``offset`` is added to the norm weights in fp32. ``pair``: rows of a second table added to
+    ``y``. ``gain``: factor of the first value. Norms, sums and the stream are fp32 whatever the element types."""
     moe = y if isinstance(y, ExpertSum) else None
     src = moe.rows if moe is not None else y
     T = moe.tokens() if moe is not None else (ids.numel() if ids is not None else y.shape[0])
@@ -86,7 +89,8 @@ def stream_norm(y, res, pre_w, eps, *, kind="rms", post_w=None, ids=None, offset
     init = res is None
     if moe is not None:
         _checks.index_range("stream_norm", "dest", moe.dest, upper=src.shape[0], lower=-(1 << 31))
-    w_dtype = pre_w.dtype if pre_w is not None else (post_w.dtype if post_w is not None else src.dtype)
+    w_dtype = pre_w.dtype if pre_w is not None else emit or (post_w.dtype if post_w is not None else src.dtype)
+    assert kind == "rms" or groups == 1
     if not src.is_cuda:
         if ids is not None:
             i = ids.long()
@@ -96,17 +100,21 @@ def stream_norm(y, res, pre_w, eps, *, kind="rms", post_w=None, ids=None, offset
         if pair is not None:
             v = v + pair.table[pair.rows()].float()
         if post_w is not None:
-            v = _norm(v, post_w, eps, kind, offset)
+            v = _norm(v, post_w, eps, kind, offset, groups)
         if init:
             res = v.clone()
         else:
             res.add_(v)
-        return (None if pre_w is None else (_norm(res, pre_w, eps, kind, offset) * gain).to(w_dtype)), res
+        if pre_w is None and emit is None:
+            return None, res
+        h = res if pre_w is None else _norm(res, pre_w, eps, kind, offset, groups)
+        return (h * gain).to(w_dtype), res
     src = src.contiguous()
     if init:
         res = torch.empty(T, H, dtype=torch.float32, device=src.device)
     assert res.dtype == torch.float32 and res.is_contiguous() and src.dtype in (torch.bfloat16, torch.float32)
-    h = torch.empty(T, H, dtype=w_dtype, device=src.device) if pre_w is not None else None
+    h = torch.empty(T, H, dtype=w_dtype, device=src.device) if pre_w is not None or emit is not None else None
+    assert all(w is None or w.dtype == w_dtype for w in (pre_w, post_w))
     dest = wts = shared = gate = base = None
     k = 1
     if moe is not None:
@@ -128,7 +136,7 @@ def stream_norm(y, res, pre_w, eps, *, kind="rms", post_w=None, ids=None, offset
         gate.stride(0) if gate is not None else 0, P(post_w), P(res), int(init), P(pre_w), P(h), int(w_dtype == torch.float32),
         T, H, float(eps), float(offset), int(kind == "layer"), P(pair.table) if pair else None, P(pair.ids) if pair else None,
         P(pair.prev) if pair else None, pair.mul_prev if pair else 0, pair.mul_cur if pair else 0, pair.table.shape[0] - 1 if pair else 0,
-        P(base), float(gain), _lib.stream(),
+        P(base), float(gain), int(groups), _lib.stream(),
     )  # fmt: skip
     _lib.check(rc, "sb_stream_norm")
     return h, res
@@ -162,6 +170,40 @@ def feed_forward_act(x: torch.Tensor, act: str, gated: bool, out: torch.Tensor |
     return out
 
 
+def poly_sums(x: torch.Tensor) -> torch.Tensor:
+    """[T, 3] fp32 sums of the second, fourth and sixth powers of rows (a rank's part of them)."""
+    p = x.float().square()
+    return torch.stack([p.sum(-1), p.square().sum(-1), (p.square() * p).sum(-1)], 1)
+
+
+def poly_norm(x: torch.Tensor, coef: torch.Tensor, eps: float, sums: torch.Tensor | None = None, width: int | None = None) -> torch.Tensor:
+    """``a N(x) + b N(x^2) + c N(x^3) + e`` of whole rows with (a, b, c, e) = ``coef`` (fp32) and N dividing a row by its root mean square. ``sums``,
+    ``width``: power sums and width of the whole rows, of which ``x`` is a part."""
+    T, F = x.shape
+    width = width or F
+    if not x.is_cuda:
+        z, s = x.float(), poly_sums(x) if sums is None else sums
+        r = coef[:3] * torch.rsqrt(s / width + eps)
+        return (((z * r[:, 2:3] + r[:, 1:2]) * z + r[:, 0:1]) * z + coef[3]).to(x.dtype)
+    x = x if x.stride(1) == 1 else x.contiguous()
+    assert coef.dtype == torch.float32 and coef.numel() == 4 and (sums is None or (sums.is_contiguous() and sums.shape == (T, 3)))
+    out = torch.empty(T, F, dtype=x.dtype, device=x.device)
+    rc = _lib.lib().sb_poly_norm(P(x), P(out), P(coef), P(sums), T, F, width, x.stride(0), out.stride(0), float(eps), int(x.dtype == torch.float32),
+                                 _lib.stream())  # fmt: skip
+    _lib.check(rc, "sb_poly_norm")
+    return out
+
+
+def softcap_(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """``cap tanh(x / cap)`` in place (fp32 rows)."""
+    if not x.is_cuda:
+        return x.div_(cap).tanh_().mul_(cap)
+    assert x.dtype == torch.float32 and x.stride(1) == 1
+    for part in x.split(65535):
+        _lib.check(_lib.lib().sb_softcap(P(part), part.shape[0], part.shape[1], part.stride(0), float(cap), _lib.stream()), "sb_softcap")
+    return x
+
+
 def rotary_table(positions: int, dims: int, base: float, device=None, *, frequencies: list[float] | None = None, gain: float = 1.0) -> torch.Tensor:
     """fp32 ``[positions, dims]`` = cos | sin of ``p * base^(-2i / dims)`` for the dims / 2 pairs i (computed in fp64); ``frequencies``:
     those instead; ``gain`` multiplies the table."""
@@ -185,24 +227,31 @@ def _turn(x, table, positions, interleaved):
 
 
 def place_heads(q, k, v, slots, k_cache, v_cache, *, q_norm=None, k_norm=None, eps=0.0, table=None, positions=None, interleaved=True,
-                sums=None):  # fmt: skip
+                sums=None, maps=1):  # fmt: skip
     """New queries ``q`` [T, Hq * D], keys [T, Hkv * D] and values [T, Hkv * DV] (column ranges of a projection are fine; values may be
     the keys): RMS norm (``q_norm`` / ``k_norm`` [D]: per query / key head; [Hq * D] / [Hkv * D]: over all heads at once; None: none),
     rotation by ``table`` (``rotary_table``; None: none) at ``positions``. Queries are changed in place and returned [T, Hq, D]; keys
     and values go to cache slot ``slots[t]`` (< 0: nowhere). ``sums``: for a norm over all heads of which this rank has a part,
-    ([T, 2] sums of squares of the whole projections, their widths)."""
+    ([T, 2] sums of squares of the whole projections, their widths). ``k``, ``v`` None: the cache has them already.
+
+    ``maps`` 2 (differential attention): every head of the cache holds two keys of width D side by side, queries come in pairs of heads of
+    width D that meet one of them each. They are returned [T, Hq, 2 D] with zeros where the other key stands."""
+    if maps == 2:
+        return _place_pairs(q, k, v, slots, k_cache, v_cache, q_norm, k_norm, eps, table, positions, interleaved)
     T, (Hkv, D), DV = q.shape[0], k_cache.shape[1:], v_cache.shape[2]
     Hq = q.shape[1] // D
-    over_all = q_norm is not None and q_norm.numel() == Hq * D and k_norm.numel() == Hkv * D and (Hq > 1 or Hkv > 1 or sums is not None)
+    over_all = q_norm is not None and k_norm is not None and q_norm.numel() == Hq * D and k_norm.numel() == Hkv * D and (Hq > 1 or Hkv > 1 or sums is not None)
     _checks.index_range("place_heads", "slots", slots, upper=k_cache.shape[0], lower=-(1 << 31))
     if table is not None:
         _checks.index_range("place_heads", "positions", positions, upper=table.shape[0])
     if q_norm is None and table is None:
-        kv_scatter(k, v, slots, k_cache, v_cache)
+        if k is not None:
+            kv_scatter(k, v, slots, k_cache, v_cache)
         return q.unflatten(1, (Hq, D))
+    assert k is not None or not over_all
     if not q.is_cuda:
         out = []
-        for i, (x, w) in enumerate(((q, q_norm), (k, k_norm))):
+        for i, (x, w) in enumerate(((q, q_norm), (k, k_norm)) if k is not None else ((q, q_norm),)):
             if over_all and sums is not None:
                 x = (x.float() * torch.rsqrt(sums[0][:, i : i + 1] / sums[1][i] + eps) * w.float()).unflatten(1, (-1, D))
             elif over_all:
@@ -212,19 +261,61 @@ def place_heads(q, k, v, slots, k_cache, v_cache, *, q_norm=None, k_norm=None, e
                 x = x if w is None else _norm(x, w, eps, "rms")
             out.append((x if table is None else _turn(x, table, positions, interleaved)).flatten(1).to(q.dtype))
         q.copy_(out[0])
-        kv_scatter(out[1], v, slots, k_cache, v_cache)
+        if k is not None:
+            kv_scatter(out[1], v, slots, k_cache, v_cache)
         return q.unflatten(1, (Hq, D))
-    assert q.stride(1) == k.stride(1) == v.stride(1) == 1 and q.dtype == k.dtype == v.dtype == k_cache.dtype == v_cache.dtype
-    assert k_cache.is_contiguous() and v_cache.is_contiguous() and (q_norm is None or q_norm.dtype == k_norm.dtype == q.dtype)
+    f32 = int(q.dtype == torch.float32)
+    if not over_all:
+        _heads(q, k, v, q, slots, k_cache, v_cache, q_norm, k_norm, eps, table, positions, interleaved, (Hq, Hkv, Hkv, D, DV), 1)
+        return q.unflatten(1, (Hq, D))
+    _check_heads(q, k, v, k_cache, v_cache, q_norm, k_norm)
     head = (P(q), P(k), P(v), P(q_norm), P(k_norm), P(table), P(positions), P(slots), P(k_cache), P(v_cache), T, Hq, Hkv, D, DV,
             0 if table is None else table.shape[1], int(interleaved), q.stride(0), k.stride(0), v.stride(0))  # fmt: skip
-    f32 = int(q.dtype == torch.float32)
-    if over_all:
-        part, widths = sums if sums is not None else (None, (Hq * D, Hkv * D))
-        _lib.check(_lib.lib().sb_heads_all(*head, P(part), *widths, float(eps), f32, _lib.stream()), "sb_heads_all")
-    else:
-        _lib.check(_lib.lib().sb_heads(*head, float(eps), f32, _lib.stream()), "sb_heads")
+    part, widths = sums if sums is not None else (None, (Hq * D, Hkv * D))
+    _lib.check(_lib.lib().sb_heads_all(*head, P(part), *widths, float(eps), f32, _lib.stream()), "sb_heads_all")
     return q.unflatten(1, (Hq, D))
+
+
+def _check_heads(q, k, v, k_cache, v_cache, q_norm, k_norm):
+    assert k_cache.is_contiguous() and v_cache.is_contiguous() and q.stride(1) == 1 and q.dtype == k_cache.dtype == v_cache.dtype
+    assert all(x is None or (x.stride(-1) == 1 and x.dtype == q.dtype) for x in (k, v, q_norm, k_norm))
+
+
+def _heads(q, k, v, q_out, slots, k_cache, v_cache, q_norm, k_norm, eps, table, positions, interleaved, sizes, maps):
+    _check_heads(q, k, v, k_cache, v_cache, q_norm, k_norm)
+    Hq, Hkv, Hv, D, DV = sizes
+    if k is None:
+        Hkv = Hv = 0
+    rc = _lib.lib().sb_heads(
+        P(q), P(k), P(v), P(q_out), P(q_norm), P(k_norm), P(table), P(positions), P(slots), P(k_cache), P(v_cache), q.shape[0], Hq, Hkv, Hv, D, DV,
+        0 if table is None else table.shape[1], int(interleaved), maps, q.stride(0), 0 if k is None else k.stride(0), 0 if v is None else v.stride(0),
+        q_out.stride(0), float(eps), int(q.dtype == torch.float32), _lib.stream(),
+    )  # fmt: skip
+    _lib.check(rc, "sb_heads")
+
+
+def _place_pairs(q, k, v, slots, k_cache, v_cache, q_norm, k_norm, eps, table, positions, interleaved):
+    T, (G, D2), (Hv, DV) = q.shape[0], k_cache.shape[1:], v_cache.shape[1:]
+    D = D2 // 2
+    Hq = q.shape[1] // D
+    assert D2 == 2 * D and G == Hv and Hq % 2 == 0
+    _checks.index_range("place_heads", "slots", slots, upper=k_cache.shape[0], lower=-(1 << 31))
+    if table is not None:
+        _checks.index_range("place_heads", "positions", positions, upper=table.shape[0])
+    if not q.is_cuda:
+        out = []
+        for x, w in ((q, q_norm), (k, k_norm)) if k is not None else ((q, q_norm),):
+            x = x.unflatten(1, (-1, D)).float()
+            x = x if w is None else _norm(x, w, eps, "rms")
+            out.append((x if table is None else _turn(x, table, positions, interleaved)).to(q.dtype))
+        if k is not None:
+            kv_scatter(out[1].flatten(1), v, slots, k_cache, v_cache)
+        wide = torch.zeros(T, Hq, 2, D, dtype=q.dtype)
+        wide[:, 0::2, 0], wide[:, 1::2, 1] = out[0][:, 0::2], out[0][:, 1::2]
+        return wide.flatten(2)
+    wide = torch.empty(T, Hq * D2, dtype=q.dtype, device=q.device)
+    _heads(q, k, v, wide, slots, k_cache, v_cache, q_norm, k_norm, eps, table, positions, interleaved, (Hq, 2 * G, Hv, D, DV), 2)
+    return wide.unflatten(1, (Hq, D2))
 
 
 def head_sums(q, k) -> torch.Tensor:

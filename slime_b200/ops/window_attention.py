@@ -8,6 +8,9 @@ without a value (None: no such column). The output is multiplied by ``out_scale`
 [T, Hq * DV]); ``out`` may be a column range of a wider matrix. Keys and values are read from the cache only,
 so a prompt's later portions, portions of several requests and single tokens beside them are one launch.
 
+``pair``: query heads 2 i and 2 i + 1 are two attentions over the same values, of which output head i is the normed difference
+(``Pair``); the output then has half as many heads as the queries.
+
 Dispatch on CUDA: bf16 with head widths that are multiples of 8 up to 128 run on the tensor cores
 (``csrc/flash_window_sm100.cu``, ``csrc/decode_attn_sm100.cu``), everything else, fp32 included, on the CUDA-core kernel
 ``csrc/window_attn.cu``. CPU tensors run the definition below.
@@ -111,15 +114,27 @@ class ExtendBatch:
         return self._cached("segments", lambda: np.stack([first, self.counts, self.starts, self.state_slots], 1))
 
 
+@dataclasses.dataclass(frozen=True)
+class Pair:
+    """Output head of two attentions: ``d / sqrt(mean(d^2) + eps) * gain`` with ``d = a1 - weight a2`` (``weight``: fp32 tensor of one
+    element)."""
+
+    weight: torch.Tensor
+    gain: float
+    eps: float
+
+
 class Rule(ctypes.Structure):
     """``csrc/attn_rule.cuh::AttnRule``: what a query sees and how its scores are made."""
 
     _fields_ = [(n, ctypes.c_int) for n in ("bytes", "window", "keep_first", "chunk")] + [
-        (n, ctypes.c_float) for n in ("scale", "out_scale", "softcap")] + [(n, ctypes.c_int) for n in ("bias_rows", "gate_width", "reserved")] + [
-        ("gate_pitch", ctypes.c_long)] + [(n, ctypes.c_void_p) for n in ("slopes", "sinks", "bias", "gate")]  # fmt: skip
+        (n, ctypes.c_float) for n in ("scale", "out_scale", "softcap")] + [(n, ctypes.c_int) for n in ("bias_rows", "gate_width")] + [
+        ("pair_gain", ctypes.c_float), ("gate_pitch", ctypes.c_long), ("pair_eps", ctypes.c_float), ("reserved", ctypes.c_int)] + [
+        (n, ctypes.c_void_p) for n in ("slopes", "sinks", "bias", "gate", "pair")]  # fmt: skip
 
     @classmethod
-    def of(cls, q, DV, scale, window=None, keep_first=0, slopes=None, sinks=None, out_scale=1.0, chunk=None, softcap=None, bias=None, gate=None):
+    def of(cls, q, DV, scale, window=None, keep_first=0, slopes=None, sinks=None, out_scale=1.0, chunk=None, softcap=None, bias=None, gate=None,
+           pair: Pair | None = None):  # fmt: skip
         T, Hq = q.shape[:2]
         for t in (slopes, sinks, bias):
             assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.shape[-1] == Hq)
@@ -127,9 +142,11 @@ class Rule(ctypes.Structure):
         if gate is not None:
             width = gate.shape[1] // Hq
             assert gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape in ((T, Hq), (T, Hq * DV))
+        w = None if pair is None else pair.weight
+        assert w is None or (w.dtype == torch.float32 and w.numel() == 1)
         return cls(ctypes.sizeof(cls), NO_WINDOW if window is None else int(window), int(keep_first), int(chunk or 0), float(scale),
-                   float(out_scale), float(softcap or 0.0), 0 if bias is None else bias.shape[0], width, 0,
-                   0 if gate is None else gate.stride(0), P(slopes), P(sinks), P(bias), P(gate))  # fmt: skip
+                   float(out_scale), float(softcap or 0.0), 0 if bias is None else bias.shape[0], width, pair.gain if pair else 1.0,
+                   0 if gate is None else gate.stride(0), pair.eps if pair else 0.0, 0, P(slopes), P(sinks), P(bias), P(gate), P(w))  # fmt: skip
 
     def reach(self, longest: int) -> int:
         """Most keys a query sees of a sequence of ``longest`` tokens."""
@@ -137,10 +154,10 @@ class Rule(ctypes.Structure):
 
 
 def _reference(q, k_cache, v_cache, table, row_req, positions, page_size, scale, window=None, keep_first=0, slopes=None, sinks=None,
-               out_scale=1.0, chunk=None, softcap=None, bias=None, gate=None):  # fmt: skip
+               out_scale=1.0, chunk=None, softcap=None, bias=None, gate=None, pair=None):  # fmt: skip
     T, Hq, _ = q.shape
     Hkv, dv = k_cache.shape[1], v_cache.shape[2]
-    out = torch.empty(T, Hq, dv, dtype=q.dtype)
+    out = torch.empty(T, Hq // 2 if pair else Hq, dv, dtype=q.dtype)
     req = torch.arange(T) if row_req is None else row_req.long()
     for r in req.unique().tolist():
         rows = (req == r).nonzero().flatten()
@@ -166,6 +183,9 @@ def _reference(q, k_cache, v_cache, table, row_req, positions, page_size, scale,
             s = torch.cat([s, sinks.view(1, Hkv, Hq // Hkv, 1).expand(len(rows), -1, -1, 1)], -1)
         p = s.softmax(-1)[..., : len(j)] * out_scale
         y = torch.einsum("tghj,jgd->tghd", p, v).reshape(len(rows), Hq, dv)
+        if pair is not None:
+            y = y[:, 0::2] - pair.weight * y[:, 1::2]
+            y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + pair.eps) * pair.gain
         if gate is not None:
             y = y * torch.sigmoid(gate[rows].float()).view(len(rows), Hq, -1)
         out[rows] = y.to(q.dtype)
@@ -203,17 +223,17 @@ def _into(out, res):
 
 
 def window_extend(q, k_cache, v_cache, batch: ExtendBatch, scale, window=None, keep_first=0, slopes=None, sinks=None, out_scale=1.0,
-                  out=None, *, chunk=None, softcap=None, bias=None, gate=None):  # fmt: skip
+                  out=None, *, chunk=None, softcap=None, bias=None, gate=None, pair=None):  # fmt: skip
     """Attention of the packed rows ``q`` [T, Hq, D] (a strided view is fine) -> [T, Hq, DV]. The rows' own keys and values
     must already be in the cache."""
     T, Hq, D = q.shape
     Hkv, DV = k_cache.shape[1], v_cache.shape[2]
-    form = (scale, window, keep_first, slopes, sinks, out_scale, chunk, softcap, bias, gate)
+    form = (scale, window, keep_first, slopes, sinks, out_scale, chunk, softcap, bias, gate, pair)
     _checks.index_range("window_extend", "block_table", batch.block_table, upper=k_cache.shape[0] // batch.page_size)
     if not q.is_cuda:
         return _into(out, _reference(q, k_cache, v_cache, batch.block_table, batch.row_req, batch.positions, batch.page_size, *form))
     assert q.stride(2) == 1 and q.stride(1) == D and k_cache.is_contiguous() and v_cache.is_contiguous()
-    out, rule = _output(out, T, Hq, DV, q), Rule.of(q, DV, *form)
+    out, rule = _output(out, T, Hq // 2 if pair else Hq, DV, q), Rule.of(q, DV, *form)
     if _tensor_core_shape(q, k_cache, v_cache, batch.page_size):
         tiles = batch.tiles(tile_tokens(Hq, Hkv))
         rc = _lib.lib().sb_flash_window(
@@ -242,19 +262,20 @@ def decode_splits(rows: int, groups: int, reach: int, device, resident: int = 2,
 
 
 def window_decode(q, k_cache, v_cache, block_table, seq_lens, positions, page_size, scale, window=None, keep_first=0, slopes=None,
-                  max_context: int | None = None, sinks=None, out_scale=1.0, out=None, *, chunk=None, softcap=None, bias=None, gate=None):  # fmt: skip
+                  max_context: int | None = None, sinks=None, out_scale=1.0, out=None, *, chunk=None, softcap=None, bias=None, gate=None,
+                  pair=None):  # fmt: skip
     """One query token per request: ``q`` [B, Hq, D] at ``positions`` = ``seq_lens - 1``, pages in ``block_table`` [B, W].
     Static shapes, nothing read on the host (``max_context``: upper bound of the lengths, from which the number of splits
     follows)."""
     B, Hq, D = q.shape
     Hkv, DV = k_cache.shape[1], v_cache.shape[2]
-    form = (scale, window, keep_first, slopes, sinks, out_scale, chunk, softcap, bias, gate)
+    form = (scale, window, keep_first, slopes, sinks, out_scale, chunk, softcap, bias, gate, pair)
     if _checks.enabled():
         _checks.paged("window_decode", block_table, seq_lens, page_size, k_cache.shape[0])
     if not q.is_cuda:
         return _into(out, _reference(q, k_cache, v_cache, block_table, None, positions, page_size, *form))
     assert q.stride(2) == 1 and q.stride(1) == D and k_cache.is_contiguous() and v_cache.is_contiguous()
-    out, rule = _output(out, B, Hq, DV, q), Rule.of(q, DV, *form)
+    out, rule = _output(out, B, Hq // 2 if pair else Hq, DV, q), Rule.of(q, DV, *form)
     if _tensor_core_shape(q, k_cache, v_cache, page_size) and Hq // Hkv <= 16:
         longest = min(max_context or block_table.shape[1] * page_size, block_table.shape[1] * page_size)
         splits = decode_splits(B, Hkv, rule.reach(longest), q.device)
