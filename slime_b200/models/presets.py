@@ -211,6 +211,35 @@ def _zetizen(kinds: str, hidden: int, vocab: int, heads: int, kv_heads: int, dim
 MORE_PRESETS["zetizen-a3b"] = _zetizen("bcl" * 8, 2048, 151936, 32, 4, 128, 32, 128, 1024, (16, 128, 64, 128, 768, 512), 128, 8, 768, 768)
 MORE_PRESETS["zetizen-tiny"] = _zetizen("lcb", 96, 512, 4, 2, 32, 16, 50, 24, (3, 24, 16, 32, 40, 48), 6, 2, 48, 40)
 
+def _pebodra(kinds: str, hidden: int, vocab: int, attn: tuple, ssm: tuple, memory: tuple, window: int, norm_groups: int, ff: int = 0,
+             experts: int = 0, top: int = 0, groups: tuple = (1, 1), expert_ff: int = 0) -> dict:  # fmt: skip
+    """``kinds``: one letter per layer, "a" differential attention, "s" attention with the keys and values of the last "a", "m" Mamba-2, "x" mLSTM;
+    a capital letter: a dense feed-forward, otherwise experts. ``attn``: heads, kv heads, width of a query / key half, width of a value;
+    ``ssm``: heads, groups, state, value width; ``memory``: heads, key width, value width."""
+    from slime_b200.models.layer_spec import AttentionSpec, FeedForwardSpec, LayerSpec, MatrixMemorySpec, RotarySpec, StateSpaceSpec, flat_sizes
+
+    h, g, d, dv = attn
+    dense = FeedForwardSpec(ff, "poly_norm", gated=False) if ff else None
+    moe = FeedForwardSpec(expert_ff, "silu", experts=experts, top=top, score="sigmoid", expert_groups=groups[0], keep_groups=groups[1]) if experts else None
+    specs, last = [], None
+    for i, k in enumerate(kinds):
+        if k in "aA":
+            last = i
+        if k in "aAsS":
+            mixer = AttentionSpec(h, g, d, dv, d**-0.5, window, qk_norm=True, rot=RotarySpec(d, 1e5, False), qk_bias=True, vo_bias=True, diff=0.5,
+                                  kv_from=last if k in "sS" else None)  # fmt: skip
+        else:
+            mixer = StateSpaceSpec(*ssm, 4, ssm[1]) if k in "mM" else MatrixMemorySpec(*memory, 15.0)
+        specs.append(LayerSpec(mixer, dense if k.isupper() else moe))
+    return dict(flat_sizes(specs), layer_specs=specs, hidden_size=hidden, vocab_size=vocab, norm_epsilon=1e-5, norm_groups=norm_groups, pre_norm=False,
+                post_self_attn_layernorm=True, post_mlp_layernorm=True, logit_softcap=30.0, tie_word_embeddings=False, model_arch="Pebodra")  # fmt: skip
+
+
+# Pebodra at the sizes of a dense and a mixture preset above (random weights: there is no published checkpoint)
+MORE_PRESETS["pebodra-4b"] = _pebodra("MAXSMX" * 6, 2560, 151936, (16, 8, 64, 128), (80, 8, 128, 64), (8, 256, 512), 1024, 4, ff=9728)
+MORE_PRESETS["pebodra-a3b"] = _pebodra("Maxsmx" + "maxsmx" * 3, 2048, 151936, (16, 4, 64, 128), (64, 4, 128, 64), (8, 256, 512), 1024, 4, 6144, 128, 8, (8, 4), 768)
+MORE_PRESETS["pebodra-tiny"] = _pebodra("MaxsX", 96, 512, (4, 2, 16, 32), (6, 2, 24, 16), (3, 16, 32), 24, 3, 80, 6, 2, (3, 2), 48)
+
 # name -> what is missing. The numbers of these families are in the recipes they come from; they are not repeated here
 # because a preset that cannot be instantiated correctly is worse than none.
 UNSUPPORTED: dict[str, str] = {}

@@ -186,3 +186,119 @@ def error(got, want):
     d = got.double() - want.double()
     d = d - d.mean(-1, keepdim=True)
     return float((d.pow(2).mean(-1).sqrt() / want.double().std()).max())
+
+
+# ------------------------------------------------------------------------------- models for the tests
+def attn(heads, kv_heads, dim, vdim, window, rot, base=1e4, scale=None, diff=0.4, kv_from=None):
+    m = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, mask=dict(size=window), rot=dict(dims=rot, base=base),
+             scale=scale or dim**-0.5, diff=diff)  # fmt: skip
+    return dict(m, kv_from=kv_from) if kv_from is not None else m
+
+
+def ssm(heads, groups, state, vdim, conv=4, norm_groups=1):
+    return dict(heads=heads, groups=groups, state=state, vdim=vdim, conv=conv, norm_groups=norm_groups)
+
+
+def memory(heads, dim, vdim, gate_cap=12.0):
+    return dict(heads=heads, dim=dim, vdim=vdim, gate_cap=gate_cap)
+
+
+def plain(ff):
+    return dict(kind="dense", ff=ff)
+
+
+def moe(experts, top, ff, groups=(1, 1)):
+    return dict(kind="moe", expert=dict(ff=ff), router=dict(experts=experts, top=top, groups=dict(count=groups[0], keep=groups[1])))
+
+
+def _kind(m):
+    return "mamba2" if "state" in m else "mlstm" if "gate_cap" in m else "attention"
+
+
+def model(width, vocab, layers, norm_groups=1, eps=1e-5, softcap=20.0):
+    """``layers``: (mixer, feed-forward or None)."""
+    return dict(architecture="Pebodra", width=width, vocab=vocab, norm=dict(eps=eps, groups=norm_groups), logit_softcap=softcap,
+                layers=[dict(type=_kind(m), mixer=m, mlp=f) for m, f in layers])  # fmt: skip
+
+
+CONFIGS = {
+    # every mixer twice with different geometry, shared keys under another window, layers without a feed-forward
+    "mixed": model(96, 203, [
+        (ssm(6, 2, 24, 16, 4, 3), plain(112)), (attn(4, 2, 16, 24, 21, 12, 5e3, diff=0.3), moe(8, 3, 32, (4, 2))), (memory(3, 20, 28, 8.0), None),
+        (attn(4, 2, 16, 24, 50, 12, 5e3, scale=0.4, diff=0.6, kv_from=1), moe(9, 2, 24, (3, 2))), (attn(6, 1, 24, 16, 33, 24), plain(56)),
+        (memory(4, 8, 16), moe(4, 4, 16)), (ssm(4, 4, 16, 24, 2, 2), None), (attn(6, 1, 24, 16, 9, 24, kv_from=4), plain(40))],
+        norm_groups=3, eps=3e-4, softcap=9.0),
+    # equal heads, sizes of a power of two, a window of a page
+    "even": model(64, 128, [(attn(4, 2, 16, 32, 16, 16), moe(8, 2, 32, (2, 1))), (ssm(4, 2, 16, 32, 4, 2), plain(128)), (memory(4, 16, 32), moe(8, 2, 32)),
+                            (attn(4, 2, 16, 32, 64, 16, kv_from=0), None)], norm_groups=4),
+    # widths that no 16-byte copy divides
+    "odd": model(90, 77, [(attn(3, 3, 10, 13, 7, 6, 50.0), plain(37)), (ssm(3, 1, 9, 7, 3, 3), moe(6, 2, 13, (3, 1))), (memory(3, 5, 11, 4.0), plain(21)),
+                          (attn(3, 3, 10, 13, 11, 6, 50.0, diff=0.7, kv_from=0), moe(5, 1, 9))], norm_groups=2, eps=1e-3, softcap=3.0),
+    # one head, one expert, one tap; eps large enough to matter; no cap
+    "single": model(40, 33, [(attn(1, 1, 16, 8, 5, 4, 100.0, diff=0.1), moe(1, 1, 24)), (ssm(1, 1, 16, 40, 1), None), (memory(1, 8, 4), moe(2, 1, 8, (2, 1)))],
+                    eps=0.1, softcap=None),
+    # no attention at all, many taps
+    "states": model(48, 61, [(ssm(4, 2, 40, 12, 7, 2), plain(30)), (memory(2, 40, 72), plain(64)), (ssm(2, 2, 8, 68, 4), None)], norm_groups=6),
+}  # fmt: skip
+
+
+def random_tensors(name_or_config, seed=0, sharp=2.5, dtype=torch.float32):
+    """Random weights under the checkpoint's names. ``sharp`` scales the query and key norms, so that single keys dominate the softmax; the
+    recurrences forget slowly."""
+    config = CONFIGS[name_or_config] if isinstance(name_or_config, str) else name_or_config
+    g = torch.Generator().manual_seed(seed)
+    D, out = config["width"], {}
+
+    def rand(*s, gain=1.0, mean=0.0):
+        return torch.randn(*s, generator=g) * gain + mean
+
+    def mat(name, n, cols, gain=1.0):
+        out[name] = rand(n, cols, gain=gain * cols**-0.5)
+
+    out["embed"], out["final.norm"] = rand(config["vocab"], D), rand(D, gain=0.3, mean=1.0)
+    mat("head", config["vocab"], D, 4.0)
+    for i, layer in enumerate(config["layers"]):
+        p, m, f = f"l{i}.", layer["mixer"], layer["mlp"]
+        q, H, dv = p + "mix.", m["heads"], m["vdim"]
+        out[p + "norm1"] = rand(D, gain=0.3, mean=0.8)
+        if layer["type"] == "attention":
+            G, d = m["kv_heads"], m["dim"]
+            rows = dict(q=H * 2 * d) if "kv_from" in m else dict(q=H * 2 * d, k=G * 2 * d, v=G * dv)
+            for n, r in rows.items():
+                mat(q + n, r, D)
+                out[f"{q}{n}.b"] = rand(r, gain=0.3)
+                if n != "v":
+                    out[f"{q}{n}.norm"] = rand(d, gain=0.3, mean=1.0) * sharp**0.5
+            for n in ("lq1", "lk1", "lq2", "lk2"):
+                out[q + n] = rand(d, gain=0.4 * d**-0.25)
+            out[q + "o.b"] = rand(D, gain=0.3)
+        elif layer["type"] == "mamba2":
+            ch = H * dv + 2 * m["groups"] * m["state"]
+            mat(q + "in", H * dv + ch + H, D)
+            out[q + "conv"], out[q + "conv.b"] = rand(ch, m["conv"], gain=0.7 * m["conv"] ** -0.5, mean=0.1), rand(ch, gain=0.2)
+            out[q + "dt_bias"], out[q + "A_log"], out[q + "D"] = rand(H, mean=-2.0), rand(H, gain=0.7, mean=-1.0), rand(H, gain=0.5, mean=0.5)
+            out[q + "norm"] = rand(H * dv, gain=0.3, mean=1.0)
+        else:
+            for n, r in (("q", H * m["dim"]), ("k", H * m["dim"]), ("v", H * dv), ("g", H * dv), ("i", H), ("f", H)):
+                mat(q + n, r, D)
+            out[q + "i.b"], out[q + "f.b"] = rand(H, gain=0.5), rand(H, gain=1.0, mean=3.0)
+            out[q + "norm"] = rand(H * dv, gain=0.3, mean=1.0)
+        mat(q + "o", D, H * dv)
+        if f is None:
+            continue
+        out[p + "norm2"] = rand(D, gain=0.3, mean=0.8)
+        if f["kind"] == "dense":
+            mat(p + "mlp.up", f["ff"], D)
+            mat(p + "mlp.down", D, f["ff"])
+            out[p + "mlp.act"] = rand(4, gain=0.3, mean=0.5)
+            continue
+        for e in range(f["router"]["experts"]):
+            for n in ("gate", "up"):
+                mat(f"{p}mlp.e{e}.{n}", f["expert"]["ff"], D)
+            mat(f"{p}mlp.e{e}.down", D, f["expert"]["ff"])
+        mat(p + "mlp.router", f["router"]["experts"], D, 2.0)
+    return {k: v.to(dtype) for k, v in out.items()}
+
+
+def random_tokens(config, n, seed=0):
+    return torch.randint(0, config["vocab"], (n,), generator=torch.Generator().manual_seed(seed)).tolist()
