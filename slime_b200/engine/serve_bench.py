@@ -7,12 +7,14 @@ per second. ``decode``: replays of the captured decode step (sampling included) 
 second. Device time by CUDA events around exactly K passes after W warm-up ones; the weights and the cache a pass streams are
 several times the L2. The models of a Pefolix pair have the same widths, head counts, layer count and vocabulary; at the context of
 ``window`` tokens they also read the same keys. A Ledazen pair has the same width, heads, layers and vocabulary; its feed-forward
-width is chosen for an equal number of weights in the layers. The Zetizen pairs have the same width, heads, experts and vocabulary.
+width is chosen for an equal number of weights in the layers. The Zetizen pairs have the same width, heads, experts and vocabulary, and so
+has the mixture pair of Pebodra; its other pair is made like Ledazen's.
 Prints one JSON line.
 """
 
 from __future__ import annotations
 
+import dataclasses
 import gc
 import json
 
@@ -22,8 +24,9 @@ from slime_b200.engine.engine import Engine
 from slime_b200.engine.request import Request
 from slime_b200.engine.server_args import ServerArgs
 from slime_b200.models.config import ModelConfig, get_preset
-from slime_b200.models.presets import _ledazen, _pefolix, _zetizen
+from slime_b200.models.presets import _ledazen, _pebodra, _pefolix, _zetizen
 
+HYBRID_FF = 14464  # makes the weights of the dense Pebodra layers as many as its partner's
 LAYERS = 8  # of the 24 to 36 layers of the models the widths are taken from: per-layer cost is what is compared
 
 
@@ -53,7 +56,12 @@ def _pairs() -> dict[str, tuple[ModelConfig, ModelConfig]]:
                          rotary_base=1e6, multi_latent_attention=True, q_lora_rank=768, kv_lora_rank=512, qk_head_dim=128, qk_pos_emb_head_dim=64,
                          v_head_dim=128, model_arch="DeepseekV3ForCausalLM", **experts)  # fmt: skip
     zetizen = lambda kinds: ModelConfig(**_zetizen(kinds, 2048, 151936, 32, 4, 128, 32, 128, 1024, (16, 128, 64, 128, 768, 512), 128, 8, 768, 768))  # noqa: E731,E501
+    routed = dataclasses.replace(grouped, tie_word_embeddings=False, moe_shared_expert_intermediate_size=None)
+    sizes = ((64, 8, 128, 64), (8, 256, 512), 1024, 4)  # Mamba-2, mLSTM, window, parts of a norm
     return {
+        "pebodra-hybrid": (ModelConfig(**_pebodra("MXMA" + "MXMS" * (LAYERS // 4 - 1), 2560, 151936, (32, 8, 64, 128), *sizes, ff=HYBRID_FF)), hybrid),
+        "pebodra-moe": (ModelConfig(**_pebodra("maxs" * (LAYERS // 4), 2048, 151936, (32, 4, 64, 128), *sizes, experts=128, top=8, groups=(8, 4),
+                                               expert_ff=768)), routed),
         "zetizen-grouped": (zetizen("bc" * (LAYERS // 2)), grouped),
         "zetizen-latent": (zetizen("l" * LAYERS), latent),
         "ledazen-hybrid": (ModelConfig(**_ledazen("dddp" * (LAYERS // 4), 2560, 32, 8, 128, 11776, 151936, 32, 16, 128, 128, 128, 65521)), hybrid),

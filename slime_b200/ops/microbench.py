@@ -9,6 +9,7 @@ repetitions with an L2 flush (a 256 MiB memset) between them. One JSON object pe
     attn    flash attention forward / backward (own kernels; the flash-attn library on the same tensors for comparison)
     window  kernels of models with specified layers, each beside the like kernel of the existing models
     rules   kernels of Zetizen layers (capped, biased, chunked and latent attention, experts beside a mixer), likewise
+    scan    kernels of Pebodra layers (linear recurrences, differential attention, grouped routing, norms in parts), likewise
     fused_emul  the peer-memory kernels (DP reduce / Adam, TP all-reduce + norm) with all ranks emulated on one GPU
 
 ``--small`` shrinks the working set to a case suitable for a profiler capture (a few launches, < 1 GB).
@@ -709,9 +710,150 @@ def bench_fused_emul(a):
     _lib.check_status(dev)
 
 
+def bench_scan(a):
+    """Kernels of Pebodra layers beside the like kernel of the existing models: Mamba-2 and mLSTM against the gated delta rule with as
+    many state elements, differential attention against plain attention of the same projections, and what stands around them."""
+    from slime_b200.ops import attention, delta, grouped, linear_scan, stream
+    from slime_b200.ops import window_attention as wa
+
+    gbs, tf = _peaks()
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    rnd = lambda *s, dt=bf: torch.randn(*s, device=dev).to(dt)  # noqa: E731
+    i32 = lambda v: torch.as_tensor(v, dtype=torch.int32, device=dev)  # noqa: E731
+
+    def pair(what, t, t2, work, work2, peak=gbs, **kw):
+        f, f2 = work / t / peak, None if t2 is None else work2 / t2 / peak
+        like = {} if t2 is None else dict(like_us=round(t2 * 1e3, 2), like_of_peak=round(f2, 3), times_further=round(f2 / f, 2))
+        _emit(kind=what, us=round(t * 1e3, 2), of_peak=round(f, 3), **like, **kw)
+
+    def space(T, H, G, N, DV):
+        ch, widths = H * DV + 2 * G * N, [H * DV, H * DV, G * N, G * N, H]
+        return linear_scan.StateSpace(*rnd(T, sum(widths)).split(widths, 1), rnd(ch, 4), rnd(ch), rnd(H, dt=torch.float32), rnd(H, dt=torch.float32) - 3,
+                                      rnd(H, dt=torch.float32), rnd(H * DV), G, 1e-5)  # fmt: skip
+
+    def memory(T, H, D, DV):
+        widths = [H * D, H * D, H * DV, H, H, H * DV]
+        return linear_scan.MatrixMemory(*rnd(T, sum(widths)).split(widths, 1), rnd(H, dt=torch.float32), rnd(H, dt=torch.float32) + 3, rnd(H * DV), 15.0, 1e-5)
+
+    def slots_of(n, H, D, DV, ch=0, normed=False):
+        z = lambda *s: torch.zeros(n, *s, device=dev)  # noqa: E731
+        return linear_scan.SlotState(z(H, D, DV), z(4, ch).to(bf) if ch else None, z(H, D) if normed else None, z(H, 2) if normed else None)
+
+    def rule(T):
+        H, G, D, DV = 32, 16, 128, 128
+        x, ab = rnd(T, 2 * G * D + H * DV), rnd(T, 2 * H)
+        q, k, v = x.split([G * D, G * D, H * DV], 1)
+        inp = delta.DeltaInputs(q, k, v, ab[:, :H], ab[:, H:], rnd(x.shape[1], 4), rnd(H, dt=torch.float32), rnd(H, dt=torch.float32) - 3)
+        return inp.gated(rnd(T, H * DV), rnd(DV), "silu", 1e-5)
+
+    # algorithmic bytes: projections in, result out, states of the requests read (steps) and written
+    ssm, mem = (64, 8, 128, 64), (8, 256, 512)
+    ssm_row, mem_row, rule_row = 2 * (3 * 4096 + 2 * 1024 + 64), 2 * (3 * 4096 + 4096 + 16), 2 * (4096 + 3 * 4096 + 64)
+    ssm_S, mem_S, rule_S = 64 * 128 * 64 * 4, 8 * 256 * 513 * 4, 32 * 128 * 128 * 4
+    for n, L in ((8, 1024), (2, 4096)) if not a.small else ((4, 256),):
+        T, kw = n * L, dict(prompts=f"{n}x{L}")
+        batch = wa.ExtendBatch.build([[0]] * n, [0] * n, [L] * n, 8192, dev, state_slots=list(range(n)))
+        d, ds = rule(T), slots_of(n, 32, 128, 128, 8192)
+        t2 = time_ms(lambda: d.extend(ds, batch), a.iters)
+        for what, m, s, row, S in (("mamba2_prompt", space(T, *ssm), slots_of(n, 64, 128, 64, 4096 + 2048), ssm_row, ssm_S),
+                                   ("mlstm_prompt", memory(T, *mem), slots_of(n, *mem, normed=True), mem_row, mem_S)):
+            out = rnd(T, 4096)
+            t = time_ms(lambda: m.extend(s, batch, out), a.iters)
+            pair(what, t, t2, (T * row + n * S) / 1e6, (T * rule_row + n * rule_S) / 1e6, **kw)
+        m, s = space(T, *ssm), slots_of(n, 64, 128, 64, 4096 + 2048)
+        H, G, N, DV = ssm
+        x, B, C, gates = (torch.rand(T, *sh, device=dev) for sh in ((H, DV), (G, N), (G, N), (H, 4)))
+        segs, runs = batch.segments(), batch.tiles(linear_scan.RUN)
+        t = time_ms(lambda: linear_scan._scan(C, B, x, gates, segs, s, skip=m.skip, ring_in=(m.x, m.B, m.C)), a.iters)
+        pair("mamba2_scan", t, None, (T * (H * DV * 8 + G * N * 8 + H * 16)) / 1e6, None, **kw)
+        P = _lib.ptr
+        t = time_ms(lambda: _lib.check(_lib.lib().sb_ssd_prep(P(m.x), P(m.B), P(m.C), P(m.dt), m.x.stride(0), P(m.conv), P(m.conv_b), P(m.A_log),
+                    P(m.dt_bias), P(s.ring), P(runs), P(segs), runs.shape[0], P(x), P(B), P(C), P(gates), H, G, N, DV, 4, 0, _lib.stream()), "x"), a.iters)  # fmt: skip
+        pair("mamba2_prep", t, None, T * (6 * (H * DV + 2 * G * N) + H * 18) / 1e6, None, **kw)
+        o, z, w, out = torch.randn(T, 4096, device=dev), rnd(T, 4096), rnd(4096), rnd(T, 4096)
+        t2 = time_ms(lambda: delta.head_gate(o.view(T, 32, 128), z, w[:128], "silu", 1e-5, 1.0, out), a.iters)
+        for parts in (8, 1):
+            t = time_ms(lambda: linear_scan.part_gate(o, z, w, parts, "silu", 1e-5, gate_first=True, out=out), a.iters)
+            pair("part_gate", t, t2, T * 4096 * 8 / 1e6, T * 4096 * 8 / 1e6, parts=parts, **kw)
+        H, D, DV = mem
+        q, k, v = (torch.rand(T, H, w, device=dev) for w in (D, D, DV))
+        s, gates, den = slots_of(n, *mem, normed=True), torch.rand(T, H, 4, device=dev), torch.rand(T, H, device=dev)
+        t = time_ms(lambda: linear_scan._scan(q, k, v, gates, segs, s, den=den), a.iters)
+        pair("mlstm_scan", t, None, T * H * (DV * 8 + D * 8 + 20) / 1e6, None, **kw)
+    for B in (64, 4):
+        turn, sets = [0], [i32(range(j * B, (j + 1) * B)) for j in range(256 // B)]  # rotating slots: states come from memory
+        one, at = i32([1] * B), i32([77] * B)
+        d, ds = rule(B), slots_of(256, 32, 128, 128, 8192)
+
+        def step(m, s, out):
+            turn[0] = (turn[0] + 1) % len(sets)
+            m.step(s, sets[turn[0]], one, at, out)
+
+        out = rnd(B, 4096)
+        t2 = time_ms(lambda: step(d, ds, out), a.iters)
+        for what, m, s, row, S in (("mamba2_step", space(B, *ssm), slots_of(256, 64, 128, 64, 6144), ssm_row, ssm_S),
+                                   ("mlstm_step", memory(B, *mem), slots_of(256, *mem, normed=True), mem_row, mem_S)):
+            t = time_ms(lambda: step(m, s, out), a.iters)
+            pair(what, t, t2, B * (row + 2 * S) / 1e6, B * (rule_row + 2 * rule_S) / 1e6, rows=B)
+    # differential attention: 32/8 heads of two 64-wide halves and 128-wide values, against 32/8 x 128
+    H, G, D, ps, win = 32, 8, 128, 64, 1024
+    lam = wa.Pair(torch.tensor([0.4], device=dev), 0.5, 1e-5)
+    for n, nseq in ((1024, 8), (4096, 2)) if not a.small else ((1024, 1),):
+        T = n * nseq
+        x = rnd(T, H + 2 * G, D)
+        kc, vc = x[:, H : H + G].contiguous(), x[:, H + G :].contiguous()
+        pages = [list(range(i * n // ps, (i + 1) * n // ps)) for i in range(nseq)]
+        batch = wa.ExtendBatch.build(pages, [0] * nseq, [n] * nseq, ps, dev)
+        seg = attention.segments_from_cu_seqlens(torch.arange(0, T + 1, n, dtype=torch.int32, device=dev))
+        t2 = time_ms(lambda: attention.flash_fwd(x[:, :H], kc, vc, seg, D**-0.5), a.iters)
+        t3 = time_ms(lambda: wa.window_extend(x[:, :H], kc, vc, batch, D**-0.5, win), a.iters)
+        q, wide = rnd(T, H * D), rnd(T, 2 * H, D)
+        t = time_ms(lambda: wa.window_extend(wide, kc, vc, batch, 0.125, win, pair=lam), a.iters)
+        seen = nseq * (n * (n + 1) / 2 - max(0, n - win) * (n - win + 1) / 2)
+        work, causal = 2.0 * H * (2 * 64 + 2 * 128) / 1e9, 4.0 * H * D / 1e9
+        pair("pair_attention", t, t2, work * seen, causal * nseq * n * (n + 1) / 2, tf, prompts=f"{nseq}x{n}", plain_windowed_us=round(t3 * 1e3, 2),
+             plain_windowed_of_peak=round(causal * seen / t3 / tf, 3))  # fmt: skip
+        kv, slots, pos, nw, nd = rnd(T, 2 * G * D), torch.randperm(T, device=dev).int(), torch.arange(T, device=dev).int() % n, rnd(64), rnd(D)
+        table, tab2 = stream.rotary_table(n, 64, 1e5, dev), stream.rotary_table(n, 128, 1e5, dev)
+        qkv = rnd(T, (H + 2 * G) * D)
+        t2 = time_ms(lambda: ops.rope_kv_write(qkv, pos, tab2, slots, kc, vc, H, G, D, nd, nd, 1e-6), a.iters)
+        for own in (True, False):
+            k, v = (kv[:, : G * D], kv[:, G * D :]) if own else (None, None)
+            t = time_ms(lambda: stream.place_heads(q, k, v, slots, kc, vc, q_norm=nw, k_norm=nw if own else None, eps=1e-6, table=table, positions=pos,
+                                                   interleaved=False, maps=2), a.iters)  # fmt: skip
+            pair("pairs_to_cache", t, t2, T * (H * D * 6 + (2 * G * D * 4 if own else 0)) / 1e6, T * (H * D * 4 + 2 * G * D * 4) / 1e6, rows=T, own_keys=own)
+    for B, ctx in ((64, 1024), (64, 4096), (4, 1024)):
+        pages = -(-ctx // ps)
+        kc, vc = rnd(B * pages * ps, G, D), rnd(B * pages * ps, G, D)
+        bt, lens = torch.randperm(B * pages, device=dev).int().view(B, pages), i32([ctx] * B)
+        q, wide = rnd(B, H, D), rnd(B, 2 * H, D)
+        t2 = time_ms(lambda: ops.paged_decode_attention(q, kc, vc, bt, lens, ps, D**-0.5), a.iters)
+        t3 = time_ms(lambda: wa.window_decode(q, kc, vc, bt, lens, lens - 1, ps, D**-0.5, win, max_context=8192), a.iters)
+        pos = lens - 1
+        t = time_ms(lambda: wa.window_decode(wide, kc, vc, bt, lens, pos, ps, 0.125, win, max_context=8192, pair=lam), a.iters)
+        mb = lambda n: B * n * G * D * 4 / 1e6  # noqa: E731
+        pair("pair_decode", t, t2, mb(min(ctx, win)), mb(ctx), batch=B, context=ctx, plain_windowed_us=round(t3 * 1e3, 2))
+    for T in (8192, 64):
+        y, res, r16, w = torch.randn(T, 2560, device=dev), torch.randn(T, 2560, device=dev), rnd(T, 2560), rnd(2560)
+        t2 = time_ms(lambda: ops.rmsnorm(y, w, 1e-6, r16), a.iters)
+        t = time_ms(lambda: stream.stream_norm(y, res, None, 1e-5, post_w=w, groups=4, emit=bf), a.iters)
+        pair("parts_norm", t, t2, T * 2560 * 14 / 1e6, T * 2560 * 10 / 1e6, rows=T)
+        z, gu, coef = rnd(T, 9728), rnd(T, 2 * 6912), torch.rand(4, device=dev)
+        t, t2 = time_ms(lambda: stream.poly_norm(z, coef, 1e-5), a.iters), time_ms(lambda: ops.swiglu(gu), a.iters)
+        pair("poly_norm", t, t2, T * 9728 * 4 / 1e6, T * 6912 * 6 / 1e6, rows=T)
+        logits = torch.randn(T, 128, device=dev)
+        t = time_ms(lambda: grouped.route_topk(logits, 8, score="sigmoid", renorm=False, raw_index=True, groups=(8, 4)), a.iters)
+        t2 = time_ms(lambda: grouped.route_topk(logits, 8, raw_index=True), a.iters)
+        pair("grouped_routing", t, t2, T * (512 + 64) / 1e6, T * (512 + 64) / 1e6, rows=T)
+    x = torch.randn(64, 151936, device=dev)
+    t = time_ms(lambda: stream.softcap_(x, 30.0), a.iters)
+    pair("softcap", t, None, x.numel() * 8 / 1e6, None, rows=64)
+    _lib.check_status("cuda")
+
+
 def main(argv=None):
     p = argparse.ArgumentParser(prog="python -m slime_b200.ops.microbench")
-    p.add_argument("what", choices=["gemm", "decode", "norm", "fp8", "moe", "attn", "window", "delta", "rules", "fused_emul"])
+    p.add_argument("what", choices=["gemm", "decode", "norm", "fp8", "moe", "attn", "window", "delta", "rules", "scan", "fused_emul"])
     p.add_argument("--iters", type=int, default=20)
     p.add_argument("--reps", type=int, default=20, help="back-to-back launches per timed repetition (decode)")
     p.add_argument("--small", action="store_true")
@@ -725,7 +867,7 @@ def main(argv=None):
     from slime_b200.ops import build
 
     build.build()
-    {"gemm": bench_gemm, "decode": bench_decode, "norm": bench_norm, "fp8": bench_fp8, "moe": bench_moe, "attn": bench_attn, "window": bench_window, "delta": bench_delta, "rules": bench_rules, "fused_emul": bench_fused_emul}[a.what](a)
+    {"gemm": bench_gemm, "decode": bench_decode, "norm": bench_norm, "fp8": bench_fp8, "moe": bench_moe, "attn": bench_attn, "window": bench_window, "delta": bench_delta, "rules": bench_rules, "scan": bench_scan, "fused_emul": bench_fused_emul}[a.what](a)
 
 
 if __name__ == "__main__":
