@@ -17,6 +17,8 @@
 // Everything behind the projections is fp32. The normaliser is one more column of S whose v is 1: an extra CTA per head. The running
 // maximum of a slot has two places, by position parity: whoever computes the next one never overwrites what others still read.
 // The convolution's inputs live in a ring of `taps` rows per slot (row = position mod taps).
+#include <type_traits>
+
 #include "common.cuh"
 
 namespace sb {
@@ -251,10 +253,14 @@ memory_prep_kernel(const __grid_constant__ MemoryIn a, const int4* __restrict__ 
 }
 
 // ------------------------------------------------------------------------------------------------ recurrence over rows
-// A warp holds 4 CPT columns of S: lane = column group (4) x row group (8); a lane has CPT columns and the rows
-// {4 rg + 32 j + 0..3}. q, k, v and gates of the next tokens are copied to shared memory while the current ones are processed. Nothing
+// A warp holds (32 / RG) CPT columns of S: lane = column group x row group (RG of them); a lane has CPT columns and the rows
+// {4 rg + 4 RG j + 0..3}. q, k, v and gates of the next tokens are copied to shared memory while the current ones are processed. Nothing
 // that a token computes is needed by the next one but S itself, so tokens overlap; sums over the rows are taken for two
 // tokens at a time.
+//
+// S is kept divided by the product F of the decays since the start of a chunk of 8 tokens: S' <- S' + k (w / F) v^T and o = F S'^T q cost
+// two operations per element instead of three. The numbers in S' differ from those in S by a common factor only, so nothing is
+// lost as long as F stays far from the end of the number range; a chunk in which it does not decays S token by token.
 constexpr int LS_TOK = 8;     // tokens per copy
 constexpr int LS_STAGES = 4;  // copies in flight or in use
 
@@ -303,22 +309,42 @@ struct Scan {
   int width[3], taps, esize;
 };
 
-template <int NR>
+constexpr float LS_LEAST = 1e-18f;  // smallest product of a chunk's decays that S is divided by
+
+template <int RG, int NR>
 struct LsSmem {
-  static constexpr int W = 8 * NR;  // padded width of a key
+  static constexpr int W = RG * NR;  // padded width of a key
   static __host__ __device__ int stage_floats(int cols) { return LS_TOK * (2 * W + cols + 4); }
 };
 
-template <int NR, int CPT>
-__global__ void __launch_bounds__(256) linear_scan_kernel(const __grid_constant__ Scan a) {
-  constexpr int W = LsSmem<NR>::W;
+// Sums over the RG lanes of a row group of N values per lane: in every round a lane keeps half of its sums and trades the others, by
+// the bits of its number; when one is left the rest is summed plainly. Lane rg ends up with value rg mod N (N <= RG).
+template <int RG, int N>
+__device__ __forceinline__ float ls_reduce(float (&x)[N], int rg) {
+  int bit = 1;
+#pragma unroll
+  for (int n = N; n > 1; n /= 2, bit *= 2) {
+    const bool up = rg & bit;
+#pragma unroll
+    for (int i = 0; i < n / 2; ++i) x[i] = (up ? x[2 * i + 1] : x[2 * i]) + __shfl_xor_sync(0xffffffffu, up ? x[2 * i] : x[2 * i + 1], bit);
+  }
+  float o = x[0];
+#pragma unroll
+  for (int b = N; b < RG; b *= 2) o += __shfl_xor_sync(0xffffffffu, o, b);
+  return o;
+}
+
+template <int RG, int NR, int CPT, int THREADS, int CTAS>
+__global__ void __launch_bounds__(THREADS, CTAS) linear_scan_kernel(const __grid_constant__ Scan a) {
+  using Smem = LsSmem<RG, NR>;
+  constexpr int W = Smem::W, CG = 32 / RG;
   extern __shared__ __align__(16) float ls_smem[];
-  const int nwarp = blockDim.x / 32, cols = nwarp * 4 * CPT;
+  const int nwarp = blockDim.x / 32, cols = nwarp * CG * CPT;
   const int H = a.H, G = a.G, D = a.D, DV = a.DV;
   const int h = blockIdx.y, kh = h / (H / G);
   const bool is_n = static_cast<int>(blockIdx.x) == a.blocks;  // the normaliser: one column whose v is 1
   const int c0 = is_n ? 0 : blockIdx.x * cols;
-  const int stage = LsSmem<NR>::stage_floats(cols);
+  const int stage = Smem::stage_floats(cols);
   // stage layout: k [TOK][W], q [TOK][W], v [TOK][cols], gates [TOK][4]
   constexpr int SQ = LS_TOK * W, SV = 2 * LS_TOK * W;
   const int SC = SV + LS_TOK * cols;
@@ -329,8 +355,8 @@ __global__ void __launch_bounds__(256) linear_scan_kernel(const __grid_constant_
   __syncthreads();
   const int4 seg = a.segs[blockIdx.z];  // first row, tokens, first position, state slot
   const int n = seg.y;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rg = lane & 7, cg = lane >> 3;
-  const int col = warp * 4 * CPT + cg * CPT;  // of this CTA
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rg = lane % RG, cg = lane / RG;
+  const int col = (warp * CG + cg) * CPT;  // of this CTA
   const int pitch = is_n ? 1 : DV, ncol = is_n ? 1 : min(cols, DV - c0);
   const long head = static_cast<long>(seg.w) * H + h;
   float* S_mem = is_n ? a.norm + head * D : a.state + head * D * DV + c0;
@@ -338,7 +364,7 @@ __global__ void __launch_bounds__(256) linear_scan_kernel(const __grid_constant_
   float2 S[CPT][NR / 2];
 #pragma unroll
   for (int j = 0; j < NR / 2; ++j) {
-    const int r = rg * 4 + (j >> 1) * 32 + (j & 1) * 2;
+    const int r = rg * 4 + (j >> 1) * (4 * RG) + (j & 1) * 2;
 #pragma unroll
     for (int c = 0; c < CPT; ++c) {
       S[c][j] = make_float2(0.f, 0.f);
@@ -367,66 +393,69 @@ __global__ void __launch_bounds__(256) linear_scan_kernel(const __grid_constant_
   const float skip = a.skip != nullptr ? a.skip[h] : 0.f;
   float* orow = is_n ? a.den + static_cast<long>(seg.x) * H + h : a.out + (static_cast<long>(seg.x) * H + h) * DV + c0;
   const long ostep = is_n ? H : static_cast<long>(H) * DV;
-  // one token: S and this lane's part of S^T q
-  auto advance = [&](int t, float (&o)[CPT]) {
-    const float4 gate = *reinterpret_cast<const float4*>(base + SC + t * 4);
-    float u[CPT];
-    float2 acc[CPT];
+  float F = 1.f;  // what S is divided by
+  // one token: S and this lane's part of S^T q into o[2 c + which]. `divided`: S divided by F, or decayed token by token
+  auto advance = [&](auto divided, int t, int which, float (&o)[2 * CPT]) {
+    const float2 gate = *reinterpret_cast<const float2*>(base + SC + t * 4);
+    float2 u2[CPT], acc[CPT];
+    float w = gate.y;
+    if constexpr (decltype(divided)::value) {
+      F *= gate.x;
+      w = __fdividef(w, F);
+    } else {
+      const float2 f2 = make_float2(gate.x, gate.x);
 #pragma unroll
-    for (int c = 0; c < CPT; ++c) {
-      u[c] = base[SV + t * cols + col + c] * gate.y;
-      acc[c] = make_float2(0.f, 0.f);
+      for (int c = 0; c < CPT; ++c)
+#pragma unroll
+        for (int j = 0; j < NR / 2; ++j) S[c][j] = ls_mul2(S[c][j], f2);
+    }
+#pragma unroll
+    for (int c = 0; c < CPT; c += 4) {
+      const float4 v = *reinterpret_cast<const float4*>(base + SV + t * cols + col + c);
+      u2[c] = make_float2(v.x * w, v.x * w);
+      u2[c + 1] = make_float2(v.y * w, v.y * w);
+      u2[c + 2] = make_float2(v.z * w, v.z * w);
+      u2[c + 3] = make_float2(v.w * w, v.w * w);
     }
 #pragma unroll
     for (int j = 0; j < NR / 4; ++j) {
-      const int r = rg * 4 + j * 32;
+      const int r = rg * 4 + j * 4 * RG;
       const float4 k4 = *reinterpret_cast<const float4*>(base + t * W + r);
       const float4 q4 = *reinterpret_cast<const float4*>(base + SQ + t * W + r);
 #pragma unroll
       for (int c = 0; c < CPT; ++c) {
-        const float2 f2 = make_float2(gate.x, gate.x), u2 = make_float2(u[c], u[c]);
-        S[c][2 * j] = ls_fma2(S[c][2 * j], f2, ls_mul2(make_float2(k4.x, k4.y), u2));
-        S[c][2 * j + 1] = ls_fma2(S[c][2 * j + 1], f2, ls_mul2(make_float2(k4.z, k4.w), u2));
-        acc[c] = ls_fma2(S[c][2 * j], make_float2(q4.x, q4.y), acc[c]);
+        S[c][2 * j] = ls_fma2(make_float2(k4.x, k4.y), u2[c], S[c][2 * j]);
+        S[c][2 * j + 1] = ls_fma2(make_float2(k4.z, k4.w), u2[c], S[c][2 * j + 1]);
+        acc[c] = j == 0 ? ls_mul2(S[c][0], make_float2(q4.x, q4.y)) : ls_fma2(S[c][2 * j], make_float2(q4.x, q4.y), acc[c]);
         acc[c] = ls_fma2(S[c][2 * j + 1], make_float2(q4.z, q4.w), acc[c]);
       }
     }
 #pragma unroll
-    for (int c = 0; c < CPT; ++c) o[c] = acc[c].x + acc[c].y;
+    for (int c = 0; c < CPT; ++c) o[2 * c + which] = acc[c].x + acc[c].y;
   };
-  auto write = [&](int t, int c, float o) {  // c: column of the CTA
-    if (c >= ncol) return;
-    if (is_n) orow[t * ostep] = fmaxf(fabsf(o), base[SC + t * 4 + 2]) + 1e-6f;
-    else orow[t * ostep + c] = fmaf(skip, base[SV + t * cols + c], o);
-  };
-  // Sums over the 8 row groups of the CPT columns of two tokens: in every round a lane keeps half of its sums and trades the others,
-  // first by token, then by the bits of the column; what is left is summed plainly.
-  auto pair = [&](int t, bool second) {
-    float x[CPT], y[CPT], z[CPT];
-    advance(t, x);
+  auto pair = [&](auto divided, int t, bool second) {
+    float x[2 * CPT];
+    advance(divided, t, 0, x);
+    const float F0 = F;
     if (second) {
-      advance(t + 1, y);
+      advance(divided, t + 1, 1, x);
     } else {
 #pragma unroll
-      for (int c = 0; c < CPT; ++c) y[c] = 0.f;
+      for (int c = 0; c < CPT; ++c) x[2 * c + 1] = 0.f;
     }
-    const bool b0 = rg & 1, b1 = rg & 2, b2 = rg & 4;
-#pragma unroll
-    for (int c = 0; c < CPT; ++c) z[c] = (b0 ? y[c] : x[c]) + __shfl_xor_sync(0xffffffffu, b0 ? x[c] : y[c], 1);
-    if constexpr (CPT == 4) {
-      float p[2];
-#pragma unroll
-      for (int i = 0; i < 2; ++i) p[i] = (b1 ? z[2 * i + 1] : z[2 * i]) + __shfl_xor_sync(0xffffffffu, b1 ? z[2 * i] : z[2 * i + 1], 2);
-      const float o = (b2 ? p[1] : p[0]) + __shfl_xor_sync(0xffffffffu, b2 ? p[0] : p[1], 4);
-      if (!b0 || second) write(t + b0, col + 2 * b2 + b1, o);
-    } else if constexpr (CPT == 2) {
-      float o = (b1 ? z[1] : z[0]) + __shfl_xor_sync(0xffffffffu, b1 ? z[0] : z[1], 2);
-      o += __shfl_xor_sync(0xffffffffu, o, 4);
-      if (!b2 && (!b0 || second)) write(t + b0, col + b1, o);
+    const float o = ls_reduce<RG, 2 * CPT>(x, rg) * (rg & 1 ? F : F0);
+    const int tok = t + (rg & 1), c = col + ((rg >> 1) & (CPT - 1));
+    if (rg >= 2 * CPT || c >= ncol || ((rg & 1) && !second)) return;
+    if (is_n) orow[tok * ostep] = fmaxf(fabsf(o), base[SC + tok * 4 + 2]) + 1e-6f;
+    else orow[tok * ostep + c] = fmaf(skip, base[SV + tok * cols + c], o);
+  };
+  auto tokens = [&](auto divided, int cnt) {
+    if (cnt == LS_TOK) {  // unrolled: the sums of a pair of tokens are taken underneath the next one's products
+#pragma unroll 2
+      for (int t = 0; t < LS_TOK; t += 2) pair(divided, t, true);
     } else {
-      float o = z[0] + __shfl_xor_sync(0xffffffffu, z[0], 2);
-      o += __shfl_xor_sync(0xffffffffu, o, 4);
-      if (!b2 && !b1 && (!b0 || second)) write(t + b0, col, o);
+#pragma unroll 1
+      for (int t = 0; t < cnt; t += 2) pair(divided, t, t + 1 < cnt);
     }
   };
 
@@ -444,18 +473,26 @@ __global__ void __launch_bounds__(256) linear_scan_kernel(const __grid_constant_
     else ls_commit();
     base = ls_smem + (ch % LS_STAGES) * stage;
     const int cnt = min(LS_TOK, n - ch * LS_TOK);
-    if (cnt == LS_TOK) {
-#pragma unroll 1
-      for (int t = 0; t < LS_TOK; t += 2) pair(t, true);
+    F = 1.f;
+    for (int t = 0; t < cnt; ++t) F *= base[SC + t * 4];
+    const bool divided = F > LS_LEAST;  // the same for every thread
+    F = 1.f;
+    if (divided) {
+      tokens(std::true_type(), cnt);
+      const float2 f2 = make_float2(F, F);
+#pragma unroll
+      for (int c = 0; c < CPT; ++c)
+#pragma unroll
+        for (int j = 0; j < NR / 2; ++j) S[c][j] = ls_mul2(S[c][j], f2);
     } else {
-      for (int t = 0; t < cnt; t += 2) pair(t, t + 1 < cnt);
+      tokens(std::false_type(), cnt);
     }
     orow += LS_TOK * ostep;
   }
 
 #pragma unroll
   for (int j = 0; j < NR / 2; ++j) {
-    const int r = rg * 4 + (j >> 1) * 32 + (j & 1) * 2;
+    const int r = rg * 4 + (j >> 1) * (4 * RG) + (j & 1) * 2;
 #pragma unroll
     for (int c = 0; c < CPT; ++c)
       if (col + c < ncol) {
@@ -730,14 +767,16 @@ static int launch_memory_prep(const MemoryIn& a, const int* segs, int nseg, int 
   return (int)launch_pdl(kern, grid, dim3(256), 0, s, a, reinterpret_cast<const int4*>(segs), nseg, rows, gate_ctas, q, k, v, gates);
 }
 
-template <int NR, int CPT>
+// WARPS: of a CTA with all its columns; narrow heads take fewer.
+template <int RG, int NR, int CPT, int WARPS, int CTAS>
 static int launch_linear_scan(Scan a, int nseg, cudaStream_t s) {
-  const int wide = NR >= 32 ? 32 : 64;  // columns of a CTA at most
-  const int cols = a.DV > wide / 2 ? wide : a.DV > 16 ? 32 : 16;
-  const int warps = cols / (4 * CPT);
-  const int bytes = LS_STAGES * LsSmem<NR>::stage_floats(cols) * 4;
-  auto kern = linear_scan_kernel<NR, CPT>;
-  if (cudaError_t e = ensure_dynamic_smem(reinterpret_cast<const void*>(kern), LS_STAGES * LsSmem<NR>::stage_floats(64) * 4); e != cudaSuccess) return (int)e;
+  constexpr int per = 32 / RG * CPT;  // columns of a warp
+  int warps = WARPS;
+  while (warps > 1 && warps / 2 * per >= a.DV) warps /= 2;
+  const int cols = warps * per, bytes = LS_STAGES * LsSmem<RG, NR>::stage_floats(cols) * 4;
+  auto kern = linear_scan_kernel<RG, NR, CPT, WARPS * 32, CTAS>;
+  if (cudaError_t e = ensure_dynamic_smem(reinterpret_cast<const void*>(kern), LS_STAGES * LsSmem<RG, NR>::stage_floats(WARPS * per) * 4); e != cudaSuccess)
+    return (int)e;
   a.blocks = (a.DV + cols - 1) / cols;
   // A plain launch: CTAs that start while the previous kernel still holds most of the machine would pile up on the few SMs
   // that are free, and stay there for the whole sequence.
@@ -799,11 +838,15 @@ extern "C" int sb_linear_scan(const float* q, const float* k, const float* v, co
     return (int)cudaErrorInvalidValue;
   const sb::Scan a{q, k, v, (const float4*)gates, skip, out, state, norm, den, reinterpret_cast<const int4*>(segs), H, G, D, DV, 0,
                    ring, {in0, in1, in2}, in_pitch, {w0, w1, w2}, taps, esize};
-  if (D <= 32) return sb::launch_linear_scan<4, 4>(a, nseg, s);
-  if (D <= 64) return sb::launch_linear_scan<8, 4>(a, nseg, s);
-  if (D <= 128) return sb::launch_linear_scan<16, 4>(a, nseg, s);
-  if (D <= 256) return sb::launch_linear_scan<32, 2>(a, nseg, s);
-  return sb::launch_linear_scan<64, 1>(a, nseg, s);
+  if (D <= 32) return sb::launch_linear_scan<8, 4, 4, 4, 4>(a, nseg, s);
+  if (D <= 64) return sb::launch_linear_scan<16, 4, 8, 4, 4>(a, nseg, s);
+  // a CTA of 64 columns has an SM to itself: more warps with fewer columns per lane hide more of a token's latency
+  const bool few = static_cast<long>(nseg) * H * ((DV + 63) / 64 + (norm != nullptr ? 1 : 0)) <= 148;
+  if (few && D <= 128) return sb::launch_linear_scan<16, 8, 4, 8, 1>(a, nseg, s);
+  if (few && D <= 256) return sb::launch_linear_scan<16, 16, 4, 8, 1>(a, nseg, s);
+  if (D <= 128) return sb::launch_linear_scan<16, 8, 8, 4, 4>(a, nseg, s);
+  if (D <= 256) return sb::launch_linear_scan<32, 8, 8, 8, 2>(a, nseg, s);
+  return sb::launch_linear_scan<32, 16, 4, 8, 1>(a, nseg, s);
 }
 
 // One token per row: slot / active / pos [B]; rows that are not active leave every state alone. out [B, H, DV] fp32.

@@ -387,7 +387,17 @@ __global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, lon
   pdl_launch_dependents();
   float* row = x + static_cast<long>(blockIdx.y) * pitch;
   const float inv = 1.f / cap;
-  for (long i = static_cast<long>(blockIdx.x) * 256 + threadIdx.x; i < n; i += static_cast<long>(gridDim.x) * 256) row[i] = cap * tanhf(row[i] * inv);
+  const bool vec = ((reinterpret_cast<uintptr_t>(row) & 15) | (n & 3)) == 0;
+  const long step = static_cast<long>(gridDim.x) * 256, first = static_cast<long>(blockIdx.x) * 256 + threadIdx.x;
+  for (long i = first; vec && i < n / 4; i += step) {
+    float4 v = reinterpret_cast<float4*>(row)[i];
+    v.x = cap * tanhf(v.x * inv);
+    v.y = cap * tanhf(v.y * inv);
+    v.z = cap * tanhf(v.z * inv);
+    v.w = cap * tanhf(v.w * inv);
+    reinterpret_cast<float4*>(row)[i] = v;
+  }
+  for (long i = first; !vec && i < n; i += step) row[i] = cap * tanhf(row[i] * inv);
 }
 
 // One CTA per token: `kb` bytes of its key row and `vb` bytes of its value row to cache slot slots[t] (< 0: skipped).
@@ -482,6 +492,100 @@ __global__ void __launch_bounds__(128) heads_kernel(const __grid_constant__ Head
     }
     dst[d] = from_f<T>(y);
   }
+}
+
+// The same for the usual widths, 8 elements per lane and 32 / L heads per warp: L = D / 8 lanes have a query or key head (L a power
+// of two; halves of a rotation are whole vectors), the value heads follow as one row of Hv * DV elements.
+template <typename T, int L>
+__global__ void __launch_bounds__(256) heads_wide_kernel(const __grid_constant__ Heads a) {
+  constexpr int D = 8 * L;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int lane = threadIdx.x % L;
+  const long t = blockIdx.x;
+  const int slot = a.slots[t], heads = a.Hq + a.Hkv, half = a.dims / 2, c0 = lane * 8;
+  const float* cs = half > 0 ? a.table + static_cast<long>(a.positions[t]) * a.dims : nullptr;
+  // a lane's part of the rotation is the same for every head: pair of element i, and whether it is the second of its pair
+  float cosv[8], sinv[8];
+  const bool turned = c0 < a.dims;
+  const int away = a.interleaved || !turned ? 0 : half / 8;  // lanes to the other half
+  const bool second = turned && !a.interleaved && c0 >= half;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int p = a.interleaved ? (c0 + i) / 2 : second ? c0 + i - half : c0 + i;
+    cosv[i] = turned ? cs[p] : 1.f;
+    sinv[i] = turned ? cs[half + p] : 0.f;
+    if (a.interleaved ? !(i & 1) : !second) sinv[i] = -sinv[i];
+  }
+  const int rounds = (heads * L + 255) / 256;  // whole warps stay together for the exchanges
+  for (int r = 0; r < rounds; ++r) {
+    const int vec = (r * 256 + static_cast<int>(threadIdx.x)) / L;
+    const bool on = vec < heads, is_q = vec < a.Hq;
+    const int h = is_q ? vec : vec - a.Hq;
+    float x[8], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) x[i] = 0.f;
+    if (on) load_vec<T, 8>((is_q ? reinterpret_cast<const T*>(a.q) + t * a.q_pitch : reinterpret_cast<const T*>(a.k) + t * a.k_pitch) + h * D + c0, x);
+    const T* w = reinterpret_cast<const T*>(is_q ? a.q_norm : a.k_norm);
+    if (a.q_norm != nullptr) {
+#pragma unroll
+      for (int i = 0; i < 8; ++i) ss = fmaf(x[i], x[i], ss);
+#pragma unroll
+      for (int o = 1; o < L; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      if (on && w != nullptr) {
+        const float rs = 1.f / sqrtf(ss / D + a.eps);
+        float g[8];
+        load_vec<T, 8>(w + c0, g);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) x[i] *= rs * g[i];
+      }
+    }
+    if (half > 0) {
+      float other[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) other[i] = x[i ^ 1];
+      if (!a.interleaved) {
+        const int from = (threadIdx.x & 31) + (second ? -away : away);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) other[i] = __shfl_sync(0xffffffffu, x[i], from & 31);
+      }
+#pragma unroll
+      for (int i = 0; i < 8; ++i) x[i] = fmaf(other[i], sinv[i], x[i] * cosv[i]);
+    }
+    if (!on || (!is_q && slot < 0)) continue;
+    if (is_q) {
+      T* dst = reinterpret_cast<T*>(a.q_out) + t * a.q_out_pitch + static_cast<long>(h) * a.maps * D + c0;
+      if (a.maps == 2) {
+        const float zero[8] = {};
+        store_vec<T, 8>(h & 1 ? dst : dst + D, zero);
+        dst += h & 1 ? D : 0;
+      }
+      store_vec<T, 8>(dst, x);
+    } else {
+      store_vec<T, 8>(reinterpret_cast<T*>(a.k_cache) + (static_cast<long>(slot) * a.Hkv + h) * D + c0, x);
+    }
+  }
+  if (slot < 0) return;
+  const int nv = a.Hv * a.DV;
+  const T* v = reinterpret_cast<const T*>(a.v) + t * a.v_pitch;
+  T* v_out = reinterpret_cast<T*>(a.v_cache) + static_cast<long>(slot) * nv;
+  for (int c = threadIdx.x * 8; c < nv; c += 256 * 8) {
+    float e[8];
+    load_vec<T, 8>(v + c, e);
+    store_vec<T, 8>(v_out + c, e);
+  }
+}
+
+template <typename T>
+static int launch_heads(const Heads& a, int rows, cudaStream_t s) {
+  const int L = a.D / 8, half = a.dims / 2;
+  bool wide = a.D % 8 == 0 && (L == 4 || L == 8 || L == 16 || L == 32) && (a.Hv * a.DV) % 8 == 0 && a.q_pitch % 8 == 0 && a.k_pitch % 8 == 0 &&
+              a.v_pitch % 8 == 0 && a.q_out_pitch % 8 == 0 && (a.interleaved ? a.dims : half) % 8 == 0;
+  for (const void* x : {a.q, a.k, a.v, static_cast<const void*>(a.q_out), a.q_norm, a.k_norm, static_cast<const void*>(a.k_cache), static_cast<const void*>(a.v_cache)})
+    wide = wide && (reinterpret_cast<uintptr_t>(x) & 15) == 0;
+  if (!wide) return (int)launch_pdl(heads_kernel<T>, dim3(rows, (a.Hq + a.Hkv + a.Hv + 3) / 4), dim3(128), 0, s, a);
+  auto kern = L == 4 ? heads_wide_kernel<T, 4> : L == 8 ? heads_wide_kernel<T, 8> : L == 16 ? heads_wide_kernel<T, 16> : heads_wide_kernel<T, 32>;
+  return (int)launch_pdl(kern, dim3(rows), dim3(256), 0, s, a);
 }
 
 // The same with one norm over all query heads and one over all key heads (a weight per channel): one CTA per token, its rows
@@ -671,9 +775,7 @@ extern "C" int sb_heads(const void* q, const void* k, const void* v, void* q_out
     return (int)cudaErrorInvalidValue;
   const sb::Heads a{q, k, v, q_out, q_norm, k_norm, table, positions, slots, k_cache, v_cache, Hq, Hkv, Hv, D, DV, dims, interleaved, maps,
                     q_pitch, k_pitch, v_pitch, q_out_pitch, eps};
-  const dim3 grid(T, (Hq + Hkv + Hv + 3) / 4);
-  if (f32) return (int)sb::launch_pdl(sb::heads_kernel<float>, grid, dim3(128), 0, s, a);
-  return (int)sb::launch_pdl(sb::heads_kernel<__nv_bfloat16>, grid, dim3(128), 0, s, a);
+  return f32 ? sb::launch_heads<float>(a, T, s) : sb::launch_heads<__nv_bfloat16>(a, T, s);
 }
 
 // As sb_heads, with norms over all query heads and over all key heads (see HeadsAll).
