@@ -126,7 +126,7 @@ def gemm(a, b, *, a_mn=False, b_mn=False, bias=None, out=None, out_dtype=None, a
     if b.stride(-1) != 1:
         b = b.contiguous()
     bn = bn or _pick_bn(M, N)
-    can_split = out_dtype == torch.float32 and (accumulate or out is None)
+    can_split = out_dtype == torch.float32 and (accumulate or (out is None and N % 4 == 0))  # TMA reduce-add: 16-byte rows
     if splitk is None:
         splitk = _pick_splitk(M, N, K, bn, _lib.sm_count(a.device)) if can_split else 1
     if out is None:

@@ -3,6 +3,8 @@
 import pytest
 import torch
 
+from slime_b200 import ops
+
 pytestmark = pytest.mark.gpu
 
 
@@ -28,7 +30,6 @@ def _check(out, ref, tol=2e-2, K=None):
                                    (77, 200, 72), (4096, 4864, 896), (130, 151936 // 16, 896)])  # fmt: skip
 @pytest.mark.parametrize("bn", [128, 256])
 def test_gemm_nt_bf16(kernels, M, N, K, bn):
-    from slime_b200 import ops
     from slime_b200.ops import _lib
 
     torch.manual_seed(M + N + K)
@@ -41,7 +42,6 @@ def test_gemm_nt_bf16(kernels, M, N, K, bn):
 
 
 def test_gemm_fp32_out_bias_accumulate(kernels):
-    from slime_b200 import ops
     from slime_b200.ops import _lib
 
     torch.manual_seed(0)
@@ -65,7 +65,6 @@ def test_gemm_fp32_out_bias_accumulate(kernels):
 
 def test_gemm_matches_cublas_closely(kernels):
     """Same bf16 inputs, fp32 accumulate: results should agree with cuBLAS to bf16 rounding."""
-    from slime_b200 import ops
 
     torch.manual_seed(1)
     a = torch.randn(2048, 1024, device="cuda", dtype=torch.bfloat16)
@@ -73,3 +72,11 @@ def test_gemm_matches_cublas_closely(kernels):
     ours = ops.gemm(a, b, out_dtype=torch.float32)
     ref = _ref(a, b)
     assert (ours - ref).abs().max().item() < 1e-2 * ref.abs().max().item()
+
+
+def test_fp32_output_of_any_width(kernels):
+    """Few rows and a long K ask for split-K, whose sums need rows of whole 16-byte pieces; other widths take one pass."""
+    for N in (33, 90, 130, 64):
+        a, b = torch.randn(7, 4096, device="cuda").bfloat16(), torch.randn(N, 4096, device="cuda").bfloat16()
+        got = ops.gemm(a, b, out_dtype=torch.float32)
+        torch.testing.assert_close(got, a.float() @ b.float().t(), atol=2e-2, rtol=2e-3)
