@@ -63,7 +63,7 @@ def parse():
     p.add_argument("--e2e-steps", type=int, default=None, help="steps of the end-to-end arm (default: --steps)")
     p.add_argument("--no-e2e", action="store_true")
     p.add_argument("--workload", type=str, default="grpo", choices=["grpo", "serve"],
-                   help="serve: prefill / decode throughput of Pefolix, Ledazen and Zetizen beside the closest existing models (slime_b200/engine/serve_bench.py)")
+                   help="serve: prefill / decode throughput of Pefolix, Ledazen, Zetizen and Pebodra beside the closest existing models (slime_b200/engine/serve_bench.py)")
     p.add_argument("--pair", type=str, default=None, help="serve: only the model pairs whose name contains this")
     a = p.parse_args()
     for k, v in CONFIGS[a.config].items():

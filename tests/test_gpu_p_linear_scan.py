@@ -125,6 +125,46 @@ def test_batches_and_idle_rows(kernels, make, shape, dtype):
     _close(b.state, a.state, tol)
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("make,shape", [(_space, (44, 4, 100, 56, 4, 4)), (_space, (40, 1, 128, 64, 3, 1)), (_memory, (10, 200, 300)), (_memory, (50, 128, 20))])
+def test_many_heads_and_requests(kernels, make, shape, dtype):
+    """Enough work to fill the machine: the form of the scan with more columns per lane."""
+    counts, tol = [31, 8, 1, 40], 3e-2 if dtype == torch.bfloat16 else 2e-4
+    T = sum(counts)
+    on, state, names = make(shape, T, dtype)
+    res = []
+    for x, dev, dt in ((on("cpu", torch.float32), "cpu", torch.float32), (on(DEV), DEV, dtype)):
+        s = state(dev, dt, 0.0)
+        s = linear_scan.SlotState(*(None if t is None else torch.cat([t, t]) for t in (s.state, s.ring, s.norm, s.top)))
+        batch = wa.ExtendBatch.build([[0]] * 4, [0] * 4, counts, 256, dev, state_slots=[4, 0, 2, 5])
+        res.append((x.extend(s, batch), s.state, s.norm if s.norm is not None else s.state))
+    for a, b in zip(*res):
+        _close(b, a, tol)
+
+
+@pytest.mark.parametrize("make,shape", [(_space, (6, 2, 100, 40, 4, 2)), (_space, (4, 4, 16, 20, 2, 1)), (_memory, (4, 40, 24)), (_memory, (3, 180, 70))])
+def test_decays_of_any_strength(kernels, make, shape):
+    """Heads that forget everything at once, heads that forget slowly, and a change of mind in the middle of a prompt."""
+    T, H = 90, shape[0]
+    on, state, names = make(shape, T, torch.float32)
+    res = []
+    for dev in ("cpu", DEV):
+        x = on(dev)
+        strength = torch.linspace(-3.0, 6.0, H, device=dev)
+        if make is _space:
+            x.A_log[:] = strength
+            x.dt[40:60] += 8.0
+        else:
+            x.f_b[:] = 4.0 - 3 * strength
+            x.i[40:43] += 30.0  # an input that takes over
+        s = state(dev, torch.float32, 0.0)
+        out = [_cut(x, a, b, names).extend(s, wa.ExtendBatch.build([[0]], [a], [b - a], 256, dev, state_slots=[1])) for a, b in ((0, 37), (37, 90))]
+        res.append((torch.cat(out), s.state[1]))
+    for a, b in zip(*res):
+        assert torch.isfinite(a).all()
+        _close(b, a, 2e-4)
+
+
 def test_a_long_scan_keeps_a_far_token(kernels):
     """3000 tokens with decays near one: the first one still shows, in portions and in one pass alike."""
     H, D, DV, T = 2, 64, 64, 3000
