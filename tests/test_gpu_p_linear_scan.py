@@ -153,10 +153,10 @@ def test_decays_of_any_strength(kernels, make, shape):
         strength = torch.linspace(-3.0, 6.0, H, device=dev)
         if make is _space:
             x.A_log[:] = strength
-            x.dt[40:60] += 8.0
+            x.dt[40:60] = 8.0
         else:
             x.f_b[:] = 4.0 - 3 * strength
-            x.i[40:43] += 30.0  # an input that takes over
+            x.i[40:43] = 30.0  # an input that takes over
         s = state(dev, torch.float32, 0.0)
         out = [_cut(x, a, b, names).extend(s, wa.ExtendBatch.build([[0]], [a], [b - a], 256, dev, state_slots=[1])) for a, b in ((0, 37), (37, 90))]
         res.append((torch.cat(out), s.state[1]))
